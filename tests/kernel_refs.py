@@ -36,7 +36,8 @@ def add_rms_norm(resid, delta, weight, eps, out, rows=None) -> None:
 
 
 def post_norm_add_rms_norm(resid, delta, post_weight, layer_scale, post_eps, post_offset, weight, offset, eps, out,
-                           rows=None, post_mult=1.0, delta_bias=None) -> None:
+                           rows=None, post_mult=1.0, delta_bias=None, second=None, second_scale=1.0, add_rows=None,
+                           add_vec=None) -> None:
     x = resid if rows is None else resid[rows.long()]
     if delta is not None:
         y = (delta if rows is None else delta[rows.long()]).float()
@@ -44,20 +45,27 @@ def post_norm_add_rms_norm(resid, delta, post_weight, layer_scale, post_eps, pos
             y = y + delta_bias.float()
         if post_weight is not None:
             g = post_weight.float()
-            y = y * torch.rsqrt(y.pow(2).mean(-1, keepdim=True) + post_eps) * (1 + g if post_offset else g) * post_mult
+            y = y * torch.rsqrt(y.pow(2).mean(-1, keepdim=True) + post_eps) * (1 + g if post_offset else g)
+        y = y * post_mult
         if layer_scale is not None:
             y = y * layer_scale.float()
         x = x + y
-        if rows is None:
-            resid.copy_(x)
+        if second is not None:
+            x = x + second_scale * (second if rows is None else second[rows.long()]).float()
+    if add_rows is not None:
+        x = x + (add_rows if rows is None else add_rows[rows.long()])
+    if add_vec is not None:
+        x = x + add_vec.float()
+    if rows is None:
+        resid.copy_(x)
     g = weight.float()
     out.copy_((x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps) * (1 + g if offset else g)).to(out.dtype))
 
 
-def rope_tables(positions, inv_freq, cos, sin) -> None:
+def rope_tables(positions, inv_freq, cos, sin, mult=1.0) -> None:
     a = positions.double()[:, None] * inv_freq[None, :]
-    cos.copy_(a.cos().float())
-    sin.copy_(a.sin().float())
+    cos.copy_((a.cos() * mult).float())
+    sin.copy_((a.sin() * mult).float())
 
 
 def silu_mul(gate_up, out) -> None:
@@ -144,6 +152,36 @@ def paged_attention(q, k_cache, v_cache, page_size, block_tables, ctx: Any, scal
             p = torch.softmax(s, -1)
         res[r0: r0 + n] = torch.einsum("hij,jhd->ihd", p, v)
     out.copy_(res.view(t, hq * dv).to(out.dtype))
+
+
+def talking_attention(q, k_cache, v_cache, page_size, block_tables, ctx: Any, scale, window, softcap, talk, out,
+                      sinks=None) -> None:
+    t, hq, d = q.shape
+    group, dv = hq // k_cache.shape[1], v_cache.shape[3]
+    res = torch.zeros(t, hq, dv, dtype=torch.float32, device=q.device)
+    cu, lens = ctx.cu_query_lens.tolist(), ctx.context_lens_dev.tolist()
+    for b in range(ctx.num_seqs):
+        r0, n, total = cu[b], cu[b + 1] - cu[b], lens[b]
+        lo = max(0, (total - n) - window + 1) if window else 0      # pages before this may be gone
+        pos = torch.arange(lo, total, device=q.device)
+        pages = block_tables[b].long()[pos // page_size]
+        k = k_cache[pages, :, pos % page_size].float().repeat_interleave(group, dim=1)
+        v = v_cache[pages, :, pos % page_size].float().repeat_interleave(group, dim=1)
+        qpos = torch.arange(total - n, total, device=q.device)
+        hidden = pos[None, :] > qpos[:, None]
+        if window:
+            hidden = hidden | (pos[None, :] <= qpos[:, None] - window)
+        s = torch.einsum("ihd,jhd->hij", q[r0: r0 + n].float(), k) * scale
+        if softcap is not None:
+            s = softcap * torch.tanh(s / softcap)
+        s = s.masked_fill(hidden, float("-inf"))
+        if sinks is not None:
+            s = torch.cat([s, sinks.float()[:, None, None].expand(hq, n, 1)], dim=-1)
+        p = torch.softmax(s, -1)[..., : pos.shape[0]]
+        if talk is not None:
+            p = torch.einsum("hg,gij->hij", talk.float(), p)
+        res[r0: r0 + n] = torch.einsum("hij,jhd->ihd", p, v)
+    out.copy_(res.reshape(out.shape).to(out.dtype))
 
 
 def gemm(x, w, out) -> None:
@@ -309,6 +347,20 @@ def moe_route(logits, top, counts, arena=None, tile_rows=64, rule=None, outputs=
         order = torch.sort(-choice, dim=-1, stable=True).indices[:, :top]
         picked = torch.gather(scores, 1, order)
         weights = picked / (picked.sum(-1, keepdim=True) + 1e-20) * rule.scale
+        if getattr(rule, "sigmoid", False):
+            choice = scores = torch.sigmoid(z)
+            if rule.correction is not None:
+                choice = scores + rule.correction.float()
+            if rule.groups > 1:
+                best = choice.view(t, rule.groups, -1).max(-1).values
+                kept = torch.sort(-best, dim=-1, stable=True).indices[:, : rule.keep]
+                allowed = torch.zeros(t, rule.groups, dtype=torch.bool, device=z.device).scatter_(1, kept, True)
+                choice = choice.masked_fill(~allowed.repeat_interleave(e // rule.groups, dim=1), float("-inf"))
+            order = torch.sort(-choice, dim=-1, stable=True).indices[:, :top]
+            picked = torch.gather(scores, 1, order)
+            weights = picked / (picked.sum(-1, keepdim=True) + 1e-20) * rule.scale
+        if not getattr(rule, "normalise", True):
+            weights = picked * rule.scale
     real = e - identity
     ids = order.reshape(-1)
     queued = torch.nonzero(ids < real).reshape(-1)                     # picks of experts with matrices
@@ -319,19 +371,28 @@ def moe_route(logits, top, counts, arena=None, tile_rows=64, rule=None, outputs=
     token_of[: by_expert.numel()] = by_expert // top
     sizes = torch.bincount(ids[queued], minlength=real)
     offsets = torch.cat([sizes.new_zeros(1), sizes.cumsum(0)])
-    return {"top": top, "experts": real, "picks": ids.numel(), "ids": ids.int(), "weights": weights.reshape(-1),
+    row_weight = None
+    if rule is not None and getattr(rule, "on_input", False):
+        row_weight = torch.zeros(ids.numel(), device=z.device)
+        row_weight[: by_expert.numel()] = weights.reshape(-1)[by_expert]
+    return {"top": top, "experts": real, "picks": ids.numel(), "ids": ids.int(), "weights": weights.reshape(-1), "row_weight": row_weight,
             "row_of": row_of.int(), "token_of": token_of.int(), "offsets": offsets.int(), "logits": logits, "identity": identity,
             "max_tiles": moe_max_tiles(t, top, real, tile_rows), "tile_rows": tile_rows}
 
 
-def moe_gemm(x, w, out, plan, gated, gather, arena=None) -> None:
+def moe_gemm(x, w, out, plan, gated, gather, arena=None, limit=0.0) -> None:
     off = plan["offsets"].tolist()
     src = x[plan["token_of"].long()] if gather else x
     n = out.shape[1]
     for e in range(plan["experts"]):
         if off[e + 1] > off[e]:
             z = src[off[e]: off[e + 1]].float() @ w[e].float().t()
-            if gated:
+            if gated and plan.get("row_weight") is not None:
+                z = z * plan["row_weight"][off[e]: off[e + 1], None]
+            if gated and limit > 0:
+                g, u = z[:, :n].clamp(max=limit), z[:, n:].clamp(-limit, limit)
+                z = g * torch.sigmoid(1.702 * g) * (u + 1)
+            elif gated:
                 z = z[:, :n] * torch.sigmoid(z[:, :n]) * z[:, n:]
             out[off[e]: off[e + 1]] = z.to(out.dtype)
 
@@ -342,7 +403,7 @@ def moe_combine(y, plan, shared_out, out, x=None, shared_gate=None) -> None:
     picked = y[rows.clamp(min=0)].float().reshape(t, top, -1)
     if x is not None:                       # an identity pick's output is the token's input
         picked = torch.where((rows < 0).reshape(t, top, 1), x.float().reshape(t, 1, -1), picked)
-    total = (picked * plan["weights"].reshape(t, top, 1)).sum(1)
+    total = picked.sum(1) if plan.get("row_weight") is not None else (picked * plan["weights"].reshape(t, top, 1)).sum(1)
     if shared_out is not None:
         g = 1.0 if shared_gate is None else torch.sigmoid(shared_gate.float()).reshape(t, 1)
         total = total + g * shared_out.float()
@@ -446,6 +507,35 @@ def qkv_prepare(q_in, k_in, v_in, q_weight, k_weight, eps, cos, sin, rotary_dim,
     v_cache[page, :, off] = v
 
 
+def qkv_rotate(proj, taps, state, ctx, cos, sin, rotary_dim, interleaved, unit_eps, slots, k_cache, v_cache, page_size, heads,
+               kv_heads, d, dv, q_out) -> None:
+    t = q_out.shape[0]
+    channels = (heads + kv_heads) * d + kv_heads * dv
+    x = proj[:, :channels].float()
+    if taps is not None:
+        k = taps.shape[0]
+        cu, rows = ctx.cu_query_lens.tolist(), None if k == 1 else ctx.state_slots.tolist()
+        y = torch.empty_like(x)
+        for b in range(ctx.num_seqs):
+            lo, hi = cu[b], cu[b + 1]
+            before = x[:0] if k == 1 else state[rows[b]].view(k - 1, channels).float()
+            seq = torch.cat([before, x[lo:hi]])
+            y[lo:hi] = sum(seq[j: j + hi - lo] * taps[j].float()[None, :] for j in range(k))
+            if k > 1:
+                state[rows[b]] = seq[-(k - 1):].reshape(-1)
+        x = y
+
+    def prep(z, n):
+        z = _rotate(z.reshape(t, n, d), cos, sin, rotary_dim, interleaved)
+        return z if unit_eps is None else z * torch.rsqrt(z.pow(2).mean(-1, keepdim=True) + unit_eps)
+
+    q, k_, v = x[:, : heads * d], x[:, heads * d: (heads + kv_heads) * d], x[:, (heads + kv_heads) * d:]
+    q_out.copy_(prep(q, heads).to(q_out.dtype))
+    page, off = slots.long() // page_size, slots.long() % page_size
+    k_cache[page, :, off] = prep(k_, kv_heads).to(k_cache.dtype)
+    v_cache[page, :, off] = v.reshape(t, kv_heads, dv).to(v_cache.dtype)
+
+
 # ------------------------------------------------- linear attention without a correction term
 def _silu(z):
     return z * torch.sigmoid(z)
@@ -496,6 +586,21 @@ def linear_scan_gated(q, k, v, w_pre, w_bias, tau, q_scale, state, ctx, heads, d
                 S = alpha[:, None] * S + torch.outer(kk, vv)
                 out[t, h] = S.t() @ qq
             st[h] = S
+
+
+def linear_scan_rotated(q, k, v, decay, cos, sin, rotary_dim, interleaved, k_scale, state, ctx, heads, d, dv, out) -> None:
+    cu, slots = ctx.cu_query_lens.tolist(), ctx.state_slots.tolist()
+    t, dt = q.shape[0], state.dtype
+    qq = _rotate(q.to(dt).reshape(t, heads, d), cos, sin, rotary_dim, interleaved)
+    kk = _rotate(k.to(dt).reshape(t, heads, d), cos, sin, rotary_dim, interleaved) * k_scale
+    vv = v.to(dt).reshape(t, heads, dv)
+    for b in range(ctx.num_seqs):
+        st = state[slots[b]].view(heads, d, dv)
+        S = st.clone()
+        for i in range(cu[b], cu[b + 1]):
+            S = decay.to(dt)[:, None, None] * S + kk[i][:, :, None] * vv[i][:, None, :]
+            out[i] = torch.einsum("hkv,hk->hv", S, qq[i])
+        st.copy_(S)
 
 
 def rms_norm_rows(x, weight, eps, out) -> None:
@@ -622,7 +727,7 @@ _NAMES = ["embed", "add_rms_norm", "rope_tables", "silu_mul", "qk_norm_rope_writ
           "post_norm_add_rms_norm", "latent_prepare", "latent_attention", "bmm", "transpose01", "moe_max_tiles", "moe_tile_rows", "moe_route_from",
           "moe_route", "moe_gemm", "moe_combine", "linear_scan_bonus", "linear_scan_decay", "token_shift_mix",
           "embed_pos_norm", "stream_sum", "add_bias", "tanh_", "act_mul_gather", "gemm_biased_swiglu", "linear_scan_gated",
-          "rms_norm_rows"]
+          "rms_norm_rows", "qkv_rotate", "talking_attention", "linear_scan_rotated"]
 
 
 @contextmanager

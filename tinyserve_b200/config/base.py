@@ -49,6 +49,8 @@ class LayerSpec:
     parts: Mapping[str, PartSpec]
     position: PartSpec | None = None  # position encoding the mixers apply; None = none
     block_args: Mapping[str, Any] = field(default_factory=dict)   # constants of the block itself
+    # Position encodings by mixer role, for a layer whose mixers rotate differently (instead of ``position``).
+    positions: Mapping[str, PartSpec] = field(default_factory=dict)
 
 
 @dataclass(frozen=True)
@@ -58,10 +60,13 @@ class LayerCall:
     ``layer`` indexes ``ModelSpec.layers``. ``reads_cache_of`` is ``None`` when the call
     owns a cache entry of its own (it writes this step's keys/values or state there), or
     the index of an EARLIER call in the order whose cache entry it reads without writing.
+    ``stream_input``: a part (family "stream input") that adds something to the residual stream
+    right before the call, such as what marks the passes of layers that run several times.
     """
 
     layer: int
     reads_cache_of: int | None = None
+    stream_input: PartSpec | None = None
 
 
 @dataclass(frozen=True)

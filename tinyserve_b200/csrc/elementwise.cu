@@ -133,10 +133,10 @@ __global__ void add_rms_norm_vec_kernel(float* __restrict__ resid, const T* __re
 }
 
 // ------------------------------------------------------------ rotary tables
-// angle = position * inv_freq in float64; cos and sin in float64, rounded to float32.
+// angle = position * inv_freq in float64; cos and sin (times a constant) in float64, rounded to float32.
 __global__ void rope_tables_kernel(const int* __restrict__ positions, const double* __restrict__ inv_freq,
                                    float* __restrict__ cos_out, float* __restrict__ sin_out,
-                                   int num_tokens, int half) {
+                                   int num_tokens, int half, double mult) {
   pdl_trigger();
   pdl_wait();
   const int idx = blockIdx.x * blockDim.x + threadIdx.x;
@@ -145,8 +145,8 @@ __global__ void rope_tables_kernel(const int* __restrict__ positions, const doub
   const double a = (double)positions[t] * inv_freq[i];
   double s, c;
   sincos(a, &s, &c);
-  cos_out[idx] = (float)c;
-  sin_out[idx] = (float)s;
+  cos_out[idx] = (float)(c * mult);
+  sin_out[idx] = (float)(s * mult);
 }
 
 // ------------------------------------------------------------- SiLU-multiply
@@ -366,11 +366,11 @@ extern "C" int ts_add_rms_norm(float* resid, const void* delta, const void* weig
 }
 
 extern "C" int ts_rope_tables(const int* positions, const double* inv_freq, float* cos_out, float* sin_out,
-                              int num_tokens, int half, cudaStream_t stream) {
+                              int num_tokens, int half, double mult, cudaStream_t stream) {
   const int total = num_tokens * half;
   if (total <= 0) return 0;
   return launch(rope_tables_kernel, (total + 255) / 256, 256, 0, stream, positions, inv_freq, cos_out, sin_out,
-                num_tokens, half);
+                num_tokens, half, mult);
 }
 
 extern "C" int ts_silu_mul(const void* gate_up, void* out, int num_tokens, int inter, int dtype,

@@ -45,9 +45,14 @@ constexpr int GATED_SILU = 1, GATED_GELU_TANH = 2, GATED_CLAMPED_SWISH = 3, GATE
 
 template <int BN, typename TOut, int SWIGLU>
 __device__ __forceinline__ void drain_tile(uint32_t tmem_acc, int row, int M, int N, int n0, TOut* __restrict__ out,
-                                           float act_limit, const bf16* __restrict__ act_bias) {
+                                           float act_limit, const bf16* __restrict__ act_bias, const float* row_weight = nullptr) {
   constexpr int BN_OUT = SWIGLU ? BN / 2 : BN;
   if constexpr (SWIGLU) {
+    // a factor of the row on both sums before the activation (clamped form only)
+    [[maybe_unused]] float rw = 1.f;
+    if constexpr (SWIGLU == GATED_CLAMPED_SWISH) {
+      if (row_weight != nullptr && row < M) rw = *(const volatile float*)(row_weight + row);
+    }
 #pragma unroll 1
     for (int c = 0; c < BN_OUT / 32; ++c) {
       uint32_t g[32], u[32];
@@ -96,8 +101,8 @@ __device__ __forceinline__ void drain_tile(uint32_t tmem_acc, int row, int M, in
             const float gv = __uint_as_float(g[j]) + bg[j % 8];
             f[j] = __fdividef(gv, 1.f + __expf(-gv)) * (__uint_as_float(u[j]) + bu[j % 8]);
           } else if constexpr (SWIGLU == GATED_CLAMPED_SWISH) {
-            const float gv = fminf(__uint_as_float(g[j]), act_limit);
-            const float uv = fminf(fmaxf(__uint_as_float(u[j]), -act_limit), act_limit);
+            const float gv = fminf(__uint_as_float(g[j]) * rw, act_limit);
+            const float uv = fminf(fmaxf(__uint_as_float(u[j]) * rw, -act_limit), act_limit);
             f[j] = __fdividef(gv, 1.f + __expf(-1.702f * gv)) * (uv + 1.f);
           } else {
             const float gv = round_to<bf16>(__uint_as_float(g[j])), uv = round_to<bf16>(__uint_as_float(u[j]));
@@ -160,6 +165,7 @@ struct GemmGroup {
   const int* offsets = nullptr;      // [experts + 1] first sorted row of every expert
   const int* num_tiles = nullptr;    // [1] row tiles in the list
   int w_rows = 0;
+  const float* row_weight = nullptr; // a factor per sorted row on its sums (clamped activation only)
 };
 
 // Persistent, warp-specialised: a CTA loops over output tiles (tile = blockIdx.x + i * gridDim.x,
@@ -293,7 +299,8 @@ __global__ void __launch_bounds__(TG_THREADS) gemm_tcgen05_kernel(const __grid_c
       }
       tc_fence_after();
       const int row = m0 + quad * 32 + lane;
-      drain_tile<BN, TOut, SWIGLU>(tmem_base + ((uint32_t)(quad * 32) << 16) + (uint32_t)(b * BN), row, m_end, N, n0, out, act_limit, act_bias);
+      drain_tile<BN, TOut, SWIGLU>(tmem_base + ((uint32_t)(quad * 32) << 16) + (uint32_t)(b * BN), row, m_end, N, n0, out, act_limit, act_bias,
+                                   grp.row_weight);
       // this warp has read its part of the accumulator: hand the buffer back to the MMA warp
       tc_fence_before();
       __syncwarp();
@@ -581,9 +588,10 @@ extern "C" int ts_gemm_tcgen05_gated(const void* x, const void* w, void* out, in
 
 // The experts' products of a routed feed-forward over rows sorted by expert (GemmGroup above): x is
 // [picks, K] in the sorted order, w [experts, N (gated: 2 N), K], out [picks, N] bf16; gated: out =
-// silu(gate) * up. The tile list must have been made for tiles of 128 rows. K % 8 == 0.
+// silu(gate) * up, or with a limit > 0 the clamped form, whose sums are first multiplied by row_weight[row] when it is
+// given. The tile list must have been made for tiles of 128 rows. K % 8 == 0.
 extern "C" int ts_moe_gemm_tcgen05(const void* x, const void* w, void* out, int picks, int N, int K, int experts, int gated,
-                                   const int* offsets, const int* tile_expert, const int* tile_row0, const int* num_tiles,
+                                   const float* row_weight, float limit, const int* offsets, const int* tile_expert, const int* tile_row0, const int* num_tiles,
                                    int max_tiles, int* error_flag, cudaStream_t stream) {
   if (picks <= 0 || N <= 0 || max_tiles <= 0) return 0;
   if (K <= 0 || K % 8 != 0 || error_flag == nullptr || experts <= 0) return TS_ERR_UNSUPPORTED;
@@ -591,11 +599,15 @@ extern "C" int ts_moe_gemm_tcgen05(const void* x, const void* w, void* out, int 
   GemmGroup grp;
   grp.tile_expert = tile_expert; grp.tile_row0 = tile_row0; grp.offsets = offsets; grp.num_tiles = num_tiles;
   grp.w_rows = gated ? 2 * N : N;
+  if (row_weight && !(gated && limit > 0.f)) return TS_ERR_UNSUPPORTED;
+  grp.row_weight = row_weight;
   const long long w_total = (long long)experts * grp.w_rows;
   if (w_total > 0x7fffffffLL) return TS_ERR_UNSUPPORTED;
   CUtensorMap mx, mw;
   if (gated) {
     if (!make_map(&mx, x, picks, K, TG_BM) || !make_map(&mw, w, (int)w_total, K, 128)) return TS_ERR_UNSUPPORTED;
+    if (limit > 0.f)
+      return launch_tc<256, 4, bf16, GATED_CLAMPED_SWISH>(mx, mw, (bf16*)out, picks, N, K, error_flag, stream, limit, grp, max_tiles);
     return launch_tc<256, 4, bf16, GATED_SILU>(mx, mw, (bf16*)out, picks, N, K, error_flag, stream, 0.f, grp, max_tiles);
   }
   if (!make_map(&mx, x, picks, K, TG_BM) || !make_map(&mw, w, (int)w_total, K, 256)) return TS_ERR_UNSUPPORTED;

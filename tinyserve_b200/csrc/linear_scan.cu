@@ -10,6 +10,9 @@
 //  * MODE_GATED (gated linear attention): a decay per key channel and token,
 //    alpha = sigmoid(z)^(1/tau) = exp(logsigmoid(z) / tau) with z = w_pre + w_0; q is multiplied by a constant;
 //    S <- diag(alpha) S + k v^T; o = S^T q (the read-out sees the current token's write).
+//  * MODE_ROTATED (retention): a constant decay per head; the first `rotary_dim` elements of q and k turn by the
+//    token's angles (pairs i, i + rotary_dim / 2 or neighbours), k is then multiplied by a constant; S <- decay_h S + k v^T;
+//    o = S^T q. The rotation happens where the chunk is staged, so the turned values are never rounded.
 //
 // Work split as in the other recurrent kernels: a CTA owns (request, head, block of 32 value
 // columns); compute warp w owns key rows [w * RPT, (w + 1) * RPT) and lane c column c, so a thread
@@ -40,7 +43,7 @@ constexpr int LIN_MAX_KEY_DIM = 256;
 constexpr int LIN_LOADER_WARPS = 4;
 constexpr int LIN_LOADS = 8;
 constexpr int LIN_RPT = 16;
-constexpr int MODE_BONUS = 0, MODE_DECAY = 1, MODE_GATED = 2;
+constexpr int MODE_BONUS = 0, MODE_DECAY = 1, MODE_GATED = 2, MODE_ROTATED = 3;
 constexpr int SCAN_WHOLE = 0, SCAN_LOCAL = 1, SCAN_FINAL = 2;
 
 __device__ __forceinline__ float siluf(float z) { return z / (1.f + expf(-z)); }
@@ -55,7 +58,10 @@ struct LinScanArgs {
   const float* w_bias;              // MODE_BONUS, MODE_GATED: [H * d]
   float inv_tau, q_scale;           // MODE_GATED: 1 / tau of the decay, and the constant on q
   const float* bonus;               // MODE_BONUS: [H * d]
-  const float* decay;               // MODE_DECAY: [H]
+  const float* decay;               // MODE_DECAY, MODE_ROTATED: [H]
+  const float* cos_tab; const float* sin_tab;   // MODE_ROTATED: [T, rotary_dim / 2]
+  int rotary_dim, interleaved;      // MODE_ROTATED
+  float k_scale;                    // MODE_ROTATED: the constant on k
   float* state; int state_stride;   // [slots, H * d * dv]
   const int* cu_q; const int* state_slots;
   int H, d, dv;
@@ -107,32 +113,70 @@ __device__ __forceinline__ void linear_scan_body(const LinScanArgs& a) {
     float* v_s = q_s + NARR * CH * dpad;
     const int t0 = start + c * CH, nt = min(CH, end - t0);
     const int lt = own_loads ? tid : tid - W * 32, ln = (own_loads ? W : LIN_LOADER_WARPS) * 32;
-    for (int base = lt; base < nt * dpad; base += ln * LIN_LOADS) {
-      float qv[LIN_LOADS], kv[LIN_LOADS], wv[LIN_LOADS];
+    if constexpr (MODE == MODE_ROTATED) {
+      // pair by pair: the rotated pairs first, then the elements behind them two by two (zeros from d on)
+      const int pairs = dpad >> 1, half = a.rotary_dim >> 1;
+      constexpr int U = LIN_LOADS / 2;
+      for (int base = lt; base < nt * pairs; base += ln * U) {
+        float q0[U], q1[U], k0[U], k1[U], cs[U], sn[U];
+        int at0[U], at1[U];
 #pragma unroll
-      for (int u = 0; u < LIN_LOADS; ++u) {
-        const int idx = base + u * ln;
-        const int tok = idx / dpad, r = idx - tok * dpad;
-        const bool ok = idx < nt * dpad && r < d;
-        qv[u] = ok ? to_float(qp[(size_t)(t0 + tok) * a.q_stride + h * d + r]) : 0.f;
-        kv[u] = ok ? to_float(kp[(size_t)(t0 + tok) * a.k_stride + h * d + r]) : 0.f;
-        if (CHANNEL_DECAY) wv[u] = ok ? a.w_pre[(size_t)(t0 + tok) * a.w_stride + h * d + r] + a.w_bias[h * d + r] : 0.f;
+        for (int u = 0; u < U; ++u) {
+          const int idx = base + u * ln;
+          const int tok = idx / pairs, p = idx - tok * pairs;
+          const bool in = idx < nt * pairs, turns = p < half;
+          const int r0 = !turns ? a.rotary_dim + 2 * (p - half) : a.interleaved ? 2 * p : p;
+          const int r1 = !turns ? r0 + 1 : a.interleaved ? r0 + 1 : p + half;
+          const size_t row = (size_t)(t0 + tok);
+          const T* qr = qp + row * a.q_stride + h * d;
+          const T* kr = kp + row * a.k_stride + h * d;
+          q0[u] = in && r0 < d ? to_float(qr[r0]) : 0.f;
+          q1[u] = in && r1 < d ? to_float(qr[r1]) : 0.f;
+          k0[u] = in && r0 < d ? to_float(kr[r0]) : 0.f;
+          k1[u] = in && r1 < d ? to_float(kr[r1]) : 0.f;
+          cs[u] = in && turns ? a.cos_tab[row * half + p] : 1.f;
+          sn[u] = in && turns ? a.sin_tab[row * half + p] : 0.f;
+          at0[u] = in ? tok * dpad + r0 : -1;
+          at1[u] = tok * dpad + r1;
+        }
+#pragma unroll
+        for (int u = 0; u < U; ++u) {
+          if (at0[u] >= 0) {
+            q_s[at0[u]] = q0[u] * cs[u] - q1[u] * sn[u];
+            q_s[at1[u]] = q1[u] * cs[u] + q0[u] * sn[u];
+            k_s[at0[u]] = (k0[u] * cs[u] - k1[u] * sn[u]) * a.k_scale;
+            k_s[at1[u]] = (k1[u] * cs[u] + k0[u] * sn[u]) * a.k_scale;
+          }
+        }
       }
+    } else {
+      for (int base = lt; base < nt * dpad; base += ln * LIN_LOADS) {
+        float qv[LIN_LOADS], kv[LIN_LOADS], wv[LIN_LOADS];
 #pragma unroll
-      for (int u = 0; u < LIN_LOADS; ++u) {
-        const int idx = base + u * ln;
-        if (idx < nt * dpad) {
-          if (MODE == MODE_DECAY) {
-            q_s[idx] = siluf(qv[u]);
-            k_s[idx] = siluf(kv[u]);
-          } else if (MODE == MODE_GATED) {
-            q_s[idx] = qv[u] * a.q_scale;
-            k_s[idx] = kv[u];
-            w_s[idx] = expf(logsigmoidf(wv[u]) * a.inv_tau);
-          } else {
-            q_s[idx] = qv[u];
-            k_s[idx] = kv[u];
-            w_s[idx] = expf(-expf(wv[u]));
+        for (int u = 0; u < LIN_LOADS; ++u) {
+          const int idx = base + u * ln;
+          const int tok = idx / dpad, r = idx - tok * dpad;
+          const bool ok = idx < nt * dpad && r < d;
+          qv[u] = ok ? to_float(qp[(size_t)(t0 + tok) * a.q_stride + h * d + r]) : 0.f;
+          kv[u] = ok ? to_float(kp[(size_t)(t0 + tok) * a.k_stride + h * d + r]) : 0.f;
+          if (CHANNEL_DECAY) wv[u] = ok ? a.w_pre[(size_t)(t0 + tok) * a.w_stride + h * d + r] + a.w_bias[h * d + r] : 0.f;
+        }
+#pragma unroll
+        for (int u = 0; u < LIN_LOADS; ++u) {
+          const int idx = base + u * ln;
+          if (idx < nt * dpad) {
+            if (MODE == MODE_DECAY) {
+              q_s[idx] = siluf(qv[u]);
+              k_s[idx] = siluf(kv[u]);
+            } else if (MODE == MODE_GATED) {
+              q_s[idx] = qv[u] * a.q_scale;
+              k_s[idx] = kv[u];
+              w_s[idx] = expf(logsigmoidf(wv[u]) * a.inv_tau);
+            } else {
+              q_s[idx] = qv[u];
+              k_s[idx] = kv[u];
+              w_s[idx] = expf(-expf(wv[u]));
+            }
           }
         }
       }
@@ -161,7 +205,7 @@ __device__ __forceinline__ void linear_scan_body(const LinScanArgs& a) {
     if (MODE == MODE_BONUS) {
 #pragma unroll
       for (int i = 0; i < RPT; ++i) u[i] = (r0 + i < d) ? a.bonus[h * d + r0 + i] : 0.f;
-    } else if (MODE == MODE_DECAY) {
+    } else if (MODE == MODE_DECAY || MODE == MODE_ROTATED) {
       decay = a.decay[h];
     }
   }
@@ -298,7 +342,8 @@ __global__ void linear_scan_combine_kernel(LinScanArgs a) {
   const int r = idx / a.dv;
   float s = a.state[(size_t)a.state_slots[b] * a.state_stride + (size_t)h * per_head + idx];
   float p_const = 1.f;
-  if (MODE == MODE_DECAY && nsegs > 1) {
+  constexpr bool CONSTANT = MODE == MODE_DECAY || MODE == MODE_ROTATED;
+  if (CONSTANT && nsegs > 1) {
     const float dec = a.decay[h];
     for (int t = 0; t < a.seg_len; ++t) p_const *= dec;
   }
@@ -311,7 +356,7 @@ __global__ void linear_scan_combine_kernel(LinScanArgs a) {
     for (int j = 0; j < 8; ++j) {
       const bool more = s0 + j + 1 < nsegs;
       left[j] = more ? p0[(size_t)(s0 + j) * seg_stride] : 0.f;
-      pp[j] = !more ? 0.f : MODE != MODE_DECAY ? d0[(size_t)(s0 + j) * a.H * a.d] : p_const;
+      pp[j] = !more ? 0.f : !CONSTANT ? d0[(size_t)(s0 + j) * a.H * a.d] : p_const;
     }
 #pragma unroll
     for (int j = 0; j < 8; ++j) {
@@ -375,7 +420,7 @@ static int lin_allow_smem(K kern, size_t smem, size_t& allowed) {
 template <typename T, int MODE, int PASS>
 static int launch_linear_pass(const LinScanArgs& a, dim3 grid, cudaStream_t stream) {
   const int dpad = a.W * LIN_RPT;
-  const int narr = MODE == MODE_DECAY ? 2 : 3;
+  const int narr = MODE == MODE_DECAY || MODE == MODE_ROTATED ? 2 : 3;
   const size_t smem = sizeof(float) * (2 * (size_t)a.CH * (narr * dpad + 32) + (size_t)a.CH * a.W * 32);
   static size_t allowed = 0;
   if constexpr (PASS == SCAN_WHOLE) {
@@ -394,7 +439,7 @@ static int launch_linear(const LinScanArgs& a, int num_seqs, cudaStream_t stream
   const int col_blocks = (a.dv + 31) / 32;
   if (a.max_segs <= 1) return launch_linear_pass<T, MODE, SCAN_WHOLE>(a, dim3(num_seqs, a.H, col_blocks), stream);
   const dim3 grid(num_seqs * a.max_segs, a.H, col_blocks);
-  if (MODE != MODE_DECAY)
+  if constexpr (MODE == MODE_BONUS || MODE == MODE_GATED)
     if (int e = launch(linear_scan_seg_decay_kernel<MODE>, dim3(num_seqs * a.max_segs, (a.H * a.d + 127) / 128), 128, 0, stream, a)) return e;
   if (int e = launch_linear_pass<T, MODE, SCAN_LOCAL>(a, grid, stream)) return e;
   if (int e = launch(linear_scan_combine_kernel<MODE>, dim3(num_seqs, a.H, (a.d * a.dv + 255) / 256), 256, 0, stream, a)) return e;
@@ -402,7 +447,8 @@ static int launch_linear(const LinScanArgs& a, int num_seqs, cudaStream_t stream
 }
 
 // mode 0: bonus read-out with a decay per key channel and token; mode 1: constant decay per head, SiLU on q, k, v;
-// mode 2: decay sigmoid(w_pre + w_bias)^(inv_tau) per key channel and token, q times q_scale, read-out after the write.
+// mode 2: decay sigmoid(w_pre + w_bias)^(inv_tau) per key channel and token, q times q_scale, read-out after the write;
+// mode 3: constant decay per head, q and k rotated (cos_tab / sin_tab [T, rotary_dim / 2]), then k times k_scale.
 // max_segs > 1 cuts every request's tokens into segments of seg_len (max_segs * seg_len covers the longest) that
 // run side by side (max_query_len = the most tokens any request brings): seg_state [num_seqs * max_segs, heads * d * dv] and, for modes 0 and 2, seg_decay
 // [num_seqs * max_segs, heads * d] are scratch.
@@ -411,24 +457,30 @@ extern "C" int ts_linear_scan(int mode, const void* q, int q_stride, const void*
                               const float* decay, float* state, int state_stride, const int* cu_q,
                               const int* state_slots, int num_seqs, int heads, int d, int dv, float* out, int dtype,
                               int max_query_len, int seg_len, int max_segs, float* seg_state, float* seg_decay,
-                              float inv_tau, float q_scale, cudaStream_t stream) {
+                              float inv_tau, float q_scale, const float* cos_tab, const float* sin_tab, int rotary_dim,
+                              int interleaved, float k_scale, cudaStream_t stream) {
   if (num_seqs <= 0) return 0;
   if (d <= 0 || dv <= 0 || d > LIN_MAX_KEY_DIM) return TS_ERR_UNSUPPORTED;
   if (mode == MODE_BONUS ? (!w_pre || !w_bias || !bonus) : mode == MODE_GATED ? (!w_pre || !w_bias || !(inv_tau > 0.f))
-                                                             : (mode != MODE_DECAY || !decay)) return TS_ERR_BAD_ARGUMENT;
+                                                             : ((mode != MODE_DECAY && mode != MODE_ROTATED) || !decay)) return TS_ERR_BAD_ARGUMENT;
+  if (mode == MODE_ROTATED && (rotary_dim < 0 || rotary_dim > d || (rotary_dim & 1) || (rotary_dim && (!cos_tab || !sin_tab))))
+    return TS_ERR_BAD_ARGUMENT;
   if (dtype != TS_DTYPE_F32 && dtype != TS_DTYPE_BF16) return TS_ERR_BAD_ARGUMENT;
-  if (max_segs > 1 && (seg_len <= 0 || !seg_state || (mode != MODE_DECAY && !seg_decay))) return TS_ERR_BAD_ARGUMENT;
+  if (max_segs > 1 && (seg_len <= 0 || !seg_state || ((mode == MODE_BONUS || mode == MODE_GATED) && !seg_decay))) return TS_ERR_BAD_ARGUMENT;
   LinScanArgs a;
   a.q = q; a.q_stride = q_stride; a.k = k; a.k_stride = k_stride; a.v = v; a.v_stride = v_stride;
   a.w_pre = w_pre; a.w_stride = w_stride; a.w_bias = w_bias; a.bonus = bonus; a.decay = decay;
   a.state = state; a.state_stride = state_stride; a.cu_q = cu_q; a.state_slots = state_slots;
   a.H = heads; a.d = d; a.dv = dv; a.out = out; a.inv_tau = inv_tau; a.q_scale = q_scale;
+  a.cos_tab = cos_tab; a.sin_tab = sin_tab; a.rotary_dim = rotary_dim; a.interleaved = interleaved; a.k_scale = k_scale;
   a.W = (d + LIN_RPT - 1) / LIN_RPT;
   a.CH = a.W * LIN_RPT <= 128 ? 16 : 8;
   a.loader_warps = (max_query_len > 0 && max_query_len <= a.CH) ? 0 : LIN_LOADER_WARPS;
   a.seg_len = seg_len; a.max_segs = max_segs > 1 ? max_segs : 1; a.seg_state = seg_state; a.seg_decay = seg_decay;
   if (mode == MODE_BONUS)
     return dtype == TS_DTYPE_F32 ? launch_linear<float, MODE_BONUS>(a, num_seqs, stream) : launch_linear<bf16, MODE_BONUS>(a, num_seqs, stream);
+  if (mode == MODE_ROTATED)
+    return dtype == TS_DTYPE_F32 ? launch_linear<float, MODE_ROTATED>(a, num_seqs, stream) : launch_linear<bf16, MODE_ROTATED>(a, num_seqs, stream);
   if (mode == MODE_GATED)
     return dtype == TS_DTYPE_F32 ? launch_linear<float, MODE_GATED>(a, num_seqs, stream) : launch_linear<bf16, MODE_GATED>(a, num_seqs, stream);
   return dtype == TS_DTYPE_F32 ? launch_linear<float, MODE_DECAY>(a, num_seqs, stream) : launch_linear<bf16, MODE_DECAY>(a, num_seqs, stream);

@@ -6,12 +6,16 @@
 //            ALL outputs first, picks by score + correction inside the best groups of neighbouring
 //            outputs only, and weights the picks by their scores over the picks' sum, times a constant;
 //            the last outputs may be identity experts, which have no matrices and no queue: their
-//            picks carry the token's own input to the combine step;
+//            picks carry the token's own input to the combine step. A third rule scores every output by
+//            its sigmoid; the weights may be left as the scores are, and may belong to the experts' input
+//            instead of their output (`row_weight`: the sorted row's weight, applied where the gate and up
+//            sums are finished, since W (w x) = w (W x); the combine step then adds the rows as they are);
 //   plan     one thread turns the counters into the experts' row ranges of the sorted order and
 //            into a list of row tiles (expert, first row), and clears the counters for the next step;
 //   scatter  every (token, pick) learns its row of the sorted order; the row learns its token;
 //   products tile by tile over that list: act[row, :] = silu(x[token] Wgate_e^T) * (x[token] Wup_e^T)
-//            (the token's row of x is fetched through the list, nothing is copied), then
+//            (or the clamped form of the activation; the token's row of x is fetched through the list,
+//            nothing is copied), then
 //            y[row, :] = act[row, :] Wdown_e^T;
 //   combine  out[token] = sum_j weight_j y[row_j] (+ the shared expert's output, optionally times the sigmoid
 //            of a gate logit per token), 32-bit, rounded once; an identity pick's y is the token's input.
@@ -26,19 +30,30 @@
 namespace ts {
 
 // ------------------------------------------------------------------------- route
-// One token by one warp: picks, weights, and a place in each picked expert's queue (`counts` may be
-// in shared memory).
 // How a token's picks and weights follow from its router outputs.
 struct RouteRule {
   int scored;               // 0: the largest logits, weighted by the softmax over the picks alone
                             // 1: softmax over all outputs; picks by score + correction within the best groups;
                             //    weights = scores of the picks / (their sum + 1e-20) * scale
+                            // 2: the same with sigmoid(z) as an output's score
+  int normalise;            // scored: 0 leaves the weights at score * scale
   int real;                 // outputs that are experts with matrices (the first ones); the rest are identity experts
   int groups, keep;         // scored: equal groups of neighbouring outputs, of which the `keep` best may be picked from
   float scale;              // scored: constant on the weights
   const float* correction;  // scored: [E] added to the scores for the choice only, or null
   int ld;                   // floats between two tokens' rows of router outputs
 };
+
+// The score of an output with logit z under a scored rule.
+__device__ __forceinline__ float route_score(const RouteRule& rule, float z, float zmax, float inv_sum) {
+  return rule.scored == 2 ? 1.f / (1.f + expf(-z)) : expf(z - zmax) * inv_sum;
+}
+// What the choice compares. Sigmoid scores without a correction rise with the logit, so the logit stands for
+// them (near 1 neighbouring scores round to the same value, their logits do not).
+__device__ __forceinline__ float route_choice(const RouteRule& rule, float z, int e, float zmax, float inv_sum) {
+  if (rule.scored == 2 && !rule.correction) return z;
+  return route_score(rule, z, zmax, inv_sum) + (rule.correction ? rule.correction[e] : 0.f);
+}
 
 // One token by one warp: picks, weights, and a place in each picked expert's queue (`counts` may be
 // in shared memory). A pick of an identity expert (id >= rule.real) takes no place (-1).
@@ -49,19 +64,21 @@ __device__ __forceinline__ void route_token(const float* __restrict__ z, int t, 
   unsigned allowed = 0xffffffffu;          // bit g: group g may be picked from
   int group_size = E;
   if (rule.scored) {
-    float mx = -INFINITY;
-    for (int e = lane; e < E; e += 32) mx = fmaxf(mx, z[e]);
-    zmax = warp_max(mx);
-    float sum = 0.f;
-    for (int e = lane; e < E; e += 32) sum += expf(z[e] - zmax);
-    inv_sum = 1.f / warp_sum(sum);
+    if (rule.scored == 1) {
+      float mx = -INFINITY;
+      for (int e = lane; e < E; e += 32) mx = fmaxf(mx, z[e]);
+      zmax = warp_max(mx);
+      float sum = 0.f;
+      for (int e = lane; e < E; e += 32) sum += expf(z[e] - zmax);
+      inv_sum = 1.f / warp_sum(sum);
+    }
     if (rule.groups > 1) {
       // lane g: the best choice score of group g, then its rank among the groups (value down, index up)
       group_size = E / rule.groups;
       float best = -INFINITY;
       if (lane < rule.groups)
         for (int e = lane * group_size; e < (lane + 1) * group_size; ++e)
-          best = fmaxf(best, expf(z[e] - zmax) * inv_sum + (rule.correction ? rule.correction[e] : 0.f));
+          best = fmaxf(best, route_choice(rule, z[e], e, zmax, inv_sum));
       int rank = 0;
       for (int g = 0; g < rule.groups; ++g) {
         const float other = __shfl_sync(0xffffffffu, best, g);
@@ -79,7 +96,7 @@ __device__ __forceinline__ void route_token(const float* __restrict__ z, int t, 
     for (int e = lane; e < E; e += 32) {
       float v = z[e];
       if (rule.scored) {
-        v = expf(v - zmax) * inv_sum + (rule.correction ? rule.correction[e] : 0.f);
+        v = route_choice(rule, v, e, zmax, inv_sum);
         if (!((allowed >> (e / group_size)) & 1u)) continue;
       }
       const bool after = (v < prev_v) || (v == prev_v && e > prev_e);
@@ -98,7 +115,7 @@ __device__ __forceinline__ void route_token(const float* __restrict__ z, int t, 
   const bool picked = lane < top && my_e >= 0 && my_e < E;   // fewer finite candidates than picks: the pick is dropped
   float p;
   if (rule.scored) {
-    p = picked ? expf(z[my_e] - zmax) * inv_sum : 0.f;        // the score itself, without the correction
+    p = picked ? route_score(rule, z[my_e], zmax, inv_sum) : 0.f;        // the score itself, without the correction
   } else {
     const float head = __shfl_sync(0xffffffffu, my_v, 0);
     p = lane < top ? expf(my_v - head) : 0.f;
@@ -106,7 +123,7 @@ __device__ __forceinline__ void route_token(const float* __restrict__ z, int t, 
   const float sum = warp_sum(p);
   if (lane < top) {
     const int e = picked ? my_e : 0;
-    const float w = rule.scored ? p / (sum + 1e-20f) * rule.scale : p / sum;
+    const float w = !rule.scored ? p / sum : rule.normalise ? p / (sum + 1e-20f) * rule.scale : p * rule.scale;
     ids[(size_t)t * top + lane] = e;
     weights[(size_t)t * top + lane] = picked ? w : 0.f;
     place[(size_t)t * top + lane] = e < rule.real ? atomicAdd(&counts[e], 1) : -1;
@@ -133,7 +150,7 @@ __global__ void __launch_bounds__(ROUTE_SMALL_THREADS) moe_route_small_kernel(
     float* logits, int num_tokens, int E, int top, int tile_rows, int* __restrict__ ids,
     float* __restrict__ weights, int* __restrict__ place, int* __restrict__ offsets, int* __restrict__ tile_expert,
     int* __restrict__ tile_row0, int* __restrict__ num_tiles, int max_tiles, int* __restrict__ row_of,
-    int* __restrict__ token_of, RouteRule rule) {
+    int* __restrict__ token_of, float* __restrict__ row_weight, RouteRule rule) {
   __shared__ int counts[ROUTE_SMALL_MAX_EXPERTS];
   __shared__ int offs[ROUTE_SMALL_MAX_EXPERTS + 1];
   pdl_trigger();
@@ -195,6 +212,7 @@ __global__ void __launch_bounds__(ROUTE_SMALL_THREADS) moe_route_small_kernel(
     const int row = offs[ids[idx]] + place[idx];
     row_of[idx] = row;
     token_of[row] = idx / top;
+    if (row_weight) row_weight[row] = weights[idx];
   }
 }
 
@@ -223,7 +241,8 @@ __global__ void moe_plan_kernel(int* __restrict__ counts, int E, int tile_rows, 
 
 // ----------------------------------------------------------------------- scatter
 __global__ void moe_scatter_kernel(const int* __restrict__ ids, const int* __restrict__ place, const int* __restrict__ offsets,
-                                   int total, int top, int* __restrict__ row_of, int* __restrict__ token_of) {
+                                   int total, int top, int* __restrict__ row_of, int* __restrict__ token_of,
+                                   const float* __restrict__ weights, float* __restrict__ row_weight) {
   pdl_trigger();
   pdl_wait();
   const int idx = blockIdx.x * blockDim.x + threadIdx.x;
@@ -235,6 +254,7 @@ __global__ void moe_scatter_kernel(const int* __restrict__ ids, const int* __res
   const int row = offsets[ids[idx]] + place[idx];
   row_of[idx] = row;
   token_of[row] = idx / top;
+  if (row_weight) row_weight[row] = weights[idx];
 }
 
 // --------------------------------------------------------- products, CUDA cores
@@ -242,12 +262,28 @@ constexpr int SG_M = 64, SG_N = 64, SG_K = 16, SG_THREADS = 256;
 
 __device__ __forceinline__ float silu_f(float z) { return z / (1.f + expf(-z)); }
 
-// GATED: w holds, per expert, N gate rows then N up rows; out[row, n] = silu(g) * u.
+// How the finished gate and up sums of a gated product become one value.
+struct GateForm {
+  const float* row_weight;   // [sorted rows] factor on both sums, or null
+  float limit;               // > 0: g = min(g, limit), u = clamp(u, -limit, limit), g sigmoid(1.702 g) (u + 1)
+};
+__device__ __forceinline__ float gate_value(float g, float u, float w, float limit) {
+  g *= w;
+  u *= w;
+  if (limit > 0.f) {
+    g = fminf(g, limit);
+    u = fminf(fmaxf(u, -limit), limit);
+    return g / (1.f + expf(-1.702f * g)) * (u + 1.f);
+  }
+  return silu_f(g) * u;
+}
+
+// GATED: w holds, per expert, N gate rows then N up rows; out[row, n] = silu(g) * u (or another GateForm).
 template <typename T, bool GATED>
 __global__ void __launch_bounds__(SG_THREADS) moe_gemm_simt_kernel(
     const T* __restrict__ x, const int* __restrict__ token_of, const T* __restrict__ w, T* __restrict__ out,
     const int* __restrict__ offsets, const int* __restrict__ tile_expert, const int* __restrict__ tile_row0,
-    const int* __restrict__ num_tiles, int N, int K) {
+    const int* __restrict__ num_tiles, int N, int K, GateForm form) {
   __shared__ float As[SG_K][SG_M + 4];
   __shared__ float Bs[GATED ? 2 : 1][SG_K][SG_N + 4];
   pdl_trigger();
@@ -308,12 +344,13 @@ __global__ void __launch_bounds__(SG_THREADS) moe_gemm_simt_kernel(
   for (int i = 0; i < 4; ++i) {
     const int m = r0 + ty * 4 + i;
     if (m >= rend) continue;
+    const float rw = GATED && form.row_weight ? form.row_weight[m] : 1.f;
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int n = n0 + tx * 4 + j;
       if (n >= N) continue;
       float v = acc[0][i][j];
-      if (GATED) v = silu_f(v) * acc[1][i][j];
+      if (GATED) v = gate_value(v, acc[1][i][j], rw, form.limit);
       out[(size_t)m * N + n] = from_float<T>(v);
     }
   }
@@ -351,7 +388,7 @@ template <bool GATED>
 __global__ void __launch_bounds__(TG_THREADS) moe_gemm_mma_kernel(
     const bf16* __restrict__ x, const int* __restrict__ token_of, const bf16* __restrict__ w, bf16* __restrict__ out,
     const int* __restrict__ offsets, const int* __restrict__ tile_expert, const int* __restrict__ tile_row0,
-    const int* __restrict__ num_tiles, int N, int K) {
+    const int* __restrict__ num_tiles, int N, int K, GateForm form) {
   constexpr int NB = GATED ? 2 : 1;
   extern __shared__ __align__(16) unsigned char raw[];
   bf16* As = (bf16*)raw;                                   // [STAGES][TG_M][TG_LD]
@@ -434,6 +471,12 @@ __global__ void __launch_bounds__(TG_THREADS) moe_gemm_mma_kernel(
   cp_async_wait<0>();
   // accumulator layout: rows lane / 4 and + 8, columns (lane % 4) * 2 and + 1 of each 8-wide block
   const int mrow = r0 + warp * 16 + (lane >> 2);
+  float rw[2] = {1.f, 1.f};
+  if (GATED && form.row_weight) {
+#pragma unroll
+    for (int half = 0; half < 2; ++half)
+      if (mrow + half * 8 < rend) rw[half] = form.row_weight[mrow + half * 8];
+  }
 #pragma unroll
   for (int j = 0; j < 8; ++j) {
     const int n = n0 + j * 8 + (lane & 3) * 2;
@@ -443,7 +486,10 @@ __global__ void __launch_bounds__(TG_THREADS) moe_gemm_mma_kernel(
       const int m = mrow + half * 8;
       if (m >= rend) continue;
       float v0 = acc[0][j][half * 2], v1 = acc[0][j][half * 2 + 1];
-      if (GATED) { v0 = silu_f(v0) * acc[NB - 1][j][half * 2]; v1 = silu_f(v1) * acc[NB - 1][j][half * 2 + 1]; }
+      if (GATED) {
+        v0 = gate_value(v0, acc[NB - 1][j][half * 2], rw[half], form.limit);
+        v1 = gate_value(v1, acc[NB - 1][j][half * 2 + 1], rw[half], form.limit);
+      }
       const __nv_bfloat162 pk = __floats2bfloat162_rn(v0, v1);
       *reinterpret_cast<__nv_bfloat162*>(out + (size_t)m * N + n) = pk;
     }
@@ -482,7 +528,7 @@ __global__ void moe_combine_kernel(const T* __restrict__ y, const int* __restric
     float v = 0.f;
     for (int j = 0; j < top; ++j) {
       const int row = row_of[(size_t)t * top + j];
-      v = fmaf(weights[(size_t)t * top + j], to_float(row >= 0 ? y[(size_t)row * hidden + c] : x[(size_t)t * hidden + c]), v);
+      v = fmaf(weights ? weights[(size_t)t * top + j] : 1.f, to_float(row >= 0 ? y[(size_t)row * hidden + c] : x[(size_t)t * hidden + c]), v);
     }
     if (shared_out) v = fmaf(sg, to_float(shared_out[(size_t)t * hidden + c]), v);
     out[(size_t)t * hidden + c] = from_float<T>(v);
@@ -502,7 +548,7 @@ __global__ void moe_combine_vec_kernel(const T* __restrict__ y, const int* __res
   // volatile: this read stands right behind the wait and depends on nothing, so as a plain read it could be moved in front of it
   const float sg = shared_gate ? 1.f / (1.f + expf(-*(const volatile float*)(shared_gate + (size_t)t * gate_stride))) : 1.f;
   const int* rows = row_of + (size_t)t * top;
-  const float* wt = weights + (size_t)t * top;
+  const float* wt = weights ? weights + (size_t)t * top : nullptr;     // null: the rows are added as they are
   for (int c = threadIdx.x * VEC; c < hidden; c += blockDim.x * VEC) {
     float acc[VEC];
 #pragma unroll
@@ -517,7 +563,7 @@ __global__ void moe_combine_vec_kernel(const T* __restrict__ y, const int* __res
         if (j0 + u < top) {
           float f[VEC];
           part[u].unpack(f);
-          const float a = wt[j0 + u];
+          const float a = wt ? wt[j0 + u] : 1.f;
 #pragma unroll
           for (int e = 0; e < VEC; ++e) acc[e] = fmaf(a, f[e], acc[e]);
         }
@@ -543,35 +589,37 @@ using namespace ts;
 extern "C" int ts_moe_tile_rows() { return SG_M; }      // both product forms use tiles of 64 rows
 
 // The rule's arguments, checked: E outputs of which the first `real` are experts with matrices.
-static int make_rule(RouteRule& r, int E, int real, int top, int scored, int groups, int keep, float scale,
+static int make_rule(RouteRule& r, int E, int real, int top, int scored, int normalise, int groups, int keep, float scale,
                      const float* correction, int ld) {
+  if (scored < 0 || scored > 2) return TS_ERR_BAD_ARGUMENT;
   if (E <= 0 || real <= 0 || real > E || top <= 0 || top > 32 || top > E || ld < E) return TS_ERR_BAD_ARGUMENT;
   if (!scored && (real != E || groups > 1 || correction)) return TS_ERR_BAD_ARGUMENT;
   if (groups < 1) groups = 1;
   if (groups > 32 || E % groups || keep < 1 || keep > groups || (E / groups) * keep < top) return TS_ERR_BAD_ARGUMENT;
-  r.scored = scored; r.real = real; r.groups = groups; r.keep = keep; r.scale = scale; r.correction = correction; r.ld = ld;
+  r.scored = scored; r.normalise = normalise; r.real = real; r.groups = groups; r.keep = keep; r.scale = scale; r.correction = correction; r.ld = ld;
   return 0;
 }
 
 // logits [T, ld >= E] float -> ids / weights / place [T, top]; counts [real] (zero on entry, zero again after the plan);
 // offsets [real + 1]; tile_expert / tile_row0 [max_tiles]; num_tiles [1]; row_of [T * top]; token_of [T * top].
 // tile_rows: rows of a tile of the list (64 for the products of this file, 128 for the tcgen05 product).
-// scored / groups / keep / scale / correction / real: see RouteRule (scored 0 wants real = E, groups <= 1).
-extern "C" int ts_moe_route(const float* logits, int ld, int num_tokens, int E, int real, int top, int scored, int groups,
-                            int keep, float scale, const float* correction, int* ids, float* weights, int* place,
+// scored / normalise / groups / keep / scale / correction / real: see RouteRule (scored 0 wants real = E, groups <= 1).
+// row_weight [T * top], may be null: receives the weight of every sorted row.
+extern "C" int ts_moe_route(const float* logits, int ld, int num_tokens, int E, int real, int top, int scored, int normalise,
+                            int groups, int keep, float scale, const float* correction, int* ids, float* weights, int* place,
                             int* counts, int* offsets, int* tile_expert, int* tile_row0, int* num_tiles, int max_tiles,
-                            int* row_of, int* token_of, int tile_rows, cudaStream_t stream) {
+                            int* row_of, int* token_of, float* row_weight, int tile_rows, cudaStream_t stream) {
   if (num_tokens <= 0) return 0;
   if (tile_rows != 64 && tile_rows != 128) return TS_ERR_BAD_ARGUMENT;
   RouteRule rule;
-  if (int e = make_rule(rule, E, real, top, scored, groups, keep, scale, correction, ld)) return e;
+  if (int e = make_rule(rule, E, real, top, scored, normalise, groups, keep, scale, correction, ld)) return e;
   const int picks = num_tokens * top;
   const int most = picks < picks / tile_rows + real ? picks : picks / tile_rows + real;   // every tile has a row; an expert one ragged tile
   if (max_tiles < most) return TS_ERR_BAD_ARGUMENT;
   if (num_tokens <= 64 && E <= ROUTE_SMALL_MAX_EXPERTS)
     return launch(moe_route_small_kernel<float>, 1, ROUTE_SMALL_THREADS, 0, stream, (const float*)nullptr, (const float*)nullptr, 0,
                   const_cast<float*>(logits), num_tokens, E, top, tile_rows, ids, weights, place, offsets, tile_expert, tile_row0,
-                  num_tiles, max_tiles, row_of, token_of, rule);
+                  num_tiles, max_tiles, row_of, token_of, row_weight, rule);
   int st = launch(moe_route_kernel, (num_tokens * 32 + 127) / 128, 128, 0, stream, logits, num_tokens, E, top, ids,
                   weights, place, counts, rule);
   if (st != 0) return st;
@@ -579,7 +627,7 @@ extern "C" int ts_moe_route(const float* logits, int ld, int num_tokens, int E, 
   if (st != 0) return st;
   const int total = num_tokens * top;
   return launch(moe_scatter_kernel, (total + 255) / 256, 256, 0, stream, (const int*)ids, (const int*)place,
-                (const int*)offsets, total, top, row_of, token_of);
+                (const int*)offsets, total, top, row_of, token_of, (const float*)weights, row_weight);
 }
 
 // The same for a step of up to 64 tokens with the router's product inside: logits (scratch, [T, E] float) are
@@ -591,7 +639,7 @@ extern "C" int ts_moe_route_fused(const void* x, const void* w_router, int hidde
   if (num_tokens <= 0) return 0;
   if (tile_rows != 64 && tile_rows != 128) return TS_ERR_BAD_ARGUMENT;
   RouteRule rule;
-  if (int e = make_rule(rule, E, E, top, 0, 1, 1, 1.f, nullptr, E)) return e;
+  if (int e = make_rule(rule, E, E, top, 0, 1, 1, 1, 1.f, nullptr, E)) return e;
   const int picks = num_tokens * top;
   const int most = picks < picks / tile_rows + E ? picks : picks / tile_rows + E;
   if (max_tiles < most || hidden <= 0 || !x || !w_router) return TS_ERR_BAD_ARGUMENT;
@@ -599,20 +647,25 @@ extern "C" int ts_moe_route_fused(const void* x, const void* w_router, int hidde
   if (dtype == TS_DTYPE_F32)
     return launch(moe_route_small_kernel<float>, 1, ROUTE_SMALL_THREADS, 0, stream, (const float*)x, (const float*)w_router, hidden,
                   logits, num_tokens, E, top, tile_rows, ids, weights, place, offsets, tile_expert, tile_row0, num_tiles, max_tiles,
-                  row_of, token_of, rule);
+                  row_of, token_of, (float*)nullptr, rule);
   if (dtype == TS_DTYPE_BF16)
     return launch(moe_route_small_kernel<bf16>, 1, ROUTE_SMALL_THREADS, 0, stream, (const bf16*)x, (const bf16*)w_router, hidden,
                   logits, num_tokens, E, top, tile_rows, ids, weights, place, offsets, tile_expert, tile_row0, num_tiles, max_tiles,
-                  row_of, token_of, rule);
+                  row_of, token_of, (float*)nullptr, rule);
   return TS_ERR_BAD_ARGUMENT;
 }
 
 // out[row, :] for every row of the sorted order: x rows are taken through `token_of` when it is
-// given (else row by row). w is [E, N (gated: 2 N), K]. `use_mma` 0 forces the CUDA-core form.
+// given (else row by row). w is [E, N (gated: 2 N), K]. `use_mma` 0 forces the CUDA-core form. gated: row_weight
+// and limit as in GateForm (null and 0 for silu(g) * u).
 extern "C" int ts_moe_gemm(const void* x, const int* token_of, const void* w, void* out, const int* offsets,
                            const int* tile_expert, const int* tile_row0, const int* num_tiles, int max_tiles, int N,
-                           int K, int gated, int dtype, int use_mma, cudaStream_t stream) {
+                           int K, int gated, const float* row_weight, float limit, int dtype, int use_mma,
+                           cudaStream_t stream) {
   if (max_tiles <= 0) return 0;
+  GateForm form;
+  form.row_weight = row_weight;
+  form.limit = limit;
   if (N <= 0 || K <= 0) return TS_ERR_BAD_ARGUMENT;
   if (dtype == TS_DTYPE_BF16 && use_mma && K % TG_K == 0 && N % 8 == 0 &&
       (((uintptr_t)x | (uintptr_t)w | (uintptr_t)out) & 15) == 0) {
@@ -624,18 +677,18 @@ extern "C" int ts_moe_gemm(const void* x, const int* token_of, const void* w, vo
       cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
       if (e != cudaSuccess) return (int)e;
       return launch(kern, grid, TG_THREADS, smem, stream, (const bf16*)x, token_of, (const bf16*)w, (bf16*)out, offsets,
-                    tile_expert, tile_row0, num_tiles, N, K);
+                    tile_expert, tile_row0, num_tiles, N, K, form);
     }
     auto kern = moe_gemm_mma_kernel<false>;
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
     return launch(kern, grid, TG_THREADS, smem, stream, (const bf16*)x, token_of, (const bf16*)w, (bf16*)out, offsets,
-                  tile_expert, tile_row0, num_tiles, N, K);
+                  tile_expert, tile_row0, num_tiles, N, K, form);
   }
   dim3 grid((N + SG_N - 1) / SG_N, max_tiles);
 #define TS_MOE_CASE(T_, G_)                                                                                     \
   return launch(moe_gemm_simt_kernel<T_, G_>, grid, SG_THREADS, 0, stream, (const T_*)x, token_of, (const T_*)w, \
-                (T_*)out, offsets, tile_expert, tile_row0, num_tiles, N, K)
+                (T_*)out, offsets, tile_expert, tile_row0, num_tiles, N, K, form)
   if (dtype == TS_DTYPE_F32) { if (gated) TS_MOE_CASE(float, true); TS_MOE_CASE(float, false); }
   if (dtype == TS_DTYPE_BF16) { if (gated) TS_MOE_CASE(bf16, true); TS_MOE_CASE(bf16, false); }
 #undef TS_MOE_CASE
@@ -655,7 +708,7 @@ extern "C" int ts_moe_gather(const void* x, const int* token_of, void* xs, int p
 }
 
 // x [T, hidden] (the tokens' inputs) is read for identity picks (row_of < 0) and may be null when there are none;
-// shared_gate (float, one logit per token, gate_stride floats apart) multiplies the shared output by its sigmoid.
+// weights null: the picked rows are added as they are; shared_gate (float, one logit per token, gate_stride floats apart) multiplies the shared output by its sigmoid.
 extern "C" int ts_moe_combine(const void* y, const int* row_of, const float* weights, const void* shared_out, void* out,
                               int num_tokens, int top, int hidden, const void* x, const float* shared_gate, int gate_stride,
                               int dtype, cudaStream_t stream) {

@@ -3,9 +3,13 @@
 //
 //   y   = d / sqrt(mean(d^2) + eps_post) * gain(post_weight) * layer_scale * m  (when a post norm is pending;
 //                                                                                  m a constant multiplier)
-//   y   = (d + bias) * layer_scale                                               (a layer scale alone, with the
-//                                                                                  sub-layer's output bias, if any)
-//   x  <- x + y                                                                   (written back unless `rows`)
+//   y   = (d + bias) * m * layer_scale                                           (without a post norm: a constant and
+//                                                                                  a layer scale, with the sub-layer's
+//                                                                                  output bias, if any)
+//   x  <- x + y + s d2 + rows + vec                                               (written back unless `rows`; d2 the
+//                                                                                  output of a sub-layer side by side with
+//                                                                                  d and its constant, rows 32-bit and vec
+//                                                                                  one value per column; each if given)
 //   out = x / sqrt(mean(x^2) + eps) * gain(weight)
 //
 // gain(w) = 1 + w when the weight is stored around zero (`unit_offset`), else w. Everything is
@@ -26,7 +30,11 @@ struct PostNormArgs {
   const void* weight;
   void* out;
   const int* rows;
+  const void* second;       // may be null: a second pending output, model dtype, times second_scale
+  const float* add_rows;    // may be null: 32-bit rows added to the stream
+  const void* add_vec;      // may be null: one value per column added to the stream
   int num_rows, hidden;
+  float second_scale;
   float post_eps, eps;
   float post_mult;          // a constant on the normed pending output
   int post_offset, offset;  // 1: the gain is 1 + weight
@@ -48,7 +56,10 @@ __global__ void post_norm_add_rms_norm_kernel(PostNormArgs a) {
   const T* ls = (const T*)a.layer_scale;
   const T* db = (const T*)a.delta_bias;
   const T* w = (const T*)a.weight;
-  const bool write_back = (a.rows == nullptr) && (d != nullptr);
+  const T* d2 = a.second ? (const T*)a.second + (size_t)row * hidden : nullptr;
+  const float* ar = a.add_rows ? a.add_rows + (size_t)row * hidden : nullptr;
+  const T* av = (const T*)a.add_vec;
+  const bool write_back = (a.rows == nullptr) && (d != nullptr || ar != nullptr || av != nullptr);
   float post_rstd = 1.f;
   if (d && pw) {
     float ss = 0.f;
@@ -80,6 +91,8 @@ __global__ void post_norm_add_rms_norm_kernel(PostNormArgs a) {
 #pragma unroll
           for (int e = 0; e < VEC; ++e) y[e] += b[e];
         }
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) y[e] *= a.post_mult;
       }
       if (ls) {
         float s[VEC];
@@ -89,9 +102,26 @@ __global__ void post_norm_add_rms_norm_kernel(PostNormArgs a) {
       }
 #pragma unroll
       for (int e = 0; e < VEC; ++e) v[e] += y[e];
-      if (write_back) {
-        if constexpr (VEC == 4) Quad<float>::store(x + i, v); else x[i] = v[0];
+      if (d2) {
+        if constexpr (VEC == 4) Quad<T>::load(d2 + i, y); else y[0] = to_float(d2[i]);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) v[e] = fmaf(a.second_scale, y[e], v[e]);
       }
+    }
+    if (ar) {
+      float y[VEC];
+      if constexpr (VEC == 4) Quad<float>::load(ar + i, y); else y[0] = ar[i];
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) v[e] += y[e];
+    }
+    if (av) {
+      float y[VEC];
+      if constexpr (VEC == 4) Quad<T>::load(av + i, y); else y[0] = to_float(av[i]);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) v[e] += y[e];
+    }
+    if (write_back) {
+      if constexpr (VEC == 4) Quad<float>::store(x + i, v); else x[i] = v[0];
     }
 #pragma unroll
     for (int e = 0; e < VEC; ++e) { xs[i + e] = v[e]; ss = fmaf(v[e], v[e], ss); }
@@ -115,19 +145,22 @@ using namespace ts;
 extern "C" int ts_post_norm_add_rms_norm(float* resid, const void* delta, const void* post_weight, const void* layer_scale,
                                          float post_eps, int post_offset, float post_mult, const void* weight, int offset,
                                          float eps, void* out, const int* rows, int num_rows, int hidden, const void* delta_bias,
+                                         const void* second, float second_scale, const float* add_rows, const void* add_vec,
                                          int dtype, cudaStream_t stream) {
   if (num_rows <= 0) return 0;
   if (hidden <= 0 || hidden > 12288 || !weight || !out || !resid) return TS_ERR_BAD_ARGUMENT;
   if (dtype != TS_DTYPE_F32 && dtype != TS_DTYPE_BF16) return TS_ERR_BAD_ARGUMENT;
-  if ((post_weight || layer_scale || delta_bias) && !delta) return TS_ERR_BAD_ARGUMENT;
+  if ((post_weight || layer_scale || delta_bias || second) && !delta) return TS_ERR_BAD_ARGUMENT;
   if (delta_bias && post_weight) return TS_ERR_UNSUPPORTED;
   PostNormArgs a;
   a.resid = resid; a.delta = delta; a.post_weight = post_weight; a.layer_scale = layer_scale; a.delta_bias = delta_bias; a.weight = weight;
   a.out = out; a.rows = rows; a.num_rows = num_rows; a.hidden = hidden; a.post_eps = post_eps; a.eps = eps;
   a.post_offset = post_offset; a.offset = offset; a.post_mult = post_mult;
+  a.second = second; a.second_scale = second_scale; a.add_rows = add_rows; a.add_vec = add_vec;
   const size_t smem = sizeof(float) * (size_t)hidden;
   const bool aligned = hidden % 4 == 0 &&
-      (((uintptr_t)resid | (uintptr_t)delta | (uintptr_t)post_weight | (uintptr_t)layer_scale | (uintptr_t)delta_bias | (uintptr_t)weight | (uintptr_t)out) & 15) == 0;
+      (((uintptr_t)resid | (uintptr_t)delta | (uintptr_t)post_weight | (uintptr_t)layer_scale | (uintptr_t)delta_bias | (uintptr_t)weight | (uintptr_t)out |
+        (uintptr_t)second | (uintptr_t)add_rows | (uintptr_t)add_vec) & 15) == 0;
   const int per = aligned ? 4 : 1;
   int threads = 64;
   while (threads < 512 && threads * per * 2 <= hidden) threads <<= 1;

@@ -31,7 +31,7 @@ class KernelError(RuntimeError):
 _SIGNATURES: dict[str, list[Any]] = {
     "ts_embed": [_vp, _vp, _vp, _i, _i, _i, _i, _f, _vp],
     "ts_add_rms_norm": [_vp, _vp, _vp, _vp, _vp, _i, _i, _f, _i, _vp],
-    "ts_rope_tables": [_vp, _vp, _vp, _vp, _i, _i, _vp],
+    "ts_rope_tables": [_vp, _vp, _vp, _vp, _i, _i, _c.c_double, _vp],
     "ts_silu_mul": [_vp, _vp, _i, _i, _i, _vp],
     "ts_qk_norm_rope_write": [_vp, _vp, _vp, _vp, _f, _vp, _vp, _i, _i, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _vp],
     "ts_paged_attention_simt": [_vp, _vp, _vp, _vp, _vp, _i, _vp, _vp, _vp, _i, _vp, _i, _i, _i, _i, _i, _i,
@@ -45,17 +45,21 @@ _SIGNATURES: dict[str, list[Any]] = {
     "ts_add_bias": [_vp, _vp, _i, _i, _i, _vp],
     "ts_tanh": [_vp, _c.c_size_t, _i, _vp],
     "ts_linear_scan": [_i, _vp, _i, _vp, _i, _vp, _i, _vp, _i, _vp, _vp, _vp, _vp, _i, _vp, _vp, _i, _i, _i, _i, _vp, _i, _i, _i, _i, _vp, _vp,
-                       _f, _f, _vp],
+                       _f, _f, _vp, _vp, _i, _i, _f, _vp],
     "ts_token_shift_mix": [_vp, _i, _vp, _i, _vp, _i, _vp, _vp, _i, _i, _i, _vp, _i, _vp],
     "ts_softcap": [_vp, _c.c_size_t, _f, _vp],
     "ts_rms_norm_rows": [_vp, _c.c_longlong, _vp, _f, _vp, _i, _i, _i, _vp],
     "ts_head_norm_gate": [_vp, _i, _vp, _i, _vp, _i, _vp, _i, _i, _i, _i, _f, _i, _i, _i, _vp],
-    "ts_post_norm_add_rms_norm": [_vp, _vp, _vp, _vp, _f, _i, _f, _vp, _i, _f, _vp, _vp, _i, _i, _vp, _i, _vp],
+    "ts_post_norm_add_rms_norm": [_vp, _vp, _vp, _vp, _f, _i, _f, _vp, _i, _f, _vp, _vp, _i, _i, _vp, _vp, _f, _vp, _vp, _i, _vp],
     "ts_mlstm_scan": [_vp, _i, _i, _i, _i, _vp, _vp, _f, _f, _vp, _i, _vp, _vp, _i, _i, _i, _i, _vp, _i, _vp],
     "ts_delta_scan": [_vp, _i, _i, _i, _i, _vp, _i, _i, _vp, _vp, _vp, _i, _f, _vp, _i, _vp, _vp, _i, _i, _i, _i, _i, _vp, _vp],
     "ts_causal_conv_silu": [_vp, _i, _vp, _vp, _i, _vp, _vp, _i, _i, _i, _i, _vp, _i, _vp],
     "ts_qkv_prepare": [_vp, _i, _vp, _i, _vp, _i, _vp, _vp, _vp, _vp, _vp, _f, _vp, _vp, _i, _vp, _vp, _vp, _i, _i, _i, _i,
                        _i, _i, _vp, _i, _i, _vp],
+    "ts_qkv_rotate": [_vp, _i, _vp, _i, _vp, _i, _vp, _vp, _i, _vp, _vp, _i, _i, _i, _f, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _vp,
+                      _i, _i, _vp],
+    "ts_talking_attention": [_vp, _vp, _vp, _vp, _vp, _i, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _f, _i, _f, _vp, _vp, _i, _vp, _vp,
+                             _i, _vp],
     "ts_prefill_attention_mma": [_vp, _vp, _vp, _vp, _vp, _i, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _f, _i, _vp],
     "ts_decode_attention_mma": [_vp, _vp, _vp, _vp, _vp, _i, _vp, _vp, _vp, _i, _i, _i, _i, _i, _f, _i, _i, _vp, _vp,
                                 _vp, _vp],
@@ -87,11 +91,12 @@ _SIGNATURES: dict[str, list[Any]] = {
                           _i, _i, _i, _vp],
     "ts_latent_attention": [_vp, _vp, _vp, _vp, _i, _vp, _vp, _i, _i, _i, _i, _i, _i, _f, _i, _i, _i, _i, _vp, _vp, _i, _vp, _vp],
     "ts_latent_attention_mma_takes": [_i, _i],
-    "ts_moe_route": [_vp, _i, _i, _i, _i, _i, _i, _i, _i, _f, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _vp, _vp, _i, _vp],
+    "ts_moe_route": [_vp, _i, _i, _i, _i, _i, _i, _i, _i, _i, _f, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _vp, _vp, _vp, _i,
+                     _vp],
     "ts_moe_route_fused": [_vp, _vp, _i, _i, _vp, _i, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _vp, _vp, _i, _vp],
     "ts_moe_gather": [_vp, _vp, _vp, _i, _i, _vp, _vp],
-    "ts_moe_gemm_tcgen05": [_vp, _vp, _vp, _i, _i, _i, _i, _i, _vp, _vp, _vp, _vp, _i, _vp, _vp],
-    "ts_moe_gemm": [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _vp],
+    "ts_moe_gemm_tcgen05": [_vp, _vp, _vp, _i, _i, _i, _i, _i, _vp, _f, _vp, _vp, _vp, _vp, _i, _vp, _vp],
+    "ts_moe_gemm": [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _vp, _f, _i, _i, _vp],
     "ts_moe_combine": [_vp, _vp, _vp, _vp, _vp, _i, _i, _i, _vp, _vp, _i, _i, _vp],
     "ts_sample": [_vp, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp],
 }
@@ -238,11 +243,15 @@ def add_rms_norm(resid: torch.Tensor, delta: torch.Tensor | None, weight: torch.
 def post_norm_add_rms_norm(resid: torch.Tensor, delta: torch.Tensor | None, post_weight: torch.Tensor | None,
                            layer_scale: torch.Tensor | None, post_eps: float, post_offset: bool, weight: torch.Tensor,
                            offset: bool, eps: float, out: torch.Tensor, rows: torch.Tensor | None = None,
-                           post_mult: float = 1.0, delta_bias: torch.Tensor | None = None) -> None:
+                           post_mult: float = 1.0, delta_bias: torch.Tensor | None = None,
+                           second: torch.Tensor | None = None, second_scale: float = 1.0,
+                           add_rows: torch.Tensor | None = None, add_vec: torch.Tensor | None = None) -> None:
     """The residual sum with a norm on the pending sub-layer output, and the next norm, in one pass,
     all in 32-bit: ``y = post_mult * delta / sqrt(mean(delta^2) + post_eps) * gain(post_weight) * layer_scale``
     (``post_weight`` / ``layer_scale`` ``None``: that factor is left out; without a ``post_weight``, ``delta_bias``
-    (one value per column, dt) is added to ``delta`` first: ``y = (delta + delta_bias) * layer_scale``), ``x = resid + y``,
+    (one value per column, dt) is added to ``delta`` first: ``y = (delta + delta_bias) * post_mult * layer_scale``),
+    ``x = resid + y`` (``+ second_scale * second``, a second pending output like ``delta``; ``+ add_rows``, float32
+    ``[T, h]``; ``+ add_vec``, one value per column, dt; each when given),
     ``out = dt(x / sqrt(mean(x^2) + eps) * gain(weight))`` with ``gain(w) = 1 + w`` when the matching
     ``offset`` flag is set, else ``w``. Without ``rows`` the sum is written back to ``resid``; with
     ``rows`` (int32) only those rows are read and ``resid`` stays."""
@@ -256,22 +265,27 @@ def post_norm_add_rms_norm(resid: torch.Tensor, delta: torch.Tensor | None, post
     for name, v in (("post_weight", post_weight), ("layer_scale", layer_scale), ("delta_bias", delta_bias)):
         if v is not None and (delta is None or v.shape != (h,)):
             raise KernelError(f"post_norm_add_rms_norm: {name} needs a pending output and one value per column")
+    if second is not None and (delta is None or second.shape != resid.shape):
+        raise KernelError("post_norm_add_rms_norm: a second pending output goes beside the first, with its shape")
+    if (add_rows is not None and add_rows.shape != resid.shape) or (add_vec is not None and add_vec.shape != (h,)):
+        raise KernelError("post_norm_add_rms_norm: add_rows must have the stream's shape, add_vec one value per column")
     if (rows is None and n != resid.shape[0]) or (rows is not None and rows.shape != (n,)):
         raise KernelError("post_norm_add_rms_norm: out must have one row per row of resid, or per entry of rows")
     _check(_fn("ts_post_norm_add_rms_norm")(
         _dev(resid, "resid", torch.float32), _opt(delta, "delta", dt), _opt(post_weight, "post_weight", dt),
         _opt(layer_scale, "layer_scale", dt), float(post_eps), int(bool(post_offset)), float(post_mult), _dev(weight, "weight", dt),
         int(bool(offset)), float(eps), _dev(out, "out"), _opt(rows, "rows", torch.int32), n, h, _opt(delta_bias, "delta_bias", dt),
-        _code(dt), _stream()), "post_norm_add_rms_norm")
+        _opt(second, "second", dt), float(second_scale), _opt(add_rows, "add_rows", torch.float32),
+        _opt(add_vec, "add_vec", dt), _code(dt), _stream()), "post_norm_add_rms_norm")
 
 
-def rope_tables(positions: torch.Tensor, inv_freq: torch.Tensor, cos: torch.Tensor, sin: torch.Tensor) -> None:
-    """``cos/sin[t, i] = float32(cos/sin(float64(positions[t]) * inv_freq[i]))``."""
+def rope_tables(positions: torch.Tensor, inv_freq: torch.Tensor, cos: torch.Tensor, sin: torch.Tensor, mult: float = 1.0) -> None:
+    """``cos/sin[t, i] = float32(mult * cos/sin(float64(positions[t]) * inv_freq[i]))``."""
     t, half = cos.shape
     if positions.shape != (t,) or inv_freq.shape != (half,) or sin.shape != cos.shape:
         raise KernelError("rope_tables: shape mismatch")
     _check(_fn("ts_rope_tables")(_dev(positions, "positions", torch.int32), _dev(inv_freq, "inv_freq", torch.float64),
-                                 _dev(cos, "cos", torch.float32), _dev(sin, "sin", torch.float32), t, half,
+                                 _dev(cos, "cos", torch.float32), _dev(sin, "sin", torch.float32), t, half, float(mult),
                                  _stream()), "rope_tables")
 
 
@@ -1329,10 +1343,23 @@ def linear_scan_gated(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, w_pre: 
     _linear_scan(2, q, k, v, w_pre, w_bias, None, None, state, ctx, heads, d, dv, out, inv_tau=1.0 / tau, q_scale=q_scale)
 
 
+def linear_scan_rotated(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, cos: torch.Tensor | None,
+                        sin: torch.Tensor | None, rotary_dim: int, interleaved: bool, k_scale: float, state: torch.Tensor,
+                        ctx: Any, heads: int, d: int, dv: int, out: torch.Tensor) -> None:
+    """Retention: the first ``rotary_dim`` elements of every head of q and k turn by the token's angles (``cos``/``sin``
+    ``[T, rotary_dim / 2]`` float32), k is multiplied by ``k_scale``, all in 32-bit on the way into the recurrence; per
+    head ``S <- decay_h S + k v^T``, ``o = S^T q``. Shapes as for ``linear_scan_bonus``; ``decay [heads]`` float32."""
+    if rotary_dim and (cos is None or tuple(cos.shape) != (q.shape[0], rotary_dim // 2) or tuple(sin.shape) != tuple(cos.shape)):
+        raise KernelError("linear_scan_rotated: rotary tables missing or of the wrong shape")
+    _linear_scan(3, q, k, v, None, None, None, decay, state, ctx, heads, d, dv, out, cos=cos, sin=sin, rotary_dim=rotary_dim,
+                 interleaved=interleaved, k_scale=k_scale)
+
+
 def _linear_scan(mode: int, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, w_pre: torch.Tensor | None,
                  w_bias: torch.Tensor | None, bonus: torch.Tensor | None, decay: torch.Tensor | None,
                  state: torch.Tensor, ctx: Any, heads: int, d: int, dv: int, out: torch.Tensor,
-                 inv_tau: float = 0.0, q_scale: float = 1.0) -> None:
+                 inv_tau: float = 0.0, q_scale: float = 1.0, cos: torch.Tensor | None = None, sin: torch.Tensor | None = None,
+                 rotary_dim: int = 0, interleaved: bool = False, k_scale: float = 1.0) -> None:
     t, dt = q.shape[0], q.dtype
     for name, x, width in (("q", q, heads * d), ("k", k, heads * d), ("v", v, heads * dv)):
         if not x.is_cuda or x.dtype != dt or x.shape != (t, width) or x.stride(1) != 1:
@@ -1360,7 +1387,8 @@ def _linear_scan(mode: int, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, w
         _dev(ctx.state_slots, "state_slots", torch.int32), ctx.num_seqs, heads, d, dv,
         _dev(out, "out", torch.float32), _code(dt), int(ctx.max_query_len), seg_len, max_segs,
         None if seg_state is None else seg_state.data_ptr(), None if seg_decay is None else seg_decay.data_ptr(),
-        float(inv_tau), float(q_scale), _stream()),
+        float(inv_tau), float(q_scale), _opt(cos, "cos", torch.float32), _opt(sin, "sin", torch.float32), int(rotary_dim),
+        int(bool(interleaved)), float(k_scale), _stream()),
         "linear_scan", kernels=1 if max_segs <= 1 else (4 if mode in (0, 2) else 3))
 
 
@@ -1518,6 +1546,92 @@ def qkv_prepare(q_in: torch.Tensor, k_in: torch.Tensor | None, v_in: torch.Tenso
         _opt(cos, "cos", torch.float32), _opt(sin, "sin", torch.float32), int(rotary_dim),
         _opt(slots, "slots", torch.int32), _opt(k_cache, "k_cache", dt), _opt(v_cache, "v_cache", dt), page_size, t,
         heads, kv_heads, d, dv, _dev(q_out, "q_out"), int(bool(norm_whole)), _code(dt), _stream()), "qkv_prepare")
+
+
+def qkv_rotate(proj: torch.Tensor, taps: torch.Tensor | None, state: torch.Tensor | None, ctx: Any, cos: torch.Tensor | None,
+               sin: torch.Tensor | None, rotary_dim: int, interleaved: bool, unit_eps: float | None, slots: torch.Tensor,
+               k_cache: torch.Tensor, v_cache: torch.Tensor, page_size: int, heads: int, kv_heads: int, d: int, dv: int,
+               q_out: torch.Tensor) -> None:
+    """``proj [T, >= channels]`` dt holds q, k and v (``channels`` = ``(heads + kv_heads) * d + kv_heads * dv`` columns).
+    With ``taps [K, channels]`` dt every channel first passes a causal convolution over time, ``y_t = sum_j taps[j]
+    u_(t - K + 1 + j)``, whose inputs before this step come from ``state [slots, (K - 1) * channels]`` float32 (zero at a
+    request's start), left holding the last ``K - 1`` inputs. Then the first ``rotary_dim`` elements of every q and k head
+    turn (neighbours when ``interleaved``, else i with i + rotary_dim / 2), and with ``unit_eps`` every q and k head is
+    divided by its root mean square (``unit_eps`` inside the root). 32-bit, rounded once: queries to ``q_out
+    [T, heads, d]``, keys and values to the caches at the tokens' slots."""
+    t, dt = q_out.shape[0], q_out.dtype
+    channels = (heads + kv_heads) * d + kv_heads * dv
+    if proj.dim() != 2 or proj.shape[0] != t or proj.shape[1] < channels or proj.dtype != dt or proj.stride(1) != 1 or not proj.is_cuda:
+        raise KernelError(f"qkv_rotate: proj must be [T, >= {channels}] {dt} with unit column stride on the device")
+    if tuple(q_out.shape) != (t, heads, d) or slots.shape != (t,):
+        raise KernelError("qkv_rotate: q_out shape, or one slot per token")
+    if tuple(k_cache.shape[1:]) != (kv_heads, page_size, d) or tuple(v_cache.shape[1:]) != (kv_heads, page_size, dv):
+        raise KernelError("qkv_rotate: cache layout")
+    if rotary_dim and (cos is None or tuple(cos.shape) != (t, rotary_dim // 2) or tuple(sin.shape) != tuple(cos.shape)):
+        raise KernelError("qkv_rotate: rotary tables missing or of the wrong shape")
+    k, state_ptr, state_stride = 0, None, 0
+    if taps is not None:
+        k = taps.shape[0]
+        if taps.shape != (k, channels) or taps.dtype != dt:
+            raise KernelError(f"qkv_rotate: taps must be [K, {channels}] {dt}")
+        if k > 1:
+            state_ptr, state_stride = _state_rows(state, (k - 1) * channels, "qkv_rotate")
+    _check_indices("qkv_rotate", None, None, page_size, k_cache.shape[0], slots)
+    single = ctx.max_query_len == 1
+    _check(_fn("ts_qkv_rotate")(
+        proj.data_ptr(), proj.stride(0), _opt(taps, "taps", dt), k, state_ptr, state_stride,
+        _dev(ctx.cu_query_lens, "cu_query_lens", torch.int32), _opt(ctx.state_slots, "state_slots", torch.int32), ctx.num_seqs,
+        _opt(cos, "cos", torch.float32), _opt(sin, "sin", torch.float32), int(rotary_dim), int(bool(interleaved)),
+        int(unit_eps is not None), float(unit_eps or 0.0), _dev(slots, "slots", torch.int32), _dev(k_cache, "k_cache", dt),
+        _dev(v_cache, "v_cache", dt), page_size, t, heads, kv_heads, d, dv, _dev(q_out, "q_out"), int(single), _code(dt),
+        _stream()), "qkv_rotate", kernels=2 if k > 1 and not single else 1)
+
+
+# ------------------------------------- attention with weights mixed across the heads
+TALKING_MAX_SPLITS = 16
+TALKING_MIN_KEYS_PER_SPLIT = 64
+
+
+def talking_splits(num_seqs: int, keys: int) -> int:
+    """Key ranges per request for a step of single tokens: enough CTAs to give every SM one, no range shorter than
+    64 keys. Depends only on the step's shape."""
+    return max(1, min(SM_COUNT // max(1, num_seqs), keys // TALKING_MIN_KEYS_PER_SPLIT, TALKING_MAX_SPLITS))
+
+
+def talking_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, page_size: int, block_tables: torch.Tensor,
+                      ctx: Any, scale: float, window: int, softcap: float | None, talk: torch.Tensor | None, out: torch.Tensor,
+                      sinks: torch.Tensor | None = None) -> None:
+    """Causal attention (``window`` 0: all earlier positions) with optionally capped scores ``cap tanh(s / cap)`` and
+    the heads' weights mixed behind the softmax: ``w_h = sum_g talk[h, g] p_g`` (``talk [Hq, Hq]`` float32 or None), each
+    head applying its mixed weights to the values of its own key/value head. Shapes as for :func:`paged_attention`."""
+    t, hq, d = q.shape
+    hkv, dv, dt = k_cache.shape[1], v_cache.shape[3], q.dtype
+    if k_cache.dtype != dt or v_cache.dtype != dt or out.dtype != dt or out.numel() != t * hq * dv or hq % hkv:
+        raise KernelError("talking_attention: dtypes, out shape or head grouping")
+    if tuple(k_cache.shape[1:]) != (hkv, page_size, d) or tuple(v_cache.shape[:3]) != tuple(k_cache.shape[:3]):
+        raise KernelError("talking_attention: cache layout must be [pages, kv_heads, page_size, head_dim]")
+    if block_tables.dim() != 2 or block_tables.shape[0] != ctx.num_seqs:
+        raise KernelError("talking_attention: block_tables must be [requests, width]")
+    if talk is not None and (talk.shape != (hq, hq) or talk.dtype != torch.float32):
+        raise KernelError("talking_attention: talk must be float32 [heads, heads]")
+    if sinks is not None and (sinks.shape != (hq,) or sinks.dtype != torch.float32):
+        raise KernelError("talking_attention: sinks must be float32, one per query head")
+    if softcap is not None and not softcap > 0:
+        raise KernelError("talking_attention: softcap must be positive or None")
+    _check_indices("talking_attention", block_tables, ctx, page_size, k_cache.shape[0])
+    splits, part_ml, part_out = 1, None, None
+    if ctx.max_query_len == 1:
+        splits = talking_splits(ctx.num_seqs, min(ctx.max_context_len, window) if window else ctx.max_context_len)
+        if splits > 1:
+            part_ml = ctx.arena.take((t, hq, splits, 2), torch.float32)
+            part_out = ctx.arena.take((t, splits, hq * dv), torch.float32)
+    _check(_fn("ts_talking_attention")(
+        _dev(q, "q"), _dev(out, "out"), _dev(k_cache, "k_cache"), _dev(v_cache, "v_cache"),
+        _dev(block_tables, "block_tables", torch.int32), block_tables.shape[1],
+        _dev(ctx.cu_query_lens, "cu_query_lens", torch.int32), _dev(ctx.context_lens_dev, "context_lens", torch.int32),
+        ctx.num_seqs, ctx.max_query_len, t, hq, hkv, d, dv, page_size, float(scale), int(window), float(softcap or 0.0),
+        _opt(talk, "talk", torch.float32), _opt(sinks, "sinks", torch.float32), splits, _opt(part_ml, "part_ml"),
+        _opt(part_out, "part_out"), _code(dt), _stream()), "talking_attention", kernels=3 if splits > 1 else 1)
 
 
 # ------------------------------------------------------------- latent attention
@@ -1681,9 +1795,16 @@ class RouteRule:
     or None) and only inside the ``keep`` best of ``groups`` equal groups of neighbouring outputs (a group's
     value is its largest choice score; the others' count as minus infinity); the weights are the picks' scores
     over their sum (+ 1e-20), times ``scale``. ``identity``: the last outputs are experts without matrices
-    whose output is their input; their picks take no row of the sorted order."""
+    whose output is their input; their picks take no row of the sorted order. ``sigmoid`` (scored): an output's
+    score is the sigmoid of its logit instead (without a correction the choice then goes by the logits, whose
+    order is the scores'). ``normalise=False``: the weights are ``score * scale``, not divided by their sum.
+    ``on_input``: a weight multiplies its expert's input: the gated product applies it (``plan["row_weight"]``)
+    and the combine step adds the experts' outputs as they are."""
 
     scored: bool = False
+    sigmoid: bool = False
+    normalise: bool = True
+    on_input: bool = False
     groups: int = 1
     keep: int = 1
     scale: float = 1.0
@@ -1735,33 +1856,43 @@ def moe_route(logits: torch.Tensor, top: int, counts: torch.Tensor, arena: Any, 
         raise KernelError("moe_route: outputs, identity experts or the logits' layout")
     if not 0 < top <= min(e, 32) or counts.shape != (real,):
         raise KernelError("moe_route: top must be between 1 and min(outputs, 32); counts one per expert with matrices")
-    if not rule.scored and (rule.identity or rule.groups > 1 or rule.correction is not None):
-        raise KernelError("moe_route: groups, a correction and identity experts come with the scored rule")
+    if not rule.scored and (rule.identity or rule.groups > 1 or rule.correction is not None or rule.sigmoid or rule.on_input
+                            or not rule.normalise):
+        raise KernelError("moe_route: groups, a correction, identity experts and the weights' options come with the scored rule")
+    if rule.on_input and rule.identity:
+        raise KernelError("moe_route: weights on the experts' input together with identity experts")
     if rule.groups < 1 or rule.groups > 32 or e % rule.groups or not 1 <= rule.keep <= rule.groups or e // rule.groups * rule.keep < top:
         raise KernelError("moe_route: up to 32 equal groups, of which the kept ones must hold at least `top` outputs")
     if rule.correction is not None and (rule.correction.shape != (e,) or rule.correction.dtype != torch.float32):
         raise KernelError("moe_route: the correction must be float32, one value per output")
     tiles = moe_max_tiles(t, top, real, tile_rows)
     plan = _moe_plan(t, real, top, arena, tile_rows)
+    plan["row_weight"] = arena.take((t * top,), torch.float32) if rule.on_input else None
     _check(_fn("ts_moe_route")(
-        _dev(logits, "logits", torch.float32), logits.stride(0), t, e, real, top, int(rule.scored), rule.groups, rule.keep,
+        _dev(logits, "logits", torch.float32), logits.stride(0), t, e, real, top,
+        0 if not rule.scored else 2 if rule.sigmoid else 1, int(bool(rule.normalise)), rule.groups, rule.keep,
         float(rule.scale), _opt(rule.correction, "correction", torch.float32), plan["ids"].data_ptr(),
         plan["weights"].data_ptr(), plan["place"].data_ptr(), _dev(counts, "counts", torch.int32), plan["offsets"].data_ptr(),
         plan["tile_expert"].data_ptr(), plan["tile_row0"].data_ptr(), plan["num_tiles"].data_ptr(), tiles,
-        plan["row_of"].data_ptr(), plan["token_of"].data_ptr(), tile_rows, _stream()), "moe_route",
-        kernels=1 if t <= 64 else 3)
+        plan["row_of"].data_ptr(), plan["token_of"].data_ptr(), _opt(plan["row_weight"], "row_weight"), tile_rows, _stream()),
+        "moe_route", kernels=1 if t <= 64 else 3)
     plan["logits"] = logits
     plan["identity"] = rule.identity
     return plan
 
 
 def moe_gemm(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, plan: dict[str, Any], gated: bool, gather: bool,
-             arena: Any = None) -> None:
+             arena: Any = None, limit: float = 0.0) -> None:
     """The experts' products over the sorted order of ``plan``: for every sorted row r of expert e,
     ``out[r] = x_r W_e^T`` (``gated``: ``silu(x_r Wgate_e^T) * (x_r Wup_e^T)`` with ``w [E, 2 N, K]``,
     gate rows first; else ``w [E, N, K]``). ``gather``: ``x`` is ``[T, K]`` and row r reads its
-    token's row; else ``x`` is ``[picks, K]`` in the sorted order. ``out [picks, N]`` dt."""
+    token's row; else ``x`` is ``[picks, K]`` in the sorted order. ``out [picks, N]`` dt. ``limit`` > 0 (gated): the
+    clamped activation, ``g = min(gate, limit)``, ``u = clamp(up, -limit, limit)``, ``g sigmoid(1.702 g) (u + 1)``. When the
+    plan's weights belong to the experts' input, a gated product multiplies both sums of a row by its weight first."""
     picks, n = out.shape
+    row_weight = plan.get("row_weight") if gated else None
+    if limit > 0 and not gated:
+        raise KernelError("moe_gemm: the clamped activation belongs to a gated product")
     e, rows, k = w.shape
     if picks != plan["picks"] or e != plan["experts"] or rows != (2 * n if gated else n) or x.shape[1] != k:
         raise KernelError("moe_gemm: shapes")
@@ -1778,14 +1909,16 @@ def moe_gemm(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, plan: dict[str
                                         total_rows.data_ptr(), _stream()), "moe_gather")
             x = xs
         _check(_fn("ts_moe_gemm_tcgen05")(
-            _dev(x, "x"), _dev(w, "w"), _dev(out, "out"), picks, n, k, e, int(bool(gated)), plan["offsets"].data_ptr(),
-            plan["tile_expert"].data_ptr(), plan["tile_row0"].data_ptr(), plan["num_tiles"].data_ptr(), plan["max_tiles"],
+            _dev(x, "x"), _dev(w, "w"), _dev(out, "out"), picks, n, k, e, int(bool(gated)),
+            _opt(row_weight, "row_weight"), float(limit), plan["offsets"].data_ptr(), plan["tile_expert"].data_ptr(),
+            plan["tile_row0"].data_ptr(), plan["num_tiles"].data_ptr(), plan["max_tiles"],
             _error_word(x.device).data_ptr(), _stream()), "moe_gemm_tcgen05")
         return
     _check(_fn("ts_moe_gemm")(
         _dev(x, "x"), plan["token_of"].data_ptr() if gather else None, _dev(w, "w"), _dev(out, "out"),
         plan["offsets"].data_ptr(), plan["tile_expert"].data_ptr(), plan["tile_row0"].data_ptr(),
-        plan["num_tiles"].data_ptr(), plan["max_tiles"], n, k, int(bool(gated)), _code(x.dtype), int(MOE_TENSOR_CORES),
+        plan["num_tiles"].data_ptr(), plan["max_tiles"], n, k, int(bool(gated)), _opt(row_weight, "row_weight"), float(limit),
+        _code(x.dtype), int(MOE_TENSOR_CORES),
         _stream()), "moe_gemm")
 
 
@@ -1794,7 +1927,7 @@ def moe_combine(y: torch.Tensor, plan: dict[str, Any], shared_out: torch.Tensor 
     """``out[t] = dt(sum_j weight[t, j] * y[row_of[t, j]] (+ g[t] * shared_out[t]))`` in 32-bit. A pick of an
     identity expert contributes ``weight * x[t]`` (``x [T, hidden]`` dt: the experts' input; needed when the plan
     has identity experts). ``shared_gate`` (float32 ``[T]``, possibly a column of a wider matrix): ``g =
-    sigmoid(shared_gate)``; without it ``g = 1``."""
+    sigmoid(shared_gate)``; without it ``g = 1``. With weights on the experts' input the picked rows are added as they are."""
     t, h = out.shape
     if tuple(y.shape) != (plan["picks"], h) or t * plan["top"] != plan["picks"] or y.dtype != out.dtype:
         raise KernelError("moe_combine: shapes or dtypes")
@@ -1806,7 +1939,8 @@ def moe_combine(y: torch.Tensor, plan: dict[str, Any], shared_out: torch.Tensor 
         raise KernelError("moe_combine: x must be [T, hidden] dt")
     if shared_gate is not None and (shared_out is None or shared_gate.shape != (t,) or shared_gate.dtype != torch.float32):
         raise KernelError("moe_combine: the shared gate is one float32 logit per token and needs a shared output")
-    _check(_fn("ts_moe_combine")(_dev(y, "y"), plan["row_of"].data_ptr(), plan["weights"].data_ptr(),
+    _check(_fn("ts_moe_combine")(_dev(y, "y"), plan["row_of"].data_ptr(),
+                                 None if plan.get("row_weight") is not None else plan["weights"].data_ptr(),
                                  _opt(shared_out, "shared_out"), _dev(out, "out"), t, plan["top"], h, _opt(x, "x"),
                                  None if shared_gate is None else shared_gate.data_ptr(),
                                  0 if shared_gate is None else shared_gate.stride(0), _code(out.dtype), _stream()),

@@ -19,8 +19,8 @@ import torch
 from . import parts as _parts  # noqa: F401  (registers the built-in parts)
 from .config.base import LayerSpec, ModelConfig, ModelSpec
 from .parts.base import (
-    BLOCKS, EMBEDDINGS, HEADS, NORMS, PART_FAMILIES, POSITION_ENCODINGS,
-    Block, CacheNeed, PagedNeed, PositionEncoding, ResidualStream, StepContext, TensorSpec,
+    BLOCKS, EMBEDDINGS, HEADS, NORMS, PART_FAMILIES, POSITION_ENCODINGS, STREAM_INPUTS,
+    Block, CacheNeed, PagedNeed, PositionEncoding, ResidualStream, StepContext, StreamInput, TensorSpec,
 )
 from .weights.loader import load_tensors, merge_specs
 from .weights.random_init import random_bound_tensors
@@ -31,6 +31,7 @@ class Layer:
     spec: LayerSpec
     block: Block
     position: PositionEncoding | None
+    positions: dict[str, PositionEncoding]      # by mixer role, when the mixers have encodings of their own
 
 
 class ModelParts:
@@ -45,20 +46,32 @@ class ModelParts:
         self.layers: list[Layer] = []
         for n, ls in enumerate(spec.layers):
             block = self._build_block(n, ls)
-            pos = None
-            if ls.position is not None:
-                cand = POSITION_ENCODINGS.build(ls.position.kind, **ls.position.args)
-                pos = self._positions.setdefault(cand.key(), cand)
-            self.layers.append(Layer(ls, block, pos))
-        # One cache user per (call of the order, mixer role of its block), in that order: the
+            pos = None if ls.position is None else self._encoding(ls.position)
+            unknown = set(ls.positions) - set(block.mixers())
+            if unknown:
+                raise ValueError(f"layer {n}: position encodings for {sorted(unknown)}, which are no mixers of its block")
+            self.layers.append(Layer(ls, block, pos, {role: self._encoding(p) for role, p in ls.positions.items()}))
+        self.stream_inputs: list[StreamInput | None] = [
+            None if c.stream_input is None else STREAM_INPUTS.build(c.stream_input.kind, **c.stream_input.args) for c in spec.order]
+        self.keeps_origin = any(s is not None and s.needs_origin for s in self.stream_inputs)
+        # One cache user per (call of the order, mixer role of its block, need of that mixer), in that order: the
         # cache manager gets their needs as a flat list and hands back one entry for each.
         self.cache_users: list[tuple[int, str]] = []
-        self._user_index: dict[tuple[int, str], int] = {}
+        self._user_index: dict[tuple[int, str], "int | tuple[int, ...]"] = {}
+        self._needs: list[CacheNeed | None] = []
         for n, call in enumerate(spec.order):
-            for role in self.layers[call.layer].block.mixers():
-                self._user_index[(n, role)] = len(self.cache_users)
-                self.cache_users.append((n, role))
+            for role, mixer in self.layers[call.layer].block.mixers().items():
+                need = mixer.cache_need()
+                several = need if isinstance(need, tuple) else (need,)
+                first = len(self.cache_users)
+                self.cache_users += [(n, role)] * len(several)
+                self._user_index[(n, role)] = tuple(range(first, first + len(several))) if isinstance(need, tuple) else first
+                self._needs += several if call.reads_cache_of is None else (None,) * len(several)
         self._check_order()
+
+    def _encoding(self, spec: Any) -> PositionEncoding:
+        cand = POSITION_ENCODINGS.build(spec.kind, **spec.args)
+        return self._positions.setdefault(cand.key(), cand)
 
     @staticmethod
     def _build_block(n: int, ls: LayerSpec) -> Block:
@@ -103,6 +116,9 @@ class ModelParts:
         for layer in self.layers:
             for part in layer.block.parts.values():
                 yield layer.spec.prefix, part
+        for part in self.stream_inputs:
+            if part is not None:
+                yield "", part
         yield "", self.final_norm
         yield "", self.head
 
@@ -124,17 +140,10 @@ class ModelParts:
 
     # ---- cache
     def cache_needs(self) -> list[CacheNeed | None]:
-        """One entry per cache user (a call of the order and a mixer role of its block; with one
-        mixer per block, one entry per call): what it keeps between steps (``None`` for a
-        mixer that keeps nothing or a call that reads another call's cache)."""
-        needs: list[CacheNeed | None] = []
-        for n, role in self.cache_users:
-            call = self.spec.order[n]
-            if call.reads_cache_of is not None:
-                needs.append(None)
-            else:
-                needs.append(self.layers[call.layer].block.parts[role].cache_need())
-        return needs
+        """One entry per cache user (a call of the order, a mixer role of its block and a need of
+        that mixer; with one mixer per block that keeps one thing, one entry per call): what it keeps
+        between steps (``None`` for a mixer that keeps nothing or a call that reads another call's cache)."""
+        return list(self._needs)
 
     def caches_of_call(self, n: int, entries: list[Any]) -> dict[str, Any]:
         """The cache entries that call ``n`` of the order works on, by mixer role: its own, or
@@ -143,14 +152,15 @@ class ModelParts:
         src = n if call.reads_cache_of is None else call.reads_cache_of
         out = {}
         for role in self.layers[call.layer].block.mixers():
-            entry = entries[self._user_index[(src, role)]]
+            index = self._user_index[(src, role)]
+            entry = tuple(entries[i] for i in index) if isinstance(index, tuple) else entries[index]
             if entry is not None:
                 out[role] = entry
         return out
 
     def recordable(self, kind: str) -> bool:
         """Whether steps of this kind ("decode", "prefill") can be recorded: every part allows it."""
-        parts = [part for _, part in self._each_part()] + [l.position for l in self.layers if l.position is not None]
+        parts = [part for _, part in self._each_part()] + list(self._positions.values())
         return all(kind in part.recordable for part in parts)
 
 
@@ -208,22 +218,33 @@ class DecoderModel:
                 total += t.numel() * t.element_size()
         return total
 
+    @staticmethod
+    def _position_data(encoding: PositionEncoding, ctx: StepContext) -> Any:
+        key = encoding.key()
+        if key not in ctx.position_tables:
+            ctx.position_tables[key] = encoding.prepare(ctx)
+        return ctx.position_tables[key]
+
     def forward(self, ctx: StepContext, caches: list[Any], want_rows: torch.Tensor | None,
                 num_want: int) -> torch.Tensor | None:
         """Run this step's tokens; return float32 logits ``[num_want, vocab]`` at ``want_rows``
         (flat row indices into the step's tokens), or ``None`` if nothing is wanted."""
         parts = self.parts
         stream = ResidualStream(parts.embedding.forward(ctx))
+        if parts.keeps_origin:
+            stream.origin = parts.embedding.forward(ctx)      # a second copy that no layer adds to
         for n, call in enumerate(self.spec.order):
             layer = parts.layers[call.layer]
-            tables = None
-            if layer.position is not None:
-                key = layer.position.key()
-                if key not in ctx.position_tables:
-                    ctx.position_tables[key] = layer.position.prepare(ctx)
-                tables = ctx.position_tables[key]
+            if parts.stream_inputs[n] is not None:
+                parts.stream_inputs[n].forward(stream, ctx)
+            if layer.positions:
+                tables = {role: self._position_data(p, ctx) for role, p in layer.positions.items()}
+            else:
+                tables = None if layer.position is None else self._position_data(layer.position, ctx)
             ctx.upcoming_caches = parts.caches_of_call(n + 1, caches) if n + 1 < len(self.spec.order) else {}
             layer.block.forward(stream, ctx, parts.caches_of_call(n, caches), call.reads_cache_of is None, tables)
+            if stream.extra is not None:
+                raise RuntimeError(f"call {n} of the order: the block's first norm does not take what was added in front of it")
         ctx.arena.step_region()
         for join in ctx.at_step_end:
             join()

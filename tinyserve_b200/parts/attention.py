@@ -17,7 +17,7 @@ from typing import Any, Mapping
 import torch
 
 from ..kernels import ops
-from .base import (EVERY_STEP, KVCacheEntry, KVNeed, LatentNeed, LazyNormed, Mixer, ResidualStream, SplitKVNeed,
+from .base import (EVERY_STEP, KVCacheEntry, KVNeed, LatentNeed, LazyNormed, Mixer, ResidualStream, SplitKVNeed, StateNeed,
                    StepContext, TensorSpec, project, project_to_stream, register_mixer)
 
 
@@ -393,6 +393,107 @@ class LatentAttention(Mixer):
         return out
 
 
+class RotatedAttention(Mixer):
+    """Grouped-query attention without an output gate, whose q, k and v pass, in this order: the merged projection
+    (no biases); with ``conv_taps`` a short causal convolution over time on every channel (tensors ``<q>.conv``,
+    ``<k>.conv``, ``<v>.conv`` ``[channels, taps]``, no bias, no activation; the last ``taps - 1`` projected values of
+    a request are state); the rotation of q and k that the layer's position encoding asks for (either
+    pairing, tables with any constant on them); with ``unit_norm`` a division of every q and k head by its root mean
+    square, without a weight. Scores ``scale * q . k``, with ``softcap`` then ``cap * tanh(s / cap)``; causal, with
+    ``window`` only the last ``window`` positions, itself included; softmax, with ``sink`` a learned logit per head in
+    the denominator; with ``talk`` the heads' weights are mixed by a learned ``[heads, heads]`` matrix before each
+    head applies its own to the values of its key/value head; ``W_o`` on the concatenated heads.
+
+    ``names`` maps the roles "q", "k", "v", "out", "sink", "talk" to tensor names after the prefix. Convolution,
+    rotation, norm and cache write are one kernel; plain scores run on the framework's paged attention kernels,
+    capped or mixed ones on ``ops.talking_attention``."""
+
+    recordable = EVERY_STEP
+    _NAMES = {"q": "q", "k": "k", "v": "v", "out": "o", "sink": "sink", "talk": "talk"}
+
+    def __init__(self, prefix: str, hidden_size: int, num_heads: int, num_kv_heads: int, key_dim: int, value_dim: int,
+                 scale: float, window: int | None = None, unit_norm: bool = False, norm_eps: float = 1e-6, sink: bool = False,
+                 softcap: float | None = None, talk: bool = False, conv_taps: int | None = None,
+                 names: Mapping[str, str] | None = None) -> None:
+        if num_heads % num_kv_heads:
+            raise ValueError(f"num_heads={num_heads} is not a multiple of num_kv_heads={num_kv_heads}")
+        if window is not None and window <= 0:
+            raise ValueError(f"window must be positive or None, got {window}")
+        if softcap is not None and not softcap > 0:
+            raise ValueError(f"softcap must be positive or None, got {softcap}")
+        if conv_taps is not None and conv_taps < 1:
+            raise ValueError(f"conv_taps={conv_taps} must be at least 1 (None: no convolution)")
+        for what, size in (("key_dim", key_dim), ("value_dim", value_dim)):
+            if not 0 < size <= 256:
+                raise ValueError(f"{what}={size}: the attention kernels take head sizes up to 256")
+        self.prefix, self.h = prefix, int(hidden_size)
+        self.heads, self.groups, self.d, self.dv = int(num_heads), int(num_kv_heads), int(key_dim), int(value_dim)
+        self.scale, self.window = float(scale), None if window is None else int(window)
+        self.unit_eps = float(norm_eps) if unit_norm else None
+        self.has_sink, self.softcap, self.has_talk = bool(sink), None if softcap is None else float(softcap), bool(talk)
+        self.taps = None if conv_taps is None else int(conv_taps)
+        self.names = {**self._NAMES, **(names or {})}
+        self.rows = (self.heads * self.d, self.groups * self.d, self.groups * self.dv)      # of q, k and v
+        self.channels = sum(self.rows)
+        self.w_taps = self.sink = self.talk = None
+
+    def cache_need(self) -> Any:
+        kv = (KVNeed(self.groups, self.d, self.window) if self.d == self.dv
+              else SplitKVNeed(self.groups, self.d, self.dv, self.window))
+        if self.taps is None or self.taps == 1:
+            return kv
+        return kv, StateNeed(((self.taps - 1) * self.channels,), torch.float32)      # the convolution's last inputs
+
+    def tensor_specs(self, prefix: str) -> list[TensorSpec]:
+        p, n, h = prefix + self.prefix, self.names, self.h
+        qkv = tuple(p + n[r] for r in ("q", "k", "v"))
+        specs = [TensorSpec(p + "qkv", (self.channels, h), merged_from=qkv, merged_rows=self.rows),
+                 TensorSpec(p + n["out"], (h, self.heads * self.dv))]
+        if self.taps is not None:
+            specs.append(TensorSpec(p + "qkv.conv", (self.channels, self.taps), std=0.3, merged_from=tuple(x + ".conv" for x in qkv),
+                                    merged_rows=self.rows))
+        if self.has_sink:
+            specs.append(TensorSpec(p + n["sink"], (self.heads,), std=1.0))
+        if self.has_talk:
+            specs.append(TensorSpec(p + n["talk"], (self.heads, self.heads), std=0.3))
+        return specs
+
+    def bind(self, prefix: str, tensors: Mapping[str, torch.Tensor]) -> None:
+        p, n = prefix + self.prefix, self.names
+        self.w_in, self.w_o = tensors[p + "qkv"], tensors[p + n["out"]]
+        if self.taps is not None:
+            self.w_taps = tensors[p + "qkv.conv"].t().contiguous()          # tap by tap: a channel's neighbours lie together
+        if self.has_sink:
+            self.sink = tensors[p + n["sink"]].float().contiguous()
+        if self.has_talk:
+            self.talk = tensors[p + n["talk"]].float().contiguous()
+
+    def forward(self, x: torch.Tensor, ctx: StepContext, cache: Any, writes_cache: bool, position: Any) -> torch.Tensor:
+        if not writes_cache:
+            raise RuntimeError("this mixer keeps a cache of its own")
+        kv, state = cache if isinstance(cache, tuple) else (cache, None)
+        t, arena = x.shape[0], ctx.arena
+        group = ctx.kv[kv.group]
+        proj = arena.take((t, self.channels), ctx.dtype)
+        ops.gemm(x, self.w_in, proj)
+        rot = None if position is None else position.qk_rotation()
+        queries = arena.take((t, self.heads, self.d), ctx.dtype)
+        ops.qkv_rotate(proj, self.w_taps, None if state is None else state.state, ctx, None if rot is None else rot.cos,
+                       None if rot is None else rot.sin, 0 if rot is None else rot.rotary_dim, rot is not None and rot.interleaved,
+                       self.unit_eps, group.slots, kv.k, kv.v, kv.page_size, self.heads, self.groups, self.d, self.dv, queries)
+        attn = arena.take((t, self.heads * self.dv), ctx.dtype)
+        if self.softcap is None and self.talk is None:
+            ops.paged_attention(queries, kv.k, kv.v, kv.page_size, group.block_tables, ctx, self.scale, self.window or 0, attn,
+                                sinks=self.sink)
+        else:
+            ops.talking_attention(queries, kv.k, kv.v, kv.page_size, group.block_tables, ctx, self.scale, self.window or 0,
+                                  self.softcap, self.talk, attn, sinks=self.sink)
+        out = arena.take((t, self.h), ctx.dtype)
+        ops.gemm(attn, self.w_o, out)
+        return out
+
+
+register_mixer("rotated_attention", RotatedAttention)
 register_mixer("gqa_attention", GQAAttention)
 register_mixer("latent_attention", LatentAttention)
 register_mixer("gated_sink_attention", GatedSinkAttention)

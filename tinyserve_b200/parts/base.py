@@ -18,8 +18,11 @@ Kinds of part and what each must provide:
 * ``Mixer``: ``cache_need()`` says what it keeps between steps, as a ``CacheNeed``: a
   ``PagedNeed`` (pages per token: ``KVNeed`` is keys and values for all or a window of the
   positions; a mixer may define its own), a ``SlotNeed`` (``StateNeed``: a fixed-size state per
-  request), or nothing; ``forward(x, ctx, cache, writes_cache) -> [T, hidden]``.
+  request), a tuple of several needs, or nothing; ``forward(x, ctx, cache, writes_cache) -> [T, hidden]``
+  (``cache`` is then a tuple too).
 * ``FeedForward``: ``forward(x, ctx) -> [T, hidden]``.
+* ``StreamInput``: adds something to the residual stream in front of a call of the run order
+  (``LayerCall.stream_input``); it is left pending and folded in by the next norm.
 * ``Block``: names the roles it wants filled (``roles``: role -> family of part) and arranges
   those parts around the stream; ``PreNormBlock`` wants a mixer, a feed-forward and their norms.
 
@@ -277,9 +280,15 @@ class ResidualStream:
     A layer that norms a sub-layer's output before the residual sum leaves that norm pending too:
     ``post`` holds ``(weight, layer_scale | None, eps, unit_offset, mult)`` with which ``delta`` is normed
     and scaled when the next norm folds it into the stream (``parts.norm.PostRMSNorm``); a sixth element, when
-    there is one, is an output bias of the sub-layer that is added to ``delta`` first (``parts.norm.LayerScale``)."""
+    there is one, is an output bias of the sub-layer that is added to ``delta`` first (``parts.norm.LayerScale``).
 
-    __slots__ = ("resid", "delta", "sumsq", "resid16", "_sumsq_buf", "_resid16_buf", "lanes", "connection", "post")
+    Two sub-layers side by side leave two outputs: ``second`` is ``(output, constant)`` of the other one, added to
+    the stream together with ``delta``. ``extra`` is what a ``StreamInput`` has left: ``(rows [T, hidden] 32-bit or
+    None, one value per column or None)``, added after them. Norms that do not know these two leave them, and the
+    model refuses to go on. ``origin`` is the embedding output in 32-bit, kept for the calls that add it again."""
+
+    __slots__ = ("resid", "delta", "sumsq", "resid16", "_sumsq_buf", "_resid16_buf", "lanes", "connection", "post", "second",
+                 "extra", "origin")
 
     def __init__(self, resid: torch.Tensor, delta: torch.Tensor | None = None) -> None:
         self.resid = resid
@@ -287,6 +296,9 @@ class ResidualStream:
         self.lanes: torch.Tensor | None = None
         self.connection: tuple[torch.Tensor, torch.Tensor] | None = None
         self.post: tuple[torch.Tensor, torch.Tensor | None, float, bool, float] | None = None
+        self.second: tuple[torch.Tensor, float] | None = None
+        self.extra: tuple[torch.Tensor | None, torch.Tensor | None] | None = None
+        self.origin: torch.Tensor | None = None
         self.sumsq: torch.Tensor | None = None
         self.resid16: torch.Tensor | None = None
         self._sumsq_buf: torch.Tensor | None = None
@@ -433,7 +445,7 @@ class Mixer(Part):
     # True if ``forward`` has a keyword ``stream`` and may add its output to it (returning None).
     adds_to_stream: bool = False
 
-    def cache_need(self) -> CacheNeed | None:
+    def cache_need(self) -> "CacheNeed | tuple[CacheNeed, ...] | None":
         return None
 
     def forward(self, x: torch.Tensor, ctx: StepContext, cache: Any, writes_cache: bool,
@@ -463,6 +475,17 @@ class TokenInput(Part):
         raise NotImplementedError
 
 
+class StreamInput(Part):
+    """Something added to the residual stream right before a call of the run order: ``forward(stream,
+    ctx)`` leaves it in ``stream.extra``. ``needs_origin``: it adds the embedding output again
+    (``stream.origin``, which the model then keeps)."""
+
+    needs_origin: bool = False
+
+    def forward(self, stream: ResidualStream, ctx: StepContext) -> None:
+        raise NotImplementedError
+
+
 class Block:
     """Arranges the parts of one layer around the residual stream. A block class names the roles
     it wants filled: ``roles`` maps a role (a name of the block's own choosing, the key under which
@@ -486,7 +509,8 @@ class Block:
     def forward(self, stream: ResidualStream, ctx: StepContext, caches: Mapping[str, Any], writes_cache: bool,
                 position: Any) -> None:
         """``caches[role]`` is the cache entry of the mixer in that role for this call of the
-        layer (absent if it keeps nothing)."""
+        layer (absent if it keeps nothing). ``position`` is the step's position data of the layer's
+        encoding, or a mapping of mixer roles to it when the mixers have encodings of their own."""
         raise NotImplementedError
 
 
@@ -521,6 +545,7 @@ BLOCKS = _Registry("block")
 EMBEDDINGS = _Registry("embedding")
 HEADS = _Registry("output head")
 TOKEN_INPUTS = _Registry("token input")
+STREAM_INPUTS = _Registry("stream input")
 # the families a block's roles may name
 PART_FAMILIES = {"mixer": MIXERS, "feed_forward": FEED_FORWARDS, "norm": NORMS, "token_input": TOKEN_INPUTS}
 

@@ -10,14 +10,29 @@ from typing import Any, Mapping
 from .base import Block, Part, ResidualStream, StepContext, register_block
 
 
-class PreNormBlock(Block):
-    # the order is the order of the layer's tensors in ``tensor_specs``
-    roles = {"mixer_norm": "norm", "mixer": "mixer", "feed_forward_norm": "norm", "feed_forward": "feed_forward"}
+def _position_of(position: Any, role: str) -> Any:
+    return position.get(role) if isinstance(position, Mapping) else position
 
-    def __init__(self, parts: Mapping[str, Part]) -> None:
+
+class PreNormBlock(Block):
+    """``x += mixer(norm(x))``, then, when the layer has a feed-forward, ``x += feed_forward(norm(x))``. With a
+    ``second_mixer`` both mixers read the same normed input and the sum takes
+    ``mixer_scale * mixer + second_mixer_scale * second_mixer``; the two outputs stay pending side by side."""
+
+    # the order is the order of the layer's tensors in ``tensor_specs``
+    roles = {"mixer_norm": "norm", "mixer": "mixer", "second_mixer": "mixer", "feed_forward_norm": "norm",
+             "feed_forward": "feed_forward"}
+    optional_roles = frozenset({"second_mixer", "feed_forward_norm", "feed_forward"})
+
+    def __init__(self, parts: Mapping[str, Part], mixer_scale: float = 1.0, second_mixer_scale: float = 1.0) -> None:
         super().__init__(parts)
-        self.mixer, self.feed_forward = parts["mixer"], parts["feed_forward"]
-        self.mixer_norm, self.feed_forward_norm = parts["mixer_norm"], parts["feed_forward_norm"]
+        if ("feed_forward" in parts) != ("feed_forward_norm" in parts):
+            raise ValueError("a feed-forward comes with its norm")
+        self.mixer, self.second_mixer, self.feed_forward = parts["mixer"], parts.get("second_mixer"), parts.get("feed_forward")
+        self.mixer_norm, self.feed_forward_norm = parts["mixer_norm"], parts.get("feed_forward_norm")
+        self.scale_a, self.scale_b = float(mixer_scale), float(second_mixer_scale)
+        if self.second_mixer is None and (self.scale_a != 1.0 or self.scale_b != 1.0):
+            raise ValueError("constants on the mixers' outputs come with two mixers")
 
     def forward(self, stream: ResidualStream, ctx: StepContext, caches: Mapping[str, Any], writes_cache: bool,
                 position: Any) -> None:
@@ -26,13 +41,26 @@ class PreNormBlock(Block):
         ctx.arena.next_frame()
         mixer, ff = self.mixer, self.feed_forward
         cache = caches.get("mixer")
-        ctx.upcoming_weights = ff.streamed_weights()
+        if self.second_mixer is not None:
+            ctx.upcoming_weights = []
+            hn = self.mixer_norm.forward(stream, ctx)
+            a = mixer.forward(hn, ctx, cache, writes_cache, _position_of(position, "mixer"))
+            b = self.second_mixer.forward(hn, ctx, caches.get("second_mixer"), writes_cache, _position_of(position, "second_mixer"))
+            stream.delta, stream.second, stream.sumsq = a, (b, self.scale_b), None
+            stream.post = (None, None, 0.0, False, self.scale_a)
+            if ff is not None:
+                self._leave(stream, ff.forward(self.feed_forward_norm.forward(stream, ctx), ctx))
+            return
+        position = _position_of(position, "mixer")
+        ctx.upcoming_weights = [] if ff is None else ff.streamed_weights()
         hn = self.mixer_norm.lazy(stream, ctx) if mixer.takes_lazy_input else self.mixer_norm.forward(stream, ctx)
         if mixer.adds_to_stream:
             mixed = mixer.forward(hn, ctx, cache, writes_cache, position, stream=stream)
         else:
             mixed = mixer.forward(hn, ctx, cache, writes_cache, position)
         self._leave(stream, mixed)
+        if ff is None:
+            return
         hn = self.feed_forward_norm.lazy(stream, ctx) if ff.takes_lazy_input else self.feed_forward_norm.forward(stream, ctx)
         self._leave(stream, ff.forward(hn, ctx, stream=stream) if ff.adds_to_stream else ff.forward(hn, ctx))
 

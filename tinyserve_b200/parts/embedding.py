@@ -10,7 +10,8 @@ from typing import Mapping
 import torch
 
 from ..kernels import ops
-from .base import EMBEDDINGS, EVERY_STEP, HEADS, Part, StepContext, TensorSpec
+from .base import (EMBEDDINGS, EVERY_STEP, HEADS, STREAM_INPUTS, Part, ResidualStream, StepContext, StreamInput,
+                   TensorSpec)
 
 
 class TokenEmbedding(Part):
@@ -101,6 +102,33 @@ class LMHead(Part):
         return out
 
 
+class PassVector(StreamInput):
+    """In front of pass ``index`` of layers that run ``count`` times: row ``index`` of the learned table
+    ``name [count, hidden]`` is added to the stream, and with ``add_origin`` the embedding output once more.
+    Both are left pending: the pass's first norm adds them in 32-bit in the pass it makes anyway."""
+
+    recordable = EVERY_STEP
+
+    def __init__(self, name: str, hidden_size: int, index: int, count: int, add_origin: bool = False) -> None:
+        if not 0 <= index < count:
+            raise ValueError(f"pass {index} of {count}")
+        self.name, self.hidden_size, self.index, self.count = name, int(hidden_size), int(index), int(count)
+        self.needs_origin = bool(add_origin)
+        self.vector: torch.Tensor | None = None
+
+    def tensor_specs(self, prefix: str) -> list[TensorSpec]:
+        return [TensorSpec(prefix + self.name, (self.count, self.hidden_size))]
+
+    def bind(self, prefix: str, tensors: Mapping[str, torch.Tensor]) -> None:
+        self.vector = tensors[prefix + self.name][self.index]
+
+    def forward(self, stream: ResidualStream, ctx: StepContext) -> None:
+        if stream.extra is not None:
+            raise RuntimeError("something is already waiting to be added to the stream")
+        stream.extra = (stream.origin if self.needs_origin else None, self.vector)
+
+
+STREAM_INPUTS.register("pass_vector", PassVector)
 EMBEDDINGS.register("token_embedding", TokenEmbedding)
 EMBEDDINGS.register("positioned_embedding", PositionedEmbedding)
 HEADS.register("lm_head", LMHead)

@@ -139,7 +139,11 @@ class RoutedExperts(FeedForward):
     the experts' are identity experts, whose output is the token's input itself; they take part in the
     softmax, the groups and the choice, and have no tensors. ``shared_gate``: the shared expert's output is
     multiplied by ``sigmoid(w_sg . x)``, one value per token (a ``[1, hidden]`` tensor, which rides along
-    in the router's product so that it is 32-bit like the router).
+    in the router's product so that it is 32-bit like the router). ``score="sigmoid"``: an output's score is the
+    sigmoid of its logit; ``normalise=False``: the weights are the scores (times ``route_scale``) as they are;
+    ``weight_on="input"``: a weight multiplies its expert's input, ``sum_e expert_e(w_e x)``, which the gated product
+    applies to its finished sums. ``activation="clamped_swish"`` with ``limit``: the experts' activation is
+    ``g sigmoid(1.702 g) (u + 1)`` with ``g = min(gate, limit)`` and ``u = clamp(up, -limit, limit)``.
 
     The experts' matrices are stacked (``[E, 2 ff, hidden]`` gate rows then up rows, ``[E, hidden,
     ff]``); tokens are sorted by expert on the device and the products run tile by tile over that
@@ -153,14 +157,27 @@ class RoutedExperts(FeedForward):
     def __init__(self, prefix: str, hidden_size: int, num_experts: int, top: int, expert_size: int,
                  shared_size: int | None = None, names: "Mapping[str, str] | None" = None, routing: str = "top_logits",
                  correction: bool = False, groups: int = 1, group_keep: int = 1, route_scale: float = 1.0,
-                 identity: int = 0, shared_gate: bool = False) -> None:
+                 identity: int = 0, shared_gate: bool = False, score: str = "softmax", normalise: bool = True,
+                 weight_on: str = "output", activation: str = "silu", limit: float | None = None) -> None:
+        if score not in ("softmax", "sigmoid") or weight_on not in ("output", "input") or activation not in ("silu", "clamped_swish"):
+            raise ValueError(f"score={score!r} ('softmax', 'sigmoid'), weight_on={weight_on!r} ('output', 'input'), "
+                             f"activation={activation!r} ('silu', 'clamped_swish')")
+        if (activation == "clamped_swish") != (limit is not None) or (limit is not None and not limit > 0):
+            raise ValueError("'clamped_swish' takes a positive limit, 'silu' none")
+        if weight_on == "input" and (identity or activation == "silu"):
+            raise NotImplementedError("weights on the experts' input: without identity experts, with the clamped activation")
+        if activation == "clamped_swish" and shared_size is not None:
+            raise NotImplementedError("a shared expert with the clamped activation")
+        self.sigmoid, self.normalise, self.on_input = score == "sigmoid", bool(normalise), weight_on == "input"
+        self.limit = 0.0 if limit is None else float(limit)
         outputs = int(num_experts) + int(identity)
         if not 0 < top <= min(outputs, 32):
             raise ValueError(f"top={top} must be between 1 and min(router outputs={outputs}, 32)")
         if routing not in ("top_logits", "scored"):
             raise ValueError(f"routing={routing!r}: 'top_logits' or 'scored'")
-        if routing != "scored" and (correction or groups != 1 or identity or route_scale != 1.0):
-            raise ValueError("a correction, groups, identity experts and a constant on the weights come with routing='scored'")
+        if routing != "scored" and (correction or groups != 1 or identity or route_scale != 1.0 or self.sigmoid or not normalise
+                                    or self.on_input):
+            raise ValueError("a correction, groups, identity experts and the weights' options come with routing='scored'")
         if identity < 0 or not 1 <= groups <= 32 or outputs % groups or not 1 <= group_keep <= groups:
             raise ValueError(f"groups={groups} (at most 32) must divide the {outputs} router outputs, and 1 <= group_keep <= groups")
         if outputs // groups * group_keep < top:
@@ -212,7 +229,8 @@ class RoutedExperts(FeedForward):
         if self.scored:
             corr = tensors[p + n["correction"]].float().contiguous() if self.has_correction else None
             self.rule = ops.RouteRule(scored=True, groups=self.groups, keep=self.group_keep, scale=self.route_scale,
-                                      identity=self.identity, correction=corr)
+                                      identity=self.identity, correction=corr, sigmoid=self.sigmoid, normalise=self.normalise,
+                                      on_input=self.on_input)
         self.w_gate_up = tensors[p + "experts.gate+up"].view(self.experts, 2 * self.ff, self.h)
         self.w_down = tensors[p + "experts.down"].view(self.experts, self.h, self.ff)
         if self.shared_ff is not None:
@@ -227,7 +245,7 @@ class RoutedExperts(FeedForward):
         tile_rows = ops.moe_tile_rows(t, self.top, self.experts, ctx.dtype, (self.h, self.ff))
         plan = ops.moe_route_from(x, self.w_router, self.top, self.counts, arena, tile_rows, self.rule, self.outputs)
         act = arena.take((t * self.top, self.ff), ctx.dtype)
-        ops.moe_gemm(x, self.w_gate_up, act, plan, gated=True, gather=True, arena=arena)
+        ops.moe_gemm(x, self.w_gate_up, act, plan, gated=True, gather=True, arena=arena, limit=self.limit)
         y = arena.take((t * self.top, self.h), ctx.dtype)
         ops.moe_gemm(act, self.w_down, y, plan, gated=False, gather=False, arena=arena)
         shared = None

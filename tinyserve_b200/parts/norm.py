@@ -40,20 +40,27 @@ class RMSNorm(Norm):
         self.weight = tensors[prefix + self.name]
 
     def _run(self, stream: ResidualStream, out: torch.Tensor, rows: torch.Tensor | None) -> None:
+        more = {}
+        if stream.second is not None:
+            more["second"], more["second_scale"] = stream.second
+        if stream.extra is not None:
+            more["add_rows"], more["add_vec"] = stream.extra
         if stream.post is None and not self.round_once:
+            if more:
+                raise NotImplementedError("two outputs side by side or a stream input in front of a norm that rounds before its weight")
             ops.add_rms_norm(stream.resid, stream.delta, self.weight, self.eps, out, rows=rows)
             return
         post_w, post_scale, post_eps, post_offset, post_mult, *rest = \
             stream.post if stream.post is not None else (None, None, 0.0, False, 1.0)
         ops.post_norm_add_rms_norm(stream.resid, stream.delta, post_w, post_scale, post_eps, post_offset, self.weight,
                                    self.unit_offset, self.eps, out, rows=rows, post_mult=post_mult,
-                                   delta_bias=rest[0] if rest else None)
+                                   delta_bias=rest[0] if rest else None, **more)
 
     def forward(self, stream: ResidualStream, ctx: StepContext) -> torch.Tensor:
         out = ctx.arena.take((stream.resid.shape[0], self.size), ctx.dtype)
         self._run(stream, out, None)
-        if stream.delta is not None:
-            stream.delta = None
+        if stream.delta is not None or stream.extra is not None:
+            stream.delta = stream.second = stream.extra = None
             stream.post = None
             stream.sumsq = None          # the stream has changed
         return out

@@ -38,6 +38,11 @@ constant ``tau``; per head ``S <- diag(alpha) S + k v^T``, ``o = S^T q`` (the re
 token's write). Each head's ``o`` is RMS-normed with a weight shared by the heads, multiplied by
 ``silu(W_g h)`` and projected by ``W_o``.
 
+``RetentionMixer``: linear attention with a constant decay per head, a rotation and no activation: q and k
+(``heads x dim``) are rotated as the layer's position encoding asks, k is multiplied by ``dim^-1/2``; per
+head ``S <- decay_h S + k v^T``, ``o = S^T q``; each head's ``o`` is divided by its root mean square (no
+weight), the heads are concatenated, multiplied by ``silu(W_g h)`` and projected by ``W_o``.
+
 Gates, decays, step sizes, unit scalings and the state are 32-bit; the projections and the
 convolution's inputs are in the model dtype. Nothing of a step is read on the host: requests are
 found through ``cu_query_lens`` and ``state_slots`` on the device, so every kind of step can be
@@ -428,6 +433,54 @@ class GatedLinearAttention(Mixer):
         return out
 
 
+class RetentionMixer(Mixer):
+    recordable = EVERY_STEP
+    _NAMES = {"q": "q", "k": "k", "v": "v", "gate": "g", "out": "o"}
+
+    def __init__(self, prefix: str, hidden_size: int, num_heads: int, key_dim: int, value_dim: int, decay: "list[float]",
+                 norm_eps: float, names: Mapping[str, str] | None = None) -> None:
+        _check_key_dim("retention", key_dim)
+        if len(decay) != num_heads:
+            raise ValueError(f"{len(decay)} decay constants for {num_heads} heads")
+        self.prefix, self.h = prefix, int(hidden_size)
+        self.heads, self.d, self.dv, self.eps = int(num_heads), int(key_dim), int(value_dim), float(norm_eps)
+        self.decay_values = [float(x) for x in decay]
+        self.names = {**self._NAMES, **(names or {})}
+
+    def cache_need(self) -> StateNeed:
+        return StateNeed((self.heads * self.d * self.dv,), torch.float32)
+
+    def tensor_specs(self, prefix: str) -> list[TensorSpec]:
+        p, n, h = prefix + self.prefix, self.names, self.h
+        qk, vv = self.heads * self.d, self.heads * self.dv
+        return [TensorSpec(p + "qkvg", (2 * qk + 2 * vv, h), merged_from=tuple(p + n[r] for r in ("q", "k", "v", "gate")),
+                           merged_rows=(qk, qk, vv, vv)),
+                TensorSpec(p + n["out"], (h, vv))]
+
+    def bind(self, prefix: str, tensors: Mapping[str, torch.Tensor]) -> None:
+        p, n = prefix + self.prefix, self.names
+        self.w_in, self.w_o = tensors[p + "qkvg"], tensors[p + n["out"]]
+        self.decay = torch.tensor(self.decay_values, dtype=torch.float32, device=self.w_o.device)
+
+    def forward(self, x: torch.Tensor, ctx: StepContext, cache: StateCacheEntry, writes_cache: bool, position: Any) -> torch.Tensor:
+        t, arena = x.shape[0], ctx.arena
+        qk, vv = self.heads * self.d, self.heads * self.dv
+        proj = arena.take((t, 2 * qk + 2 * vv), ctx.dtype)
+        ops.gemm(x, self.w_in, proj)
+        rot = None if position is None else position.qk_rotation()
+        read = arena.take((t, self.heads, self.dv), torch.float32)
+        ops.linear_scan_rotated(proj[:, :qk], proj[:, qk: 2 * qk], proj[:, 2 * qk: 2 * qk + vv], self.decay,
+                                None if rot is None else rot.cos, None if rot is None else rot.sin,
+                                0 if rot is None else rot.rotary_dim, rot is not None and rot.interleaved, self.d ** -0.5,
+                                cache.state, ctx, self.heads, self.d, self.dv, read)
+        gated = arena.take((t, vv), ctx.dtype)
+        ops.head_norm_gate(read, None, False, proj[:, 2 * qk + vv:], True, self.eps, gated, gate_silu=True)
+        out = arena.take((t, self.h), ctx.dtype)
+        ops.gemm(gated, self.w_o, out)
+        return out
+
+
+register_mixer("retention", RetentionMixer)
 register_mixer("gated_linear_attention", GatedLinearAttention)
 register_mixer("gated_delta", GatedDeltaMixer)
 register_mixer("time_mix", TimeMixMixer)

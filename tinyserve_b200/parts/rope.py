@@ -5,8 +5,8 @@ in float64, ``angle = position * inv_freq`` in float64, cos and sin taken in flo
 rounded to float32. The rotation itself (pairs ``i`` and ``i + rotary_dim/2`` for the "half"
 pairing, neighbours ``2i, 2i+1`` for "interleaved"; src/tinyserve/layers.py:84-91 has the
 former) is applied by the mixer's fused kernel, which receives these tables. ``scaling``: the four
-keys of the rule by wavelength below, or ``{"factor": f}`` alone for linear scaling (every
-frequency divided by ``f``).
+keys of the rule by wavelength below; ``factor, original, fast, slow`` for YaRN (``scale_yarn``, which also
+puts a constant on cos and sin); or ``{"factor": f}`` alone for linear scaling (every frequency divided by ``f``).
 """
 
 from __future__ import annotations
@@ -36,6 +36,23 @@ def scale_by_wavelength(freq: torch.Tensor, factor: float, low: float, high: flo
     return torch.where(wavelength < original / high, freq, out)
 
 
+def scale_yarn(freq: torch.Tensor, dims: int, base: float, factor: float, original: float, fast: float, slow: float) -> torch.Tensor:
+    """YaRN: pair i keeps its frequency where it turns more than ``fast`` times over ``original`` positions, has it
+    divided by ``factor`` where it turns less than ``slow`` times, and moves between the two along a ramp over the
+    pairs' indices (float64). The bounds are the indices at which a pair of ``base^(-2i/dims)`` turns that often,
+    rounded outwards and kept inside ``0 .. dims - 1``."""
+    if not (factor > 0 and original > 0 and fast > 0 and slow > 0 and base > 1):
+        raise ValueError(f"YaRN needs positive factor, original, fast, slow and base > 1; got {factor}, {original}, {fast}, {slow}, {base}")
+
+    def index(turns: float) -> float:
+        return dims * math.log(original / (2.0 * math.pi * turns)) / (2.0 * math.log(base))
+
+    lo, hi = max(math.floor(index(fast)), 0), min(math.ceil(index(slow)), dims - 1)
+    i = torch.arange(freq.shape[0], dtype=torch.float64)
+    ramp = ((i - lo) / max(hi - lo, 0.001)).clamp(0.0, 1.0)
+    return freq / factor * ramp + freq * (1.0 - ramp)
+
+
 class RotaryEncoding(PositionEncoding):
     recordable = EVERY_STEP
 
@@ -50,7 +67,13 @@ class RotaryEncoding(PositionEncoding):
         two_i = torch.arange(0, self.rotary_dim, 2, dtype=torch.float64)
         self._inv_freq_host = self.theta ** (-two_i / self.rotary_dim)
         self.scaling = None
-        if scaling and set(scaling) == {"factor"}:
+        self.mult = 1.0                 # a constant on cos and sin
+        if scaling and set(scaling) == {"factor", "original", "fast", "slow"}:
+            values = [float(scaling[k]) for k in ("factor", "original", "fast", "slow")]
+            self.scaling = ("yarn", *values)
+            self._inv_freq_host = scale_yarn(self._inv_freq_host, self.rotary_dim, self.theta, *values)
+            self.mult = 0.1 * math.log(values[0]) + 1.0
+        elif scaling and set(scaling) == {"factor"}:
             # linear scaling: every frequency divided by the factor (positions stretched by it)
             if not float(scaling["factor"]) > 0:
                 raise ValueError(f"rotary scaling factor must be positive, got {scaling['factor']}")
@@ -71,7 +94,10 @@ class RotaryEncoding(PositionEncoding):
         half = self.rotary_dim // 2
         cos = ctx.arena.take_step((ctx.num_tokens, half), torch.float32)
         sin = ctx.arena.take_step((ctx.num_tokens, half), torch.float32)
-        ops.rope_tables(ctx.positions, self._inv_freq, cos, sin)
+        if self.mult == 1.0:
+            ops.rope_tables(ctx.positions, self._inv_freq, cos, sin)
+        else:
+            ops.rope_tables(ctx.positions, self._inv_freq, cos, sin, self.mult)
         return RotaryTables(cos, sin, self.rotary_dim, self.pairing == "interleaved")
 
 
