@@ -1,4 +1,4 @@
-"""``python bench.py --designs [--design fegilix|guzovik|gasavik|diderax] [--design-beside qwen3|guzovik|...]``:
+"""``python bench.py --designs [--design fegilix|guzovik|gasavik|diderax|sanevik] [--design-beside qwen3|guzovik|...]``:
 prefill and decode throughput of a design at layer sizes that resemble a real model's (random weights), beside
 the dense Qwen3 decoder (or, with ``--design-beside``, another design of the framework), with the same width,
 attention heads, (active) feed-forward size and number of layers; and where each design's step time goes, kernel class by kernel class, with the
@@ -107,11 +107,32 @@ def diderax_config(s: dict) -> dict:
                        {"type": "attention", "mlp": dense, "mixer": attn}, {"type": "gla", "mlp": moe, "mixer": gla}]}
 
 
-DESIGNS = {"fegilix": fegilix_config, "guzovik": guzovik_config, "gasavik": gasavik_config, "diderax": diderax_config}
+def sanevik_config(s: dict) -> dict:
+    """Four layers of which the first two run twice: windowed attention with sinks and unit-length q and k; the pair
+    of windowed attention behind convolutions with capped scores and mixed heads, and retention with heads of 128
+    that fill the width; the two again with weights of their own. Windows of 512; every layer with routed experts
+    of a quarter of the dense feed-forward's size, four used per token."""
+    attn = {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": s["dim"], "vdim": s["dim"], "scale": s["dim"] ** -0.5,
+            "rot": {"dims": s["dim"], "base": 5e5, "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}},
+            "mask": {"size": 512}}
+    pair = {"left": {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": s["dim"], "vdim": s["dim"], "scale": s["dim"] ** -0.5,
+                     "rot": {"dims": s["dim"], "base": 1e4}, "mask": {"size": 512}, "softcap": 30.0, "conv": 4},
+            "right": {"heads": s["rec_heads"], "dim": s["dim"], "vdim": s["dim"], "rot": {"dims": s["dim"], "base": 1e4},
+                      "decay": [1.0 - 2.0 ** -(5 + 5 * i / max(1, s["rec_heads"] - 1)) for i in range(s["rec_heads"])]},
+            "left_scale": 0.6, "right_scale": 0.5}
+    mlp = {"kind": "moe", "router": {"experts": s["experts"], "top": 4}, "expert": {"ff": s["ff"] // 4, "limit": 7.0}}
+    a, p = {"type": "attention", "mlp": mlp, "mixer": attn}, {"type": "parallel", "mlp": mlp, "mixer": pair}
+    return {"architecture": "Sanevik", "vocab": VOCAB, "width": s["width"], "norm": {"eps": 1e-6}, "max_positions": 8192,
+            "loop": {"start": 0, "stop": 2, "times": 2}, "layers": [a, p, a, p]}
+
+
+DESIGNS = {"fegilix": fegilix_config, "guzovik": guzovik_config, "gasavik": gasavik_config, "diderax": diderax_config,
+           "sanevik": sanevik_config}
 NEW_OPS = ["post_norm_add_rms_norm", "latent_prepare", "latent_attention", "bmm", "transpose01", "moe_route_from", "moe_route", "moe_gemm",
            "moe_combine", "gemm_gated", "hc_mix_norm", "hc_collapse", "act_mul", "softcap", "head_norm_gate", "mlstm_scan", "delta_scan",
            "causal_conv_silu", "qkv_prepare", "linear_scan_bonus", "linear_scan_decay", "token_shift_mix", "embed_pos_norm",
-           "stream_sum", "add_bias", "tanh_", "act_mul_gather", "gemm_biased_swiglu", "linear_scan_gated", "rms_norm_rows"]
+           "stream_sum", "add_bias", "tanh_", "act_mul_gather", "gemm_biased_swiglu", "linear_scan_gated", "rms_norm_rows",
+           "qkv_rotate", "talking_attention", "linear_scan_rotated"]
 OLD_OPS = ["embed", "add_rms_norm", "rope_tables", "silu_mul", "qk_norm_rope_write", "paged_attention",
            "decode_attention_fused", "gemm", "gemm_swiglu", "gemm_to_stream", "gemm_normed", "sample"]
 
@@ -248,6 +269,16 @@ class DesignBench(Bench):
             if name == "linear_scan_gated":   # state in and out, q, k, v and the decays' pre-activations read, the read-out written; 4 flops per state element and token
                 ctx, heads, d, dv = a[8], a[9], a[10], a[11]
                 return (2.0 * ctx.num_seqs * heads * d * dv * 4 + nbytes(a[0], a[1], a[2], a[3], a[12]), 4.0 * a[0].shape[0] * heads * d * dv)
+            if name == "linear_scan_rotated":     # state in and out, q, k, v read, the read-out written; 4 flops per state element and token
+                ctx, heads, d, dv = a[10], a[11], a[12], a[13]
+                return (2.0 * ctx.num_seqs * heads * d * dv * 4 + nbytes(a[0], a[1], a[2], a[14]), 4.0 * a[0].shape[0] * heads * d * dv)
+            if name == "qkv_rotate":          # q, k and v rows read and written
+                return 2.0 * a[0].shape[0] * ((a[13] + a[14]) * a[15] + a[14] * a[16]) * a[0].element_size(), 0.0
+            if name == "talking_attention":   # keys and values once per request; both products and the mixing of the heads
+                ctx, window, heads = a[5], a[7], a[0].shape[1]
+                rows = sum(min(c, (window or c) + n - 1) for n, c in zip(ctx.query_lens, ctx.context_lens))
+                return (float(rows) * a[1].shape[1] * (a[1].shape[3] + a[2].shape[3]) * a[1].element_size(),
+                        2.0 * heads * (a[1].shape[3] + a[2].shape[3] + heads) * seen(ctx, window))
             if name == "rms_norm_rows":
                 return 2.0 * nbytes(a[3]), 0.0
             if name == "token_shift_mix":
