@@ -1,0 +1,503 @@
+// Attention with the heads' weights mixed after the softmax (talking_attention.cuh) on the tensor cores, bf16: prompt
+// portions and single tokens, head sizes in steps of 16 up to 128, up to 64 heads.
+//
+// A CTA owns 16 queries and up to 16 heads, a warp one head; with more heads (or more key/value heads than fit in
+// shared memory) the CTAs of a thread-block cluster own a share of the heads each and hand their weights to one
+// another through distributed shared memory, so no score is computed twice. Keys and values arrive in tiles of 16
+// positions by cp.async, two tiles in flight. First visit of the keys: every head's row maxima and sums. Second visit,
+// tile by tile:
+//   S_h = Q_h K^T (mma.sync), capped, p_h = 2^(s - lse) in 32-bit, stored as two bf16 parts (value and remainder);
+//   W = T P for all positions of the tile (mma.sync with T as the A operand, both parts of P as B: the mixed weights
+//       have 32-bit sums of 16-bit-exact products and are rounded once, where they meet the values);
+//   O_h += W_h V (mma.sync), accumulators in registers.
+// Single tokens: one row of 16 is live, the keys are cut into ranges (a launch for the maxima and sums, one for the
+// values, and the ranges' outputs added up, as in the CUDA-core form).
+#define TS_PDL_CLASS PDL_ATTENTION
+#include "talking_attention.cuh"
+
+namespace ts {
+
+constexpr int TM_ROWS = 16, TM_KEYS = 16, TM_ROWP = TM_KEYS + 8, TM_POS = TM_ROWS * TM_ROWP + 8;   // padded rows
+constexpr int TM_BOTH = 0, TM_STATS = 1, TM_VALUES = 2;
+constexpr float TM_LOG2E = 1.4426950408889634f;
+
+__device__ __forceinline__ uint32_t tm_smem(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
+__device__ __forceinline__ void tm_cp16(void* smem, const void* gmem, bool valid) {
+  const int bytes = valid ? 16 : 0;
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(tm_smem(smem)), "l"(gmem), "r"(bytes) : "memory");
+}
+__device__ __forceinline__ void tm_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+__device__ __forceinline__ void tm_wait_all() { asm volatile("cp.async.wait_group 0;" ::: "memory"); }
+__device__ __forceinline__ void tm_ldm(uint32_t (&r)[4], const void* smem) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(tm_smem(smem)) : "memory");
+}
+__device__ __forceinline__ void tm_ldm_t(uint32_t (&r)[4], const void* smem) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(tm_smem(smem)) : "memory");
+}
+__device__ __forceinline__ void tm_mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ float tm_ex2(float x) { return exp2f(x); }
+__device__ __forceinline__ uint32_t tm_pack(float a, float b) {
+  const __nv_bfloat162 v = __floats2bfloat162_rn(a, b);
+  return *reinterpret_cast<const uint32_t*>(&v);
+}
+
+template <int CL>
+__device__ __forceinline__ void tm_sync() {
+  if constexpr (CL == 1) {
+    __syncthreads();
+  } else {
+    asm volatile("barrier.cluster.arrive.release.aligned;\n\tbarrier.cluster.wait.acquire.aligned;" ::: "memory");
+  }
+}
+template <int CL>
+__device__ __forceinline__ void tm_store_all(uint32_t addr, uint32_t v) {        // to this address in every CTA of the cluster
+  if constexpr (CL == 1) {
+    asm volatile("st.shared.u32 [%0], %1;" ::"r"(addr), "r"(v) : "memory");
+  } else {
+#pragma unroll
+    for (int c = 0; c < CL; ++c) {
+      uint32_t remote;
+      asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(remote) : "r"(addr), "r"(c));
+      asm volatile("st.shared::cluster.u32 [%0], %1;" ::"r"(remote), "r"(v) : "memory");
+    }
+  }
+}
+
+// The scores of a fragment in base-2 units: scale, or scale and soft cap. tanh by its Taylor series up to the 11th
+// power while every argument of the warp is small (the next term is below 2e-8 of the value at 0.35), tanhf otherwise.
+struct CapArgs { float mul, cap2; bool capped; };    // capped: cap2 * tanh(mul * s); else mul * s
+__device__ __forceinline__ void cap_scores(float (&s)[2][4], const CapArgs& c) {
+  bool big = false;
+#pragma unroll
+  for (int n = 0; n < 2; ++n)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      s[n][e] *= c.mul;
+      big |= fabsf(s[n][e]) > 0.35f;
+    }
+  if (!c.capped) return;
+  if (__any_sync(0xffffffffu, big)) {
+#pragma unroll
+    for (int n = 0; n < 2; ++n)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) s[n][e] = c.cap2 * tanhf(s[n][e]);
+    return;
+  }
+#pragma unroll
+  for (int n = 0; n < 2; ++n)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const float x = s[n][e], u = x * x;
+      float p = fmaf(u, -1382.f / 155925.f, 62.f / 2835.f);
+      p = fmaf(u, p, -17.f / 315.f);
+      p = fmaf(u, p, 2.f / 15.f);
+      p = fmaf(u, p, -1.f / 3.f);
+      s[n][e] = c.cap2 * fmaf(x * u, p, x);
+    }
+}
+
+struct TalkMmaShape {
+  int heads_per_cta;       // <= 16: a warp each
+  int kv_per_cta;          // key/value heads a CTA's heads read, at most
+  int padded_heads;        // all heads, rounded up to 16
+};
+
+template <int KD, int KV, int CL>
+__global__ void __launch_bounds__(512) talking_mma_kernel(TalkArgs a, TalkMmaShape sh, int phase) {
+  extern __shared__ __align__(16) unsigned char raw[];
+  const int H = a.num_heads, G = a.num_kv_heads, per = H / G, D = a.head_dim, DV = a.v_head_dim;
+  const int KS = D + 8, VS = DV + 8;                       // padded row strides
+  const int Hp = sh.padded_heads;
+  const size_t k_elems = (size_t)sh.kv_per_cta * TM_KEYS * KS, v_elems = (size_t)sh.kv_per_cta * TM_KEYS * VS;
+  bf16* Ks = (bf16*)raw;                                   // [2][kv][KEYS][KS]
+  bf16* Vs = Ks + 2 * k_elems;                             // [2][kv][KEYS][VS]
+  bf16* Ps = Vs + 2 * v_elems;                             // [2 parts][Hp][TM_POS]
+  bf16* Ws = Ps + (size_t)2 * Hp * TM_POS;                 // [16][TM_POS]
+  bf16* Tm = Ws + (size_t)16 * TM_POS;                     // [16][Hp + 8]
+  __shared__ int key_rows[2][TM_KEYS];
+
+  pdl_trigger();
+  pdl_wait();
+  const int rank = CL == 1 ? 0 : (int)(blockIdx.x % CL);
+  const int seq = blockIdx.y;
+  const int row0 = a.cu_q[seq], n = a.cu_q[seq + 1] - row0;
+  const int q0 = (int)(blockIdx.x / CL) * TM_ROWS;
+  if (q0 >= n) return;                                     // the same for every CTA of a cluster
+  const int ctx = a.ctx_lens[seq];
+  const int first_pos = ctx - n + q0;
+  const int nq = min(TM_ROWS, n - q0);
+  const int last_pos = first_pos + nq - 1;
+  const int lo = a.window > 0 ? max(0, first_pos - a.window + 1) : 0;
+  const int all_tiles = (last_pos + 1 - lo + TM_KEYS - 1) / TM_KEYS;
+  const int each = (all_tiles + a.num_splits - 1) / a.num_splits;
+  const int k_begin = lo + (int)blockIdx.z * each * TM_KEYS;
+  const int k_end = min(last_pos + 1, k_begin + each * TM_KEYS);
+  const int tiles = max(0, (k_end - k_begin + TM_KEYS - 1) / TM_KEYS);
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, threads = blockDim.x;
+  const int head0 = rank * sh.heads_per_cta, my_heads = min(sh.heads_per_cta, H - head0);
+  const int kv0 = head0 / per, my_kv = my_heads > 0 ? (head0 + my_heads - 1) / per - kv0 + 1 : 0;
+  const int head = head0 + warp;
+  const bool has_head = warp < my_heads;
+  const int my_g = has_head ? head / per - kv0 : 0;
+  const int* table = a.block_tables + (size_t)seq * a.table_width;
+  const bf16* kc = (const bf16*)a.k_cache;
+  const bf16* vc = (const bf16*)a.v_cache;
+  const int r = lane >> 2, c2 = (lane & 3) * 2;            // this lane's rows r, r + 8 and columns c2, c2 + 1 of a fragment
+
+  // this warp's queries as A fragments
+  uint32_t qf[KD][4];
+#pragma unroll
+  for (int kk = 0; kk < KD; ++kk)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int row = r + (j & 1) * 8, col = kk * 16 + c2 + (j >> 1) * 8;
+      qf[kk][j] = 0u;
+      if (has_head && row < nq && kk * 16 < D)
+        qf[kk][j] = *reinterpret_cast<const uint32_t*>((const bf16*)a.q + ((size_t)(row0 + q0 + row) * H + head) * D + col);
+    }
+  if (phase != TM_STATS) {
+    for (int idx = tid; idx < 16 * Hp; idx += threads) {
+      const int h = idx / Hp, g = idx - h * Hp;
+      float t = 0.f;
+      if (head0 + h < H && h < my_heads && g < H) t = a.talk ? a.talk[(size_t)(head0 + h) * H + g] : (g == head0 + h ? 1.f : 0.f);
+      Tm[h * (Hp + 8) + g] = __float2bfloat16_rn(t);
+    }
+    // rows of P of no head (H not a multiple of 16) stay zero
+    for (int idx = tid; idx < 2 * (Hp - H) * TM_POS; idx += threads) {
+      const int part = idx / ((Hp - H) * TM_POS), rest = idx - part * (Hp - H) * TM_POS;
+      Ps[((size_t)part * Hp + H) * TM_POS + rest] = __float2bfloat16_rn(0.f);
+    }
+  }
+  auto find_rows = [&](int t) {                            // the cache rows of tile t (-1: no such key), in units of kv head 0
+    if (tid < TM_KEYS) {
+      const int kpos = k_begin + t * TM_KEYS + tid;
+      key_rows[t & 1][tid] = t < tiles && kpos < k_end ? (int)talk_row(table, kpos, 0, a) : -1;
+    }
+  };
+  auto load_rows = [&](bf16* dst, const bf16* src, int t, int width, int stride) {
+    const int chunks = width >> 3, total = my_kv * TM_KEYS * chunks;
+    for (int idx = tid; idx < total; idx += threads) {
+      const int line = idx / chunks, ch = idx - line * chunks;
+      const int key = line & (TM_KEYS - 1), g = line / TM_KEYS;
+      const int row = key_rows[t & 1][key];
+      const size_t off = row < 0 ? 0 : ((size_t)row + (size_t)(kv0 + g) * a.page_size) * width + ch * 8;
+      tm_cp16(dst + (size_t)line * stride + ch * 8, src + off, row >= 0);
+    }
+  };
+  CapArgs cap;
+  cap.capped = a.softcap > 0.f;
+  cap.mul = cap.capped ? a.scale / a.softcap : a.scale * TM_LOG2E;
+  cap.cap2 = a.softcap * TM_LOG2E;
+
+  // the scores of this warp's head for tile t, in base-2 units, minus infinity where a row does not see the key
+  auto scores = [&](float (&s)[2][4], int t) {
+#pragma unroll
+    for (int j = 0; j < 2; ++j)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) s[j][e] = 0.f;
+    const bf16* kb = Ks + (size_t)(t & 1) * k_elems + ((size_t)my_g * TM_KEYS + (lane & 7) + ((lane >> 4) << 3)) * KS + ((lane >> 3) & 1) * 8;
+#pragma unroll
+    for (int kk = 0; kk < KD; ++kk) {
+      if (kk * 16 < D) {
+        uint32_t b[4];
+        tm_ldm(b, kb + kk * 16);
+        tm_mma(s[0], qf[kk], b[0], b[1]);
+        tm_mma(s[1], qf[kk], b[2], b[3]);
+      }
+    }
+    cap_scores(s, cap);
+    const int k0 = k_begin + t * TM_KEYS;
+    // the whole tile is seen by every row: no mask
+    if (k0 + TM_KEYS - 1 <= first_pos && k0 + TM_KEYS <= k_end && (a.window <= 0 || k0 > last_pos - a.window)) return;
+#pragma unroll
+    for (int j = 0; j < 2; ++j)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int kpos = k0 + j * 8 + c2 + (e & 1), qpos = first_pos + r + (e >> 1) * 8;
+        if (!(kpos < k_end && kpos <= qpos && (a.window <= 0 || kpos > qpos - a.window))) s[j][e] = -INFINITY;
+      }
+  };
+
+  float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
+  find_rows(0);
+  find_rows(1);
+  __syncthreads();
+  if (phase != TM_VALUES) {
+    if (tiles > 0) load_rows(Ks, kc, 0, D, KS);
+    tm_commit();
+    for (int t = 0; t < tiles; ++t) {
+      tm_wait_all();
+      __syncthreads();                                     // tile t has arrived, and nobody reads the other buffer any more
+      if (t + 1 < tiles) load_rows(Ks + (size_t)((t + 1) & 1) * k_elems, kc, t + 1, D, KS);
+      tm_commit();
+      find_rows(t + 2);                                    // in the place of tile t's, whose last reader was a step ago
+      if (has_head) {
+        float s[2][4];
+        scores(s, t);
+#pragma unroll
+        for (int half = 0; half < 2; ++half) {
+          float mx = fmaxf(fmaxf(s[0][half * 2], s[0][half * 2 + 1]), fmaxf(s[1][half * 2], s[1][half * 2 + 1]));
+          mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
+          mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
+          const float mn = fmaxf(m[half], mx);
+          if (mn != -INFINITY) {
+            float sum = 0.f;
+#pragma unroll
+            for (int j = 0; j < 2; ++j) sum += tm_ex2(s[j][half * 2] - mn) + tm_ex2(s[j][half * 2 + 1] - mn);
+            l[half] = l[half] * tm_ex2(m[half] - mn) + sum;
+            m[half] = mn;
+          }
+        }
+      }
+    }
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+      l[half] += __shfl_xor_sync(0xffffffffu, l[half], 1);
+      l[half] += __shfl_xor_sync(0xffffffffu, l[half], 2);
+    }
+    if (phase == TM_STATS) {
+      if (has_head && (lane & 3) == 0)
+#pragma unroll
+        for (int half = 0; half < 2; ++half)
+          if (r + half * 8 < nq) {
+            float* ml = a.part_ml + (((size_t)(row0 + q0 + r + half * 8) * H + head) * a.num_splits + blockIdx.z) * 2;
+            ml[0] = m[half];
+            ml[1] = l[half];
+          }
+      return;
+    }
+  } else if (has_head) {
+#pragma unroll
+    for (int half = 0; half < 2; ++half)
+      if (r + half * 8 < nq) {
+        const float* ml = a.part_ml + ((size_t)(row0 + q0 + r + half * 8) * H + head) * a.num_splits * 2;
+        for (int s = 0; s < a.num_splits; ++s) m[half] = fmaxf(m[half], ml[2 * s]);
+        for (int s = 0; s < a.num_splits; ++s)
+          if (ml[2 * s] != -INFINITY) l[half] += ml[2 * s + 1] * tm_ex2(ml[2 * s] - m[half]);
+      }
+  }
+  // the logarithm of each row's denominator; rows that see nothing (none that is stored) get weights of zero
+  float lse[2];
+#pragma unroll
+  for (int half = 0; half < 2; ++half) {
+    if (a.sinks && has_head) {
+      const float sink = a.sinks[head] * TM_LOG2E, top = fmaxf(m[half], sink);
+      l[half] = (m[half] == -INFINITY ? 0.f : l[half] * tm_ex2(m[half] - top)) + tm_ex2(sink - top);
+      m[half] = top;
+    }
+    lse[half] = l[half] > 0.f ? m[half] + log2f(l[half]) : INFINITY;
+  }
+
+  float o[KV * 2][4];
+#pragma unroll
+  for (int j = 0; j < KV * 2; ++j)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) o[j][e] = 0.f;
+  __syncthreads();
+  find_rows(0);
+  find_rows(1);
+  tm_sync<CL>();                                           // every CTA of the cluster is here before the first remote store
+  if (tiles > 0) {
+    load_rows(Ks, kc, 0, D, KS);
+    load_rows(Vs, vc, 0, DV, VS);
+  }
+  tm_commit();
+  const int warps = threads >> 5;
+  for (int t = 0; t < tiles; ++t) {
+    tm_wait_all();
+    __syncthreads();                                       // tile t has arrived, and nobody reads the other buffers any more
+    if (t + 1 < tiles) {
+      load_rows(Ks + (size_t)((t + 1) & 1) * k_elems, kc, t + 1, D, KS);
+      load_rows(Vs + (size_t)((t + 1) & 1) * v_elems, vc, t + 1, DV, VS);
+    }
+    tm_commit();
+    if (has_head) {
+      float s[2][4];
+      scores(s, t);
+#pragma unroll
+      for (int half = 0; half < 2; ++half) {
+        const uint32_t at = tm_smem(Ps + (size_t)head * TM_POS + (r + half * 8) * TM_ROWP + c2);
+#pragma unroll
+        for (int j = 0; j < 2; ++j) {
+          const float p0 = tm_ex2(s[j][half * 2] - lse[half]), p1 = tm_ex2(s[j][half * 2 + 1] - lse[half]);
+          const uint32_t hi = tm_pack(p0, p1);
+          const uint32_t rem = tm_pack(p0 - __uint_as_float(hi << 16), p1 - __uint_as_float(hi & 0xffff0000u));
+          tm_store_all<CL>(at + j * 16, hi);
+          tm_store_all<CL>(at + j * 16 + (uint32_t)(Hp * TM_POS * 2), rem);
+        }
+      }
+    }
+    tm_sync<CL>();
+    find_rows(t + 2);
+    // mixed weights of this CTA's heads: a query row of the tile per turn
+    for (int i = warp; i < TM_ROWS; i += warps) {
+      float w[2][4];
+#pragma unroll
+      for (int j = 0; j < 2; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) w[j][e] = 0.f;
+      for (int g0 = 0; g0 < Hp; g0 += 16) {
+        uint32_t tf[4], b[4];
+        tm_ldm(tf, Tm + (size_t)(lane & 15) * (Hp + 8) + g0 + (lane >> 4) * 8);
+        const bf16* pb = Ps + (size_t)(g0 + (lane & 7) + ((lane >> 3) & 1) * 8) * TM_POS + i * TM_ROWP + (lane >> 4) * 8;
+        tm_ldm_t(b, pb);
+        tm_mma(w[0], tf, b[0], b[1]);
+        tm_mma(w[1], tf, b[2], b[3]);
+        tm_ldm_t(b, pb + (size_t)Hp * TM_POS);
+        tm_mma(w[0], tf, b[0], b[1]);
+        tm_mma(w[1], tf, b[2], b[3]);
+      }
+#pragma unroll
+      for (int j = 0; j < 2; ++j) {
+        uint32_t* at = reinterpret_cast<uint32_t*>(Ws + (size_t)r * TM_POS + i * TM_ROWP + j * 8 + c2);
+        at[0] = tm_pack(w[j][0], w[j][1]);
+        at[(size_t)8 * TM_POS / 2] = tm_pack(w[j][2], w[j][3]);
+      }
+    }
+    tm_sync<CL>();
+    if (has_head) {
+      uint32_t wf[4];
+      tm_ldm(wf, Ws + (size_t)warp * TM_POS + (lane & 15) * TM_ROWP + (lane >> 4) * 8);
+      const bf16* vb = Vs + (size_t)(t & 1) * v_elems + ((size_t)my_g * TM_KEYS + (lane & 7) + ((lane >> 3) & 1) * 8) * VS + (lane >> 4) * 8;
+#pragma unroll
+      for (int j = 0; j < KV; ++j) {
+        if (j * 16 < DV) {
+          uint32_t b[4];
+          tm_ldm_t(b, vb + j * 16);
+          tm_mma(o[2 * j], wf, b[0], b[1]);
+          tm_mma(o[2 * j + 1], wf, b[2], b[3]);
+        }
+      }
+    }
+  }
+  if (has_head) {
+#pragma unroll
+    for (int j = 0; j < KV * 2; ++j) {
+      if (j * 8 < DV) {
+#pragma unroll
+        for (int half = 0; half < 2; ++half) {
+          const int row = r + half * 8;
+          if (row < nq) {
+            const size_t t = (size_t)(row0 + q0 + row);
+            const int col = head * DV + j * 8 + c2;
+            if (a.num_splits == 1)
+              *reinterpret_cast<uint32_t*>((bf16*)a.out + t * H * DV + col) = tm_pack(o[j][half * 2], o[j][half * 2 + 1]);
+            else
+              *reinterpret_cast<float2*>(a.part_out + (t * a.num_splits + blockIdx.z) * H * DV + col) =
+                  make_float2(o[j][half * 2], o[j][half * 2 + 1]);
+          }
+        }
+      }
+    }
+  }
+}
+
+__global__ void talking_mma_combine_kernel(const float* part, bf16* out, int splits, int width, size_t total) {
+  pdl_trigger();
+  pdl_wait();
+  for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < total; idx += (size_t)gridDim.x * blockDim.x) {
+    const size_t t = idx / width, c = idx - t * width;
+    float o = 0.f;
+    for (int s = 0; s < splits; ++s) o += part[(t * splits + s) * width + c];
+    out[idx] = __float2bfloat16_rn(o);
+  }
+}
+
+// How a cluster shares the heads: as few CTAs as hold 16 heads each and whose keys and values fit in shared memory.
+static bool talk_mma_shape(int H, int G, int D, int DV, TalkMmaShape& sh, int& cluster, size_t& smem) {
+  constexpr size_t LIMIT = 226 * 1024;
+  const int per = H / G;
+  sh.padded_heads = (H + 15) / 16 * 16;
+  if (sh.padded_heads > 64) return false;
+  for (cluster = 1; cluster <= 4; cluster *= 2) {
+    const int hc = (H + cluster - 1) / cluster;
+    if (hc > 16) continue;
+    int kv = 0;
+    for (int c = 0; c < cluster; ++c) {
+      const int h0 = c * hc, hn = H - h0 < hc ? H - h0 : hc;
+      if (hn > 0 && (h0 + hn - 1) / per - h0 / per + 1 > kv) kv = (h0 + hn - 1) / per - h0 / per + 1;
+    }
+    sh.heads_per_cta = hc;
+    sh.kv_per_cta = kv;
+    smem = sizeof(bf16) * (2 * (size_t)kv * TM_KEYS * (D + 8 + DV + 8) + (size_t)2 * sh.padded_heads * TM_POS + (size_t)16 * TM_POS +
+                           (size_t)16 * (sh.padded_heads + 8));
+    if (smem <= LIMIT) return true;
+  }
+  return false;
+}
+
+template <int KD, int KV, int CL>
+static int launch_talk_mma(const TalkArgs& a, const TalkMmaShape& sh, size_t smem, int num_seqs, int max_query_len, int phase,
+                           cudaStream_t stream) {
+  auto kern = talking_mma_kernel<KD, KV, CL>;
+  static size_t allowed = 0;
+  if (smem > 48 * 1024 && smem > allowed) {
+    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return (int)e;
+    allowed = smem;
+  }
+  const dim3 grid((unsigned)((max_query_len + TM_ROWS - 1) / TM_ROWS * CL), num_seqs, a.num_splits);
+  const int threads = sh.heads_per_cta * 32;
+  if constexpr (CL == 1) return launch(kern, grid, threads, smem, stream, a, sh, phase);
+  else return launch_cluster(kern, grid, dim3(threads), smem, stream, dim3(CL, 1, 1), a, sh, phase);
+}
+
+template <int KD, int KV>
+static int launch_talk_mma_cl(const TalkArgs& a, const TalkMmaShape& sh, int cluster, size_t smem, int num_seqs, int max_query_len,
+                              int phase, cudaStream_t stream) {
+  if (cluster == 1) return launch_talk_mma<KD, KV, 1>(a, sh, smem, num_seqs, max_query_len, phase, stream);
+  if (cluster == 2) return launch_talk_mma<KD, KV, 2>(a, sh, smem, num_seqs, max_query_len, phase, stream);
+  return launch_talk_mma<KD, KV, 4>(a, sh, smem, num_seqs, max_query_len, phase, stream);
+}
+
+}  // namespace ts
+
+using namespace ts;
+
+extern "C" int ts_talking_attention_mma_takes(int heads, int kv_heads, int d, int dv) {
+  TalkMmaShape sh;
+  int cluster;
+  size_t smem;
+  if (heads <= 0 || kv_heads <= 0 || heads % kv_heads || d <= 0 || dv <= 0 || d % 16 || dv % 16 || d > 128 || dv > 128) return 0;
+  return talk_mma_shape(heads, kv_heads, d, dv, sh, cluster, smem) ? cluster : 0;
+}
+
+// As ts_talking_attention, bf16 only; pages * kv_heads * page_size must stay below 2^31. talk is used as bf16.
+extern "C" int ts_talking_attention_mma(const void* q, void* out, const void* k_cache, const void* v_cache, const int* block_tables,
+                                        int table_width, const int* cu_q, const int* ctx_lens, int num_seqs, int max_query_len,
+                                        int num_tokens, int heads, int kv_heads, int d, int dv, int page_size, float scale,
+                                        int window, float softcap, const float* talk, const float* sinks, int num_splits,
+                                        float* part_ml, float* part_out, cudaStream_t stream) {
+  if (num_seqs <= 0 || num_tokens <= 0) return 0;
+  if (heads <= 0 || kv_heads <= 0 || heads % kv_heads || page_size <= 0 || max_query_len <= 0 || window < 0) return TS_ERR_BAD_ARGUMENT;
+  if (num_splits < 1 || (num_splits > 1 && (!part_ml || !part_out))) return TS_ERR_BAD_ARGUMENT;
+  if (((uintptr_t)q | (uintptr_t)k_cache | (uintptr_t)v_cache | (uintptr_t)out) & 15) return TS_ERR_UNSUPPORTED;
+  TalkMmaShape sh;
+  int cluster;
+  size_t smem;
+  if (!ts_talking_attention_mma_takes(heads, kv_heads, d, dv) || !talk_mma_shape(heads, kv_heads, d, dv, sh, cluster, smem))
+    return TS_ERR_UNSUPPORTED;
+  TalkArgs a;
+  a.q = q; a.out = out; a.k_cache = k_cache; a.v_cache = v_cache; a.block_tables = block_tables; a.table_width = table_width;
+  a.cu_q = cu_q; a.ctx_lens = ctx_lens; a.num_heads = heads; a.num_kv_heads = kv_heads; a.head_dim = d; a.v_head_dim = dv;
+  a.page_size = page_size; a.page_shift = page_shift_of(page_size); a.scale = scale; a.window = window; a.softcap = softcap;
+  a.talk = talk; a.sinks = sinks; a.num_splits = num_splits; a.part_ml = part_ml; a.part_out = part_out;
+  auto run = [&](int phase) {
+    if (d <= 64 && dv <= 64) return launch_talk_mma_cl<4, 4>(a, sh, cluster, smem, num_seqs, max_query_len, phase, stream);
+    return launch_talk_mma_cl<8, 8>(a, sh, cluster, smem, num_seqs, max_query_len, phase, stream);
+  };
+  if (num_splits == 1) return run(TM_BOTH);
+  if (int e = run(TM_STATS)) return e;
+  if (int e = run(TM_VALUES)) return e;
+  const int width = heads * dv;
+  const size_t total = (size_t)num_tokens * width;
+  size_t blocks = (total + 255) / 256;
+  if (blocks > 148 * 16) blocks = 148 * 16;
+  return launch(talking_mma_combine_kernel, (unsigned)blocks, 256, 0, stream, (const float*)part_out, (bf16*)out, num_splits, width, total);
+}

@@ -60,6 +60,9 @@ _SIGNATURES: dict[str, list[Any]] = {
                       _i, _i, _vp],
     "ts_talking_attention": [_vp, _vp, _vp, _vp, _vp, _i, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _f, _i, _f, _vp, _vp, _i, _vp, _vp,
                              _i, _vp],
+    "ts_talking_attention_mma": [_vp, _vp, _vp, _vp, _vp, _i, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _f, _i, _f, _vp, _vp, _i, _vp,
+                                 _vp, _vp],
+    "ts_talking_attention_mma_takes": [_i, _i, _i, _i],
     "ts_prefill_attention_mma": [_vp, _vp, _vp, _vp, _vp, _i, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _f, _i, _vp],
     "ts_decode_attention_mma": [_vp, _vp, _vp, _vp, _vp, _i, _vp, _vp, _vp, _i, _i, _i, _i, _i, _f, _i, _i, _vp, _vp,
                                 _vp, _vp],
@@ -1588,14 +1591,27 @@ def qkv_rotate(proj: torch.Tensor, taps: torch.Tensor | None, state: torch.Tenso
 
 
 # ------------------------------------- attention with weights mixed across the heads
-TALKING_MAX_SPLITS = 16
-TALKING_MIN_KEYS_PER_SPLIT = 64
+TALKING_TENSOR_CORES = True       # bf16 at sizes the mma.sync form takes; False: CUDA cores always
+TALKING_MAX_SPLITS = 32
+TALKING_MIN_KEYS_PER_SPLIT = 32
 
 
-def talking_splits(num_seqs: int, keys: int) -> int:
-    """Key ranges per request for a step of single tokens: enough CTAs to give every SM one, no range shorter than
-    64 keys. Depends only on the step's shape."""
-    return max(1, min(SM_COUNT // max(1, num_seqs), keys // TALKING_MIN_KEYS_PER_SPLIT, TALKING_MAX_SPLITS))
+def talking_splits(ctas: int, keys: int) -> int:
+    """Key ranges per request for a step of single tokens that would launch ``ctas`` CTAs unsplit: enough to give every
+    SM one, no range shorter than 32 keys. Depends only on the step's shape."""
+    return max(1, min(SM_COUNT // max(1, ctas), keys // TALKING_MIN_KEYS_PER_SPLIT, TALKING_MAX_SPLITS))
+
+
+_talking_clusters: dict[tuple[int, int, int, int], int] = {}
+
+
+def talking_cluster(heads: int, kv_heads: int, d: int, dv: int) -> int:
+    """CTAs that share the heads of a query tile in the mma.sync form (0: it does not take these sizes)."""
+    key = (heads, kv_heads, d, dv)
+    n = _talking_clusters.get(key)
+    if n is None:
+        n = _talking_clusters[key] = int(_fn("ts_talking_attention_mma_takes")(*key))
+    return n
 
 
 def talking_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, page_size: int, block_tables: torch.Tensor,
@@ -1603,7 +1619,9 @@ def talking_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Ten
                       sinks: torch.Tensor | None = None) -> None:
     """Causal attention (``window`` 0: all earlier positions) with optionally capped scores ``cap tanh(s / cap)`` and
     the heads' weights mixed behind the softmax: ``w_h = sum_g talk[h, g] p_g`` (``talk [Hq, Hq]`` float32 or None), each
-    head applying its mixed weights to the values of its own key/value head. Shapes as for :func:`paged_attention`."""
+    head applying its mixed weights to the values of its own key/value head. Shapes as for :func:`paged_attention`.
+    bf16 at head sizes in steps of 16 up to 128 and up to 64 heads runs on the tensor cores (there ``talk`` is used as
+    bf16, which it is in a bf16 model)."""
     t, hq, d = q.shape
     hkv, dv, dt = k_cache.shape[1], v_cache.shape[3], q.dtype
     if k_cache.dtype != dt or v_cache.dtype != dt or out.dtype != dt or out.numel() != t * hq * dv or hq % hkv:
@@ -1619,19 +1637,26 @@ def talking_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Ten
     if softcap is not None and not softcap > 0:
         raise KernelError("talking_attention: softcap must be positive or None")
     _check_indices("talking_attention", block_tables, ctx, page_size, k_cache.shape[0])
+    cluster = 0
+    if TALKING_TENSOR_CORES and dt == torch.bfloat16 and k_cache.shape[0] * hkv * page_size < 2 ** 31:
+        cluster = talking_cluster(hq, hkv, d, dv)
     splits, part_ml, part_out = 1, None, None
     if ctx.max_query_len == 1:
-        splits = talking_splits(ctx.num_seqs, min(ctx.max_context_len, window) if window else ctx.max_context_len)
+        splits = talking_splits(ctx.num_seqs * max(cluster, 1), min(ctx.max_context_len, window) if window else ctx.max_context_len)
         if splits > 1:
             part_ml = ctx.arena.take((t, hq, splits, 2), torch.float32)
             part_out = ctx.arena.take((t, splits, hq * dv), torch.float32)
-    _check(_fn("ts_talking_attention")(
+    args = (
         _dev(q, "q"), _dev(out, "out"), _dev(k_cache, "k_cache"), _dev(v_cache, "v_cache"),
         _dev(block_tables, "block_tables", torch.int32), block_tables.shape[1],
         _dev(ctx.cu_query_lens, "cu_query_lens", torch.int32), _dev(ctx.context_lens_dev, "context_lens", torch.int32),
         ctx.num_seqs, ctx.max_query_len, t, hq, hkv, d, dv, page_size, float(scale), int(window), float(softcap or 0.0),
         _opt(talk, "talk", torch.float32), _opt(sinks, "sinks", torch.float32), splits, _opt(part_ml, "part_ml"),
-        _opt(part_out, "part_out"), _code(dt), _stream()), "talking_attention", kernels=3 if splits > 1 else 1)
+        _opt(part_out, "part_out"))
+    if cluster:
+        _check(_fn("ts_talking_attention_mma")(*args, _stream()), "talking_attention_mma", kernels=3 if splits > 1 else 1)
+    else:
+        _check(_fn("ts_talking_attention")(*args, _code(dt), _stream()), "talking_attention", kernels=3 if splits > 1 else 1)
 
 
 # ------------------------------------------------------------- latent attention
