@@ -22,10 +22,6 @@ constexpr int TM_BOTH = 0, TM_STATS = 1, TM_VALUES = 2;
 constexpr float TM_LOG2E = 1.4426950408889634f;
 
 __device__ __forceinline__ uint32_t tm_smem(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
-__device__ __forceinline__ void tm_cp16(void* smem, const void* gmem, bool valid) {
-  const int bytes = valid ? 16 : 0;
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(tm_smem(smem)), "l"(gmem), "r"(bytes) : "memory");
-}
 __device__ __forceinline__ void tm_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
 __device__ __forceinline__ void tm_wait_all() { asm volatile("cp.async.wait_group 0;" ::: "memory"); }
 __device__ __forceinline__ void tm_ldm(uint32_t (&r)[4], const void* smem) {
@@ -41,7 +37,11 @@ __device__ __forceinline__ void tm_mma(float (&c)[4], const uint32_t (&a)[4], ui
                : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
                : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
-__device__ __forceinline__ float tm_ex2(float x) { return exp2f(x); }
+__device__ __forceinline__ float tm_ex2(float x) {         // arguments are at most 0, or small: no range handling
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
 __device__ __forceinline__ uint32_t tm_pack(float a, float b) {
   const __nv_bfloat162 v = __floats2bfloat162_rn(a, b);
   return *reinterpret_cast<const uint32_t*>(&v);
@@ -180,16 +180,26 @@ __global__ void __launch_bounds__(512) talking_mma_kernel(TalkArgs a, TalkMmaSha
       key_rows[t & 1][tid] = t < tiles && kpos < k_end ? (int)talk_row(table, kpos, 0, a) : -1;
     }
   };
-  auto load_rows = [&](bf16* dst, const bf16* src, int t, int width, int stride) {
-    const int chunks = width >> 3, total = my_kv * TM_KEYS * chunks;
-    for (int idx = tid; idx < total; idx += threads) {
-      const int line = idx / chunks, ch = idx - line * chunks;
-      const int key = line & (TM_KEYS - 1), g = line / TM_KEYS;
-      const int row = key_rows[t & 1][key];
-      const size_t off = row < 0 ? 0 : ((size_t)row + (size_t)(kv0 + g) * a.page_size) * width + ch * 8;
-      tm_cp16(dst + (size_t)line * stride + ch * 8, src + off, row >= 0);
+  // A tile's keys (or values): a line is one key of one head, `width` elements; a thread keeps its 16-byte piece of
+  // a line and goes from line to line.
+  const int k_pieces = D >> 3, v_pieces = DV >> 3, lines = my_kv * TM_KEYS;
+  const int k_step = threads / k_pieces, v_step = threads / v_pieces;
+  const int k_line = tid / k_pieces < k_step ? tid / k_pieces : lines, k_ch = (tid % k_pieces) * 8;
+  const int v_line = tid / v_pieces < v_step ? tid / v_pieces : lines, v_ch = (tid % v_pieces) * 8;
+  const int g_rows = a.page_size;                          // rows from one key/value head to the next inside a page
+  auto load_rows = [&](bf16* dst, const bf16* src, int t, int width, int stride, int line0, int step, int ch) {
+    const int* rows = key_rows[t & 1];
+    uint32_t to = tm_smem(dst) + (uint32_t)((line0 * stride + ch) * 2);
+    const uint32_t to_step = (uint32_t)(step * stride * 2);
+    for (int line = line0; line < lines; line += step, to += to_step) {
+      const int row = rows[line & (TM_KEYS - 1)];
+      const int at = row < 0 ? 0 : row + (kv0 + (line >> 4)) * g_rows;
+      const bf16* from = src + (size_t)at * width + ch;
+      asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(to), "l"(from), "r"(row < 0 ? 0 : 16) : "memory");
     }
   };
+  auto load_keys = [&](int t) { load_rows(Ks + (size_t)(t & 1) * k_elems, kc, t, D, KS, k_line, k_step, k_ch); };
+  auto load_values = [&](int t) { load_rows(Vs + (size_t)(t & 1) * v_elems, vc, t, DV, VS, v_line, v_step, v_ch); };
   CapArgs cap;
   cap.capped = a.softcap > 0.f;
   cap.mul = cap.capped ? a.scale / a.softcap : a.scale * TM_LOG2E;
@@ -224,22 +234,31 @@ __global__ void __launch_bounds__(512) talking_mma_kernel(TalkArgs a, TalkMmaSha
       }
   };
 
+  // Capped scores cannot leave +-cap: their exponentials are summed as they are, without a running maximum.
+  const bool bounded = cap.capped && cap.cap2 <= 64.f;
   float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
+  if (bounded && phase != TM_VALUES) m[0] = m[1] = 0.f;
   find_rows(0);
   find_rows(1);
   __syncthreads();
   if (phase != TM_VALUES) {
-    if (tiles > 0) load_rows(Ks, kc, 0, D, KS);
+    if (tiles > 0) load_keys(0);
     tm_commit();
     for (int t = 0; t < tiles; ++t) {
       tm_wait_all();
       __syncthreads();                                     // tile t has arrived, and nobody reads the other buffer any more
-      if (t + 1 < tiles) load_rows(Ks + (size_t)((t + 1) & 1) * k_elems, kc, t + 1, D, KS);
+      if (t + 1 < tiles) load_keys(t + 1);
       tm_commit();
       find_rows(t + 2);                                    // in the place of tile t's, whose last reader was a step ago
       if (has_head) {
         float s[2][4];
         scores(s, t);
+        if (bounded) {
+#pragma unroll
+          for (int half = 0; half < 2; ++half)
+            l[half] += (tm_ex2(s[0][half * 2]) + tm_ex2(s[0][half * 2 + 1])) + (tm_ex2(s[1][half * 2]) + tm_ex2(s[1][half * 2 + 1]));
+          continue;
+        }
 #pragma unroll
         for (int half = 0; half < 2; ++half) {
           float mx = fmaxf(fmaxf(s[0][half * 2], s[0][half * 2 + 1]), fmaxf(s[1][half * 2], s[1][half * 2 + 1]));
@@ -304,8 +323,8 @@ __global__ void __launch_bounds__(512) talking_mma_kernel(TalkArgs a, TalkMmaSha
   find_rows(1);
   tm_sync<CL>();                                           // every CTA of the cluster is here before the first remote store
   if (tiles > 0) {
-    load_rows(Ks, kc, 0, D, KS);
-    load_rows(Vs, vc, 0, DV, VS);
+    load_keys(0);
+    load_values(0);
   }
   tm_commit();
   const int warps = threads >> 5;
@@ -313,8 +332,8 @@ __global__ void __launch_bounds__(512) talking_mma_kernel(TalkArgs a, TalkMmaSha
     tm_wait_all();
     __syncthreads();                                       // tile t has arrived, and nobody reads the other buffers any more
     if (t + 1 < tiles) {
-      load_rows(Ks + (size_t)((t + 1) & 1) * k_elems, kc, t + 1, D, KS);
-      load_rows(Vs + (size_t)((t + 1) & 1) * v_elems, vc, t + 1, DV, VS);
+      load_keys(t + 1);
+      load_values(t + 1);
     }
     tm_commit();
     if (has_head) {
