@@ -22,8 +22,8 @@ constexpr int TM_BOTH = 0, TM_STATS = 1, TM_VALUES = 2;
 constexpr float TM_LOG2E = 1.4426950408889634f;
 
 __device__ __forceinline__ uint32_t tm_smem(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
-__device__ __forceinline__ void tm_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-__device__ __forceinline__ void tm_wait_all() { asm volatile("cp.async.wait_group 0;" ::: "memory"); }
+template <int N>                                           // all but this thread's last N groups of copies have arrived
+__device__ __forceinline__ void tm_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 __device__ __forceinline__ void tm_ldm(uint32_t (&r)[4], const void* smem) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
                : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(tm_smem(smem)) : "memory");
@@ -71,35 +71,57 @@ __device__ __forceinline__ void tm_store_all(uint32_t addr, uint32_t v) {       
 
 // The scores of a fragment in base-2 units: scale, or scale and soft cap. tanh by its Taylor series up to the 11th
 // power while every argument of the warp is small (the next term is below 2e-8 of the value at 0.35), tanhf otherwise.
+// Two elements an instruction (packed 32-bit arithmetic).
 struct CapArgs { float mul, cap2; bool capped; };    // capped: cap2 * tanh(mul * s); else mul * s
+__device__ __forceinline__ uint64_t tm_two(float a, float b) {
+  uint64_t r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
+  return r;
+}
+__device__ __forceinline__ void tm_split(uint64_t v, float& a, float& b) { asm("mov.b64 {%0, %1}, %2;" : "=f"(a), "=f"(b) : "l"(v)); }
+__device__ __forceinline__ uint64_t tm_fma2(uint64_t a, uint64_t b, uint64_t c) {
+  uint64_t r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+  return r;
+}
+__device__ __forceinline__ uint64_t tm_mul2(uint64_t a, uint64_t b) {
+  uint64_t r;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
 __device__ __forceinline__ void cap_scores(float (&s)[2][4], const CapArgs& c) {
-  bool big = false;
+  const uint64_t mul = tm_two(c.mul, c.mul);
+  uint64_t x[4];
+  float most = 0.f;
 #pragma unroll
-  for (int n = 0; n < 2; ++n)
-#pragma unroll
-    for (int e = 0; e < 4; ++e) {
-      s[n][e] *= c.mul;
-      big |= fabsf(s[n][e]) > 0.35f;
-    }
+  for (int p = 0; p < 4; ++p) {
+    x[p] = tm_mul2(tm_two(s[p >> 1][(p & 1) * 2], s[p >> 1][(p & 1) * 2 + 1]), mul);
+    float x0, x1;
+    tm_split(x[p], x0, x1);
+    most = fmaxf(most, fmaxf(fabsf(x0), fabsf(x1)));
+    s[p >> 1][(p & 1) * 2] = x0;
+    s[p >> 1][(p & 1) * 2 + 1] = x1;
+  }
   if (!c.capped) return;
-  if (__any_sync(0xffffffffu, big)) {
+  if (__any_sync(0xffffffffu, !(most <= 0.35f))) {
 #pragma unroll
     for (int n = 0; n < 2; ++n)
 #pragma unroll
       for (int e = 0; e < 4; ++e) s[n][e] = c.cap2 * tanhf(s[n][e]);
     return;
   }
+  const uint64_t cap2 = tm_two(c.cap2, c.cap2);
+  const uint64_t c11 = tm_two(-1382.f / 155925.f, -1382.f / 155925.f), c9 = tm_two(62.f / 2835.f, 62.f / 2835.f),
+                 c7 = tm_two(-17.f / 315.f, -17.f / 315.f), c5 = tm_two(2.f / 15.f, 2.f / 15.f), c3 = tm_two(-1.f / 3.f, -1.f / 3.f);
 #pragma unroll
-  for (int n = 0; n < 2; ++n)
-#pragma unroll
-    for (int e = 0; e < 4; ++e) {
-      const float x = s[n][e], u = x * x;
-      float p = fmaf(u, -1382.f / 155925.f, 62.f / 2835.f);
-      p = fmaf(u, p, -17.f / 315.f);
-      p = fmaf(u, p, 2.f / 15.f);
-      p = fmaf(u, p, -1.f / 3.f);
-      s[n][e] = c.cap2 * fmaf(x * u, p, x);
-    }
+  for (int p = 0; p < 4; ++p) {
+    const uint64_t u = tm_mul2(x[p], x[p]), y = tm_mul2(x[p], cap2);
+    uint64_t q = tm_fma2(u, c11, c9);
+    q = tm_fma2(u, q, c7);
+    q = tm_fma2(u, q, c5);
+    q = tm_fma2(u, q, c3);
+    tm_split(tm_fma2(tm_mul2(y, u), q, y), s[p >> 1][(p & 1) * 2], s[p >> 1][(p & 1) * 2 + 1]);
+  }
 }
 
 struct TalkMmaShape {
@@ -120,7 +142,7 @@ __global__ void __launch_bounds__(512) talking_mma_kernel(TalkArgs a, TalkMmaSha
   bf16* Ps = Vs + 2 * v_elems;                             // [2 parts][Hp][TM_POS]
   bf16* Ws = Ps + (size_t)2 * Hp * TM_POS;                 // [16][TM_POS]
   bf16* Tm = Ws + (size_t)16 * TM_POS;                     // [16][Hp + 8]
-  __shared__ int key_rows[2][TM_KEYS];
+  __shared__ int key_rows[4][TM_KEYS];
 
   pdl_trigger();
   pdl_wait();
@@ -177,29 +199,32 @@ __global__ void __launch_bounds__(512) talking_mma_kernel(TalkArgs a, TalkMmaSha
   auto find_rows = [&](int t) {                            // the cache rows of tile t (-1: no such key), in units of kv head 0
     if (tid < TM_KEYS) {
       const int kpos = k_begin + t * TM_KEYS + tid;
-      key_rows[t & 1][tid] = t < tiles && kpos < k_end ? (int)talk_row(table, kpos, 0, a) : -1;
+      key_rows[t & 3][tid] = t < tiles && kpos < k_end ? (int)talk_row(table, kpos, 0, a) : -1;
     }
   };
   // A tile's keys (or values): a line is one key of one head, `width` elements; a thread keeps its 16-byte piece of
-  // a line and goes from line to line.
+  // a line and goes from line to line. Lines of no key are zeroed.
   const int k_pieces = D >> 3, v_pieces = DV >> 3, lines = my_kv * TM_KEYS;
   const int k_step = threads / k_pieces, v_step = threads / v_pieces;
   const int k_line = tid / k_pieces < k_step ? tid / k_pieces : lines, k_ch = (tid % k_pieces) * 8;
   const int v_line = tid / v_pieces < v_step ? tid / v_pieces : lines, v_ch = (tid % v_pieces) * 8;
-  const int g_rows = a.page_size;                          // rows from one key/value head to the next inside a page
-  auto load_rows = [&](bf16* dst, const bf16* src, int t, int width, int stride, int line0, int step, int ch) {
-    const int* rows = key_rows[t & 1];
+  auto load_lines = [&](bf16* dst, const bf16* src, int t, int width, int stride, int line0, int step, int ch) {
+    const int* rows = key_rows[t & 3];
     uint32_t to = tm_smem(dst) + (uint32_t)((line0 * stride + ch) * 2);
     const uint32_t to_step = (uint32_t)(step * stride * 2);
+    const bf16* base = src + (size_t)kv0 * a.page_size * width + ch;
+#pragma unroll 4
     for (int line = line0; line < lines; line += step, to += to_step) {
       const int row = rows[line & (TM_KEYS - 1)];
-      const int at = row < 0 ? 0 : row + (kv0 + (line >> 4)) * g_rows;
-      const bf16* from = src + (size_t)at * width + ch;
+      const bf16* from = base + (size_t)(row < 0 ? 0 : row + (line / TM_KEYS) * a.page_size) * width;
       asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(to), "l"(from), "r"(row < 0 ? 0 : 16) : "memory");
     }
   };
-  auto load_keys = [&](int t) { load_rows(Ks + (size_t)(t & 1) * k_elems, kc, t, D, KS, k_line, k_step, k_ch); };
-  auto load_values = [&](int t) { load_rows(Vs + (size_t)(t & 1) * v_elems, vc, t, DV, VS, v_line, v_step, v_ch); };
+  auto load_tiles = [&](int tk, int tv) {                  // one group: keys of tile tk and values of tile tv (none outside 0 .. tiles - 1)
+    if (tk >= 0 && tk < tiles) load_lines(Ks + (size_t)(tk & 1) * k_elems, kc, tk, D, KS, k_line, k_step, k_ch);
+    if (tv >= 0 && tv < tiles) load_lines(Vs + (size_t)(tv & 1) * v_elems, vc, tv, DV, VS, v_line, v_step, v_ch);
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
   CapArgs cap;
   cap.capped = a.softcap > 0.f;
   cap.mul = cap.capped ? a.scale / a.softcap : a.scale * TM_LOG2E;
@@ -238,18 +263,15 @@ __global__ void __launch_bounds__(512) talking_mma_kernel(TalkArgs a, TalkMmaSha
   const bool bounded = cap.capped && cap.cap2 <= 64.f;
   float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
   if (bounded && phase != TM_VALUES) m[0] = m[1] = 0.f;
-  find_rows(0);
-  find_rows(1);
+  for (int t = 0; t < 3; ++t) find_rows(t);
   __syncthreads();
   if (phase != TM_VALUES) {
-    if (tiles > 0) load_keys(0);
-    tm_commit();
+    load_tiles(0, -1);
     for (int t = 0; t < tiles; ++t) {
-      tm_wait_all();
+      tm_wait<0>();
       __syncthreads();                                     // tile t has arrived, and nobody reads the other buffer any more
-      if (t + 1 < tiles) load_keys(t + 1);
-      tm_commit();
-      find_rows(t + 2);                                    // in the place of tile t's, whose last reader was a step ago
+      load_tiles(t + 1, -1);
+      find_rows(t + 3);
       if (has_head) {
         float s[2][4];
         scores(s, t);
@@ -257,8 +279,7 @@ __global__ void __launch_bounds__(512) talking_mma_kernel(TalkArgs a, TalkMmaSha
 #pragma unroll
           for (int half = 0; half < 2; ++half)
             l[half] += (tm_ex2(s[0][half * 2]) + tm_ex2(s[0][half * 2 + 1])) + (tm_ex2(s[1][half * 2]) + tm_ex2(s[1][half * 2 + 1]));
-          continue;
-        }
+        } else {
 #pragma unroll
         for (int half = 0; half < 2; ++half) {
           float mx = fmaxf(fmaxf(s[0][half * 2], s[0][half * 2 + 1]), fmaxf(s[1][half * 2], s[1][half * 2 + 1]));
@@ -272,6 +293,7 @@ __global__ void __launch_bounds__(512) talking_mma_kernel(TalkArgs a, TalkMmaSha
             l[half] = l[half] * tm_ex2(m[half] - mn) + sum;
             m[half] = mn;
           }
+        }
         }
       }
     }
@@ -319,23 +341,14 @@ __global__ void __launch_bounds__(512) talking_mma_kernel(TalkArgs a, TalkMmaSha
 #pragma unroll
     for (int e = 0; e < 4; ++e) o[j][e] = 0.f;
   __syncthreads();
-  find_rows(0);
-  find_rows(1);
+  for (int t = 0; t < 3; ++t) find_rows(t);
   tm_sync<CL>();                                           // every CTA of the cluster is here before the first remote store
-  if (tiles > 0) {
-    load_keys(0);
-    load_values(0);
-  }
-  tm_commit();
+  load_tiles(0, -1);
+  load_tiles(1, 0);
+  tm_wait<1>();
+  __syncthreads();                                         // the first keys have arrived
   const int warps = threads >> 5;
   for (int t = 0; t < tiles; ++t) {
-    tm_wait_all();
-    __syncthreads();                                       // tile t has arrived, and nobody reads the other buffers any more
-    if (t + 1 < tiles) {
-      load_keys(t + 1);
-      load_values(t + 1);
-    }
-    tm_commit();
     if (has_head) {
       float s[2][4];
       scores(s, t);
@@ -352,8 +365,9 @@ __global__ void __launch_bounds__(512) talking_mma_kernel(TalkArgs a, TalkMmaSha
         }
       }
     }
-    tm_sync<CL>();
-    find_rows(t + 2);
+    tm_sync<CL>();                                         // all weights are there; keys of tile t and values of t - 1 are done with
+    load_tiles(t + 2, t + 1);
+    find_rows(t + 3);
     // mixed weights of this CTA's heads: a query row of the tile per turn
     for (int i = warp; i < TM_ROWS; i += warps) {
       float w[2][4];
@@ -379,6 +393,7 @@ __global__ void __launch_bounds__(512) talking_mma_kernel(TalkArgs a, TalkMmaSha
         at[(size_t)8 * TM_POS / 2] = tm_pack(w[j][2], w[j][3]);
       }
     }
+    tm_wait<1>();                                          // keys of tile t + 1 and values of tile t
     tm_sync<CL>();
     if (has_head) {
       uint32_t wf[4];
