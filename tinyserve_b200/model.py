@@ -53,6 +53,11 @@ class ModelParts:
             self.layers.append(Layer(ls, block, pos, {role: self._encoding(p) for role, p in ls.positions.items()}))
         self.stream_inputs: list[StreamInput | None] = [
             None if c.stream_input is None else STREAM_INPUTS.build(c.stream_input.kind, **c.stream_input.args) for c in spec.order]
+        for n, (call, part) in enumerate(zip(spec.order, self.stream_inputs)):
+            block = self.layers[call.layer].block
+            first_norm = next((block.parts[r] for r, family in type(block).roles.items() if family == "norm" and r in block.parts), None)
+            if part is not None and not getattr(first_norm, "folds_stream_input", False):
+                raise ValueError(f"order[{n}] has a stream input, but the first norm of its block does not add it")
         self.keeps_origin = any(s is not None and s.needs_origin for s in self.stream_inputs)
         # One cache user per (call of the order, mixer role of its block, need of that mixer), in that order: the
         # cache manager gets their needs as a flat list and hands back one entry for each.
@@ -243,8 +248,6 @@ class DecoderModel:
                 tables = None if layer.position is None else self._position_data(layer.position, ctx)
             ctx.upcoming_caches = parts.caches_of_call(n + 1, caches) if n + 1 < len(self.spec.order) else {}
             layer.block.forward(stream, ctx, parts.caches_of_call(n, caches), call.reads_cache_of is None, tables)
-            if stream.extra is not None:
-                raise RuntimeError(f"call {n} of the order: the block's first norm does not take what was added in front of it")
         ctx.arena.step_region()
         for join in ctx.at_step_end:
             join()

@@ -284,8 +284,8 @@ class ResidualStream:
 
     Two sub-layers side by side leave two outputs: ``second`` is ``(output, constant)`` of the other one, added to
     the stream together with ``delta``. ``extra`` is what a ``StreamInput`` has left: ``(rows [T, hidden] 32-bit or
-    None, one value per column or None)``, added after them. Norms that do not know these two leave them, and the
-    model refuses to go on. ``origin`` is the embedding output in 32-bit, kept for the calls that add it again."""
+    None, one value per column or None)``, added after them by the norm that follows (``Norm.folds_stream_input``: the
+    model is refused where that norm does not). ``origin`` is the embedding output in 32-bit, kept for the calls that add it again."""
 
     __slots__ = ("resid", "delta", "sumsq", "resid16", "_sumsq_buf", "_resid16_buf", "lanes", "connection", "post", "second",
                  "extra", "origin")
@@ -399,6 +399,9 @@ class Part:
 
 
 class Norm(Part):
+    # True if ``forward`` adds ``stream.extra`` (what a ``StreamInput`` has left) to the stream before it norms it.
+    folds_stream_input: bool = False
+
     def forward(self, stream: ResidualStream, ctx: StepContext) -> torch.Tensor:
         raise NotImplementedError
 

@@ -31,6 +31,7 @@ class RMSNorm(Norm):
         self.name, self.size, self.eps = name, int(size), float(eps)
         self.unit_offset = bool(unit_offset)
         self.round_once = bool(round_once) or self.unit_offset
+        self.folds_stream_input = self.round_once
         self.weight: torch.Tensor | None = None
 
     def tensor_specs(self, prefix: str) -> list[TensorSpec]:
