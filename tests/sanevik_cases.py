@@ -149,4 +149,17 @@ def oracle(folder: Path, tokens: list[int]) -> tuple[torch.Tensor, torch.Tensor]
     return want.float(), row_errors(low, want)
 
 
-assert_rows_close = _assert_rows_close
+def assert_rows_close(rows: torch.Tensor, want: torch.Tensor, cond: torch.Tensor, dtype: torch.dtype, what: str = "") -> None:
+    """float32: as for Diderax (a limit per position that grows with its conditioning: the retention's normed read-out
+    loses the digits that cancel at a request's first tokens). bfloat16: a token whose best router logits lie closer
+    together than the rounding of its input takes another expert than the oracle, and its row (and, diluted, rows that
+    attend to it) differs by much more than rounding; so the rows are judged by their median and their upper quartile
+    (a handful of rows by the median alone), and the float32 run of the same schedule carries the exactness."""
+    if dtype == torch.float32:
+        _assert_rows_close(rows, want, cond, dtype, what)
+        return
+    assert not rows.isnan().any(), f"{what}: NaN in the logits"
+    err = row_errors(rows, want).sort().values
+    median, upper = float(err[len(err) // 2]), float(err[(3 * len(err)) // 4])
+    assert median < (0.05 if len(err) >= 20 else 0.15), f"{what}: median relative error {median:.3g} over {len(err)} rows"
+    assert len(err) < 20 or upper < 0.12, f"{what}: upper quartile {upper:.3g} over {len(err)} rows"
