@@ -19,14 +19,11 @@
 // ranges (arrival counter), so there is no second kernel.
 // Every mbarrier wait is bounded; a wait that runs out sets *error_flag and the CTA leaves.
 #define TS_PDL_CLASS PDL_ATTENTION
-#include <cuda.h>
 
-#include <map>
-#include <mutex>
-#include <tuple>
 
 #include "attention.cuh"
 #include "bounded_wait.cuh"
+#include "cache_map.cuh"
 
 namespace ts {
 
@@ -623,46 +620,6 @@ __global__ void __launch_bounds__(WARPS * 32) decode_attn_tma_kernel(const __gri
 }
 
 // ---------------------------------------------------------------- host side
-typedef CUresult (*DtEncodeFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*,
-                               const cuuint64_t*, const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave,
-                               CUtensorMapSwizzle, CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
-
-static DtEncodeFn dt_encode_fn() {
-  static DtEncodeFn fn = nullptr;
-  if (fn == nullptr) {
-    void* p = nullptr;
-    cudaDriverEntryPointQueryResult q;
-    if (cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &p, cudaEnableDefault, &q) == cudaSuccess &&
-        q == cudaDriverEntryPointSuccess)
-      fn = (DtEncodeFn)p;
-  }
-  return fn;
-}
-
-// The descriptor of one cache tensor ([rows, head_dim] bf16, boxes of box_rows x 64, 128-byte
-// swizzle). Descriptors are kept per (address, rows, head_dim, box_rows): a cache tensor is
-// allocated once and used for every step.
-static const CUtensorMap* cache_map(const void* base, long long rows, int head_dim, int box_rows) {
-  static std::mutex mu;
-  static std::map<std::tuple<const void*, long long, int, int>, CUtensorMap> maps;
-  std::lock_guard<std::mutex> lock(mu);
-  auto key = std::make_tuple(base, rows, head_dim, box_rows);
-  auto it = maps.find(key);
-  if (it != maps.end()) return &it->second;
-  DtEncodeFn fn = dt_encode_fn();
-  if (fn == nullptr) return nullptr;
-  CUtensorMap m;
-  cuuint64_t dims[2] = {(cuuint64_t)head_dim, (cuuint64_t)rows};
-  cuuint64_t strides[1] = {(cuuint64_t)head_dim * 2};
-  cuuint32_t box[2] = {64u, (cuuint32_t)box_rows};
-  cuuint32_t elem[2] = {1, 1};
-  if (fn(&m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(base), dims, strides, box, elem,
-         CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B,
-         CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) != CUDA_SUCCESS)
-    return nullptr;
-  return &maps.emplace(key, m).first->second;
-}
-
 static int g_decode_cluster_merge = 1;
 
 template <int D64, int BR, bool FUSED, int WARPS, bool CLUSTER>

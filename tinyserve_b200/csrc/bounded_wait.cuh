@@ -22,7 +22,7 @@
 namespace ts {
 
 constexpr int WAIT_FAILED_GEMM_TCGEN05 = 1, WAIT_FAILED_PREFILL_TCGEN05 = 2, WAIT_FAILED_PREFILL_TMA = 3,
-              WAIT_FAILED_DECODE_TMA = 4, WAIT_FAILED_DECODE_BULK = 5;
+              WAIT_FAILED_DECODE_TMA = 4, WAIT_FAILED_DECODE_BULK = 5, WAIT_FAILED_TALKING = 6;
 
 static __constant__ long long c_wait_cycles = 2000000000ll;
 static __constant__ int c_wait_unarmed = 0;

@@ -4,7 +4,9 @@
 // A CTA owns 16 queries and up to 16 heads, a warp one head; with more heads (or more key/value heads than fit in
 // shared memory) the CTAs of a thread-block cluster own a share of the heads each and hand their weights to one
 // another through distributed shared memory, so no score is computed twice. Keys and values arrive in tiles of 16
-// positions by cp.async, two tiles in flight. First visit of the keys: every head's row maxima and sums. Second visit,
+// positions, two tiles in flight: by the TMA unit where keys and values are 64 or 128 wide and a tile lies in one page
+// (boxes of 64 columns, 128-byte swizzle, one lane of every warp asks for its share), else by cp.async into padded rows
+// (which the warps stall on: an SM takes in some 30 bytes a cycle). First visit of the keys: every head's row maxima and sums. Second visit,
 // tile by tile:
 //   S_h = Q_h K^T (mma.sync), capped, p_h = 2^(s - lse) in 32-bit, stored as two bf16 parts (value and remainder);
 //   W = T P for all positions of the tile (mma.sync with T as the A operand, both parts of P as B: the mixed weights
@@ -14,6 +16,8 @@
 // values, and the ranges' outputs added up, as in the CUDA-core form).
 #define TS_PDL_CLASS PDL_ATTENTION
 #include "talking_attention.cuh"
+#include "bounded_wait.cuh"
+#include "cache_map.cuh"
 
 namespace ts {
 
@@ -22,6 +26,15 @@ constexpr int TM_BOTH = 0, TM_STATS = 1, TM_VALUES = 2;
 constexpr float TM_LOG2E = 1.4426950408889634f;
 
 __device__ __forceinline__ uint32_t tm_smem(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
+__device__ __forceinline__ void tm_arm(uint64_t* bar, uint32_t bytes) {
+  asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;" ::"r"(tm_smem(bar)), "r"(bytes) : "memory");
+}
+// A box of 16 rows x 64 columns of the cache matrix into shared memory, 128-byte swizzled.
+__device__ __forceinline__ void tm_tensor(void* dst, const CUtensorMap* map, int x, int y, uint64_t* bar) {
+  asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4}], [%2];"
+               ::"r"(tm_smem(dst)), "l"(map), "r"(tm_smem(bar)), "r"(x), "r"(y) : "memory");
+}
+constexpr int TM_BOX = TM_KEYS * 64;                       // elements of a box
 template <int N>                                           // all but this thread's last N groups of copies have arrived
 __device__ __forceinline__ void tm_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 __device__ __forceinline__ void tm_ldm(uint32_t (&r)[4], const void* smem) {
@@ -130,11 +143,13 @@ struct TalkMmaShape {
   int padded_heads;        // all heads, rounded up to 16
 };
 
-template <int KD, int KV, int CL>
-__global__ void __launch_bounds__(512) talking_mma_kernel(TalkArgs a, TalkMmaShape sh, int phase) {
-  extern __shared__ __align__(16) unsigned char raw[];
-  const int H = a.num_heads, G = a.num_kv_heads, per = H / G, D = a.head_dim, DV = a.v_head_dim;
-  const int KS = D + 8, VS = DV + 8;                       // padded row strides
+template <int KD, int KV, int CL, bool TMA>
+__global__ void __launch_bounds__(512) talking_mma_kernel(TalkArgs a, TalkMmaShape sh, int phase, const __grid_constant__ CUtensorMap map_k,
+                                                          const __grid_constant__ CUtensorMap map_v, int* error_flag) {
+  extern __shared__ __align__(16) unsigned char raw_smem[];
+  unsigned char* raw = TMA ? (unsigned char*)(((uintptr_t)raw_smem + 1023) & ~(uintptr_t)1023) : raw_smem;
+  const int H = a.num_heads, G = a.num_kv_heads, per = H / G, D = TMA ? KD * 16 : a.head_dim, DV = TMA ? KV * 16 : a.v_head_dim;
+  const int KS = TMA ? D : D + 8, VS = TMA ? DV : DV + 8;  // padded row strides (TMA: boxes of 64 columns one after the other)
   const int Hp = sh.padded_heads;
   const size_t k_elems = (size_t)sh.kv_per_cta * TM_KEYS * KS, v_elems = (size_t)sh.kv_per_cta * TM_KEYS * VS;
   bf16* Ks = (bf16*)raw;                                   // [2][kv][KEYS][KS]
@@ -143,6 +158,7 @@ __global__ void __launch_bounds__(512) talking_mma_kernel(TalkArgs a, TalkMmaSha
   bf16* Ws = Ps + (size_t)2 * Hp * TM_POS;                 // [16][TM_POS]
   bf16* Tm = Ws + (size_t)16 * TM_POS;                     // [16][Hp + 8]
   __shared__ int key_rows[4][TM_KEYS];
+  __shared__ __align__(8) uint64_t bars[4];                // TMA: keys of even and odd tiles, values of even and odd tiles
 
   pdl_trigger();
   pdl_wait();
@@ -155,7 +171,8 @@ __global__ void __launch_bounds__(512) talking_mma_kernel(TalkArgs a, TalkMmaSha
   const int first_pos = ctx - n + q0;
   const int nq = min(TM_ROWS, n - q0);
   const int last_pos = first_pos + nq - 1;
-  const int lo = a.window > 0 ? max(0, first_pos - a.window + 1) : 0;
+  int lo = a.window > 0 ? max(0, first_pos - a.window + 1) : 0;
+  if (TMA) lo &= ~(TM_KEYS - 1);                           // a tile does not cross a page
   const int all_tiles = (last_pos + 1 - lo + TM_KEYS - 1) / TM_KEYS;
   const int each = (all_tiles + a.num_splits - 1) / a.num_splits;
   const int k_begin = lo + (int)blockIdx.z * each * TM_KEYS;
@@ -220,6 +237,38 @@ __global__ void __launch_bounds__(512) talking_mma_kernel(TalkArgs a, TalkMmaSha
       asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(to), "l"(from), "r"(row < 0 ? 0 : 16) : "memory");
     }
   };
+  const int warps = threads >> 5;
+  uint32_t phases = 0;                                     // bit b: the parity barrier b is waited for next
+  bool failed = false;
+  auto arrived = [&](int b) {
+    if (!failed) failed = !bounded_mbar_wait(tm_smem(&bars[b]), (phases >> b) & 1u);
+    phases ^= 1u << b;
+    __syncwarp();
+  };
+  auto give_up = [&]() {                                   // a wait ran out: say so, and give the copies in flight the same time again
+    if (!failed) return;
+    atomicExch(error_flag, WAIT_FAILED_TALKING);
+    if (tid == 0)
+      for (int b = 0; b < 4; ++b) bounded_mbar_wait(tm_smem(&bars[b]), (phases >> b) & 1u);
+  };
+  auto copy_tiles = [&](int tk, int tv) {                  // the same by the TMA unit
+    const bool with_k = tk >= 0 && tk < tiles, with_v = tv >= 0 && tv < tiles;
+    if (wait_test_unarmed()) return;
+    if (tid == 0) {
+      if (with_k) tm_arm(&bars[tk & 1], (uint32_t)(my_kv * (KD / 4) * TM_BOX * 2));
+      if (with_v) tm_arm(&bars[2 + (tv & 1)], (uint32_t)(my_kv * (KV / 4) * TM_BOX * 2));
+    }
+    if (lane == 0) {
+      for (int idx = warp; idx < my_kv * (KD / 4 + KV / 4); idx += warps) {
+        const bool is_v = idx >= my_kv * (KD / 4);
+        if (is_v ? !with_v : !with_k) continue;
+        const int i = is_v ? idx - my_kv * (KD / 4) : idx, t = is_v ? tv : tk, parts = is_v ? KV / 4 : KD / 4;
+        const int g = i / parts, part = i - g * parts;
+        bf16* to = (is_v ? Vs + (size_t)(t & 1) * v_elems : Ks + (size_t)(t & 1) * k_elems) + (size_t)i * TM_BOX;
+        tm_tensor(to, is_v ? &map_v : &map_k, part * 64, key_rows[t & 3][0] + (kv0 + g) * a.page_size, &bars[(is_v ? 2 : 0) + (t & 1)]);
+      }
+    }
+  };
   auto load_tiles = [&](int tk, int tv) {                  // one group: keys of tile tk and values of tile tv (none outside 0 .. tiles - 1)
     if (tk >= 0 && tk < tiles) load_lines(Ks + (size_t)(tk & 1) * k_elems, kc, tk, D, KS, k_line, k_step, k_ch);
     if (tv >= 0 && tv < tiles) load_lines(Vs + (size_t)(tv & 1) * v_elems, vc, tv, DV, VS, v_line, v_step, v_ch);
@@ -236,12 +285,13 @@ __global__ void __launch_bounds__(512) talking_mma_kernel(TalkArgs a, TalkMmaSha
     for (int j = 0; j < 2; ++j)
 #pragma unroll
       for (int e = 0; e < 4; ++e) s[j][e] = 0.f;
-    const bf16* kb = Ks + (size_t)(t & 1) * k_elems + ((size_t)my_g * TM_KEYS + (lane & 7) + ((lane >> 4) << 3)) * KS + ((lane >> 3) & 1) * 8;
+    const int krow = (lane & 7) + ((lane >> 4) << 3), khalf = (lane >> 3) & 1;
+    const bf16* kb = Ks + (size_t)(t & 1) * k_elems + (size_t)my_g * TM_KEYS * KS + (TMA ? krow * 64 : krow * KS + khalf * 8);
 #pragma unroll
     for (int kk = 0; kk < KD; ++kk) {
       if (kk * 16 < D) {
         uint32_t b[4];
-        tm_ldm(b, kb + kk * 16);
+        tm_ldm(b, TMA ? kb + (kk >> 2) * TM_BOX + (((2 * (kk & 3) + khalf) ^ (lane & 7)) << 3) : kb + kk * 16);
         tm_mma(s[0], qf[kk], b[0], b[1]);
         tm_mma(s[1], qf[kk], b[2], b[3]);
       }
@@ -264,14 +314,27 @@ __global__ void __launch_bounds__(512) talking_mma_kernel(TalkArgs a, TalkMmaSha
   float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
   if (bounded && phase != TM_VALUES) m[0] = m[1] = 0.f;
   for (int t = 0; t < 3; ++t) find_rows(t);
+  if (TMA && tid == 0) {
+    for (int b = 0; b < 4; ++b) asm volatile("mbarrier.init.shared::cta.b64 [%0], 1;" ::"r"(tm_smem(&bars[b])));
+    asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+  }
   __syncthreads();
   if (phase != TM_VALUES) {
-    load_tiles(0, -1);
+    if (TMA) {
+      copy_tiles(0, -1);
+      copy_tiles(1, -1);
+    } else {
+      load_tiles(0, -1);
+    }
     for (int t = 0; t < tiles; ++t) {
-      tm_wait<0>();
-      __syncthreads();                                     // tile t has arrived, and nobody reads the other buffer any more
-      load_tiles(t + 1, -1);
-      find_rows(t + 3);
+      if (TMA) {
+        arrived(t & 1);
+      } else {
+        tm_wait<0>();
+        __syncthreads();                                   // tile t has arrived, and nobody reads the other buffer any more
+        load_tiles(t + 1, -1);
+        find_rows(t + 3);
+      }
       if (has_head) {
         float s[2][4];
         scores(s, t);
@@ -296,6 +359,11 @@ __global__ void __launch_bounds__(512) talking_mma_kernel(TalkArgs a, TalkMmaSha
         }
         }
       }
+      if (TMA) {
+        __syncthreads();                                   // nobody reads this tile's buffer any more
+        copy_tiles(t + 2, -1);
+        find_rows(t + 3);
+      }
     }
 #pragma unroll
     for (int half = 0; half < 2; ++half) {
@@ -311,6 +379,7 @@ __global__ void __launch_bounds__(512) talking_mma_kernel(TalkArgs a, TalkMmaSha
             ml[0] = m[half];
             ml[1] = l[half];
           }
+      give_up();
       return;
     }
   } else if (has_head) {
@@ -343,12 +412,17 @@ __global__ void __launch_bounds__(512) talking_mma_kernel(TalkArgs a, TalkMmaSha
   __syncthreads();
   for (int t = 0; t < 3; ++t) find_rows(t);
   tm_sync<CL>();                                           // every CTA of the cluster is here before the first remote store
-  load_tiles(0, -1);
-  load_tiles(1, 0);
-  tm_wait<1>();
-  __syncthreads();                                         // the first keys have arrived
-  const int warps = threads >> 5;
+  if (TMA) {
+    copy_tiles(0, 0);
+    copy_tiles(1, -1);
+  } else {
+    load_tiles(0, -1);
+    load_tiles(1, 0);
+    tm_wait<1>();
+    __syncthreads();                                       // the first keys have arrived
+  }
   for (int t = 0; t < tiles; ++t) {
+    if (TMA) arrived(t & 1);
     if (has_head) {
       float s[2][4];
       scores(s, t);
@@ -366,7 +440,7 @@ __global__ void __launch_bounds__(512) talking_mma_kernel(TalkArgs a, TalkMmaSha
       }
     }
     tm_sync<CL>();                                         // all weights are there; keys of tile t and values of t - 1 are done with
-    load_tiles(t + 2, t + 1);
+    if (TMA) copy_tiles(t + 2, t + 1); else load_tiles(t + 2, t + 1);
     find_rows(t + 3);
     // mixed weights of this CTA's heads: a query row of the tile per turn
     for (int i = warp; i < TM_ROWS; i += warps) {
@@ -393,17 +467,30 @@ __global__ void __launch_bounds__(512) talking_mma_kernel(TalkArgs a, TalkMmaSha
         at[(size_t)8 * TM_POS / 2] = tm_pack(w[j][2], w[j][3]);
       }
     }
-    tm_wait<1>();                                          // keys of tile t + 1 and values of tile t
+    if (TMA) {
+      arrived(2 + (t & 1));
+      const int live = k_end - k_begin - t * TM_KEYS;      // rows from here on hold whatever the page held: their weights are zero, but a
+      if (live < TM_KEYS) {                                // number that is none would stay one
+        const int per_box = (TM_KEYS - live) * 8;          // 16-byte pieces of the dead rows of a box
+        for (int idx = tid; idx < my_kv * (KV / 4) * per_box; idx += threads) {
+          const int box = idx / per_box, rest = idx - box * per_box;
+          *reinterpret_cast<uint4*>(Vs + (size_t)(t & 1) * v_elems + (size_t)box * TM_BOX + live * 64 + rest * 8) = make_uint4(0u, 0u, 0u, 0u);
+        }
+      }
+    } else {
+      tm_wait<1>();                                        // keys of tile t + 1 and values of tile t
+    }
     tm_sync<CL>();
     if (has_head) {
       uint32_t wf[4];
       tm_ldm(wf, Ws + (size_t)warp * TM_POS + (lane & 15) * TM_ROWP + (lane >> 4) * 8);
-      const bf16* vb = Vs + (size_t)(t & 1) * v_elems + ((size_t)my_g * TM_KEYS + (lane & 7) + ((lane >> 3) & 1) * 8) * VS + (lane >> 4) * 8;
+      const int vrow = (lane & 7) + ((lane >> 3) & 1) * 8;
+      const bf16* vb = Vs + (size_t)(t & 1) * v_elems + (size_t)my_g * TM_KEYS * VS + (TMA ? vrow * 64 : vrow * VS + (lane >> 4) * 8);
 #pragma unroll
       for (int j = 0; j < KV; ++j) {
         if (j * 16 < DV) {
           uint32_t b[4];
-          tm_ldm_t(b, vb + j * 16);
+          tm_ldm_t(b, TMA ? vb + (j >> 2) * TM_BOX + (((2 * (j & 3) + (lane >> 4)) ^ (lane & 7)) << 3) : vb + j * 16);
           tm_mma(o[2 * j], wf, b[0], b[1]);
           tm_mma(o[2 * j + 1], wf, b[2], b[3]);
         }
@@ -430,6 +517,7 @@ __global__ void __launch_bounds__(512) talking_mma_kernel(TalkArgs a, TalkMmaSha
       }
     }
   }
+  give_up();
 }
 
 __global__ void talking_mma_combine_kernel(const float* part, bf16* out, int splits, int width, size_t total) {
@@ -444,7 +532,7 @@ __global__ void talking_mma_combine_kernel(const float* part, bf16* out, int spl
 }
 
 // How a cluster shares the heads: as few CTAs as hold 16 heads each and whose keys and values fit in shared memory.
-static bool talk_mma_shape(int H, int G, int D, int DV, TalkMmaShape& sh, int& cluster, size_t& smem) {
+static bool talk_mma_shape(int H, int G, int D, int DV, bool tma, TalkMmaShape& sh, int& cluster, size_t& smem) {
   constexpr size_t LIMIT = 226 * 1024;
   const int per = H / G;
   sh.padded_heads = (H + 15) / 16 * 16;
@@ -459,17 +547,19 @@ static bool talk_mma_shape(int H, int G, int D, int DV, TalkMmaShape& sh, int& c
     }
     sh.heads_per_cta = hc;
     sh.kv_per_cta = kv;
-    smem = sizeof(bf16) * (2 * (size_t)kv * TM_KEYS * (D + 8 + DV + 8) + (size_t)2 * sh.padded_heads * TM_POS + (size_t)16 * TM_POS +
+    smem = (tma ? 1024 : 0) + sizeof(bf16) * (2 * (size_t)kv * TM_KEYS * (tma ? D + DV : D + 8 + DV + 8) + (size_t)2 * sh.padded_heads * TM_POS + (size_t)16 * TM_POS +
                            (size_t)16 * (sh.padded_heads + 8));
     if (smem <= LIMIT) return true;
   }
   return false;
 }
 
-template <int KD, int KV, int CL>
+struct TalkMaps { CUtensorMap k, v; int* error_flag; };
+
+template <int KD, int KV, int CL, bool TMA>
 static int launch_talk_mma(const TalkArgs& a, const TalkMmaShape& sh, size_t smem, int num_seqs, int max_query_len, int phase,
-                           cudaStream_t stream) {
-  auto kern = talking_mma_kernel<KD, KV, CL>;
+                           const TalkMaps& maps, cudaStream_t stream) {
+  auto kern = talking_mma_kernel<KD, KV, CL, TMA>;
   static size_t allowed = 0;
   if (smem > 48 * 1024 && smem > allowed) {
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -478,16 +568,16 @@ static int launch_talk_mma(const TalkArgs& a, const TalkMmaShape& sh, size_t sme
   }
   const dim3 grid((unsigned)((max_query_len + TM_ROWS - 1) / TM_ROWS * CL), num_seqs, a.num_splits);
   const int threads = sh.heads_per_cta * 32;
-  if constexpr (CL == 1) return launch(kern, grid, threads, smem, stream, a, sh, phase);
-  else return launch_cluster(kern, grid, dim3(threads), smem, stream, dim3(CL, 1, 1), a, sh, phase);
+  if constexpr (CL == 1) return launch(kern, grid, threads, smem, stream, a, sh, phase, maps.k, maps.v, maps.error_flag);
+  else return launch_cluster(kern, grid, dim3(threads), smem, stream, dim3(CL, 1, 1), a, sh, phase, maps.k, maps.v, maps.error_flag);
 }
 
-template <int KD, int KV>
+template <int KD, int KV, bool TMA>
 static int launch_talk_mma_cl(const TalkArgs& a, const TalkMmaShape& sh, int cluster, size_t smem, int num_seqs, int max_query_len,
-                              int phase, cudaStream_t stream) {
-  if (cluster == 1) return launch_talk_mma<KD, KV, 1>(a, sh, smem, num_seqs, max_query_len, phase, stream);
-  if (cluster == 2) return launch_talk_mma<KD, KV, 2>(a, sh, smem, num_seqs, max_query_len, phase, stream);
-  return launch_talk_mma<KD, KV, 4>(a, sh, smem, num_seqs, max_query_len, phase, stream);
+                              int phase, const TalkMaps& maps, cudaStream_t stream) {
+  if (cluster == 1) return launch_talk_mma<KD, KV, 1, TMA>(a, sh, smem, num_seqs, max_query_len, phase, maps, stream);
+  if (cluster == 2) return launch_talk_mma<KD, KV, 2, TMA>(a, sh, smem, num_seqs, max_query_len, phase, maps, stream);
+  return launch_talk_mma<KD, KV, 4, TMA>(a, sh, smem, num_seqs, max_query_len, phase, maps, stream);
 }
 
 }  // namespace ts
@@ -499,23 +589,34 @@ extern "C" int ts_talking_attention_mma_takes(int heads, int kv_heads, int d, in
   int cluster;
   size_t smem;
   if (heads <= 0 || kv_heads <= 0 || heads % kv_heads || d <= 0 || dv <= 0 || d % 16 || dv % 16 || d > 128 || dv > 128) return 0;
-  return talk_mma_shape(heads, kv_heads, d, dv, sh, cluster, smem) ? cluster : 0;
+  return talk_mma_shape(heads, kv_heads, d, dv, false, sh, cluster, smem) ? cluster : 0;
 }
 
-// As ts_talking_attention, bf16 only; pages * kv_heads * page_size must stay below 2^31. talk is used as bf16.
+// As ts_talking_attention, bf16 only; cache_rows = pages * kv_heads * page_size must stay below 2^31. talk is used as bf16.
 extern "C" int ts_talking_attention_mma(const void* q, void* out, const void* k_cache, const void* v_cache, const int* block_tables,
                                         int table_width, const int* cu_q, const int* ctx_lens, int num_seqs, int max_query_len,
                                         int num_tokens, int heads, int kv_heads, int d, int dv, int page_size, float scale,
                                         int window, float softcap, const float* talk, const float* sinks, int num_splits,
-                                        float* part_ml, float* part_out, cudaStream_t stream) {
+                                        float* part_ml, float* part_out, long long cache_rows, int* error_flag,
+                                        cudaStream_t stream) {
   if (num_seqs <= 0 || num_tokens <= 0) return 0;
+  if (!error_flag || cache_rows <= 0 || cache_rows >= (1ll << 31)) return TS_ERR_BAD_ARGUMENT;
   if (heads <= 0 || kv_heads <= 0 || heads % kv_heads || page_size <= 0 || max_query_len <= 0 || window < 0) return TS_ERR_BAD_ARGUMENT;
   if (num_splits < 1 || (num_splits > 1 && (!part_ml || !part_out))) return TS_ERR_BAD_ARGUMENT;
   if (((uintptr_t)q | (uintptr_t)k_cache | (uintptr_t)v_cache | (uintptr_t)out) & 15) return TS_ERR_UNSUPPORTED;
   TalkMmaShape sh;
   int cluster;
   size_t smem;
-  if (!ts_talking_attention_mma_takes(heads, kv_heads, d, dv) || !talk_mma_shape(heads, kv_heads, d, dv, sh, cluster, smem))
+  TalkMaps maps = {};
+  maps.error_flag = error_flag;
+  bool tma = d == dv && (d == 64 || d == 128) && page_size % TM_KEYS == 0;
+  if (tma) {
+    const CUtensorMap* mk = cache_map(k_cache, cache_rows, d, TM_KEYS);
+    const CUtensorMap* mv = cache_map(v_cache, cache_rows, dv, TM_KEYS);
+    tma = mk && mv;
+    if (tma) { maps.k = *mk; maps.v = *mv; }
+  }
+  if (!ts_talking_attention_mma_takes(heads, kv_heads, d, dv) || !talk_mma_shape(heads, kv_heads, d, dv, tma, sh, cluster, smem))
     return TS_ERR_UNSUPPORTED;
   TalkArgs a;
   a.q = q; a.out = out; a.k_cache = k_cache; a.v_cache = v_cache; a.block_tables = block_tables; a.table_width = table_width;
@@ -523,8 +624,11 @@ extern "C" int ts_talking_attention_mma(const void* q, void* out, const void* k_
   a.page_size = page_size; a.page_shift = page_shift_of(page_size); a.scale = scale; a.window = window; a.softcap = softcap;
   a.talk = talk; a.sinks = sinks; a.num_splits = num_splits; a.part_ml = part_ml; a.part_out = part_out;
   auto run = [&](int phase) {
-    if (d <= 64 && dv <= 64) return launch_talk_mma_cl<4, 4>(a, sh, cluster, smem, num_seqs, max_query_len, phase, stream);
-    return launch_talk_mma_cl<8, 8>(a, sh, cluster, smem, num_seqs, max_query_len, phase, stream);
+    const bool small = d <= 64 && dv <= 64;
+    if (tma) return small ? launch_talk_mma_cl<4, 4, true>(a, sh, cluster, smem, num_seqs, max_query_len, phase, maps, stream)
+                          : launch_talk_mma_cl<8, 8, true>(a, sh, cluster, smem, num_seqs, max_query_len, phase, maps, stream);
+    return small ? launch_talk_mma_cl<4, 4, false>(a, sh, cluster, smem, num_seqs, max_query_len, phase, maps, stream)
+                 : launch_talk_mma_cl<8, 8, false>(a, sh, cluster, smem, num_seqs, max_query_len, phase, maps, stream);
   };
   if (num_splits == 1) return run(TM_BOTH);
   if (int e = run(TM_STATS)) return e;

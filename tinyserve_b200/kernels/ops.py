@@ -61,7 +61,7 @@ _SIGNATURES: dict[str, list[Any]] = {
     "ts_talking_attention": [_vp, _vp, _vp, _vp, _vp, _i, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _f, _i, _f, _vp, _vp, _i, _vp, _vp,
                              _i, _vp],
     "ts_talking_attention_mma": [_vp, _vp, _vp, _vp, _vp, _i, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _f, _i, _f, _vp, _vp, _i, _vp,
-                                 _vp, _vp],
+                                 _vp, _c.c_longlong, _vp, _vp],
     "ts_talking_attention_mma_takes": [_i, _i, _i, _i],
     "ts_prefill_attention_mma": [_vp, _vp, _vp, _vp, _vp, _i, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _f, _i, _vp],
     "ts_decode_attention_mma": [_vp, _vp, _vp, _vp, _vp, _i, _vp, _vp, _vp, _i, _i, _i, _i, _i, _f, _i, _i, _vp, _vp,
@@ -715,7 +715,7 @@ def _error_word(device: torch.device) -> torch.Tensor:
 
 # What a non-zero error word says (csrc/bounded_wait.cuh).
 WAIT_FAILURES = {1: "gemm_tcgen05", 2: "prefill_attention_tcgen05", 3: "prefill_attention_tma",
-                 4: "decode_attention_tma", 5: "decode_attention_mma"}
+                 4: "decode_attention_tma", 5: "decode_attention_mma", 6: "talking_attention_mma"}
 
 
 def raise_for_status(code: int, device: torch.device | str | None = None) -> None:
@@ -1654,7 +1654,8 @@ def talking_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Ten
         _opt(talk, "talk", torch.float32), _opt(sinks, "sinks", torch.float32), splits, _opt(part_ml, "part_ml"),
         _opt(part_out, "part_out"))
     if cluster:
-        _check(_fn("ts_talking_attention_mma")(*args, _stream()), "talking_attention_mma", kernels=3 if splits > 1 else 1)
+        _check(_fn("ts_talking_attention_mma")(*args, k_cache.shape[0] * hkv * page_size, _error_word(q.device).data_ptr(), _stream()),
+               "talking_attention_mma", kernels=3 if splits > 1 else 1)
     else:
         _check(_fn("ts_talking_attention")(*args, _code(dt), _stream()), "talking_attention", kernels=3 if splits > 1 else 1)
 
