@@ -34,6 +34,7 @@ __device__ __forceinline__ void tm_tensor(void* dst, const CUtensorMap* map, int
   asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4}], [%2];"
                ::"r"(tm_smem(dst)), "l"(map), "r"(tm_smem(bar)), "r"(x), "r"(y) : "memory");
 }
+constexpr int TM_AHEAD = 64;                               // tiles whose rows are looked up together
 constexpr int TM_BOX = TM_KEYS * 64;                       // elements of a box
 template <int N>                                           // all but this thread's last N groups of copies have arrived
 __device__ __forceinline__ void tm_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
@@ -137,6 +138,126 @@ __device__ __forceinline__ void cap_scores(float (&s)[2][4], const CapArgs& c) {
   }
 }
 
+// --------------------------------------------------- maxima and sums of prompt portions
+// The first visit needs one head at a time, so it runs on tiles of 64 queries (a warp 16 of them) that share every key
+// tile of 64, a quarter of the key traffic of the tiles of 16 below. part_ml[token, head] receives the row's maximum
+// (0 where capped scores are summed as they are) and its sum, in base-2 units.
+constexpr int TS_ROWS = 64, TS_KEYS = 64, TS_THREADS = 128;
+
+template <int KD>
+__global__ void __launch_bounds__(TS_THREADS) talking_stats_kernel(TalkArgs a) {
+  extern __shared__ __align__(16) unsigned char raw_stats[];
+  const int H = a.num_heads, D = a.head_dim, KS = D + 8;
+  bf16* Ks = (bf16*)raw_stats;                             // [2][KEYS][KS]
+  pdl_trigger();
+  pdl_wait();
+  const int seq = blockIdx.y, head = blockIdx.z, kvh = head / (H / a.num_kv_heads);
+  const int row0 = a.cu_q[seq], n = a.cu_q[seq + 1] - row0;
+  const int q0 = blockIdx.x * TS_ROWS;
+  if (q0 >= n) return;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int first_pos = a.ctx_lens[seq] - n + q0, nq = min(TS_ROWS, n - q0), last_pos = first_pos + nq - 1;
+  const int lo = a.window > 0 ? max(0, first_pos - a.window + 1) : 0;
+  const int tiles = (last_pos + 1 - lo + TS_KEYS - 1) / TS_KEYS;
+  const int* table = a.block_tables + (size_t)seq * a.table_width;
+  const bf16* kc = (const bf16*)a.k_cache;
+  const int r = warp * 16 + (lane >> 2), c2 = (lane & 3) * 2;
+  uint32_t qf[KD][4];
+#pragma unroll
+  for (int kk = 0; kk < KD; ++kk)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int row = r + (j & 1) * 8, col = kk * 16 + c2 + (j >> 1) * 8;
+      qf[kk][j] = 0u;
+      if (row < nq && kk * 16 < D)
+        qf[kk][j] = *reinterpret_cast<const uint32_t*>((const bf16*)a.q + ((size_t)(row0 + q0 + row) * H + head) * D + col);
+    }
+  // a thread copies half a key of a tile, 16 bytes a request
+  const int key = tid >> 1, pieces = D >> 3, p_begin = (tid & 1) * ((pieces + 1) / 2), p_end = (tid & 1) ? pieces : (pieces + 1) / 2;
+  auto load = [&](int t) {
+    const int kpos = lo + t * TS_KEYS + key;
+    const bool valid = t < tiles && kpos <= last_pos;
+    const bf16* from = kc + (valid ? talk_row(table, kpos, kvh, a) * D : 0);
+    const uint32_t to = tm_smem(Ks + ((size_t)(t & 1) * TS_KEYS + key) * KS);
+    if (t < tiles)
+      for (int p = p_begin; p < p_end; ++p)
+        asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(to + p * 16), "l"(from + p * 8), "r"(valid ? 16 : 0) : "memory");
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  CapArgs cap;
+  cap.capped = a.softcap > 0.f;
+  cap.mul = cap.capped ? a.scale / a.softcap : a.scale * TM_LOG2E;
+  cap.cap2 = a.softcap * TM_LOG2E;
+  const bool bounded = cap.capped && cap.cap2 <= 64.f;
+  float m[2] = {bounded ? 0.f : -INFINITY, bounded ? 0.f : -INFINITY}, l[2] = {0.f, 0.f};
+  load(0);
+  for (int t = 0; t < tiles; ++t) {
+    tm_wait<0>();
+    __syncthreads();                                       // tile t has arrived, and nobody reads the other buffer any more
+    load(t + 1);
+    const bf16* kb = Ks + ((size_t)(t & 1) * TS_KEYS + (lane & 7) + ((lane >> 4) << 3)) * KS + ((lane >> 3) & 1) * 8;
+#pragma unroll
+    for (int part = 0; part < TS_KEYS / 16; ++part) {
+      const int k0 = lo + t * TS_KEYS + part * 16;
+      // no row of this warp sees any of these keys
+      if (k0 > first_pos + warp * 16 + 15 || (a.window > 0 && k0 + 15 <= first_pos + warp * 16 - a.window)) continue;
+      float s[2][4];
+#pragma unroll
+      for (int j = 0; j < 2; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) s[j][e] = 0.f;
+#pragma unroll
+      for (int kk = 0; kk < KD; ++kk) {
+        if (kk * 16 < D) {
+          uint32_t b[4];
+          tm_ldm(b, kb + (size_t)part * 16 * KS + kk * 16);
+          tm_mma(s[0], qf[kk], b[0], b[1]);
+          tm_mma(s[1], qf[kk], b[2], b[3]);
+        }
+      }
+      cap_scores(s, cap);
+      if (!(k0 + 15 <= first_pos + warp * 16 && (a.window <= 0 || k0 > first_pos + warp * 16 + 15 - a.window))) {
+#pragma unroll
+        for (int j = 0; j < 2; ++j)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            const int kpos = k0 + j * 8 + c2 + (e & 1), qpos = first_pos + r + (e >> 1) * 8;
+            if (!(kpos <= qpos && (a.window <= 0 || kpos > qpos - a.window))) s[j][e] = -INFINITY;
+          }
+      }
+#pragma unroll
+      for (int half = 0; half < 2; ++half) {
+        float mn = m[half];
+        if (!bounded) {
+          float mx = fmaxf(fmaxf(s[0][half * 2], s[0][half * 2 + 1]), fmaxf(s[1][half * 2], s[1][half * 2 + 1]));
+          mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
+          mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
+          mn = fmaxf(m[half], mx);
+          if (mn == -INFINITY) continue;
+          l[half] *= tm_ex2(m[half] - mn);
+          m[half] = mn;
+        }
+        l[half] += (tm_ex2(s[0][half * 2] - mn) + tm_ex2(s[0][half * 2 + 1] - mn)) + (tm_ex2(s[1][half * 2] - mn) + tm_ex2(s[1][half * 2 + 1] - mn));
+      }
+    }
+  }
+#pragma unroll
+  for (int half = 0; half < 2; ++half) {
+    l[half] += __shfl_xor_sync(0xffffffffu, l[half], 1);
+    l[half] += __shfl_xor_sync(0xffffffffu, l[half], 2);
+    const int row = r + half * 8;
+    if (row < nq && (lane & 3) == 0) {
+      float* ml = a.part_ml + ((size_t)(row0 + q0 + row) * H + head) * 2;
+      ml[0] = m[half];
+      ml[1] = l[half];
+    }
+  }
+}
+
+// ------------------------------------------------------------------ the mixing kernel
+constexpr int TM_MAX_COUNTERS = 1 << 14;
+static __device__ unsigned int g_talk_counters[TM_MAX_COUNTERS];     // arrivals of a request's key ranges; zero between launches
+
 struct TalkMmaShape {
   int heads_per_cta;       // <= 16: a warp each
   int kv_per_cta;          // key/value heads a CTA's heads read, at most
@@ -158,6 +279,7 @@ __global__ void __launch_bounds__(512) talking_mma_kernel(TalkArgs a, TalkMmaSha
   bf16* Ws = Ps + (size_t)2 * Hp * TM_POS;                 // [16][TM_POS]
   bf16* Tm = Ws + (size_t)16 * TM_POS;                     // [16][Hp + 8]
   __shared__ int key_rows[4][TM_KEYS];
+  __shared__ int tile_rows[2 * TM_AHEAD];                  // TMA: the cache row of each tile's first key, TM_AHEAD tiles at a time
   __shared__ __align__(8) uint64_t bars[4];                // TMA: keys of even and odd tiles, values of even and odd tiles
 
   pdl_trigger();
@@ -213,6 +335,10 @@ __global__ void __launch_bounds__(512) talking_mma_kernel(TalkArgs a, TalkMmaSha
       Ps[((size_t)part * Hp + H) * TM_POS + rest] = __float2bfloat16_rn(0.f);
     }
   }
+  auto find_tiles = [&](int t) {                           // TMA: the first cache rows of tiles t .. t + TM_AHEAD - 1, in units of kv head 0
+    for (int i = tid; i < TM_AHEAD; i += threads)
+      if (t + i < tiles) tile_rows[(t + i) & (2 * TM_AHEAD - 1)] = (int)talk_row(table, k_begin + (t + i) * TM_KEYS, 0, a);
+  };
   auto find_rows = [&](int t) {                            // the cache rows of tile t (-1: no such key), in units of kv head 0
     if (tid < TM_KEYS) {
       const int kpos = k_begin + t * TM_KEYS + tid;
@@ -265,7 +391,7 @@ __global__ void __launch_bounds__(512) talking_mma_kernel(TalkArgs a, TalkMmaSha
         const int i = is_v ? idx - my_kv * (KD / 4) : idx, t = is_v ? tv : tk, parts = is_v ? KV / 4 : KD / 4;
         const int g = i / parts, part = i - g * parts;
         bf16* to = (is_v ? Vs + (size_t)(t & 1) * v_elems : Ks + (size_t)(t & 1) * k_elems) + (size_t)i * TM_BOX;
-        tm_tensor(to, is_v ? &map_v : &map_k, part * 64, key_rows[t & 3][0] + (kv0 + g) * a.page_size, &bars[(is_v ? 2 : 0) + (t & 1)]);
+        tm_tensor(to, is_v ? &map_v : &map_k, part * 64, tile_rows[t & (2 * TM_AHEAD - 1)] + (kv0 + g) * a.page_size, &bars[(is_v ? 2 : 0) + (t & 1)]);
       }
     }
   };
@@ -313,7 +439,11 @@ __global__ void __launch_bounds__(512) talking_mma_kernel(TalkArgs a, TalkMmaSha
   const bool bounded = cap.capped && cap.cap2 <= 64.f;
   float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
   if (bounded && phase != TM_VALUES) m[0] = m[1] = 0.f;
-  for (int t = 0; t < 3; ++t) find_rows(t);
+  if (TMA) {
+    find_tiles(0);
+  } else {
+    for (int t = 0; t < 3; ++t) find_rows(t);
+  }
   if (TMA && tid == 0) {
     for (int b = 0; b < 4; ++b) asm volatile("mbarrier.init.shared::cta.b64 [%0], 1;" ::"r"(tm_smem(&bars[b])));
     asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
@@ -362,7 +492,7 @@ __global__ void __launch_bounds__(512) talking_mma_kernel(TalkArgs a, TalkMmaSha
       if (TMA) {
         __syncthreads();                                   // nobody reads this tile's buffer any more
         copy_tiles(t + 2, -1);
-        find_rows(t + 3);
+        if (((t + 8) & (TM_AHEAD - 1)) == 0) find_tiles(t + 8);      // well before the first of them is asked for
       }
     }
 #pragma unroll
@@ -410,7 +540,11 @@ __global__ void __launch_bounds__(512) talking_mma_kernel(TalkArgs a, TalkMmaSha
 #pragma unroll
     for (int e = 0; e < 4; ++e) o[j][e] = 0.f;
   __syncthreads();
-  for (int t = 0; t < 3; ++t) find_rows(t);
+  if (TMA) {
+    if (tiles > TM_AHEAD) find_tiles(0);                   // unless they are all still there
+  } else {
+    for (int t = 0; t < 3; ++t) find_rows(t);
+  }
   tm_sync<CL>();                                           // every CTA of the cluster is here before the first remote store
   if (TMA) {
     copy_tiles(0, 0);
@@ -440,8 +574,13 @@ __global__ void __launch_bounds__(512) talking_mma_kernel(TalkArgs a, TalkMmaSha
       }
     }
     tm_sync<CL>();                                         // all weights are there; keys of tile t and values of t - 1 are done with
-    if (TMA) copy_tiles(t + 2, t + 1); else load_tiles(t + 2, t + 1);
-    find_rows(t + 3);
+    if (TMA) {
+      copy_tiles(t + 2, t + 1);
+      if (((t + 8) & (TM_AHEAD - 1)) == 0) find_tiles(t + 8);
+    } else {
+      load_tiles(t + 2, t + 1);
+      find_rows(t + 3);
+    }
     // mixed weights of this CTA's heads: a query row of the tile per turn
     for (int i = warp; i < TM_ROWS; i += warps) {
       float w[2][4];
@@ -518,16 +657,17 @@ __global__ void __launch_bounds__(512) talking_mma_kernel(TalkArgs a, TalkMmaSha
     }
   }
   give_up();
-}
-
-__global__ void talking_mma_combine_kernel(const float* part, bf16* out, int splits, int width, size_t total) {
-  pdl_trigger();
-  pdl_wait();
-  for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < total; idx += (size_t)gridDim.x * blockDim.x) {
-    const size_t t = idx / width, c = idx - t * width;
-    float o = 0.f;
-    for (int s = 0; s < splits; ++s) o += part[(t * splits + s) * width + c];
-    out[idx] = __float2bfloat16_rn(o);
+  if (a.num_splits == 1) return;
+  // the CTA of a request's last range to arrive adds the ranges' outputs up, in order, for the heads it owns
+  __shared__ int last;
+  if (!cta_arrives_last(&g_talk_counters[(size_t)seq * CL + rank], (unsigned int)a.num_splits, &last)) return;
+  const int width = my_heads * DV;
+  for (int idx = tid; idx < nq * width; idx += threads) {
+    const int row = idx / width, col = head0 * DV + idx - row * width;
+    const float* part = a.part_out + (size_t)(row0 + q0 + row) * a.num_splits * H * DV + col;
+    float sum = 0.f;
+    for (int s = 0; s < a.num_splits; ++s) sum += __ldcg(part + (size_t)s * H * DV);
+    ((bf16*)a.out)[(size_t)(row0 + q0 + row) * H * DV + col] = __float2bfloat16_rn(sum);
   }
 }
 
@@ -592,7 +732,8 @@ extern "C" int ts_talking_attention_mma_takes(int heads, int kv_heads, int d, in
   return talk_mma_shape(heads, kv_heads, d, dv, false, sh, cluster, smem) ? cluster : 0;
 }
 
-// As ts_talking_attention, bf16 only; cache_rows = pages * kv_heads * page_size must stay below 2^31. talk is used as bf16.
+// As ts_talking_attention, bf16 only; num_splits > 1 for steps of single tokens only; with num_splits 1 and part_ml
+// [T, heads, 2] the maxima and sums are made by a kernel of their own (prompt portions). cache_rows = pages * kv_heads * page_size must stay below 2^31. talk is used as bf16.
 extern "C" int ts_talking_attention_mma(const void* q, void* out, const void* k_cache, const void* v_cache, const int* block_tables,
                                         int table_width, const int* cu_q, const int* ctx_lens, int num_seqs, int max_query_len,
                                         int num_tokens, int heads, int kv_heads, int d, int dv, int page_size, float scale,
@@ -602,7 +743,8 @@ extern "C" int ts_talking_attention_mma(const void* q, void* out, const void* k_
   if (num_seqs <= 0 || num_tokens <= 0) return 0;
   if (!error_flag || cache_rows <= 0 || cache_rows >= (1ll << 31)) return TS_ERR_BAD_ARGUMENT;
   if (heads <= 0 || kv_heads <= 0 || heads % kv_heads || page_size <= 0 || max_query_len <= 0 || window < 0) return TS_ERR_BAD_ARGUMENT;
-  if (num_splits < 1 || (num_splits > 1 && (!part_ml || !part_out))) return TS_ERR_BAD_ARGUMENT;
+  if (num_splits < 1 || (num_splits > 1 && (!part_ml || !part_out || max_query_len != 1))) return TS_ERR_BAD_ARGUMENT;
+  if (num_splits > 1 && (long long)num_seqs * 4 > TM_MAX_COUNTERS) return TS_ERR_UNSUPPORTED;
   if (((uintptr_t)q | (uintptr_t)k_cache | (uintptr_t)v_cache | (uintptr_t)out) & 15) return TS_ERR_UNSUPPORTED;
   TalkMmaShape sh;
   int cluster;
@@ -630,12 +772,14 @@ extern "C" int ts_talking_attention_mma(const void* q, void* out, const void* k_
     return small ? launch_talk_mma_cl<4, 4, false>(a, sh, cluster, smem, num_seqs, max_query_len, phase, maps, stream)
                  : launch_talk_mma_cl<8, 8, false>(a, sh, cluster, smem, num_seqs, max_query_len, phase, maps, stream);
   };
-  if (num_splits == 1) return run(TM_BOTH);
+  if (num_splits == 1 && !part_ml) return run(TM_BOTH);
+  if (num_splits == 1) {
+    const dim3 grid((max_query_len + TS_ROWS - 1) / TS_ROWS, num_seqs, heads);
+    const size_t ssmem = sizeof(bf16) * 2 * (size_t)TS_KEYS * (d + 8);
+    if (int e = d <= 64 ? launch(talking_stats_kernel<4>, grid, TS_THREADS, ssmem, stream, a)
+                        : launch(talking_stats_kernel<8>, grid, TS_THREADS, ssmem, stream, a)) return e;
+    return run(TM_VALUES);
+  }
   if (int e = run(TM_STATS)) return e;
-  if (int e = run(TM_VALUES)) return e;
-  const int width = heads * dv;
-  const size_t total = (size_t)num_tokens * width;
-  size_t blocks = (total + 255) / 256;
-  if (blocks > 148 * 16) blocks = 148 * 16;
-  return launch(talking_mma_combine_kernel, (unsigned)blocks, 256, 0, stream, (const float*)part_out, (bf16*)out, num_splits, width, total);
+  return run(TM_VALUES);
 }

@@ -1642,10 +1642,12 @@ def talking_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Ten
         cluster = talking_cluster(hq, hkv, d, dv)
     splits, part_ml, part_out = 1, None, None
     if ctx.max_query_len == 1:
-        splits = talking_splits(ctx.num_seqs * max(cluster, 1), min(ctx.max_context_len, window) if window else ctx.max_context_len)
+        splits = 1 if ctx.num_seqs > 4096 else talking_splits(ctx.num_seqs * max(cluster, 1), min(ctx.max_context_len, window) if window else ctx.max_context_len)
         if splits > 1:
             part_ml = ctx.arena.take((t, hq, splits, 2), torch.float32)
             part_out = ctx.arena.take((t, splits, hq * dv), torch.float32)
+    elif cluster:
+        part_ml = ctx.arena.take((t, hq, 1, 2), torch.float32)      # maxima and sums, from a kernel of their own
     args = (
         _dev(q, "q"), _dev(out, "out"), _dev(k_cache, "k_cache"), _dev(v_cache, "v_cache"),
         _dev(block_tables, "block_tables", torch.int32), block_tables.shape[1],
@@ -1655,7 +1657,7 @@ def talking_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Ten
         _opt(part_out, "part_out"))
     if cluster:
         _check(_fn("ts_talking_attention_mma")(*args, k_cache.shape[0] * hkv * page_size, _error_word(q.device).data_ptr(), _stream()),
-               "talking_attention_mma", kernels=3 if splits > 1 else 1)
+               "talking_attention_mma", kernels=1 if part_ml is None else 2)
     else:
         _check(_fn("ts_talking_attention")(*args, _code(dt), _stream()), "talking_attention", kernels=3 if splits > 1 else 1)
 
