@@ -95,6 +95,32 @@ def test_attention_gives_up_and_recovers(kernel, lens, d, page, code, monkeypatc
     torch.testing.assert_close(out.float(), want.float(), **tol(BF16))
 
 
+@pytest.mark.parametrize("heads, groups, lens, news", [(4, 2, [300, 90], [300, 1]), (24, 4, [200, 40], [70, 40]), (4, 2, [300, 40], [1, 1])])
+def test_attention_with_mixed_heads_gives_up_and_recovers(heads, groups, lens, news) -> None:
+    """One CTA for all heads, a cluster that shares them, and single tokens over key ranges."""
+    from test_diderax_gpu import Ctx, _rand, _tables
+    from test_sanevik_gpu import _stores
+
+    tables, table, pages = _tables(lens, 16, 7)
+    k, v = _stores(BF16, tables, pages, 16, lens, groups, 64, 64)
+    q, talk = _rand(sum(news), heads, 64, seed=3, dtype=BF16), _rand(heads, heads, seed=5, scale=0.3).bfloat16().float()
+    out, want = (torch.zeros(sum(news), heads * 64, dtype=BF16, device="cuda") for _ in range(2))
+    ctx = Ctx(news, lens)
+
+    def run(impl, into):
+        impl.talking_attention(q, k, v, 16, table, ctx, 0.125, 100, 20.0, talk, into)
+
+    with lost_copies():
+        run(ops, out)
+        assert error_code() == 6
+        with pytest.raises(ops.KernelError, match="talking_attention_mma"):
+            ops.check_device_errors()
+    run(ops, out)
+    ops.check_device_errors()
+    run(ref, want)
+    torch.testing.assert_close(out.float(), want.float(), **tol(BF16))
+
+
 def test_engine_and_replay_raise_instead_of_returning_tokens(tmp_path) -> None:
     """Through the entry points: the status word comes back with the sampled tokens (one copy, no
     extra synchronisation) and ``Engine.step`` raises; trace replay raises too; and a fresh engine

@@ -34,6 +34,12 @@ __device__ __forceinline__ void tm_tensor(void* dst, const CUtensorMap* map, int
   asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4}], [%2];"
                ::"r"(tm_smem(dst)), "l"(map), "r"(tm_smem(bar)), "r"(x), "r"(y) : "memory");
 }
+__device__ __forceinline__ bool tm_try(uint32_t addr, uint32_t parity) {      // the phase is complete already, or soon
+  uint32_t ok;
+  asm volatile("{\n.reg .pred p;\nmbarrier.try_wait.parity.shared::cta.b64 p, [%1], %2;\nselp.u32 %0, 1, 0, p;\n}\n"
+               : "=r"(ok) : "r"(addr), "r"(parity) : "memory");
+  return ok != 0;
+}
 constexpr int TM_AHEAD = 64;                               // tiles whose rows are looked up together
 constexpr int TM_BOX = TM_KEYS * 64;                       // elements of a box
 template <int N>                                           // all but this thread's last N groups of copies have arrived
@@ -47,7 +53,7 @@ __device__ __forceinline__ void tm_ldm_t(uint32_t (&r)[4], const void* smem) {
                : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(tm_smem(smem)) : "memory");
 }
 __device__ __forceinline__ void tm_mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+  asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
                : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
                : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
@@ -147,6 +153,7 @@ constexpr int TS_ROWS = 64, TS_KEYS = 64, TS_THREADS = 128;
 template <int KD>
 __global__ void __launch_bounds__(TS_THREADS) talking_stats_kernel(TalkArgs a) {
   extern __shared__ __align__(16) unsigned char raw_stats[];
+  __shared__ int rows[4][TS_KEYS];
   const int H = a.num_heads, D = a.head_dim, KS = D + 8;
   bf16* Ks = (bf16*)raw_stats;                             // [2][KEYS][KS]
   pdl_trigger();
@@ -172,16 +179,21 @@ __global__ void __launch_bounds__(TS_THREADS) talking_stats_kernel(TalkArgs a) {
       if (row < nq && kk * 16 < D)
         qf[kk][j] = *reinterpret_cast<const uint32_t*>((const bf16*)a.q + ((size_t)(row0 + q0 + row) * H + head) * D + col);
     }
-  // a thread copies half a key of a tile, 16 bytes a request
-  const int key = tid >> 1, pieces = D >> 3, p_begin = (tid & 1) * ((pieces + 1) / 2), p_end = (tid & 1) ? pieces : (pieces + 1) / 2;
+  // a thread copies its 16-byte piece of one key after the other; the keys' cache rows are looked up a tile ahead
+  const int pieces = D >> 3, step = TS_THREADS / pieces, line0 = tid / pieces < step ? tid / pieces : TS_KEYS, ch = (tid % pieces) * 8;
+  auto find = [&](int t) {
+    const int kpos = lo + t * TS_KEYS + tid;
+    if (tid < TS_KEYS) rows[t & 3][tid] = t < tiles && kpos <= last_pos ? (int)talk_row(table, kpos, kvh, a) : -1;
+  };
   auto load = [&](int t) {
-    const int kpos = lo + t * TS_KEYS + key;
-    const bool valid = t < tiles && kpos <= last_pos;
-    const bf16* from = kc + (valid ? talk_row(table, kpos, kvh, a) * D : 0);
-    const uint32_t to = tm_smem(Ks + ((size_t)(t & 1) * TS_KEYS + key) * KS);
-    if (t < tiles)
-      for (int p = p_begin; p < p_end; ++p)
-        asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(to + p * 16), "l"(from + p * 8), "r"(valid ? 16 : 0) : "memory");
+    if (t < tiles) {
+      uint32_t to = tm_smem(Ks + ((size_t)(t & 1) * TS_KEYS + line0) * KS + ch);
+      for (int line = line0; line < TS_KEYS; line += step, to += (uint32_t)(step * KS * 2)) {
+        const int row = rows[t & 3][line];
+        const bf16* from = kc + (size_t)(row < 0 ? 0 : row) * D + ch;
+        asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(to), "l"(from), "r"(row < 0 ? 0 : 16) : "memory");
+      }
+    }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
   CapArgs cap;
@@ -190,46 +202,52 @@ __global__ void __launch_bounds__(TS_THREADS) talking_stats_kernel(TalkArgs a) {
   cap.cap2 = a.softcap * TM_LOG2E;
   const bool bounded = cap.capped && cap.cap2 <= 64.f;
   float m[2] = {bounded ? 0.f : -INFINITY, bounded ? 0.f : -INFINITY}, l[2] = {0.f, 0.f};
+  for (int t = 0; t < 2; ++t) find(t);
+  __syncthreads();
   load(0);
   for (int t = 0; t < tiles; ++t) {
     tm_wait<0>();
     __syncthreads();                                       // tile t has arrived, and nobody reads the other buffer any more
     load(t + 1);
+    find(t + 2);
     const bf16* kb = Ks + ((size_t)(t & 1) * TS_KEYS + (lane & 7) + ((lane >> 4) << 3)) * KS + ((lane >> 3) & 1) * 8;
 #pragma unroll
-    for (int part = 0; part < TS_KEYS / 16; ++part) {
-      const int k0 = lo + t * TS_KEYS + part * 16;
+    for (int part = 0; part < TS_KEYS / 32; ++part) {
+      const int k0 = lo + t * TS_KEYS + part * 32;
       // no row of this warp sees any of these keys
-      if (k0 > first_pos + warp * 16 + 15 || (a.window > 0 && k0 + 15 <= first_pos + warp * 16 - a.window)) continue;
-      float s[2][4];
+      if (k0 > first_pos + warp * 16 + 15 || (a.window > 0 && k0 + 31 <= first_pos + warp * 16 - a.window)) continue;
+      float s[2][2][4];                                    // two blocks of 16 keys: four independent chains of products
 #pragma unroll
-      for (int j = 0; j < 2; ++j)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) s[j][e] = 0.f;
+      for (int i = 0; i < 16; ++i) s[i >> 3][(i >> 2) & 1][i & 3] = 0.f;
 #pragma unroll
       for (int kk = 0; kk < KD; ++kk) {
         if (kk * 16 < D) {
-          uint32_t b[4];
-          tm_ldm(b, kb + (size_t)part * 16 * KS + kk * 16);
-          tm_mma(s[0], qf[kk], b[0], b[1]);
-          tm_mma(s[1], qf[kk], b[2], b[3]);
+          uint32_t b[2][4];
+#pragma unroll
+          for (int x = 0; x < 2; ++x) tm_ldm(b[x], kb + (size_t)(part * 2 + x) * 16 * KS + kk * 16);
+#pragma unroll
+          for (int x = 0; x < 2; ++x) {
+            tm_mma(s[x][0], qf[kk], b[x][0], b[x][1]);
+            tm_mma(s[x][1], qf[kk], b[x][2], b[x][3]);
+          }
         }
       }
-      cap_scores(s, cap);
-      if (!(k0 + 15 <= first_pos + warp * 16 && (a.window <= 0 || k0 > first_pos + warp * 16 + 15 - a.window))) {
+      cap_scores(s[0], cap);
+      cap_scores(s[1], cap);
+      if (!(k0 + 31 <= first_pos + warp * 16 && (a.window <= 0 || k0 > first_pos + warp * 16 + 15 - a.window))) {
 #pragma unroll
-        for (int j = 0; j < 2; ++j)
-#pragma unroll
-          for (int e = 0; e < 4; ++e) {
-            const int kpos = k0 + j * 8 + c2 + (e & 1), qpos = first_pos + r + (e >> 1) * 8;
-            if (!(kpos <= qpos && (a.window <= 0 || kpos > qpos - a.window))) s[j][e] = -INFINITY;
-          }
+        for (int i = 0; i < 16; ++i) {
+          const int kpos = k0 + (i >> 3) * 16 + ((i >> 2) & 1) * 8 + c2 + (i & 1), qpos = first_pos + r + ((i >> 1) & 1) * 8;
+          if (!(kpos <= qpos && (a.window <= 0 || kpos > qpos - a.window))) s[i >> 3][(i >> 2) & 1][i & 3] = -INFINITY;
+        }
       }
 #pragma unroll
       for (int half = 0; half < 2; ++half) {
         float mn = m[half];
         if (!bounded) {
-          float mx = fmaxf(fmaxf(s[0][half * 2], s[0][half * 2 + 1]), fmaxf(s[1][half * 2], s[1][half * 2 + 1]));
+          float mx = -INFINITY;
+#pragma unroll
+          for (int i = 0; i < 8; ++i) mx = fmaxf(mx, s[i >> 2][(i >> 1) & 1][half * 2 + (i & 1)]);
           mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
           mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
           mn = fmaxf(m[half], mx);
@@ -237,7 +255,9 @@ __global__ void __launch_bounds__(TS_THREADS) talking_stats_kernel(TalkArgs a) {
           l[half] *= tm_ex2(m[half] - mn);
           m[half] = mn;
         }
-        l[half] += (tm_ex2(s[0][half * 2] - mn) + tm_ex2(s[0][half * 2 + 1] - mn)) + (tm_ex2(s[1][half * 2] - mn) + tm_ex2(s[1][half * 2 + 1] - mn));
+#pragma unroll
+        for (int x = 0; x < 2; ++x)
+          l[half] += (tm_ex2(s[x][0][half * 2] - mn) + tm_ex2(s[x][0][half * 2 + 1] - mn)) + (tm_ex2(s[x][1][half * 2] - mn) + tm_ex2(s[x][1][half * 2 + 1] - mn));
       }
     }
   }
@@ -367,7 +387,8 @@ __global__ void __launch_bounds__(512) talking_mma_kernel(TalkArgs a, TalkMmaSha
   uint32_t phases = 0;                                     // bit b: the parity barrier b is waited for next
   bool failed = false;
   auto arrived = [&](int b) {
-    if (!failed) failed = !bounded_mbar_wait(tm_smem(&bars[b]), (phases >> b) & 1u);
+    const uint32_t addr = tm_smem(&bars[b]), parity = (phases >> b) & 1u;
+    if (!failed && !tm_try(addr, parity)) failed = !bounded_mbar_wait(addr, parity);
     phases ^= 1u << b;
     __syncwarp();
   };
@@ -377,23 +398,21 @@ __global__ void __launch_bounds__(512) talking_mma_kernel(TalkArgs a, TalkMmaSha
     if (tid == 0)
       for (int b = 0; b < 4; ++b) bounded_mbar_wait(tm_smem(&bars[b]), (phases >> b) & 1u);
   };
-  auto copy_tiles = [&](int tk, int tv) {                  // the same by the TMA unit
-    const bool with_k = tk >= 0 && tk < tiles, with_v = tv >= 0 && tv < tiles;
-    if (wait_test_unarmed()) return;
-    if (tid == 0) {
-      if (with_k) tm_arm(&bars[tk & 1], (uint32_t)(my_kv * (KD / 4) * TM_BOX * 2));
-      if (with_v) tm_arm(&bars[2 + (tv & 1)], (uint32_t)(my_kv * (KV / 4) * TM_BOX * 2));
-    }
+  // The same by the TMA unit: box i is columns 64 (i % (KD / 4)) of key/value head i / (KD / 4); one lane of every warp asks
+  // for its share of the boxes (KD == KV).
+  const bool lost = TMA && wait_test_unarmed();
+  auto copy_boxes = [&](bf16* dst, const CUtensorMap* map, uint64_t* bar, int t) {
+    if (tid == 0) tm_arm(bar, (uint32_t)(my_kv * (KD / 4) * TM_BOX * 2));
     if (lane == 0) {
-      for (int idx = warp; idx < my_kv * (KD / 4 + KV / 4); idx += warps) {
-        const bool is_v = idx >= my_kv * (KD / 4);
-        if (is_v ? !with_v : !with_k) continue;
-        const int i = is_v ? idx - my_kv * (KD / 4) : idx, t = is_v ? tv : tk, parts = is_v ? KV / 4 : KD / 4;
-        const int g = i / parts, part = i - g * parts;
-        bf16* to = (is_v ? Vs + (size_t)(t & 1) * v_elems : Ks + (size_t)(t & 1) * k_elems) + (size_t)i * TM_BOX;
-        tm_tensor(to, is_v ? &map_v : &map_k, part * 64, tile_rows[t & (2 * TM_AHEAD - 1)] + (kv0 + g) * a.page_size, &bars[(is_v ? 2 : 0) + (t & 1)]);
-      }
+      const int row = tile_rows[t & (2 * TM_AHEAD - 1)] + kv0 * a.page_size;
+      for (int i = warp; i < my_kv * (KD / 4); i += warps)
+        tm_tensor(dst + (size_t)i * TM_BOX, map, (i % (KD / 4)) * 64, row + i / (KD / 4) * a.page_size, bar);
     }
+  };
+  auto copy_tiles = [&](int tk, int tv) {
+    if (lost) return;
+    if (tk >= 0 && tk < tiles) copy_boxes(Ks + (size_t)(tk & 1) * k_elems, &map_k, &bars[tk & 1], tk);
+    if (tv >= 0 && tv < tiles) copy_boxes(Vs + (size_t)(tv & 1) * v_elems, &map_v, &bars[2 + (tv & 1)], tv);
   };
   auto load_tiles = [&](int tk, int tv) {                  // one group: keys of tile tk and values of tile tv (none outside 0 .. tiles - 1)
     if (tk >= 0 && tk < tiles) load_lines(Ks + (size_t)(tk & 1) * k_elems, kc, tk, D, KS, k_line, k_step, k_ch);
