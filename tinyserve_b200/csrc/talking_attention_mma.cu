@@ -5,7 +5,7 @@
 // shared memory) the CTAs of a thread-block cluster own a share of the heads each and hand their weights to one
 // another through distributed shared memory, so no score is computed twice. Keys and values arrive in tiles of 16
 // positions, two tiles in flight: by the TMA unit where keys and values are 64 or 128 wide and a tile lies in one page
-// (boxes of 64 columns, 128-byte swizzle, one lane of every warp asks for its share), else by cp.async into padded rows
+// (boxes of 64 columns of all heads at once, 128-byte swizzle, the warps ask for them in turn), else by cp.async into padded rows
 // (which the warps stall on: an SM takes in some 30 bytes a cycle). First visit of the keys: every head's row maxima and sums. Second visit,
 // tile by tile:
 //   S_h = Q_h K^T (mma.sync), capped, p_h = 2^(s - lse) in 32-bit, stored as two bf16 parts (value and remainder);
@@ -29,10 +29,10 @@ __device__ __forceinline__ uint32_t tm_smem(const void* p) { return (uint32_t)__
 __device__ __forceinline__ void tm_arm(uint64_t* bar, uint32_t bytes) {
   asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;" ::"r"(tm_smem(bar)), "r"(bytes) : "memory");
 }
-// A box of 16 rows x 64 columns of the cache matrix into shared memory, 128-byte swizzled.
-__device__ __forceinline__ void tm_tensor(void* dst, const CUtensorMap* map, int x, int y, uint64_t* bar) {
-  asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4}], [%2];"
-               ::"r"(tm_smem(dst)), "l"(map), "r"(tm_smem(bar)), "r"(x), "r"(y) : "memory");
+// A box of several heads x 16 rows x 64 columns of a page into shared memory, 128-byte swizzled.
+__device__ __forceinline__ void tm_tensor(void* dst, const CUtensorMap* map, int x, int y, int z, uint64_t* bar) {
+  asm volatile("cp.async.bulk.tensor.3d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4, %5}], [%2];"
+               ::"r"(tm_smem(dst)), "l"(map), "r"(tm_smem(bar)), "r"(x), "r"(y), "r"(z) : "memory");
 }
 __device__ __forceinline__ bool tm_try(uint32_t addr, uint32_t parity) {      // the phase is complete already, or soon
   uint32_t ok;
@@ -44,13 +44,14 @@ constexpr int TM_AHEAD = 64;                               // tiles whose rows a
 constexpr int TM_BOX = TM_KEYS * 64;                       // elements of a box
 template <int N>                                           // all but this thread's last N groups of copies have arrived
 __device__ __forceinline__ void tm_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
-__device__ __forceinline__ void tm_ldm(uint32_t (&r)[4], const void* smem) {
+// Shared memory is addressed in its own 32-bit window throughout.
+__device__ __forceinline__ void tm_ldm(uint32_t (&r)[4], uint32_t smem) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(tm_smem(smem)) : "memory");
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem) : "memory");
 }
-__device__ __forceinline__ void tm_ldm_t(uint32_t (&r)[4], const void* smem) {
+__device__ __forceinline__ void tm_ldm_t(uint32_t (&r)[4], uint32_t smem) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(tm_smem(smem)) : "memory");
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem) : "memory");
 }
 __device__ __forceinline__ void tm_mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
   asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
@@ -154,7 +155,8 @@ template <int KD>
 __global__ void __launch_bounds__(TS_THREADS) talking_stats_kernel(TalkArgs a) {
   extern __shared__ __align__(16) unsigned char raw_stats[];
   __shared__ int rows[4][TS_KEYS];
-  const int H = a.num_heads, D = a.head_dim, KS = D + 8;
+  constexpr int KS = KD * 16 + 8;                          // padded row stride
+  const int H = a.num_heads, D = a.head_dim;
   bf16* Ks = (bf16*)raw_stats;                             // [2][KEYS][KS]
   pdl_trigger();
   pdl_wait();
@@ -210,7 +212,7 @@ __global__ void __launch_bounds__(TS_THREADS) talking_stats_kernel(TalkArgs a) {
     __syncthreads();                                       // tile t has arrived, and nobody reads the other buffer any more
     load(t + 1);
     find(t + 2);
-    const bf16* kb = Ks + ((size_t)(t & 1) * TS_KEYS + (lane & 7) + ((lane >> 4) << 3)) * KS + ((lane >> 3) & 1) * 8;
+    const uint32_t kb = tm_smem(Ks) + (uint32_t)((((t & 1) * TS_KEYS + (lane & 7) + ((lane >> 4) << 3)) * KS + ((lane >> 3) & 1) * 8) * 2);
 #pragma unroll
     for (int part = 0; part < TS_KEYS / 32; ++part) {
       const int k0 = lo + t * TS_KEYS + part * 32;
@@ -224,7 +226,7 @@ __global__ void __launch_bounds__(TS_THREADS) talking_stats_kernel(TalkArgs a) {
         if (kk * 16 < D) {
           uint32_t b[2][4];
 #pragma unroll
-          for (int x = 0; x < 2; ++x) tm_ldm(b[x], kb + (size_t)(part * 2 + x) * 16 * KS + kk * 16);
+          for (int x = 0; x < 2; ++x) tm_ldm(b[x], kb + (uint32_t)((part * 2 + x) * 16 * KS * 2) + kk * 32);
 #pragma unroll
           for (int x = 0; x < 2; ++x) {
             tm_mma(s[x][0], qf[kk], b[x][0], b[x][1]);
@@ -398,15 +400,18 @@ __global__ void __launch_bounds__(512) talking_mma_kernel(TalkArgs a, TalkMmaSha
     if (tid == 0)
       for (int b = 0; b < 4; ++b) bounded_mbar_wait(tm_smem(&bars[b]), (phases >> b) & 1u);
   };
-  // The same by the TMA unit: box i is columns 64 (i % (KD / 4)) of key/value head i / (KD / 4); one lane of every warp asks
-  // for its share of the boxes (KD == KV).
+  // The same by the TMA unit (KD == KV): a box holds 64 columns of the tile's rows of kv_per_cta heads (heads beyond this
+  // CTA's own are fetched and not read); the warps take turns in asking.
+  const int boxes = sh.kv_per_cta;
   const bool lost = TMA && wait_test_unarmed();
   auto copy_boxes = [&](bf16* dst, const CUtensorMap* map, uint64_t* bar, int t) {
-    if (tid == 0) tm_arm(bar, (uint32_t)(my_kv * (KD / 4) * TM_BOX * 2));
-    if (lane == 0) {
-      const int row = tile_rows[t & (2 * TM_AHEAD - 1)] + kv0 * a.page_size;
-      for (int i = warp; i < my_kv * (KD / 4); i += warps)
-        tm_tensor(dst + (size_t)i * TM_BOX, map, (i % (KD / 4)) * 64, row + i / (KD / 4) * a.page_size, bar);
+    if (lane == 0 && warp == t % warps) {
+      tm_arm(bar, (uint32_t)(boxes * (KD / 4) * TM_BOX * 2));
+      const int row = tile_rows[t & (2 * TM_AHEAD - 1)];
+      const int z = a.page_shift >= 0 ? row >> a.page_shift : row / a.page_size;
+#pragma unroll
+      for (int part = 0; part < KD / 4; ++part)
+        tm_tensor(dst + (size_t)part * boxes * TM_BOX, map, part * 64, row - z * a.page_size, z + min(kv0, G - 1), bar);
     }
   };
   auto copy_tiles = [&](int tk, int tv) {
@@ -424,19 +429,30 @@ __global__ void __launch_bounds__(512) talking_mma_kernel(TalkArgs a, TalkMmaSha
   cap.mul = cap.capped ? a.scale / a.softcap : a.scale * TM_LOG2E;
   cap.cap2 = a.softcap * TM_LOG2E;
 
+  // This lane's places in the shared arrays (ldmatrix rows, fragment positions). A swizzled box: a row is 128 bytes, its
+  // 16-byte pieces permuted by the row's low three bits; piece 2 k + h of row x lies at (h ^ x) ^ 2 k.
+  const int krow = (lane & 7) + ((lane >> 4) << 3), khalf = (lane >> 3) & 1, vrow = (lane & 7) + ((lane >> 3) & 1) * 8, vhalf = lane >> 4;
+  const uint32_t part_bytes = (uint32_t)(boxes * TM_BOX * 2);          // from 64 columns of all heads to the next 64
+  const uint32_t s_k = tm_smem(Ks) + (uint32_t)(my_g * TM_KEYS * (TMA ? 64 : KS) * 2) + (uint32_t)(TMA ? krow * 128 + ((khalf ^ (lane & 7)) << 4) : (krow * KS + khalf * 8) * 2);
+  const uint32_t s_v = tm_smem(Vs) + (uint32_t)(my_g * TM_KEYS * (TMA ? 64 : VS) * 2) + (uint32_t)(TMA ? vrow * 128 + ((vhalf ^ (lane & 7)) << 4) : (vrow * VS + vhalf * 8) * 2);
+  const uint32_t s_p = tm_smem(Ps), s_w = tm_smem(Ws), k_stage = (uint32_t)(k_elems * 2), v_stage = (uint32_t)(v_elems * 2), rest = (uint32_t)(Hp * TM_POS * 2);
+  const uint32_t s_p_out = s_p + (uint32_t)((head * TM_POS + r * TM_ROWP + c2) * 2);
+  const uint32_t s_p_mix = s_p + (uint32_t)((((lane & 7) + ((lane >> 3) & 1) * 8) * TM_POS + (lane >> 4) * 8) * 2);
+  const uint32_t s_t_mix = tm_smem(Tm) + (uint32_t)(((lane & 15) * (Hp + 8) + (lane >> 4) * 8) * 2);
+  const uint32_t s_w_out = s_w + (uint32_t)((r * TM_POS + c2) * 2), s_w_in = s_w + (uint32_t)((warp * TM_POS + (lane & 15) * TM_ROWP + (lane >> 4) * 8) * 2);
+
   // the scores of this warp's head for tile t, in base-2 units, minus infinity where a row does not see the key
   auto scores = [&](float (&s)[2][4], int t) {
 #pragma unroll
     for (int j = 0; j < 2; ++j)
 #pragma unroll
       for (int e = 0; e < 4; ++e) s[j][e] = 0.f;
-    const int krow = (lane & 7) + ((lane >> 4) << 3), khalf = (lane >> 3) & 1;
-    const bf16* kb = Ks + (size_t)(t & 1) * k_elems + (size_t)my_g * TM_KEYS * KS + (TMA ? krow * 64 : krow * KS + khalf * 8);
+    const uint32_t kb = s_k + (t & 1 ? k_stage : 0u);
 #pragma unroll
     for (int kk = 0; kk < KD; ++kk) {
       if (kk * 16 < D) {
         uint32_t b[4];
-        tm_ldm(b, TMA ? kb + (kk >> 2) * TM_BOX + (((2 * (kk & 3) + khalf) ^ (lane & 7)) << 3) : kb + kk * 16);
+        tm_ldm(b, TMA ? (kb ^ (uint32_t)((kk & 3) << 5)) + (kk >> 2) * part_bytes : kb + kk * 32);
         tm_mma(s[0], qf[kk], b[0], b[1]);
         tm_mma(s[1], qf[kk], b[2], b[3]);
       }
@@ -581,14 +597,14 @@ __global__ void __launch_bounds__(512) talking_mma_kernel(TalkArgs a, TalkMmaSha
       scores(s, t);
 #pragma unroll
       for (int half = 0; half < 2; ++half) {
-        const uint32_t at = tm_smem(Ps + (size_t)head * TM_POS + (r + half * 8) * TM_ROWP + c2);
+        const uint32_t at = s_p_out + half * (8 * TM_ROWP * 2);
 #pragma unroll
         for (int j = 0; j < 2; ++j) {
           const float p0 = tm_ex2(s[j][half * 2] - lse[half]), p1 = tm_ex2(s[j][half * 2 + 1] - lse[half]);
           const uint32_t hi = tm_pack(p0, p1);
           const uint32_t rem = tm_pack(p0 - __uint_as_float(hi << 16), p1 - __uint_as_float(hi & 0xffff0000u));
           tm_store_all<CL>(at + j * 16, hi);
-          tm_store_all<CL>(at + j * 16 + (uint32_t)(Hp * TM_POS * 2), rem);
+          tm_store_all<CL>(at + j * 16 + rest, rem);
         }
       }
     }
@@ -609,20 +625,20 @@ __global__ void __launch_bounds__(512) talking_mma_kernel(TalkArgs a, TalkMmaSha
         for (int e = 0; e < 4; ++e) w[j][e] = 0.f;
       for (int g0 = 0; g0 < Hp; g0 += 16) {
         uint32_t tf[4], b[4];
-        tm_ldm(tf, Tm + (size_t)(lane & 15) * (Hp + 8) + g0 + (lane >> 4) * 8);
-        const bf16* pb = Ps + (size_t)(g0 + (lane & 7) + ((lane >> 3) & 1) * 8) * TM_POS + i * TM_ROWP + (lane >> 4) * 8;
+        tm_ldm(tf, s_t_mix + g0 * 2);
+        const uint32_t pb = s_p_mix + g0 * (TM_POS * 2) + i * (TM_ROWP * 2);
         tm_ldm_t(b, pb);
         tm_mma(w[0], tf, b[0], b[1]);
         tm_mma(w[1], tf, b[2], b[3]);
-        tm_ldm_t(b, pb + (size_t)Hp * TM_POS);
+        tm_ldm_t(b, pb + rest);
         tm_mma(w[0], tf, b[0], b[1]);
         tm_mma(w[1], tf, b[2], b[3]);
       }
 #pragma unroll
       for (int j = 0; j < 2; ++j) {
-        uint32_t* at = reinterpret_cast<uint32_t*>(Ws + (size_t)r * TM_POS + i * TM_ROWP + j * 8 + c2);
-        at[0] = tm_pack(w[j][0], w[j][1]);
-        at[(size_t)8 * TM_POS / 2] = tm_pack(w[j][2], w[j][3]);
+        const uint32_t at = s_w_out + i * (TM_ROWP * 2) + j * 16;
+        tm_store_all<1>(at, tm_pack(w[j][0], w[j][1]));
+        tm_store_all<1>(at + 8 * TM_POS * 2, tm_pack(w[j][2], w[j][3]));
       }
     }
     if (TMA) {
@@ -630,7 +646,7 @@ __global__ void __launch_bounds__(512) talking_mma_kernel(TalkArgs a, TalkMmaSha
       const int live = k_end - k_begin - t * TM_KEYS;      // rows from here on hold whatever the page held: their weights are zero, but a
       if (live < TM_KEYS) {                                // number that is none would stay one
         const int per_box = (TM_KEYS - live) * 8;          // 16-byte pieces of the dead rows of a box
-        for (int idx = tid; idx < my_kv * (KV / 4) * per_box; idx += threads) {
+        for (int idx = tid; idx < boxes * (KV / 4) * per_box; idx += threads) {
           const int box = idx / per_box, rest = idx - box * per_box;
           *reinterpret_cast<uint4*>(Vs + (size_t)(t & 1) * v_elems + (size_t)box * TM_BOX + live * 64 + rest * 8) = make_uint4(0u, 0u, 0u, 0u);
         }
@@ -641,14 +657,13 @@ __global__ void __launch_bounds__(512) talking_mma_kernel(TalkArgs a, TalkMmaSha
     tm_sync<CL>();
     if (has_head) {
       uint32_t wf[4];
-      tm_ldm(wf, Ws + (size_t)warp * TM_POS + (lane & 15) * TM_ROWP + (lane >> 4) * 8);
-      const int vrow = (lane & 7) + ((lane >> 3) & 1) * 8;
-      const bf16* vb = Vs + (size_t)(t & 1) * v_elems + (size_t)my_g * TM_KEYS * VS + (TMA ? vrow * 64 : vrow * VS + (lane >> 4) * 8);
+      tm_ldm(wf, s_w_in);
+      const uint32_t vb = s_v + (t & 1 ? v_stage : 0u);
 #pragma unroll
       for (int j = 0; j < KV; ++j) {
         if (j * 16 < DV) {
           uint32_t b[4];
-          tm_ldm_t(b, TMA ? vb + (j >> 2) * TM_BOX + (((2 * (j & 3) + (lane >> 4)) ^ (lane & 7)) << 3) : vb + j * 16);
+          tm_ldm_t(b, TMA ? (vb ^ (uint32_t)((j & 3) << 5)) + (j >> 2) * part_bytes : vb + j * 32);
           tm_mma(o[2 * j], wf, b[0], b[1]);
           tm_mma(o[2 * j + 1], wf, b[2], b[3]);
         }
@@ -772,8 +787,9 @@ extern "C" int ts_talking_attention_mma(const void* q, void* out, const void* k_
   maps.error_flag = error_flag;
   bool tma = d == dv && (d == 64 || d == 128) && page_size % TM_KEYS == 0;
   if (tma) {
-    const CUtensorMap* mk = cache_map(k_cache, cache_rows, d, TM_KEYS);
-    const CUtensorMap* mv = cache_map(v_cache, cache_rows, dv, TM_KEYS);
+    tma = talk_mma_shape(heads, kv_heads, d, dv, true, sh, cluster, smem);
+    const CUtensorMap* mk = tma ? cache_heads_map(k_cache, cache_rows / page_size, page_size, d, TM_KEYS, sh.kv_per_cta) : nullptr;
+    const CUtensorMap* mv = tma ? cache_heads_map(v_cache, cache_rows / page_size, page_size, dv, TM_KEYS, sh.kv_per_cta) : nullptr;
     tma = mk && mv;
     if (tma) { maps.k = *mk; maps.v = *mv; }
   }
@@ -794,7 +810,7 @@ extern "C" int ts_talking_attention_mma(const void* q, void* out, const void* k_
   if (num_splits == 1 && !part_ml) return run(TM_BOTH);
   if (num_splits == 1) {
     const dim3 grid((max_query_len + TS_ROWS - 1) / TS_ROWS, num_seqs, heads);
-    const size_t ssmem = sizeof(bf16) * 2 * (size_t)TS_KEYS * (d + 8);
+    const size_t ssmem = sizeof(bf16) * 2 * (size_t)TS_KEYS * ((d <= 64 ? 64 : 128) + 8);
     if (int e = d <= 64 ? launch(talking_stats_kernel<4>, grid, TS_THREADS, ssmem, stream, a)
                         : launch(talking_stats_kernel<8>, grid, TS_THREADS, ssmem, stream, a)) return e;
     return run(TM_VALUES);
