@@ -117,11 +117,21 @@ def qk_norm_rope_write(qkv, q_out, q_weight, k_weight, eps, cos, sin, rotary_dim
 
 
 def paged_attention(q, k_cache, v_cache, page_size, block_tables, ctx: Any, scale, window, out, sinks=None,
-                    keep_first=0) -> None:
+                    keep_first=0, chunk=0, maps=1, finish=None) -> None:
     """Per request: gather its keys and values from the pages in position order, then plain
     causal (windowed) attention for its new tokens (upstream src/tinyserve/attention.py:62-111)."""
     t, hq, d = q.shape
     hkv = k_cache.shape[1]
+    if maps == 2:          # each map alone, with its half of the query and key rows, then their difference
+        finished, factor, mult, eps = finish
+        res = torch.empty(t, hq, 2, v_cache.shape[3], dtype=torch.float32, device=q.device)
+        for n in (0, 1):
+            half = slice(n * d // 2, (n + 1) * d // 2)
+            one = torch.empty(t, hq * v_cache.shape[3], dtype=torch.float32, device=q.device)
+            paged_attention(q[..., half], k_cache[..., half], v_cache, page_size, block_tables, ctx, scale, window, one, chunk=chunk)
+            res[:, :, n] = one.view(t, hq, -1)
+        pair_combine(res, factor, eps, mult, finished, hq, v_cache.shape[3])
+        return
     group = hq // hkv
     dv = v_cache.shape[3]
     res = torch.zeros(t, hq, dv, dtype=torch.float32, device=q.device)
@@ -133,6 +143,8 @@ def paged_attention(q, k_cache, v_cache, page_size, block_tables, ctx: Any, scal
         lo = 0
         if window:
             lo = max(0, (total - n) - window + 1)      # pages before this may be gone
+        if chunk:
+            lo = (total - n) // chunk * chunk
         kept = min(int(keep_first), lo) if window else 0    # first positions that stay visible below the window
         pos = torch.cat([pos[:kept], pos[lo:]])
         pages = block_tables[b].long()[pos // page_size]
@@ -142,6 +154,8 @@ def paged_attention(q, k_cache, v_cache, page_size, block_tables, ctx: Any, scal
         hidden = pos[None, :] > qpos[:, None]
         if window:
             hidden = hidden | ((pos[None, :] <= qpos[:, None] - window) & (pos[None, :] >= int(keep_first)))
+        if chunk:
+            hidden = hidden | (pos[None, :] // chunk != qpos[:, None] // chunk)
         s = torch.einsum("ihd,jhd->hij", q[r0: r0 + n].float(), k) * scale
         s = s.masked_fill(hidden, float("-inf"))
         if sinks is not None:
@@ -152,6 +166,18 @@ def paged_attention(q, k_cache, v_cache, page_size, block_tables, ctx: Any, scal
             p = torch.softmax(s, -1)
         res[r0: r0 + n] = torch.einsum("hij,jhd->ihd", p, v)
     out.copy_(res.view(t, hq * dv).to(out.dtype))
+
+
+def pair_combine(x, factor, eps, mult, out, heads, dv, rows_of=None) -> None:
+    y = x.float().reshape(-1, heads, 2, dv)
+    o = y[:, :, 0] - factor.float() * y[:, :, 1]
+    o = o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + eps) * mult
+    flat = out.view(-1, heads, dv)
+    if rows_of is None:
+        flat.copy_(o.to(out.dtype))
+    else:
+        rows = rows_of[1].cu_query_lens.long()[rows_of[0].long()]
+        flat[rows] = o[rows].to(out.dtype)
 
 
 def talking_attention(q, k_cache, v_cache, page_size, block_tables, ctx: Any, scale, window, softcap, talk, out,
@@ -236,6 +262,23 @@ def act_mul(gate_up, out, activation, limit=0.0, bias=None) -> None:
     out.copy_((a * u).to(out.dtype))
 
 
+def activate(x, activation) -> None:
+    z = x.float()
+    if activation == "gelu":
+        y = 0.5 * z * (1 + torch.erf(z / math.sqrt(2)))
+    elif activation == "gelu_tanh":
+        y = 0.5 * z * (1 + torch.tanh(math.sqrt(2 / math.pi) * (z + 0.044715 * z ** 3)))
+    else:
+        y = z * torch.sigmoid(z)
+    x.copy_(y.to(x.dtype))
+
+
+def gemm_activated(x, w, out, activation) -> None:
+    y = x.float() @ w.float().t()
+    activate(y, activation)
+    out.copy_(y.to(out.dtype))
+
+
 def gemm_biased_swiglu(x, w_gate_up, bias, out, arena=None) -> None:
     act_mul(x.float() @ w_gate_up.float().t(), out, "silu", bias=bias)
 
@@ -252,9 +295,12 @@ def softcap(logits, cap) -> None:
     logits.copy_(cap * torch.tanh(logits / cap))
 
 
-def head_norm_gate(x, weight, weight_per_head, gate, normalise, eps, out, gate_per_head=False, gate_silu=False) -> None:
+def head_norm_gate(x, weight, weight_per_head, gate, normalise, eps, out, gate_per_head=False, gate_silu=False, gate_first=False) -> None:
     t, heads, w = x.shape
     y = x.float()
+    if gate_first:
+        z = gate.float().reshape(t, heads, w)
+        y, gate = y * (z * torch.sigmoid(z) if gate_silu else torch.sigmoid(z)), None
     if normalise:
         y = y * torch.rsqrt(y.pow(2).mean(-1, keepdim=True) + eps)
     if weight is not None:
@@ -470,20 +516,22 @@ def delta_scan(qkv, q_off, k_off, v_off, a, dt_bias, a_log, beta_pre, q_scale, s
             st[h] = S
 
 
-def causal_conv_silu(x, taps, state, ctx, out) -> None:
+def causal_conv_silu(x, taps, state, ctx, out, bias=None) -> None:
     cu, slots = ctx.cu_query_lens.tolist(), ctx.state_slots.tolist()
     c, k = taps.shape
     for b in range(ctx.num_seqs):
         lo, hi = cu[b], cu[b + 1]
         seq = torch.cat([state[slots[b]].view(k - 1, c), x[lo:hi].float()])
         y = sum(seq[j: j + hi - lo] * taps[:, j].float()[None, :] for j in range(k))
+        if bias is not None:
+            y = y + bias.float()
         out[lo:hi] = y * torch.sigmoid(y)
         if k > 1:
             state[slots[b]] = seq[-(k - 1):].reshape(-1)
 
 
 def qkv_prepare(q_in, k_in, v_in, q_weight, k_weight, eps, cos, sin, rotary_dim, slots, k_cache, v_cache, page_size,
-                heads, kv_heads, d, dv, q_out, q_bias=None, k_bias=None, v_bias=None, norm_whole=False) -> None:
+                heads, kv_heads, d, dv, q_out, q_bias=None, k_bias=None, v_bias=None, norm_whole=False, maps=1) -> None:
     t = q_out.shape[0]
 
     def prep(x, w, n, bias=None):
@@ -500,7 +548,7 @@ def qkv_prepare(q_in, k_in, v_in, q_weight, k_weight, eps, cos, sin, rotary_dim,
     if k_in is None:
         return
     page, off = slots.long() // page_size, slots.long() % page_size
-    k_cache[page, :, off] = prep(k_in, k_weight, kv_heads, k_bias).to(k_cache.dtype)
+    k_cache[page, :, off] = prep(k_in, k_weight, kv_heads * maps, k_bias).reshape(t, kv_heads, maps * d).to(k_cache.dtype)
     v = v_in.reshape(t, kv_heads, dv)
     if v_bias is not None:
         v = (v.float() + v_bias.float().view(kv_heads, dv)).to(v_cache.dtype)
@@ -603,6 +651,22 @@ def linear_scan_rotated(q, k, v, decay, cos, sin, rotary_dim, interleaved, k_sca
         st.copy_(S)
 
 
+def state_space_scan(c, b, x, dt_pre, dt_bias, a_log, skip, state, ctx, heads, groups, d, dv, out) -> None:
+    cu, slots = ctx.cu_query_lens.tolist(), ctx.state_slots.tolist()
+    t, ty, per = c.shape[0], state.dtype, heads // groups
+    cc = c.to(ty).reshape(t, groups, d).repeat_interleave(per, 1)
+    bb = b.to(ty).reshape(t, groups, d).repeat_interleave(per, 1)
+    xx = x.to(ty).reshape(t, heads, dv)
+    dt = torch.nn.functional.softplus(dt_pre.to(ty) + dt_bias.to(ty), threshold=50.0)
+    decay = torch.exp(-torch.exp(a_log.to(ty)) * dt)
+    for n in range(ctx.num_seqs):
+        S = state[slots[n]].view(heads, d, dv).clone()
+        for i in range(cu[n], cu[n + 1]):
+            S = decay[i][:, None, None] * S + (dt[i][:, None] * bb[i])[:, :, None] * xx[i][:, None, :]
+            out[i] = torch.einsum("hkv,hk->hv", S, cc[i]) + skip.to(ty)[:, None] * xx[i]
+        state[slots[n]] = S.reshape(-1)
+
+
 def rms_norm_rows(x, weight, eps, out) -> None:
     y = x.float()
     out.copy_((y * torch.rsqrt(y.pow(2).mean(-1, keepdim=True) + eps) * weight.float()).to(out.dtype))
@@ -621,8 +685,11 @@ def token_shift_mix(x, mu, state, ctx, out) -> None:
 
 
 # ------------------------------------------------------- around the residual stream
-def embed_pos_norm(tokens, positions, table, pos_table, norm_weight, eps, out, scale=1.0) -> None:
+def embed_pos_norm(tokens, positions, table, pos_table, norm_weight, eps, out, scale=1.0, freq=None) -> None:
     x = table[tokens.long()].float() * scale
+    if freq is not None:
+        a = positions.double()[:, None] * freq[None, :]
+        x = x + torch.stack([a.sin(), a.cos()], -1).flatten(1)[:, : x.shape[1]].float()
     if pos_table is not None:
         x = x + pos_table[positions.long()].float()
     if norm_weight is not None:
@@ -639,6 +706,11 @@ def stream_sum(resid, terms, scales, bias=None, bias_scale=1.0, copy=None) -> No
     resid.copy_(x)
     if copy is not None:
         copy.copy_(x.to(copy.dtype))
+
+
+def stream_beside(resid, delta, origin, out) -> None:
+    x = resid if delta is None else resid + delta.float()
+    out.copy_(torch.cat([x, origin], -1).to(out.dtype))
 
 
 def add_bias(y, bias) -> None:
@@ -727,7 +799,8 @@ _NAMES = ["embed", "add_rms_norm", "rope_tables", "silu_mul", "qk_norm_rope_writ
           "post_norm_add_rms_norm", "latent_prepare", "latent_attention", "bmm", "transpose01", "moe_max_tiles", "moe_tile_rows", "moe_route_from",
           "moe_route", "moe_gemm", "moe_combine", "linear_scan_bonus", "linear_scan_decay", "token_shift_mix",
           "embed_pos_norm", "stream_sum", "add_bias", "tanh_", "act_mul_gather", "gemm_biased_swiglu", "linear_scan_gated",
-          "rms_norm_rows", "qkv_rotate", "talking_attention", "linear_scan_rotated"]
+          "rms_norm_rows", "qkv_rotate", "talking_attention", "linear_scan_rotated", "pair_combine", "activate", "gemm_activated", "state_space_scan",
+          "stream_beside"]
 
 
 @contextmanager

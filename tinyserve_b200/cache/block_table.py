@@ -4,7 +4,8 @@ Position ``p`` lives in ``pages[p // page_size]`` at offset ``p % page_size`` (u
 src/tinyserve/block_table.py:19-89). For a group that only needs a window of the positions,
 pages the window has passed are given back early and their entries become ``RELEASED``;
 pages that hold any of the first ``keep_first`` positions (which stay visible whatever the window)
-are never given back early.
+are never given back early. Where positions read only their own run of ``chunk`` positions, the pages
+of finished runs are given back.
 """
 
 from __future__ import annotations
@@ -17,12 +18,13 @@ RELEASED = -1
 
 
 class BlockTable:
-    def __init__(self, allocator: PageAllocator, page_size: int, window: int | None = None, keep_first: int = 0) -> None:
+    def __init__(self, allocator: PageAllocator, page_size: int, window: int | None = None, keep_first: int = 0,
+                 chunk: int | None = None) -> None:
         if page_size <= 0:
             raise ValueError(f"page_size must be positive, got {page_size}")
         self.allocator = allocator
         self.page_size = page_size
-        self.window = window
+        self.window, self.chunk = window, chunk
         self.kept_pages = -(-max(int(keep_first), 0) // page_size)    # pages at the front that a window never drops
         self.pages: list[int] = []
         self.num_tokens = 0
@@ -78,10 +80,14 @@ class BlockTable:
 
     def release_passed(self) -> int:
         """Give back pages that no later query can see: the next query is at position
-        ``num_tokens`` and sees positions above ``num_tokens - window``. Returns how many."""
-        if self.window is None:
+        ``num_tokens`` and sees positions above ``num_tokens - window``, or those of its own chunk.
+        Returns how many."""
+        if self.window is not None:
+            first_needed = self.num_tokens - self.window + 1     # lowest position still visible
+        elif self.chunk is not None:
+            first_needed = self.num_tokens // self.chunk * self.chunk
+        else:
             return 0
-        first_needed = self.num_tokens - self.window + 1     # lowest position still visible
         if first_needed <= 0:
             return 0
         upto = min(first_needed // self.page_size, len(self.pages))

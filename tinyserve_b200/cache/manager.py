@@ -7,7 +7,7 @@ manager serves the two families through their own methods (``allocate``, ``entry
 
 Users with equal paged needs share a **page group**: one pool of pages, one allocator and, per
 request, one block table. Groups with different needs (all positions, a window of them, another
-layout) have pages of their own, so a window group can give pages back early without disturbing
+layout) have pages of their own, so a window (or chunk) group can give pages back early without disturbing
 the others, and a pool of its own size: a request never holds more pages of a window group than
 its window and one step's tokens cover, so such a group is given only as many pages as
 ``max_requests`` requests can hold at once (when the step's token budget is known). Every user of
@@ -68,9 +68,9 @@ class PageGroup:
         with a window, those that the window and one step's tokens cover (before the pages the
         window has passed are given back after the step)."""
         pages = -(-num_tokens // self.page_size)
-        if self.need.window is not None:
+        if self.need.span is not None:
             kept = -(-self.need.keep_first // self.page_size)
-            pages = min(pages, -(-(self.need.window + min(step_tokens, num_tokens)) // self.page_size) + 1 + kept)
+            pages = min(pages, -(-(self.need.span + min(step_tokens, num_tokens)) // self.page_size) + 1 + kept)
         return pages
 
 
@@ -127,8 +127,8 @@ class CacheManager:
             sizes = [num_pages] * len(distinct)
             if max_step_tokens is not None:
                 for i, need in enumerate(distinct):
-                    if need.window is not None:
-                        per_request = -(-(need.window + max_step_tokens) // page_size) + 1 + -(-need.keep_first // page_size)
+                    if need.span is not None:
+                        per_request = -(-(need.span + max_step_tokens) // page_size) + 1 + -(-need.keep_first // page_size)
                         sizes[i] = min(num_pages, max_requests * per_request)
         else:
             sizes = [int(n) for n in num_pages]
@@ -200,7 +200,7 @@ class CacheManager:
             slot = self.state_pool.allocate()
             for storage in self._slot_storage:
                 storage[slot].zero_()
-        tables = [BlockTable(g.allocator, g.page_size, g.need.window, g.need.keep_first) for g in self.groups]
+        tables = [BlockTable(g.allocator, g.page_size, g.need.window, g.need.keep_first, g.need.chunk) for g in self.groups]
         self._next_uid += 1
         return RequestCache(tables, slot, uid=self._next_uid)
 
@@ -235,8 +235,8 @@ class CacheManager:
 
     @property
     def capacity_tokens(self) -> int:
-        """Tokens of one request that the smallest group without a window holds."""
-        full = [g.num_pages for g in self.groups if g.need.window is None]
+        """Tokens of one request that the smallest group without a window or chunks holds."""
+        full = [g.num_pages for g in self.groups if g.need.span is None]
         return (min(full) if full else self.num_pages) * self.page_size
 
     def append(self, req: RequestCache, n: int) -> None:

@@ -27,7 +27,29 @@ struct AttnArgs {
   const float* sinks = nullptr;  // [num_heads] a logit per head that joins the softmax's denominator without a value
   int v_head_dim = 0;            // size of a value head when it differs from head_dim (0: the same)
   int keep_first = 0;            // with a window: positions below this stay visible to every later query
+  int chunk = 0;                 // c > 0 (without a window): a query sees its own run of c positions, counted from position 0
+  // 2: every query head and every cached key row holds two maps side by side (head_dim / 2 elements each) over the same
+  // values. `num_heads` counts (head, map) pairs, map innermost; a pair scores with its own half of both rows.
+  int maps = 1;
+  // Two maps, kernels that finish a head themselves: out = (a1 - *mix_factor a2) / rms(.) * mix_mult per head
+  const float* mix_factor = nullptr;
+  float mix_mult = 1.f, mix_eps = 0.f;
 };
+
+// The row of q (in rows of head_dim elements) that holds a (head, map) pair of a token, and whether column c of it
+// (all of an aligned run of 8 columns alike) belongs to that pair.
+__device__ __forceinline__ size_t q_row_of(size_t token, int pair, const AttnArgs& a) {
+  return a.maps == 2 ? token * (a.num_heads >> 1) + (pair >> 1) : token * a.num_heads + pair;
+}
+__device__ __forceinline__ bool q_col_lives(int pair, int c, int head_dim, const AttnArgs& a) {
+  return a.maps != 2 || (2 * c >= head_dim) == ((pair & 1) != 0);
+}
+
+// The first position that a query at position p sees (the kept first positions of a window apart).
+__device__ __forceinline__ int first_visible(int p, const AttnArgs& a) {
+  if (a.window > 0) return max(0, p - a.window + 1);
+  return a.chunk > 0 ? p / a.chunk * a.chunk : 0;
+}
 
 // The finished row: num / den, where the denominator also takes 2^(sink - max) when the head has
 // a sink logit (given in natural units; the running maximum `mx` is in base-2 units).

@@ -93,7 +93,7 @@ __global__ void __launch_bounds__(DM_THREADS) decode_attn_mma_kernel(AttnArgs a,
   const int seq = a.seq_ids[si];
   const int ctx = a.ctx_lens[seq];
   const int qrow = a.cu_q[seq];
-  const int lo = (a.window > 0) ? max(0, ctx - a.window) : 0;
+  const int lo = first_visible(ctx - 1, a);
   const int lo_al = lo & ~(DM_TK - 1);
   const int ntiles_all = (ctx - lo_al + DM_TK - 1) / DM_TK;
   const int tiles_per = (ntiles_all + a.num_splits - 1) / a.num_splits;
@@ -106,7 +106,6 @@ __global__ void __launch_bounds__(DM_THREADS) decode_attn_mma_kernel(AttnArgs a,
   // ---- Q fragments: row r = query head g0 + r of the group (rows beyond the group are zero)
   uint32_t qf[D16][4];
   {
-    const bf16* qbase = (const bf16*)a.q + ((size_t)qrow * a.num_heads + kvh * G + g0) * D;
 #pragma unroll
     for (int kk = 0; kk < D16; ++kk) {
 #pragma unroll
@@ -114,8 +113,10 @@ __global__ void __launch_bounds__(DM_THREADS) decode_attn_mma_kernel(AttnArgs a,
         const int r = g + 8 * h;
         uint32_t lo_w = 0u, hi_w = 0u;
         if (r < ng) {
-          lo_w = *reinterpret_cast<const uint32_t*>(qbase + (size_t)r * D + kk * 16 + 2 * t);
-          hi_w = *reinterpret_cast<const uint32_t*>(qbase + (size_t)r * D + kk * 16 + 8 + 2 * t);
+          const int pair = kvh * G + g0 + r;
+          const bf16* qr = (const bf16*)a.q + q_row_of(qrow, pair, a) * D;
+          if (q_col_lives(pair, kk * 16, D, a)) lo_w = *reinterpret_cast<const uint32_t*>(qr + kk * 16 + 2 * t);
+          if (q_col_lives(pair, kk * 16 + 8, D, a)) hi_w = *reinterpret_cast<const uint32_t*>(qr + kk * 16 + 8 + 2 * t);
         }
         qf[kk][h] = lo_w;
         qf[kk][2 + h] = hi_w;
@@ -317,11 +318,12 @@ using namespace ts;
 extern "C" int ts_decode_attention_mma(
     const void* q, void* out, const void* k_cache, const void* v_cache, const int* block_tables,
     int table_width, const int* cu_q, const int* ctx_lens, const int* decode_seqs, int num_decode,
-    int num_heads, int num_kv_heads, int head_dim, int page_size, float scale, int window, int num_splits,
+    int num_heads, int num_kv_heads, int head_dim, int page_size, float scale, int window, int chunk, int maps, int num_splits,
     float* part_acc, float* part_ml, int* error_flag, cudaStream_t stream) {
   if (num_decode <= 0) return 0;
   if (head_dim <= 0 || head_dim % 16 != 0 || head_dim > 128 || error_flag == nullptr) return TS_ERR_UNSUPPORTED;
-  if (num_kv_heads <= 0 || num_heads % num_kv_heads != 0 || page_size <= 0 || window < 0 || num_splits < 1 || num_splits > ATTN_MAX_SPLITS)
+  if (maps != 1 && (maps != 2 || num_heads % 2)) return TS_ERR_BAD_ARGUMENT;
+  if (num_kv_heads <= 0 || num_heads % num_kv_heads != 0 || page_size <= 0 || window < 0 || chunk < 0 || (window > 0 && chunk > 0) || num_splits < 1 || num_splits > ATTN_MAX_SPLITS)
     return TS_ERR_BAD_ARGUMENT;
   if (num_splits > 1 && (part_acc == nullptr || part_ml == nullptr)) return TS_ERR_BAD_ARGUMENT;
   if ((((uintptr_t)k_cache) | ((uintptr_t)v_cache)) & 15) return TS_ERR_UNSUPPORTED;
@@ -332,7 +334,7 @@ extern "C" int ts_decode_attention_mma(
   a.num_heads = num_heads; a.num_kv_heads = num_kv_heads; a.head_dim = head_dim; a.page_size = page_size;
   a.page_shift = page_shift_of(page_size);
   a.scale_log2 = scale * 1.4426950408889634f;
-  a.window = window;
+  a.window = window; a.chunk = chunk; a.maps = maps;
   a.num_splits = num_splits; a.part_acc = part_acc; a.part_ml = part_ml;
   switch (head_dim / 16) {
     case 1: return launch_dm<1>(a, error_flag, stream);

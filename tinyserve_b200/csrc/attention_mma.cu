@@ -76,7 +76,7 @@ __global__ void __launch_bounds__(MA_THREADS) prefill_attn_mma_kernel(AttnArgs a
 
   const int qpos_first = first_pos + q0;
   const int qpos_last = first_pos + q0 + ntok - 1;
-  const int k_lo = (a.window > 0) ? max(0, qpos_first - a.window + 1) : 0;
+  const int k_lo = first_visible(qpos_first, a);
   const int k_begin = (k_lo / MA_BN) * MA_BN;
   const int num_tiles = (qpos_last - k_begin) / MA_BN + 1;
 
@@ -86,7 +86,7 @@ __global__ void __launch_bounds__(MA_THREADS) prefill_attn_mma_kernel(AttnArgs a
     uint4 v = make_uint4(0u, 0u, 0u, 0u);
     if (r < nrows) {
       const int tok = q0 + r / ge, head = head0 + r % ge;
-      v = *reinterpret_cast<const uint4*>(q + ((size_t)(row0 + tok) * a.num_heads + head) * D + c * 8);
+      if (q_col_lives(head, c * 8, D, a)) v = *reinterpret_cast<const uint4*>(q + q_row_of(row0 + tok, head, a) * D + c * 8);
     }
     *reinterpret_cast<uint4*>(Qs + r * DS + c * 8) = v;
   }
@@ -123,16 +123,18 @@ __global__ void __launch_bounds__(MA_THREADS) prefill_attn_mma_kernel(AttnArgs a
   }
 
   // rows of this thread: warp * 16 + g and + 8
-  int qpos[2];
+  int qpos[2], qfirst[2];                                // position, and the first position seen from it
   bool rvalid[2];
 #pragma unroll
   for (int h = 0; h < 2; ++h) {
     const int r = warp * 16 + g + 8 * h;
     rvalid[h] = r < nrows;
     qpos[h] = first_pos + q0 + r / ge;
+    qfirst[h] = first_visible(qpos[h], a);
   }
   const int warp_last_row = min(warp * 16 + 15, nrows - 1);
   const int warp_qpos_max = first_pos + q0 + max(warp_last_row, 0) / ge;
+  const int warp_first_max = first_visible(warp_qpos_max, a);
   const bool warp_active = warp * 16 < nrows;
   const int warp_qpos_min = first_pos + q0 + (warp * 16) / ge;
 
@@ -173,7 +175,7 @@ __global__ void __launch_bounds__(MA_THREADS) prefill_attn_mma_kernel(AttnArgs a
       // ---- scale, mask, online softmax. A tile that every row of the warp sees whole needs no
       //      mask (rows beyond the tile's last have zero queries and finite scores).
       float mx[2] = {-INFINITY, -INFINITY};
-      const bool whole = (k0 + MA_BN - 1 <= warp_qpos_min) && (a.window == 0 || k0 > warp_qpos_max - a.window);
+      const bool whole = (k0 + MA_BN - 1 <= warp_qpos_min) && k0 >= warp_first_max;
       if (whole) {
 #pragma unroll
         for (int i = 0; i < 8; ++i)
@@ -190,8 +192,7 @@ __global__ void __launch_bounds__(MA_THREADS) prefill_attn_mma_kernel(AttnArgs a
           for (int e = 0; e < 4; ++e) {
             const int h = e >> 1;
             const int kpos = k0 + i * 8 + 2 * t + (e & 1);
-            bool ok = rvalid[h] && kpos <= qpos[h];
-            if (a.window > 0) ok = ok && (kpos > qpos[h] - a.window);
+            const bool ok = rvalid[h] && kpos <= qpos[h] && kpos >= qfirst[h];
             const float v = ok ? s[i][e] * a.scale_log2 : -INFINITY;
             s[i][e] = v;
             mx[h] = fmaxf(mx[h], v);
@@ -289,10 +290,11 @@ extern "C" int ts_prefill_attention_mma(
     const void* q, void* out, const void* k_cache, const void* v_cache, const int* block_tables,
     int table_width, const int* cu_q, const int* ctx_lens, const int* prefill_seqs, int num_prefill,
     int max_query_len, int num_heads, int num_kv_heads, int head_dim, int page_size, float scale,
-    int window, cudaStream_t stream) {
+    int window, int chunk, int maps, cudaStream_t stream) {
   if (num_prefill <= 0) return 0;
   if (head_dim <= 0 || head_dim % 16 != 0 || head_dim > 128) return TS_ERR_UNSUPPORTED;
-  if (num_kv_heads <= 0 || num_heads % num_kv_heads != 0 || page_size <= 0 || window < 0) return TS_ERR_BAD_ARGUMENT;
+  if (maps != 1 && (maps != 2 || num_heads % 2)) return TS_ERR_BAD_ARGUMENT;
+  if (num_kv_heads <= 0 || num_heads % num_kv_heads != 0 || page_size <= 0 || window < 0 || chunk < 0 || (window > 0 && chunk > 0)) return TS_ERR_BAD_ARGUMENT;
   AttnArgs a;
   a.q = q; a.out = out; a.k_cache = k_cache; a.v_cache = v_cache;
   a.block_tables = block_tables; a.table_width = table_width; a.cu_q = cu_q; a.ctx_lens = ctx_lens;
@@ -300,7 +302,7 @@ extern "C" int ts_prefill_attention_mma(
   a.num_heads = num_heads; a.num_kv_heads = num_kv_heads; a.head_dim = head_dim; a.page_size = page_size;
   a.page_shift = page_shift_of(page_size);
   a.scale_log2 = scale * 1.4426950408889634f;
-  a.window = window;
+  a.window = window; a.chunk = chunk; a.maps = maps;
   a.num_splits = 1; a.part_acc = nullptr; a.part_ml = nullptr;
   switch (head_dim / 16) {
     case 1: return launch_mma<1>(a, max_query_len, stream);

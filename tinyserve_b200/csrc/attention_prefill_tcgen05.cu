@@ -80,10 +80,15 @@ __device__ __forceinline__ bool fa_warp_wait(uint64_t* bar, uint32_t parity, vol
   return __all_sync(0xffffffffu, mbar_wait_or_fail(bar, parity, failed) ? 1 : 0) != 0;
 }
 
-template <int D64, int NQ>
+// PAIR: the two "heads" of a CTA are the two maps of one query head (AttnArgs::maps). Its row of q and every key row hold
+// both maps side by side, 64 columns each, and the values are shared, so the tiles are those of one head of 128; map q's
+// scores come from the q-th 64 columns of both operands (half the instructions of a head of 128). The head is finished
+// here: O1 / l1 - factor O2 / l2, divided by its root mean square over the head.
+template <int D64, int NQ, bool PAIR = false>
 struct FaLayout {
   static constexpr int D = 64 * D64;
-  static constexpr int STAGES = NQ == 1 ? 3 : 2;              // K / V tiles in flight
+  static_assert(!PAIR || (D64 == 2 && NQ == 2), "two maps of 64 columns over values of 128");
+  static constexpr int STAGES = NQ == 1 || PAIR ? 3 : 2;      // K / V tiles in flight
   static constexpr int SPB = NQ == 1 ? 2 : 1;                 // score / probability buffers per head
   // softmax warps per quarter of the rows, each with BN / HS of a tile's columns: two with one head (the
   // softmax of a tile is the pace there, and two threads per row halve it); with two heads the register
@@ -95,7 +100,7 @@ struct FaLayout {
   static constexpr uint32_t Q_BYTES = FA_BM * D * 2;          // per head
   static constexpr uint32_t KV_BYTES = FA_BN * D * 2;         // one K or V tile
   static constexpr uint32_t OFF_Q = 0;
-  static constexpr uint32_t OFF_K = OFF_Q + NQ * Q_BYTES;
+  static constexpr uint32_t OFF_K = OFF_Q + (PAIR ? 1 : NQ) * Q_BYTES;
   static constexpr uint32_t OFF_V = OFF_K + STAGES * KV_BYTES;
   static constexpr uint32_t TOTAL = OFF_V + STAGES * KV_BYTES;
   // tensor memory columns: the score / probability buffers of every head, then the outputs
@@ -104,12 +109,13 @@ struct FaLayout {
 };
 
 // D64 = head_dim / 64; BR = rows of a tensor box (16, or 8 for pages of 8); NQ = heads per CTA.
+// CHUNKED: compiled with the mask of chunks too (AttnArgs::chunk); the others, which are short of registers, are not.
 // blockIdx = (group of NQ query heads, tile of 128 tokens counted from the end, request in the list).
-template <int D64, int BR, int NQ>
+template <int D64, int BR, int NQ, bool PAIR, bool CHUNKED>
 __global__ void __launch_bounds__((4 * (NQ == 1 ? 2 : 1) * NQ + 2 * (NQ == 1 ? 2 : 1) + 1) * 32) prefill_attn_tc_kernel(const __grid_constant__ CUtensorMap map_k,
                                                                             const __grid_constant__ CUtensorMap map_v,
                                                                             AttnArgs a, int* error_flag) {
-  using L = FaLayout<D64, NQ>;
+  using L = FaLayout<D64, NQ, PAIR>;
   constexpr int D = L::D, BN = FA_BN, FA_KV_STAGES = L::STAGES, SPB = L::SPB, FA_SOFTMAX_WARPS = L::SOFTMAX_WARPS, HS = L::HS, PW = L::PW;
   constexpr int HC = BN / HS;                                  // score columns of one softmax thread
   // instruction descriptors: D = f32, A = B = bf16, M = 128; S: N = BN, both operands K-major;
@@ -138,7 +144,7 @@ __global__ void __launch_bounds__((4 * (NQ == 1 ? 2 : 1) * NQ + 2 * (NQ == 1 ? 2
   const int valid = min(FA_BM, q_len - q0);
   const int p_lo = ctx - q_len + q0;                          // position of row 0
   const int p_hi = p_lo + valid - 1;                          // position of the last live row
-  const int lo = a.window > 0 ? max(0, p_lo - a.window + 1) : 0;   // first key any row sees
+  const int lo = CHUNKED ? first_visible(p_lo, a) : a.window > 0 ? max(0, p_lo - a.window + 1) : 0;   // first key any row sees
   const int t_begin = lo / BN;
   // With kept first keys (positions below keep_first stay visible whatever the window) the tiles that
   // hold any of them and lie in front of the window's first tile come first; the others follow.
@@ -146,7 +152,7 @@ __global__ void __launch_bounds__((4 * (NQ == 1 ? 2 : 1) * NQ + 2 * (NQ == 1 ? 2
   const int kept_tiles = min(t_begin, (kept + BN - 1) / BN);
   const int n_tiles = (p_hi + 1 + BN - 1) / BN - t_begin + kept_tiles;     // >= 1
   auto tile_of = [&](int j) -> int { return j < kept_tiles ? j : t_begin + j - kept_tiles; };
-  const int head0 = (int)blockIdx.x * NQ;
+  const int head0 = (int)blockIdx.x * NQ;                     // PAIR: the (head, map) pairs 2 head and 2 head + 1
   const int kvh = head0 / (a.num_heads / a.num_kv_heads);
 
   pdl_trigger();
@@ -175,21 +181,23 @@ __global__ void __launch_bounds__((4 * (NQ == 1 ? 2 : 1) * NQ + 2 * (NQ == 1 ? 2
     const int q = warp / (4 * HS), half = (warp / 4) % HS, quad = warp & 3;
     const int head = head0 + q;
     const int r = quad * 32 + lane;                            // this thread's row
-    unsigned char* q_tile = smem + L::OFF_Q + q * L::Q_BYTES;
+    unsigned char* q_tile = smem + L::OFF_Q + (PAIR ? 0 : q) * L::Q_BYTES;
     {
       // Q rows into the swizzled operand layout: 16 (or 8) threads fetch a row, 16 bytes each
       constexpr int TPH = 128 * HS;                            // softmax threads of a head
-      constexpr int CPR = D / 8;                               // 16-byte chunks per row
+      constexpr int CPR = (PAIR ? D / 2 : D) / 8;              // 16-byte chunks per row (PAIR: of this map)
       constexpr int RPP = TPH / CPR, PASSES = FA_BM / RPP;     // rows per pass of the head's threads
       const int tq = threadIdx.x % TPH;
-      const int c = tq % CPR, row0 = tq / CPR;
+      const int c = tq % CPR + (PAIR ? q * CPR : 0), row0 = tq / CPR;
       uint4 v[PASSES];
 #pragma unroll
       for (int i = 0; i < PASSES; ++i) {                       // every load in flight before the first store
         const int row = row0 + i * RPP;
         v[i] = make_uint4(0u, 0u, 0u, 0u);
         if (row < valid)
-          v[i] = *reinterpret_cast<const uint4*>((const bf16*)a.q + ((size_t)(q_start + q0 + row) * a.num_heads + head) * D + c * 8);
+          v[i] = *reinterpret_cast<const uint4*>(
+              (const bf16*)a.q + (PAIR ? (size_t)(q_start + q0 + row) * (a.num_heads >> 1) + (head >> 1)
+                                       : (size_t)(q_start + q0 + row) * a.num_heads + head) * D + c * 8);
       }
 #pragma unroll
       for (int i = 0; i < PASSES; ++i) {
@@ -245,10 +253,11 @@ __global__ void __launch_bounds__((4 * (NQ == 1 ? 2 : 1) * NQ + 2 * (NQ == 1 ? 2
 #pragma unroll
         for (int c = 0; c < HC / 32; ++c) tmem_ld_32_nowait(tmem_sp + half * HC + c * 32, sraw + c * 32);
         tmem_ld_wait();
-        const bool edge = (k0 + HC - 1 > p_lo) || (a.window > 0 && k0 < p_lo + FA_BM - a.window);
+        const bool edge = (k0 + HC - 1 > p_lo) || (CHUNKED ? k0 < first_visible(p_lo + FA_BM - 1, a)
+                                                           : a.window > 0 && k0 < p_lo + FA_BM - a.window);
         float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};      // four chains: the maxima do not wait on one another
         if (edge) {
-          const int first = a.window > 0 ? p_abs - a.window + 1 : 0;
+          const int first = CHUNKED ? first_visible(p_abs, a) : a.window > 0 ? p_abs - a.window + 1 : 0;
 #pragma unroll
           for (int i = 0; i < HC; ++i) {
             const int kpos = k0 + i;
@@ -321,7 +330,59 @@ __global__ void __launch_bounds__((4 * (NQ == 1 ? 2 : 1) * NQ + 2 * (NQ == 1 ? 2
 #pragma unroll
       for (int h2 = 0; h2 < HS; ++h2) l_sum += sums[h2];      // in the order of the columns, the same in every warp
     }
-    if (ok && !stopped) {
+    if constexpr (PAIR) {
+      // Both maps' sums of a row meet; each of the two warps of a row quarter then finishes 64 of its 128 columns.
+      if (ok && !fa_warp_wait(&pv_done[q ^ 1][(n_tiles - 1) % SPB], ((n_tiles - 1) / SPB) & 1, failed)) ok = false;
+      auto meet = [&](float mine, bool mine_ok, float (&both)[2]) -> bool {
+        pair_value[q][quad][0][lane] = mine;
+        if (lane == 0) pair_ok[q][quad][0] = mine_ok ? 1 : 0;
+        pair_sync();
+        bool all_ok = true;
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+          both[i] = pair_value[i][quad][0][lane];
+          all_ok = all_ok && pair_ok[i][quad][0] != 0;
+        }
+        pair_sync();
+        return all_ok;
+      };
+      float inv[2], squares[2];
+      ok = meet(1.f / l_sum, ok, inv);
+      tc_fence_after();
+      const float minus = -*a.mix_factor * inv[1];
+      const uint32_t tmem_row = tmem_base + lane_addr + L::TMEM_O + (uint32_t)(q * (D / 2));
+      float val[D / 2];
+      float ss = 0.f;
+      if (ok) {
+#pragma unroll
+        for (int c = 0; c < D / 64; ++c) {
+          uint32_t o1[32], o2[32];
+          tmem_ld_32_nowait(tmem_row + c * 32, o1);
+          tmem_ld_32_nowait(tmem_row + D + c * 32, o2);
+          tmem_ld_wait();
+#pragma unroll
+          for (int i = 0; i < 32; ++i) {
+            const float v = fmaf(__uint_as_float(o2[i]), minus, __uint_as_float(o1[i]) * inv[0]);
+            val[c * 32 + i] = v;
+            ss = fmaf(v, v, ss);
+          }
+        }
+      }
+      ok = meet(ss, ok, squares);
+      if (ok && r < valid) {
+        const float by = rsqrtf((squares[0] + squares[1]) / (float)D + a.mix_eps) * a.mix_mult;
+        bf16* dst = (bf16*)a.out + ((size_t)(q_start + q0 + r) * (a.num_heads >> 1) + (head >> 1)) * D + q * (D / 2);
+#pragma unroll
+        for (int i = 0; i < D / 2; i += 8) {
+          uint4 v;
+          v.x = fa_pack(val[i + 0] * by, val[i + 1] * by);
+          v.y = fa_pack(val[i + 2] * by, val[i + 3] * by);
+          v.z = fa_pack(val[i + 4] * by, val[i + 5] * by);
+          v.w = fa_pack(val[i + 6] * by, val[i + 7] * by);
+          *reinterpret_cast<uint4*>(dst + i) = v;
+        }
+      }
+    } else if (ok && !stopped) {
       tc_fence_after();
       // a head's sink logit joins the denominator: 2^(sink - m) beside the sum of the 2^(s - m)
       const float inv = 1.f / (l_sum + (a.sinks ? exp2f(a.sinks[head] * 1.4426950408889634f - m_used) : 0.f));
@@ -416,10 +477,11 @@ __global__ void __launch_bounds__((4 * (NQ == 1 ? 2 : 1) * NQ + 2 * (NQ == 1 ? 2
       const int st = j % FA_KV_STAGES, bq = q * SPB + j % SPB;
       if (lane == 0) {
 #pragma unroll
-        for (int ks = 0; ks < D / 16; ++ks) {
-          const uint64_t ad = sw128_desc(q_addr + q * L::Q_BYTES + (ks >> 2) * (FA_BM * 128) + (ks & 3) * 32);
+        for (int i = 0; i < (PAIR ? 4 : D / 16); ++i) {
+          const int ks = PAIR ? 4 * q + i : i;
+          const uint64_t ad = sw128_desc(q_addr + (PAIR ? 0 : q) * L::Q_BYTES + (ks >> 2) * (FA_BM * 128) + (ks & 3) * 32);
           const uint64_t bd = sw128_desc(k_addr + st * L::KV_BYTES + (ks >> 2) * (BN * 128) + (ks & 3) * 32);
-          umma_bf16(tmem_base + L::TMEM_SP + (uint32_t)(bq * BN), ad, bd, IDESC_S, ks != 0);
+          umma_bf16(tmem_base + L::TMEM_SP + (uint32_t)(bq * BN), ad, bd, IDESC_S, i != 0);
         }
         umma_commit(&s_full[q][j % SPB]);
         if (q == NQ - 1) umma_commit(&k_empty[st]);       // the K stage is free once the last head's S has read it
@@ -534,14 +596,14 @@ static const CUtensorMap* fa_cache_map(const void* base, long long rows, int hea
   return &maps.emplace(key, m).first->second;
 }
 
-template <int D64, int BR, int NQ>
+template <int D64, int BR, int NQ, bool PAIR = false, bool CHUNKED = false>
 static int launch_fa(const AttnArgs& a, long long cache_rows, int max_query_len, int* error_flag, cudaStream_t stream) {
-  using L = FaLayout<D64, NQ>;
+  using L = FaLayout<D64, NQ, PAIR>;
   const CUtensorMap* mk = fa_cache_map(a.k_cache, cache_rows, L::D, BR);
   const CUtensorMap* mv = fa_cache_map(a.v_cache, cache_rows, L::D, BR);
   if (mk == nullptr || mv == nullptr) return TS_ERR_UNSUPPORTED;
   const size_t smem = (size_t)L::TOTAL + 1024;
-  auto kern = prefill_attn_tc_kernel<D64, BR, NQ>;
+  auto kern = prefill_attn_tc_kernel<D64, BR, NQ, PAIR, CHUNKED>;
   cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   if (e != cudaSuccess) return (int)e;
   dim3 grid(a.num_heads / NQ, (max_query_len + FA_BM - 1) / FA_BM, a.num_seqs);
@@ -561,13 +623,17 @@ extern "C" int ts_prefill_attention_tcgen05(
     const void* q, void* out, const void* k_cache, const void* v_cache, long long num_pages_total,
     const int* block_tables, int table_width, const int* cu_q, const int* ctx_lens, const int* prefill_seqs,
     int num_prefill, int max_query_len, int num_heads, int num_kv_heads, int head_dim, int page_size, float scale,
-    int window, int heads_per_cta, int* error_flag, const float* sinks, int keep_first, cudaStream_t stream) {
+    int window, int heads_per_cta, int* error_flag, const float* sinks, int keep_first, int chunk, int maps,
+    const float* mix_factor, float mix_mult, float mix_eps, cudaStream_t stream) {
+  // `chunk` (without a window): a query sees its own run of that many positions. `maps` = 2 (head_dim = 128: two maps of 64):
+  // num_heads counts (head, map) pairs, q is [T, num_heads / 2, head_dim], and out [T, num_heads / 2, head_dim] receives
+  // the finished heads (AttnArgs::mix_factor).
   // `keep_first` (with a window): positions below it stay visible to every later query
   // `sinks` (optional, [num_heads] float): a logit per head that joins the softmax's denominator without a value
   if (num_prefill <= 0 || max_query_len <= 0) return 0;
   if ((head_dim != 64 && head_dim != 128) || error_flag == nullptr) return TS_ERR_UNSUPPORTED;
   if (!(page_size == 8 || (page_size > 0 && page_size % 16 == 0))) return TS_ERR_UNSUPPORTED;
-  if (num_kv_heads <= 0 || num_heads % num_kv_heads != 0 || window < 0 || keep_first < 0 || num_pages_total <= 0) return TS_ERR_BAD_ARGUMENT;
+  if (num_kv_heads <= 0 || num_heads % num_kv_heads != 0 || window < 0 || keep_first < 0 || chunk < 0 || (window > 0 && chunk > 0) || num_pages_total <= 0) return TS_ERR_BAD_ARGUMENT;
   if ((((uintptr_t)k_cache) | ((uintptr_t)v_cache) | ((uintptr_t)q) | ((uintptr_t)out)) & 15) return TS_ERR_UNSUPPORTED;
   const long long rows = num_pages_total * num_kv_heads * page_size;
   if (rows >= (1ll << 31)) return TS_ERR_UNSUPPORTED;
@@ -585,7 +651,21 @@ extern "C" int ts_prefill_attention_tcgen05(
   a.scale_log2 = scale * 1.4426950408889634f;
   a.window = window;
   a.keep_first = window > 0 ? keep_first : 0;
+  a.chunk = chunk; a.maps = maps; a.mix_factor = mix_factor; a.mix_mult = mix_mult; a.mix_eps = mix_eps;
   a.num_splits = 1; a.part_acc = nullptr; a.part_ml = nullptr;
+  if (maps == 2) {
+    if (head_dim != 128 || sinks != nullptr) return TS_ERR_UNSUPPORTED;
+    if (num_heads % 2 || mix_factor == nullptr) return TS_ERR_BAD_ARGUMENT;
+    return page_size == 8 ? launch_fa<2, 8, 2, true, true>(a, rows, max_query_len, error_flag, stream)
+                          : launch_fa<2, 16, 2, true, true>(a, rows, max_query_len, error_flag, stream);
+  }
+  if (chunk > 0) {
+    if (head_dim == 64)
+      return page_size == 8 ? launch_fa<1, 8, 1, false, true>(a, rows, max_query_len, error_flag, stream)
+                            : launch_fa<1, 16, 1, false, true>(a, rows, max_query_len, error_flag, stream);
+    return page_size == 8 ? launch_fa<2, 8, 1, false, true>(a, rows, max_query_len, error_flag, stream)
+                          : launch_fa<2, 16, 1, false, true>(a, rows, max_query_len, error_flag, stream);
+  }
 #define TS_FA(D64_, BR_)                                                                                \
   return heads_per_cta == 2 ? launch_fa<D64_, BR_, 2>(a, rows, max_query_len, error_flag, stream)       \
                             : launch_fa<D64_, BR_, 1>(a, rows, max_query_len, error_flag, stream)

@@ -117,7 +117,7 @@ __global__ void __launch_bounds__(PT_THREADS, 4) prefill_attn_tma_kernel(const _
     const int nrows = ntok * ge;
     const int qpos_first = first_pos + q0;
     const int qpos_last = first_pos + q0 + ntok - 1;
-    const int k_lo = (a.window > 0) ? max(0, qpos_first - a.window + 1) : 0;
+    const int k_lo = first_visible(qpos_first, a);
     const int k_begin = (k_lo / PT_BN) * PT_BN;
     const int num_tiles = (qpos_last - k_begin) / PT_BN + 1;
 
@@ -161,17 +161,19 @@ __global__ void __launch_bounds__(PT_THREADS, 4) prefill_attn_tma_kernel(const _
     }
     __syncthreads();
 
-    int qpos[2];
+    int qpos[2], qfirst[2];                              // position, and the first position seen from it
     bool rvalid[2];
 #pragma unroll
     for (int h = 0; h < 2; ++h) {
       const int r = warp * 16 + g + 8 * h;
       rvalid[h] = r < nrows;
       qpos[h] = first_pos + q0 + r / ge;
+      qfirst[h] = first_visible(qpos[h], a);
     }
     const int warp_last_row = min(warp * 16 + 15, nrows - 1);
     const int warp_qpos_max = first_pos + q0 + max(warp_last_row, 0) / ge;
     const int warp_qpos_min = first_pos + q0 + (warp * 16) / ge;
+    const int warp_first_max = first_visible(warp_qpos_max, a);
     const bool warp_active = warp * 16 < nrows;
 
     float o[2 * D16][4];
@@ -219,7 +221,7 @@ __global__ void __launch_bounds__(PT_THREADS, 4) prefill_attn_tma_kernel(const _
         }
         // ---- scale, mask, online softmax (a tile that every row of the warp sees whole needs no mask)
         float mx[2] = {-INFINITY, -INFINITY};
-        const bool whole = (k0 + PT_BN - 1 <= warp_qpos_min) && (a.window == 0 || k0 > warp_qpos_max - a.window);
+        const bool whole = (k0 + PT_BN - 1 <= warp_qpos_min) && k0 >= warp_first_max;
         if (whole) {
 #pragma unroll
           for (int i = 0; i < 4; ++i)
@@ -236,8 +238,7 @@ __global__ void __launch_bounds__(PT_THREADS, 4) prefill_attn_tma_kernel(const _
             for (int e = 0; e < 4; ++e) {
               const int h = e >> 1;
               const int kpos = k0 + i * 8 + 2 * t + (e & 1);
-              bool ok = rvalid[h] && kpos <= qpos[h];
-              if (a.window > 0) ok = ok && (kpos > qpos[h] - a.window);
+              const bool ok = rvalid[h] && kpos <= qpos[h] && kpos >= qfirst[h];
               const float v = ok ? s[i][e] * a.scale_log2 : -INFINITY;
               s[i][e] = v;
               mx[h] = fmaxf(mx[h], v);
@@ -379,11 +380,11 @@ extern "C" int ts_prefill_attention_tma(
     const void* q, void* out, const void* k_cache, const void* v_cache, long long num_pages_total,
     const int* block_tables, int table_width, const int* cu_q, const int* ctx_lens, const int* prefill_seqs,
     int num_prefill, int max_query_len, int num_heads, int num_kv_heads, int head_dim, int page_size, float scale,
-    int window, int* error_flag, cudaStream_t stream) {
+    int window, int chunk, int* error_flag, cudaStream_t stream) {
   if (num_prefill <= 0) return 0;
   if ((head_dim != 64 && head_dim != 128) || error_flag == nullptr) return TS_ERR_UNSUPPORTED;
   if (!(page_size == 8 || (page_size > 0 && page_size % 16 == 0))) return TS_ERR_UNSUPPORTED;
-  if (num_kv_heads <= 0 || num_heads % num_kv_heads != 0 || window < 0 || num_pages_total <= 0) return TS_ERR_BAD_ARGUMENT;
+  if (num_kv_heads <= 0 || num_heads % num_kv_heads != 0 || window < 0 || chunk < 0 || (window > 0 && chunk > 0) || num_pages_total <= 0) return TS_ERR_BAD_ARGUMENT;
   if ((((uintptr_t)k_cache) | ((uintptr_t)v_cache) | ((uintptr_t)q)) & 15) return TS_ERR_UNSUPPORTED;
   const long long rows = num_pages_total * num_kv_heads * page_size;
   if (rows >= (1ll << 31)) return TS_ERR_UNSUPPORTED;
@@ -394,7 +395,7 @@ extern "C" int ts_prefill_attention_tma(
   a.num_heads = num_heads; a.num_kv_heads = num_kv_heads; a.head_dim = head_dim; a.page_size = page_size;
   a.page_shift = page_shift_of(page_size);
   a.scale_log2 = scale * 1.4426950408889634f;
-  a.window = window;
+  a.window = window; a.chunk = chunk;
   a.num_splits = 1; a.part_acc = nullptr; a.part_ml = nullptr;
   if (head_dim == 64)
     return page_size == 8 ? launch_pt<1, 8>(a, rows, max_query_len, error_flag, stream)

@@ -3,7 +3,7 @@
 //
 // Math (upstream src/tinyserve/attention.py:89-111): s = scale * q.k over head_dim in 32-bit,
 // causal mask (key position <= query position; optionally > query position - window, or
-// below `keep_first`: the first positions that a window never drops),
+// below `keep_first`: the first positions that a window never drops; or in the query's own chunk),
 // softmax in 32-bit (online, base 2), o = sum p v in 32-bit, cast once to the output type.
 // Query head h reads kv head h / (num_heads / num_kv_heads).
 //
@@ -63,7 +63,7 @@ __global__ void __launch_bounds__(PF_THREADS) prefill_attn_kernel(AttnArgs a) {
   for (int idx = tid; idx < PF_TQ * D; idx += PF_THREADS) {
     const int r = idx / D, d = idx - r * D;
     float v = 0.f;
-    if (r < nq) v = to_float(q[((size_t)(row0 + q0 + r) * a.num_heads + head) * D + d]) * a.scale_log2;
+    if (r < nq && q_col_lives(head, d, D, a)) v = to_float(q[q_row_of(row0 + q0 + r, head, a) * D + d]) * a.scale_log2;
     Qs[r * DS + d] = v;
   }
   if (tid < PF_TQ) { row_m[tid] = NEG_INF; row_l[tid] = 0.f; }
@@ -78,8 +78,7 @@ __global__ void __launch_bounds__(PF_THREADS) prefill_attn_kernel(AttnArgs a) {
 
   const int qpos_first = first_pos + q0;
   const int qpos_last = first_pos + q0 + nq - 1;
-  int k_lo = 0;
-  if (a.window > 0) k_lo = max(0, qpos_first - a.window + 1);
+  const int k_lo = first_visible(qpos_first, a);
   const int k_begin = (k_lo / PF_TK) * PF_TK;
   // with kept first positions the tiles below the window that hold any of them come first
   const int kept = (a.window > 0) ? min(a.keep_first, k_lo) : 0;
@@ -144,11 +143,11 @@ __global__ void __launch_bounds__(PF_THREADS) prefill_attn_kernel(AttnArgs a) {
     for (int i = 0; i < 4; ++i) {
       const int r = ty * 4 + i;
       const int qpos = first_pos + q0 + r;
+      const int first = first_visible(qpos, a);
 #pragma unroll
       for (int j = 0; j < 2; ++j) {
         const int kpos = k0 + tx * 2 + j;
-        bool ok = (r < nq) && (kpos <= qpos);
-        if (a.window > 0) ok = ok && (kpos > qpos - a.window || kpos < a.keep_first);
+        const bool ok = (r < nq) && (kpos <= qpos) && (kpos >= first || kpos < a.keep_first);
         Ss[r * (PF_TK + 1) + tx * 2 + j] = ok ? s[i][j] : NEG_INF;
       }
     }
@@ -256,7 +255,7 @@ __global__ void __launch_bounds__(DC_THREADS) decode_attn_kernel(AttnArgs a, int
   const int seq = a.seq_ids[si];
   const int ctx = a.ctx_lens[seq];
   const int qrow = a.cu_q[seq];
-  const int lo = (a.window > 0) ? max(0, ctx - a.window) : 0;
+  const int lo = first_visible(ctx - 1, a);
   // the visible keys in one run of indices: the kept first positions below the window, then the window
   const int kept = min(a.keep_first, lo);
   const int gap = lo - kept;
@@ -276,9 +275,9 @@ __global__ void __launch_bounds__(DC_THREADS) decode_attn_kernel(AttnArgs a, int
     for (int c = 0; c < CPL; ++c) {
       const int chunk = lk + c * LPK;
       float f[VEC];
-      if (g < ng && chunk < chunks) {
+      if (g < ng && chunk < chunks && q_col_lives(kvh * G + g0 + g, chunk * VEC, D, a)) {
         Vec<T> v;
-        v.load((const T*)a.q + ((size_t)qrow * a.num_heads + kvh * G + g0 + g) * D + chunk * VEC);
+        v.load((const T*)a.q + q_row_of(qrow, kvh * G + g0 + g, a) * D + chunk * VEC);
         v.unpack(f);
       } else {
 #pragma unroll

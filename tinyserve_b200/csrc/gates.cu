@@ -6,13 +6,14 @@
 
 namespace ts {
 
-constexpr int ACT_SILU = 0, ACT_GELU_TANH = 1, ACT_CLAMPED_SWISH = 2;
+constexpr int ACT_SILU = 0, ACT_GELU_TANH = 1, ACT_CLAMPED_SWISH = 2, ACT_GELU = 3;
 
 __device__ __forceinline__ float sigmoidf(float z) { return 1.f / (1.f + expf(-z)); }
 
 template <int ACT>
 __device__ __forceinline__ float activate(float z) {
   if (ACT == ACT_SILU || ACT == ACT_CLAMPED_SWISH) return z / (1.f + expf(-z));
+  if (ACT == ACT_GELU) return 0.5f * z * (1.f + erff(z * 0.7071067811865476f));      // the exact form
   // 0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3)))
   const float inner = 0.7978845608028654f * fmaf(0.044715f * z * z, z, z);
   return 0.5f * z * (1.f + tanhf(inner));
@@ -44,6 +45,15 @@ __global__ void act_mul_kernel(const T* __restrict__ gate_up, const T* __restric
   }
 }
 
+// x <- act(x), in 32-bit, rounded once: an activation that gates nothing
+template <typename T, int ACT>
+__global__ void activate_kernel(T* __restrict__ x, size_t total) {
+  pdl_trigger();
+  pdl_wait();
+  for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < total; idx += (size_t)gridDim.x * blockDim.x)
+    x[idx] = from_float<T>(activate<ACT>(to_float(x[idx])));
+}
+
 // out[t, j] = act(x[t, j]) * table[rows[t], col0 + j]: a gate on a row that is looked up per token
 // (x rows are `x_stride` apart, table rows `table_width`); a row index outside the table gives NaN.
 template <typename T, int ACT>
@@ -72,13 +82,14 @@ __global__ void softcap_kernel(float* __restrict__ x, float cap, float inv_cap, 
 // One warp per (token, head): y = x / sqrt(mean(x^2) + eps) when `normalise`, times
 // weight[head * weight_head_stride + c] when a weight is given, times sigmoid(gate[t, head, c])
 // when a gate is given (`gate_per_head`: sigmoid(gate[t, head]), one value for the whole head;
-// `gate_silu`: the gate's value is z sigmoid(z) instead of sigmoid(z)).
+// `gate_silu`: the gate's value is z sigmoid(z) instead of sigmoid(z); `gate_first`: x is multiplied by the gate
+// before the root mean square is taken).
 // x is [T, heads, width] of type IN; gate rows are `gate_stride` apart.
 template <typename IN, typename T>
 __global__ void head_norm_gate_kernel(const IN* __restrict__ x, const T* __restrict__ weight, int weight_head_stride,
                                       const T* __restrict__ gate, int gate_stride, T* __restrict__ out,
                                       int num_tokens, int heads, int width, int normalise, float eps,
-                                      int gate_per_head, int gate_silu) {
+                                      int gate_per_head, int gate_silu, int gate_first) {
   pdl_trigger();
   pdl_wait();
   const int warp = (int)(((size_t)blockIdx.x * blockDim.x + threadIdx.x) >> 5), lane = threadIdx.x & 31;
@@ -89,7 +100,11 @@ __global__ void head_norm_gate_kernel(const IN* __restrict__ x, const T* __restr
   if (normalise) {
     float ss = 0.f;
     for (int c = lane; c < width; c += 32) {
-      const float v = to_float(xr[c]);
+      float v = to_float(xr[c]);
+      if (gate_first) {
+        const float z = to_float(gate[(size_t)t * gate_stride + h * width + c]);
+        v *= gate_silu ? z * sigmoidf(z) : sigmoidf(z);
+      }
       ss = fmaf(v, v, ss);
     }
     ss = warp_sum(ss);
@@ -117,7 +132,8 @@ template <typename IN, typename T>
 __global__ void __launch_bounds__(256) head_norm_gate_wide_kernel(const IN* __restrict__ x, const T* __restrict__ weight,
                                                                   int weight_head_stride, const T* __restrict__ gate,
                                                                   int gate_stride, T* __restrict__ out, int heads, int width,
-                                                                  int normalise, float eps, int gate_per_head, int gate_silu) {
+                                                                  int normalise, float eps, int gate_per_head, int gate_silu,
+                                                                  int gate_first) {
   __shared__ float parts[8];
   pdl_trigger();
   pdl_wait();
@@ -128,7 +144,11 @@ __global__ void __launch_bounds__(256) head_norm_gate_wide_kernel(const IN* __re
   if (normalise) {
     float ss = 0.f;
     for (int c = tid; c < width; c += 256) {
-      const float v = to_float(xr[c]);
+      float v = to_float(xr[c]);
+      if (gate_first) {
+        const float z = to_float(gate[(size_t)t * gate_stride + h * width + c]);
+        v *= gate_silu ? z * sigmoidf(z) : sigmoidf(z);
+      }
       ss = fmaf(v, v, ss);
     }
     ss = warp_sum(ss);
@@ -208,6 +228,22 @@ extern "C" int ts_act_mul(const void* gate_up, const void* bias, void* out, int 
   return TS_ERR_BAD_ARGUMENT;
 }
 
+extern "C" int ts_activate(void* x, size_t total, int activation, int dtype, cudaStream_t stream) {
+  if (total == 0) return 0;
+  if (activation != ACT_SILU && activation != ACT_GELU_TANH && activation != ACT_GELU) return TS_ERR_BAD_ARGUMENT;
+  const int b = blocks_for(total, 256);
+#define TS_ACTIVATE_CASE(T_)                                                                                             \
+  {                                                                                                                      \
+    if (activation == ACT_SILU) return launch(activate_kernel<T_, ACT_SILU>, b, 256, 0, stream, (T_*)x, total);         \
+    if (activation == ACT_GELU) return launch(activate_kernel<T_, ACT_GELU>, b, 256, 0, stream, (T_*)x, total);         \
+    return launch(activate_kernel<T_, ACT_GELU_TANH>, b, 256, 0, stream, (T_*)x, total);                                \
+  }
+  if (dtype == TS_DTYPE_F32) TS_ACTIVATE_CASE(float);
+  if (dtype == TS_DTYPE_BF16) TS_ACTIVATE_CASE(bf16);
+#undef TS_ACTIVATE_CASE
+  return TS_ERR_BAD_ARGUMENT;
+}
+
 extern "C" int ts_act_mul_gather(const void* x, int x_stride, const int* rows, const void* table, int table_rows,
                                  int table_width, int col0, void* out, int num_tokens, int n, int activation, int dtype,
                                  cudaStream_t stream) {
@@ -239,33 +275,40 @@ extern "C" int ts_softcap(float* x, size_t total, float cap, cudaStream_t stream
 
 extern "C" int ts_head_norm_gate(const void* x, int x_is_f32, const void* weight, int weight_head_stride,
                                  const void* gate, int gate_stride, void* out, int num_tokens, int heads, int width,
-                                 int normalise, float eps, int gate_per_head, int gate_silu, int dtype,
+                                 int normalise, float eps, int gate_per_head, int gate_silu, int gate_first, int dtype,
                                  cudaStream_t stream) {
   const size_t warps = (size_t)num_tokens * heads;
   if (warps == 0) return 0;
+  if (gate_first && (!gate || gate_per_head)) return TS_ERR_BAD_ARGUMENT;
   if (width >= 512) {      // a CTA per row
     const int rows = (int)warps;
     if (dtype == TS_DTYPE_F32)
       return launch(head_norm_gate_wide_kernel<float, float>, rows, 256, 0, stream, (const float*)x, (const float*)weight,
-                    weight_head_stride, (const float*)gate, gate_stride, (float*)out, heads, width, normalise, eps, gate_per_head, gate_silu);
+                    weight_head_stride, (const float*)gate, gate_stride, (float*)out, heads, width, normalise, eps, gate_per_head, gate_silu,
+                  gate_first);
     if (dtype != TS_DTYPE_BF16) return TS_ERR_BAD_ARGUMENT;
     if (x_is_f32)
       return launch(head_norm_gate_wide_kernel<float, bf16>, rows, 256, 0, stream, (const float*)x, (const bf16*)weight,
-                    weight_head_stride, (const bf16*)gate, gate_stride, (bf16*)out, heads, width, normalise, eps, gate_per_head, gate_silu);
+                    weight_head_stride, (const bf16*)gate, gate_stride, (bf16*)out, heads, width, normalise, eps, gate_per_head, gate_silu,
+                  gate_first);
     return launch(head_norm_gate_wide_kernel<bf16, bf16>, rows, 256, 0, stream, (const bf16*)x, (const bf16*)weight,
-                  weight_head_stride, (const bf16*)gate, gate_stride, (bf16*)out, heads, width, normalise, eps, gate_per_head, gate_silu);
+                  weight_head_stride, (const bf16*)gate, gate_stride, (bf16*)out, heads, width, normalise, eps, gate_per_head, gate_silu,
+                  gate_first);
   }
   const int threads = 128;
   const int b = (int)((warps * 32 + threads - 1) / threads);
   if (dtype == TS_DTYPE_F32)
     return launch(head_norm_gate_kernel<float, float>, b, threads, 0, stream, (const float*)x, (const float*)weight,
-                  weight_head_stride, (const float*)gate, gate_stride, (float*)out, num_tokens, heads, width, normalise, eps, gate_per_head, gate_silu);
+                  weight_head_stride, (const float*)gate, gate_stride, (float*)out, num_tokens, heads, width, normalise, eps, gate_per_head, gate_silu,
+                  gate_first);
   if (dtype != TS_DTYPE_BF16) return TS_ERR_BAD_ARGUMENT;
   if (x_is_f32)
     return launch(head_norm_gate_kernel<float, bf16>, b, threads, 0, stream, (const float*)x, (const bf16*)weight,
-                  weight_head_stride, (const bf16*)gate, gate_stride, (bf16*)out, num_tokens, heads, width, normalise, eps, gate_per_head, gate_silu);
+                  weight_head_stride, (const bf16*)gate, gate_stride, (bf16*)out, num_tokens, heads, width, normalise, eps, gate_per_head, gate_silu,
+                  gate_first);
   return launch(head_norm_gate_kernel<bf16, bf16>, b, threads, 0, stream, (const bf16*)x, (const bf16*)weight,
-                weight_head_stride, (const bf16*)gate, gate_stride, (bf16*)out, num_tokens, heads, width, normalise, eps, gate_per_head, gate_silu);
+                weight_head_stride, (const bf16*)gate, gate_stride, (bf16*)out, num_tokens, heads, width, normalise, eps, gate_per_head, gate_silu,
+                  gate_first);
 }
 
 extern "C" int ts_rms_norm_rows(const void* x, long long x_stride, const void* weight, float eps, void* out, int num_rows,

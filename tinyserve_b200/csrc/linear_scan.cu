@@ -13,6 +13,9 @@
 //  * MODE_ROTATED (retention): a constant decay per head; the first `rotary_dim` elements of q and k turn by the
 //    token's angles (pairs i, i + rotary_dim / 2 or neighbours), k is then multiplied by a constant; S <- decay_h S + k v^T;
 //    o = S^T q. The rotation happens where the chunk is staged, so the turned values are never rounded.
+//  * MODE_STATE_SPACE (the state-space duality of Mamba-2): one decay per head AND token, exp(-exp(A_h) dt) with
+//    dt = softplus(dt_pre + dt_bias_h); k and q (B and C) are shared by the heads of a group;
+//    S <- decay S + k (dt v)^T; o = S^T q + D_h v (the read-out sees the current token's write).
 //
 // Work split as in the other recurrent kernels: a CTA owns (request, head, block of 32 value
 // columns); compute warp w owns key rows [w * RPT, (w + 1) * RPT) and lane c column c, so a thread
@@ -25,7 +28,7 @@
 //
 // A long portion is cut into segments that run side by side (SCAN_LOCAL, SCAN_FINAL): the state after a
 // segment is diag(P) S_before + L, where L is what the segment's tokens leave behind from a zero state and
-// P the product of its decays (per key channel, exp(-sum_t exp(w_pre_t + w_0)) or exp(sum_t logsigmoid(z_t) / tau), or decay_h^tokens). One
+// P the product of its decays (per key channel, exp(-sum_t exp(w_pre_t + w_0)) or exp(sum_t logsigmoid(z_t) / tau); per head, exp(-exp(A_h) sum_t dt_t); or decay_h^tokens). One
 // launch runs every segment but a request's last from zero and stores L; a small kernel walks a request's
 // segments in order and leaves each one's starting state in L's place; a last launch runs every segment
 // from its starting state, writes the read-outs, and the request's last segment stores the slot. Twice the
@@ -43,22 +46,27 @@ constexpr int LIN_MAX_KEY_DIM = 256;
 constexpr int LIN_LOADER_WARPS = 4;
 constexpr int LIN_LOADS = 8;
 constexpr int LIN_RPT = 16;
-constexpr int MODE_BONUS = 0, MODE_DECAY = 1, MODE_GATED = 2, MODE_ROTATED = 3;
+constexpr int MODE_BONUS = 0, MODE_DECAY = 1, MODE_GATED = 2, MODE_ROTATED = 3, MODE_STATE_SPACE = 4;
 constexpr int SCAN_WHOLE = 0, SCAN_LOCAL = 1, SCAN_FINAL = 2;
 
 __device__ __forceinline__ float siluf(float z) { return z / (1.f + expf(-z)); }
 // log(sigmoid(z)) = min(z, 0) - log(1 + exp(-|z|))
 __device__ __forceinline__ float logsigmoidf(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
 
+// log(1 + exp(z))
+__device__ __forceinline__ float softplusf(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
+
 struct LinScanArgs {
   const void* q; int q_stride;      // [T, H * d] rows q_stride apart (r of the time mixing)
   const void* k; int k_stride;      // [T, H * d]
   const void* v; int v_stride;      // [T, H * dv]
   const float* w_pre; int w_stride; // MODE_BONUS, MODE_GATED: [T, H * d] decay pre-activations
-  const float* w_bias;              // MODE_BONUS, MODE_GATED: [H * d]
+                                    // MODE_STATE_SPACE: [T, H] dt_pre
+  const float* w_bias;              // MODE_BONUS, MODE_GATED: [H * d]; MODE_STATE_SPACE: [H] dt_bias
   float inv_tau, q_scale;           // MODE_GATED: 1 / tau of the decay, and the constant on q
-  const float* bonus;               // MODE_BONUS: [H * d]
-  const float* decay;               // MODE_DECAY, MODE_ROTATED: [H]
+  const float* bonus;               // MODE_BONUS: [H * d]; MODE_STATE_SPACE: [H] D
+  const float* decay;               // MODE_DECAY, MODE_ROTATED: [H]; MODE_STATE_SPACE: [H] A, the logarithm of the rate
+  int heads_per_group;              // MODE_STATE_SPACE: heads that share a q / k head (rows of q and k hold H / that many)
   const float* cos_tab; const float* sin_tab;   // MODE_ROTATED: [T, rotary_dim / 2]
   int rotary_dim, interleaved;      // MODE_ROTATED
   float k_scale;                    // MODE_ROTATED: the constant on k
@@ -71,6 +79,7 @@ struct LinScanArgs {
   int seg_len, max_segs;            // segmented: tokens per segment, segments per request in the grid
   float* seg_state;                 // segmented: [num_seqs * max_segs, H * d * dv]
   float* seg_decay;                 // segmented, MODE_BONUS, MODE_GATED: [num_seqs * max_segs, H * d] products of the decays
+                                    // (MODE_STATE_SPACE: [num_seqs * max_segs, H])
 };
 
 template <typename T, int MODE, int PASS>
@@ -79,9 +88,10 @@ __device__ __forceinline__ void linear_scan_body(const LinScanArgs& a) {
   constexpr int RPT = LIN_RPT;
   constexpr bool CHANNEL_DECAY = MODE == MODE_BONUS || MODE == MODE_GATED;
   constexpr int NARR = CHANNEL_DECAY ? 3 : 2;
+  constexpr int PER_TOKEN = MODE == MODE_STATE_SPACE ? 2 : 0;     // numbers of a head and token: dt and the decay
   const int W = a.W, CH = a.CH, d = a.d, dv = a.dv, H = a.H;
   const int dpad = W * RPT;
-  const int buf_floats = CH * (NARR * dpad + 32);
+  const int buf_floats = CH * (NARR * dpad + 32 + PER_TOKEN);
   float* part = sm + 2 * buf_floats;            // [CH][W][32]
   const int b = PASS == SCAN_WHOLE ? blockIdx.x : blockIdx.x / a.max_segs;
   const int seg = PASS == SCAN_WHOLE ? 0 : blockIdx.x - b * a.max_segs;
@@ -105,12 +115,14 @@ __device__ __forceinline__ void linear_scan_body(const LinScanArgs& a) {
   const T* qp = (const T*)a.q;
   const T* kp = (const T*)a.k;
   const T* vp = (const T*)a.v;
+  const int hk = MODE == MODE_STATE_SPACE ? h / a.heads_per_group : h;      // the q / k head of this head
 
   auto load_chunk = [&](int c) {
     float* q_s = sm + (c & 1) * buf_floats;
     float* k_s = q_s + CH * dpad;
     float* w_s = k_s + CH * dpad;                       // a decay per key channel only
     float* v_s = q_s + NARR * CH * dpad;
+    float* dt_s = v_s + CH * 32;                        // per token only: dt, then the decays
     const int t0 = start + c * CH, nt = min(CH, end - t0);
     const int lt = own_loads ? tid : tid - W * 32, ln = (own_loads ? W : LIN_LOADER_WARPS) * 32;
     if constexpr (MODE == MODE_ROTATED) {
@@ -157,8 +169,8 @@ __device__ __forceinline__ void linear_scan_body(const LinScanArgs& a) {
           const int idx = base + u * ln;
           const int tok = idx / dpad, r = idx - tok * dpad;
           const bool ok = idx < nt * dpad && r < d;
-          qv[u] = ok ? to_float(qp[(size_t)(t0 + tok) * a.q_stride + h * d + r]) : 0.f;
-          kv[u] = ok ? to_float(kp[(size_t)(t0 + tok) * a.k_stride + h * d + r]) : 0.f;
+          qv[u] = ok ? to_float(qp[(size_t)(t0 + tok) * a.q_stride + hk * d + r]) : 0.f;
+          kv[u] = ok ? to_float(kp[(size_t)(t0 + tok) * a.k_stride + hk * d + r]) : 0.f;
           if (CHANNEL_DECAY) wv[u] = ok ? a.w_pre[(size_t)(t0 + tok) * a.w_stride + h * d + r] + a.w_bias[h * d + r] : 0.f;
         }
 #pragma unroll
@@ -172,6 +184,9 @@ __device__ __forceinline__ void linear_scan_body(const LinScanArgs& a) {
               q_s[idx] = qv[u] * a.q_scale;
               k_s[idx] = kv[u];
               w_s[idx] = expf(logsigmoidf(wv[u]) * a.inv_tau);
+            } else if (MODE == MODE_STATE_SPACE) {
+              q_s[idx] = qv[u];
+              k_s[idx] = kv[u];
             } else {
               q_s[idx] = qv[u];
               k_s[idx] = kv[u];
@@ -187,6 +202,13 @@ __device__ __forceinline__ void linear_scan_body(const LinScanArgs& a) {
       if (MODE == MODE_DECAY) x = siluf(x);
       v_s[idx] = x;
     }
+    if constexpr (MODE == MODE_STATE_SPACE) {
+      for (int tok = lt; tok < nt; tok += ln) {
+        const float dt = softplusf(a.w_pre[(size_t)(t0 + tok) * a.w_stride + h] + a.w_bias[h]);
+        dt_s[tok] = dt;
+        dt_s[CH + tok] = expf(-expf(a.decay[h]) * dt);
+      }
+    }
   };
 
   const int slot = a.state_slots[b];
@@ -198,7 +220,7 @@ __device__ __forceinline__ void linear_scan_body(const LinScanArgs& a) {
   float* S_out = PASS == SCAN_LOCAL ? S_seg : S;
   const int r0 = warp * RPT;
   float s[RPT], u[MODE == MODE_BONUS ? RPT : 1];
-  float decay = 1.f;
+  float decay = 1.f, skip = 0.f;
   if (!loader) {
 #pragma unroll
     for (int i = 0; i < RPT; ++i) s[i] = (PASS != SCAN_LOCAL && r0 + i < d && col_ok) ? S_in[(size_t)(r0 + i) * dv + col] : 0.f;
@@ -207,6 +229,8 @@ __device__ __forceinline__ void linear_scan_body(const LinScanArgs& a) {
       for (int i = 0; i < RPT; ++i) u[i] = (r0 + i < d) ? a.bonus[h * d + r0 + i] : 0.f;
     } else if (MODE == MODE_DECAY || MODE == MODE_ROTATED) {
       decay = a.decay[h];
+    } else if (MODE == MODE_STATE_SPACE) {
+      skip = a.bonus[h];
     }
   }
   if (loader || own_loads) load_chunk(0);
@@ -223,12 +247,17 @@ __device__ __forceinline__ void linear_scan_body(const LinScanArgs& a) {
       const float* k_s = q_s + CH * dpad;
       const float* w_s = k_s + CH * dpad;
       const float* v_s = q_s + NARR * CH * dpad;
+      const float* dt_s = v_s + CH * 32;
       const int t0 = start + c * CH, nt = min(CH, end - t0);
       for (int tok = 0; tok < nt; ++tok) {
         const float4* q4 = reinterpret_cast<const float4*>(q_s + tok * dpad + r0);
         const float4* k4 = reinterpret_cast<const float4*>(k_s + tok * dpad + r0);
         const float4* w4 = reinterpret_cast<const float4*>(w_s + tok * dpad + r0);
-        const float vv = v_s[tok * 32 + lane];
+        float vv = v_s[tok * 32 + lane];
+        if (MODE == MODE_STATE_SPACE) {
+          vv *= dt_s[tok];
+          decay = dt_s[CH + tok];
+        }
         float o0 = 0.f, o1 = 0.f;
 #pragma unroll
         for (int i = 0; i < RPT / 4; ++i) {
@@ -273,6 +302,7 @@ __device__ __forceinline__ void linear_scan_body(const LinScanArgs& a) {
         for (int tok = warp; tok < nt; tok += W) {
           float o = 0.f;
           for (int w = 0; w < W; ++w) o += part[(tok * W + w) * 32 + lane];
+          if (MODE == MODE_STATE_SPACE) o = fmaf(skip, v_s[tok * 32 + lane], o);
           if (col_ok) a.out[((size_t)(t0 + tok) * H + h) * dv + col] = o;
         }
       }
@@ -295,7 +325,8 @@ template <typename T, int MODE, int PASS>
 __global__ void __maxnreg__(80) linear_scan_segment_kernel(LinScanArgs a) { linear_scan_body<T, MODE, PASS>(a); }
 
 // The product of a segment's decays per key channel, exp(-sum_t exp(w_pre_t + w_0)) (MODE_GATED:
-// exp(sum_t logsigmoid(w_pre_t + w_0) / tau)), for every segment but a request's last. A thread per channel; grid
+// exp(sum_t logsigmoid(w_pre_t + w_0) / tau); MODE_STATE_SPACE, per head: exp(-exp(A_h) sum_t softplus(w_pre_t + w_0))),
+// for every segment but a request's last. A thread per channel (or head); grid
 // (request * max_segs + segment, blocks of 128 channels).
 template <int MODE>
 __global__ void linear_scan_seg_decay_kernel(LinScanArgs a) {
@@ -306,10 +337,14 @@ __global__ void linear_scan_seg_decay_kernel(LinScanArgs a) {
   int start = a.cu_q[b];
   const int end = a.cu_q[b + 1];
   const int nsegs = (end - start + a.seg_len - 1) / a.seg_len;
-  if (seg >= nsegs - 1 || ch >= a.H * a.d) return;
+  const int channels = MODE == MODE_STATE_SPACE ? a.H : a.H * a.d;
+  if (seg >= nsegs - 1 || ch >= channels) return;
   start += seg * a.seg_len;
   const float bias = a.w_bias[ch];
   const float* wp = a.w_pre + (size_t)start * a.w_stride + ch;
+  auto rate = [&](float z) -> float {
+    return MODE == MODE_GATED ? -logsigmoidf(z) * a.inv_tau : MODE == MODE_STATE_SPACE ? softplusf(z) : expf(z);
+  };
   float sum = 0.f;
   int t = 0;
   for (; t + 8 <= a.seg_len; t += 8) {           // eight loads in flight
@@ -317,13 +352,13 @@ __global__ void linear_scan_seg_decay_kernel(LinScanArgs a) {
 #pragma unroll
     for (int j = 0; j < 8; ++j) x[j] = wp[(size_t)(t + j) * a.w_stride];
 #pragma unroll
-    for (int j = 0; j < 8; ++j) sum += MODE == MODE_GATED ? -logsigmoidf(x[j] + bias) * a.inv_tau : expf(x[j] + bias);
+    for (int j = 0; j < 8; ++j) sum += rate(x[j] + bias);
   }
   for (; t < a.seg_len; ++t) {
-    const float z = wp[(size_t)t * a.w_stride] + bias;
-    sum += MODE == MODE_GATED ? -logsigmoidf(z) * a.inv_tau : expf(z);
+    sum += rate(wp[(size_t)t * a.w_stride] + bias);
   }
-  a.seg_decay[(size_t)blockIdx.x * a.H * a.d + ch] = expf(-sum);
+  if (MODE == MODE_STATE_SPACE) sum *= expf(a.decay[ch]);
+  a.seg_decay[(size_t)blockIdx.x * channels + ch] = expf(-sum);
 }
 
 // A request's segments in order: seg_state[segment] holds what the segment leaves from a zero state and
@@ -349,14 +384,15 @@ __global__ void linear_scan_combine_kernel(LinScanArgs a) {
   }
   const size_t seg_stride = (size_t)a.H * per_head;
   float* p0 = a.seg_state + ((size_t)b * a.max_segs * a.H + h) * per_head + idx;
-  const float* d0 = a.seg_decay + (size_t)b * a.max_segs * a.H * a.d + h * a.d + r;     // a decay per key channel only
+  const int per_seg = MODE == MODE_STATE_SPACE ? a.H : a.H * a.d;               // products of a segment
+  const float* d0 = a.seg_decay + (size_t)b * a.max_segs * per_seg + (MODE == MODE_STATE_SPACE ? h : h * a.d + r);
   for (int s0 = 0; s0 < nsegs; s0 += 8) {        // eight segments' loads in flight, then the chain
     float left[8], pp[8];
 #pragma unroll
     for (int j = 0; j < 8; ++j) {
       const bool more = s0 + j + 1 < nsegs;
       left[j] = more ? p0[(size_t)(s0 + j) * seg_stride] : 0.f;
-      pp[j] = !more ? 0.f : !CONSTANT ? d0[(size_t)(s0 + j) * a.H * a.d] : p_const;
+      pp[j] = !more ? 0.f : !CONSTANT ? d0[(size_t)(s0 + j) * per_seg] : p_const;
     }
 #pragma unroll
     for (int j = 0; j < 8; ++j) {
@@ -420,8 +456,8 @@ static int lin_allow_smem(K kern, size_t smem, size_t& allowed) {
 template <typename T, int MODE, int PASS>
 static int launch_linear_pass(const LinScanArgs& a, dim3 grid, cudaStream_t stream) {
   const int dpad = a.W * LIN_RPT;
-  const int narr = MODE == MODE_DECAY || MODE == MODE_ROTATED ? 2 : 3;
-  const size_t smem = sizeof(float) * (2 * (size_t)a.CH * (narr * dpad + 32) + (size_t)a.CH * a.W * 32);
+  const int narr = MODE == MODE_BONUS || MODE == MODE_GATED ? 3 : 2, per_token = MODE == MODE_STATE_SPACE ? 2 : 0;
+  const size_t smem = sizeof(float) * (2 * (size_t)a.CH * (narr * dpad + 32 + per_token) + (size_t)a.CH * a.W * 32);
   static size_t allowed = 0;
   if constexpr (PASS == SCAN_WHOLE) {
     auto kern = linear_scan_kernel<T, MODE>;
@@ -439,8 +475,10 @@ static int launch_linear(const LinScanArgs& a, int num_seqs, cudaStream_t stream
   const int col_blocks = (a.dv + 31) / 32;
   if (a.max_segs <= 1) return launch_linear_pass<T, MODE, SCAN_WHOLE>(a, dim3(num_seqs, a.H, col_blocks), stream);
   const dim3 grid(num_seqs * a.max_segs, a.H, col_blocks);
-  if constexpr (MODE == MODE_BONUS || MODE == MODE_GATED)
-    if (int e = launch(linear_scan_seg_decay_kernel<MODE>, dim3(num_seqs * a.max_segs, (a.H * a.d + 127) / 128), 128, 0, stream, a)) return e;
+  if constexpr (MODE == MODE_BONUS || MODE == MODE_GATED || MODE == MODE_STATE_SPACE) {
+    const int channels = MODE == MODE_STATE_SPACE ? a.H : a.H * a.d;
+    if (int e = launch(linear_scan_seg_decay_kernel<MODE>, dim3(num_seqs * a.max_segs, (channels + 127) / 128), 128, 0, stream, a)) return e;
+  }
   if (int e = launch_linear_pass<T, MODE, SCAN_LOCAL>(a, grid, stream)) return e;
   if (int e = launch(linear_scan_combine_kernel<MODE>, dim3(num_seqs, a.H, (a.d * a.dv + 255) / 256), 256, 0, stream, a)) return e;
   return launch_linear_pass<T, MODE, SCAN_FINAL>(a, grid, stream);
@@ -449,34 +487,40 @@ static int launch_linear(const LinScanArgs& a, int num_seqs, cudaStream_t stream
 // mode 0: bonus read-out with a decay per key channel and token; mode 1: constant decay per head, SiLU on q, k, v;
 // mode 2: decay sigmoid(w_pre + w_bias)^(inv_tau) per key channel and token, q times q_scale, read-out after the write;
 // mode 3: constant decay per head, q and k rotated (cos_tab / sin_tab [T, rotary_dim / 2]), then k times k_scale.
+// mode 4 (float32 only): k and q rows hold heads / heads_per_group heads; w_pre [T, heads], w_bias [heads], decay [heads] (A) and bonus [heads] (D).
 // max_segs > 1 cuts every request's tokens into segments of seg_len (max_segs * seg_len covers the longest) that
 // run side by side (max_query_len = the most tokens any request brings): seg_state [num_seqs * max_segs, heads * d * dv] and, for modes 0 and 2, seg_decay
-// [num_seqs * max_segs, heads * d] are scratch.
+// [num_seqs * max_segs, heads * d], for mode 4 [num_seqs * max_segs, heads], are scratch.
 extern "C" int ts_linear_scan(int mode, const void* q, int q_stride, const void* k, int k_stride, const void* v,
                               int v_stride, const float* w_pre, int w_stride, const float* w_bias, const float* bonus,
                               const float* decay, float* state, int state_stride, const int* cu_q,
                               const int* state_slots, int num_seqs, int heads, int d, int dv, float* out, int dtype,
                               int max_query_len, int seg_len, int max_segs, float* seg_state, float* seg_decay,
                               float inv_tau, float q_scale, const float* cos_tab, const float* sin_tab, int rotary_dim,
-                              int interleaved, float k_scale, cudaStream_t stream) {
+                              int interleaved, float k_scale, int heads_per_group, cudaStream_t stream) {
   if (num_seqs <= 0) return 0;
   if (d <= 0 || dv <= 0 || d > LIN_MAX_KEY_DIM) return TS_ERR_UNSUPPORTED;
-  if (mode == MODE_BONUS ? (!w_pre || !w_bias || !bonus) : mode == MODE_GATED ? (!w_pre || !w_bias || !(inv_tau > 0.f))
+  if (mode == MODE_STATE_SPACE) {
+    if (!w_pre || !w_bias || !bonus || !decay || heads_per_group <= 0 || heads % heads_per_group) return TS_ERR_BAD_ARGUMENT;
+    if (dtype != TS_DTYPE_F32) return TS_ERR_UNSUPPORTED;
+  } else if (mode == MODE_BONUS ? (!w_pre || !w_bias || !bonus) : mode == MODE_GATED ? (!w_pre || !w_bias || !(inv_tau > 0.f))
                                                              : ((mode != MODE_DECAY && mode != MODE_ROTATED) || !decay)) return TS_ERR_BAD_ARGUMENT;
   if (mode == MODE_ROTATED && (rotary_dim < 0 || rotary_dim > d || (rotary_dim & 1) || (rotary_dim && (!cos_tab || !sin_tab))))
     return TS_ERR_BAD_ARGUMENT;
   if (dtype != TS_DTYPE_F32 && dtype != TS_DTYPE_BF16) return TS_ERR_BAD_ARGUMENT;
-  if (max_segs > 1 && (seg_len <= 0 || !seg_state || ((mode == MODE_BONUS || mode == MODE_GATED) && !seg_decay))) return TS_ERR_BAD_ARGUMENT;
+  if (max_segs > 1 && (seg_len <= 0 || !seg_state || ((mode == MODE_BONUS || mode == MODE_GATED || mode == MODE_STATE_SPACE) && !seg_decay))) return TS_ERR_BAD_ARGUMENT;
   LinScanArgs a;
   a.q = q; a.q_stride = q_stride; a.k = k; a.k_stride = k_stride; a.v = v; a.v_stride = v_stride;
   a.w_pre = w_pre; a.w_stride = w_stride; a.w_bias = w_bias; a.bonus = bonus; a.decay = decay;
   a.state = state; a.state_stride = state_stride; a.cu_q = cu_q; a.state_slots = state_slots;
   a.H = heads; a.d = d; a.dv = dv; a.out = out; a.inv_tau = inv_tau; a.q_scale = q_scale;
   a.cos_tab = cos_tab; a.sin_tab = sin_tab; a.rotary_dim = rotary_dim; a.interleaved = interleaved; a.k_scale = k_scale;
+  a.heads_per_group = heads_per_group;
   a.W = (d + LIN_RPT - 1) / LIN_RPT;
   a.CH = a.W * LIN_RPT <= 128 ? 16 : 8;
   a.loader_warps = (max_query_len > 0 && max_query_len <= a.CH) ? 0 : LIN_LOADER_WARPS;
   a.seg_len = seg_len; a.max_segs = max_segs > 1 ? max_segs : 1; a.seg_state = seg_state; a.seg_decay = seg_decay;
+  if (mode == MODE_STATE_SPACE) return launch_linear<float, MODE_STATE_SPACE>(a, num_seqs, stream);
   if (mode == MODE_BONUS)
     return dtype == TS_DTYPE_F32 ? launch_linear<float, MODE_BONUS>(a, num_seqs, stream) : launch_linear<bf16, MODE_BONUS>(a, num_seqs, stream);
   if (mode == MODE_ROTATED)

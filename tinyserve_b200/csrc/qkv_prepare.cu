@@ -6,7 +6,8 @@
 // from rows with strides of their own, so they may be parts of one merged projection. Optional
 // biases (one value per projection row) are added first. With `norm_whole` the RMSNorm runs over the
 // whole projection row (all heads of q, or of k, together; the weight then has one value per row
-// element) instead of head by head. All arithmetic is 32-bit and the result is rounded once.
+// element) instead of head by head. `maps` > 1: a key/value head has that many keys side by side in one cache row
+// [maps * d] (its k rows lie side by side in the projection too) and one value. All arithmetic is 32-bit and the result is rounded once.
 #define TS_PDL_CLASS PDL_ELEMENTWISE
 #include "common.cuh"
 
@@ -162,12 +163,13 @@ __global__ void qkv_prepare_kernel(const T* __restrict__ q_in, int q_stride, con
                                    const T* __restrict__ k_w, float eps, const float* __restrict__ cos_tab,
                                    const float* __restrict__ sin_tab, int rotary_dim, const int* __restrict__ slots,
                                    T* __restrict__ k_cache, T* __restrict__ v_cache, int page_size, int num_tokens,
-                                   int heads, int kv_heads, int d, int dv, T* __restrict__ q_out) {
+                                   int heads, int kv_heads, int d, int dv, T* __restrict__ q_out, int maps) {
   __shared__ float rows[QP_WARPS][QP_MAX_DIM];
   float* row = rows[threadIdx.x >> 5];
   pdl_trigger();
   pdl_wait();
-  const int jobs = heads + (k_in ? 2 * kv_heads : 0);
+  const int k_heads = kv_heads * maps;
+  const int jobs = heads + (k_in ? k_heads + kv_heads : 0);
   const long long warp = ((long long)blockIdx.x * blockDim.x + threadIdx.x) >> 5;
   const int lane = threadIdx.x & 31;
   if (warp >= (long long)num_tokens * jobs) return;
@@ -181,13 +183,13 @@ __global__ void qkv_prepare_kernel(const T* __restrict__ q_in, int q_stride, con
   }
   const int slot = slots[t];
   const int page = slot / page_size, off = slot - page * page_size;
-  if (job < heads + kv_heads) {
-    const int g = job - heads;
+  if (job < heads + k_heads) {
+    const int g = job - heads, kvh = g / maps, map = g - kvh * maps;
     norm_rotate_head(k_in + (size_t)t * k_stride + g * d, k_b ? k_b + g * d : nullptr, k_w, eps, cos_t, sin_t, rotary_dim, d,
-                     k_cache + (((size_t)page * kv_heads + g) * page_size + off) * d, lane, row);
+                     k_cache + ((((size_t)page * kv_heads + kvh) * page_size + off) * maps + map) * d, lane, row);
     return;
   }
-  const int g = job - heads - kv_heads;
+  const int g = job - heads - k_heads;
   const T* src = v_in + (size_t)t * v_stride + g * dv;
   T* dst = v_cache + (((size_t)page * kv_heads + g) * page_size + off) * dv;
   const T* vb = v_b ? v_b + g * dv : nullptr;
@@ -279,11 +281,12 @@ extern "C" int ts_qkv_prepare(const void* q_in, int q_stride, const void* k_in, 
                               int v_stride, const void* q_b, const void* k_b, const void* v_b, const void* q_w, const void* k_w, float eps, const float* cos_tab,
                               const float* sin_tab, int rotary_dim, const int* slots, void* k_cache, void* v_cache,
                               int page_size, int num_tokens, int heads, int kv_heads, int d, int dv, void* q_out,
-                              int norm_whole, int dtype, cudaStream_t stream) {
+                              int norm_whole, int maps, int dtype, cudaStream_t stream) {
   if (num_tokens <= 0) return 0;
   if (d > QP_MAX_DIM) return TS_ERR_UNSUPPORTED;
   if (rotary_dim < 0 || rotary_dim > d || (rotary_dim & 1) || (rotary_dim && (!cos_tab || !sin_tab))) return TS_ERR_BAD_ARGUMENT;
   if (k_in && (!v_in || !slots || !k_cache || !v_cache || page_size <= 0)) return TS_ERR_BAD_ARGUMENT;
+  if (maps < 1 || (maps > 1 && norm_whole)) return TS_ERR_BAD_ARGUMENT;
   if (norm_whole) {
     if (dtype == TS_DTYPE_F32)
       return launch(qkv_prepare_whole_kernel<float>, num_tokens, QW_WARPS * 32, 0, stream, (const float*)q_in, q_stride,
@@ -297,18 +300,18 @@ extern "C" int ts_qkv_prepare(const void* q_in, int q_stride, const void* k_in, 
                     page_size, heads, kv_heads, d, dv, (bf16*)q_out);
     return TS_ERR_BAD_ARGUMENT;
   }
-  const long long warps = (long long)num_tokens * (heads + (k_in ? 2 * kv_heads : 0));
+  const long long warps = (long long)num_tokens * (heads + (k_in ? (maps + 1) * kv_heads : 0));
   const int threads = QP_WARPS * 32;
   const int blocks = (int)((warps * 32 + threads - 1) / threads);
   if (dtype == TS_DTYPE_F32)
     return launch(qkv_prepare_kernel<float>, blocks, threads, 0, stream, (const float*)q_in, q_stride, (const float*)k_in,
                   k_stride, (const float*)v_in, v_stride, (const float*)q_b, (const float*)k_b, (const float*)v_b, (const float*)q_w, (const float*)k_w, eps, cos_tab, sin_tab,
                   rotary_dim, slots, (float*)k_cache, (float*)v_cache, page_size, num_tokens, heads, kv_heads, d, dv,
-                  (float*)q_out);
+                  (float*)q_out, maps);
   if (dtype == TS_DTYPE_BF16)
     return launch(qkv_prepare_kernel<bf16>, blocks, threads, 0, stream, (const bf16*)q_in, q_stride, (const bf16*)k_in,
                   k_stride, (const bf16*)v_in, v_stride, (const bf16*)q_b, (const bf16*)k_b, (const bf16*)v_b, (const bf16*)q_w, (const bf16*)k_w, eps, cos_tab, sin_tab,
                   rotary_dim, slots, (bf16*)k_cache, (bf16*)v_cache, page_size, num_tokens, heads, kv_heads, d, dv,
-                  (bf16*)q_out);
+                  (bf16*)q_out, maps);
   return TS_ERR_BAD_ARGUMENT;
 }

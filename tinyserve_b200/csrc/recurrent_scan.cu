@@ -364,6 +364,7 @@ __device__ __forceinline__ float conv_input(const T* x, int x_stride, const floa
 
 template <typename T>
 __global__ void causal_conv_silu_kernel(const T* __restrict__ x, int x_stride, const T* __restrict__ taps,
+                                        const T* __restrict__ bias,
                                         const float* __restrict__ state, int state_stride,
                                         const int* __restrict__ cu_q, const int* __restrict__ state_slots, int num_seqs,
                                         int num_tokens, int C, int K, float* __restrict__ y) {
@@ -379,10 +380,38 @@ __global__ void causal_conv_silu_kernel(const T* __restrict__ x, int x_stride, c
   const int start = cu_q[lo];
   const float* st = state + (size_t)state_slots[lo] * state_stride;
   for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < C; c += gridDim.y * blockDim.x) {
-    float acc = 0.f;
+    float acc = bias ? to_float(bias[c]) : 0.f;
     for (int k = 0; k < K; ++k)
       acc = fmaf(to_float(taps[(size_t)c * K + k]), conv_input(x, x_stride, st, C, K, start, t - (K - 1 - k), c), acc);
     y[(size_t)t * C + c] = acc / (1.f + expf(-acc));
+  }
+}
+
+// A step in which no request brings more than one token: output and new state in one pass, a thread per (request, channel).
+template <typename T>
+__global__ void causal_conv_silu_single_kernel(const T* __restrict__ x, int x_stride, const T* __restrict__ taps,
+                                               const T* __restrict__ bias, float* __restrict__ state, int state_stride,
+                                               const int* __restrict__ cu_q, const int* __restrict__ state_slots, int C, int K,
+                                               float* __restrict__ y) {
+  pdl_trigger();
+  pdl_wait();
+  const int b = blockIdx.x, t = cu_q[b];
+  if (cu_q[b + 1] <= t) return;
+  float* st = state + (size_t)state_slots[b] * state_stride;
+  for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < C; c += gridDim.y * blockDim.x) {
+    const float now = to_float(x[(size_t)t * x_stride + c]);
+    float past[SCAN_MAX_TAPS];
+#pragma unroll
+    for (int k = 0; k < SCAN_MAX_TAPS; ++k) past[k] = k < K - 1 ? st[(size_t)k * C + c] : 0.f;
+    float acc = bias ? to_float(bias[c]) : 0.f;
+#pragma unroll
+    for (int k = 0; k < SCAN_MAX_TAPS; ++k)
+      if (k < K - 1) acc = fmaf(to_float(taps[(size_t)c * K + k]), past[k], acc);
+    acc = fmaf(to_float(taps[(size_t)c * K + K - 1]), now, acc);
+    y[(size_t)t * C + c] = acc / (1.f + expf(-acc));
+#pragma unroll
+    for (int k = 0; k < SCAN_MAX_TAPS; ++k)
+      if (k < K - 1) st[(size_t)k * C + c] = k + 1 < K - 1 ? past[k + 1] : now;
   }
 }
 
@@ -501,9 +530,10 @@ extern "C" int ts_delta_scan(const float* qkv, int stride, int q_off, int k_off,
 #undef TS_DELTA_CASE
 }
 
-extern "C" int ts_causal_conv_silu(const void* x, int x_stride, const void* taps, float* state, int state_stride, const int* cu_q,
+extern "C" int ts_causal_conv_silu(const void* x, int x_stride, const void* taps, const void* bias, float* state, int state_stride, const int* cu_q,
                                    const int* state_slots, int num_seqs, int num_tokens, int channels, int num_taps,
-                                   float* y, int dtype, cudaStream_t stream) {
+                                   float* y, int single, int dtype, cudaStream_t stream) {
+  // `bias` (optional, [channels]): added before the activation. `single`: no request brings more than one token.
   if (num_tokens <= 0 || num_seqs <= 0) return 0;
   if (num_taps < 1 || num_taps > SCAN_MAX_TAPS) return TS_ERR_UNSUPPORTED;
   const int threads = 128;
@@ -511,15 +541,21 @@ extern "C" int ts_causal_conv_silu(const void* x, int x_stride, const void* taps
   if (by > 64) by = 64;
   dim3 grid(num_tokens, by), sgrid(num_seqs, by);
   int st;
+  if (single && dtype == TS_DTYPE_F32)
+    return launch(causal_conv_silu_single_kernel<float>, sgrid, threads, 0, stream, (const float*)x, x_stride, (const float*)taps,
+                  (const float*)bias, state, state_stride, cu_q, state_slots, channels, num_taps, y);
+  if (single && dtype == TS_DTYPE_BF16)
+    return launch(causal_conv_silu_single_kernel<bf16>, sgrid, threads, 0, stream, (const bf16*)x, x_stride, (const bf16*)taps,
+                  (const bf16*)bias, state, state_stride, cu_q, state_slots, channels, num_taps, y);
   if (dtype == TS_DTYPE_F32) {
-    st = launch(causal_conv_silu_kernel<float>, grid, threads, 0, stream, (const float*)x, x_stride, (const float*)taps,
+    st = launch(causal_conv_silu_kernel<float>, grid, threads, 0, stream, (const float*)x, x_stride, (const float*)taps, (const float*)bias,
                 (const float*)state, state_stride, cu_q, state_slots, num_seqs, num_tokens, channels, num_taps, y);
     if (st != 0 || num_taps == 1) return st;
     return launch(conv_state_update_kernel<float>, sgrid, threads, 0, stream, (const float*)x, x_stride, state, state_stride, cu_q,
                   state_slots, channels, num_taps);
   }
   if (dtype == TS_DTYPE_BF16) {
-    st = launch(causal_conv_silu_kernel<bf16>, grid, threads, 0, stream, (const bf16*)x, x_stride, (const bf16*)taps,
+    st = launch(causal_conv_silu_kernel<bf16>, grid, threads, 0, stream, (const bf16*)x, x_stride, (const bf16*)taps, (const bf16*)bias,
                 (const float*)state, state_stride, cu_q, state_slots, num_seqs, num_tokens, channels, num_taps, y);
     if (st != 0 || num_taps == 1) return st;
     return launch(conv_state_update_kernel<bf16>, sgrid, threads, 0, stream, (const bf16*)x, x_stride, state, state_stride, cu_q,

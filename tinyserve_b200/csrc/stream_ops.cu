@@ -1,7 +1,9 @@
 // Kernels around the 32-bit residual stream for layers that are not a plain pre-norm chain:
 //
 //  * embedding with a learned position row and a norm: x = table[token] * scale + pos[position],
-//    optionally x / sqrt(mean(x^2) + eps) * weight, written to the 32-bit stream;
+//    optionally x / sqrt(mean(x^2) + eps) * weight, written to the 32-bit stream; instead of a learned row, sinusoids
+//    of the position (sine at even columns, cosine at odd ones, a frequency per pair of columns);
+//  * the stream beside the embedding output, [x + y, x0] in the model dtype, for a product that replaces the stream;
 //  * the weighted sum of several sub-layer outputs into the stream,
 //    x <- x + sum_i s_i y_i + s_b bias, with a copy of the new stream in the model dtype
 //    (for a product that reads the stream itself rather than a norm of it).
@@ -18,14 +20,14 @@ template <typename T>
 __global__ void embed_pos_norm_kernel(const int* __restrict__ tokens, const int* __restrict__ positions,
                                       const T* __restrict__ table, const T* __restrict__ pos_table,
                                       const T* __restrict__ norm_w, float* __restrict__ out, int hidden, int vocab,
-                                      int max_pos, float scale, float eps) {
+                                      int max_pos, float scale, float eps, const double* __restrict__ freq) {
   extern __shared__ float xs[];
   __shared__ float scratch[33];
   pdl_trigger();
   pdl_wait();
   const int t = blockIdx.x;
   const int id = tokens[t];
-  const int p = pos_table ? positions[t] : 0;
+  const int p = pos_table || freq ? positions[t] : 0;
   float* o = out + (size_t)t * hidden;
   if (id < 0 || id >= vocab || p < 0 || (pos_table && p >= max_pos)) {
     // an id or a position outside its table: a row of NaN, never a read out of bounds
@@ -38,6 +40,12 @@ __global__ void embed_pos_norm_kernel(const int* __restrict__ tokens, const int*
   for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
     float v = to_float(row[i]) * scale;
     if (prow) v += to_float(prow[i]);
+    if (freq) {
+      // the angle in 64-bit, reduced to [-pi, pi] before it is rounded: exact at any position
+      const double turns = (double)p * freq[i >> 1] * 0.15915494309189535;
+      const float ang = (float)((turns - rint(turns)) * 6.283185307179586);
+      v += (i & 1) ? cosf(ang) : sinf(ang);
+    }
     xs[i] = v;
     ss = fmaf(v, v, ss);
   }
@@ -96,6 +104,31 @@ __global__ void stream_sum_kernel(StreamSumArgs a) {
   }
 }
 
+// --------------------------------------------------- the stream beside the embedding output
+// out[t] = [resid[t] + delta[t], origin[t]]: the sum in 32-bit, both halves rounded once. The stream itself stays.
+template <typename T, int VEC>
+__global__ void stream_beside_kernel(const float* __restrict__ resid, const T* __restrict__ delta, const float* __restrict__ origin,
+                                     T* __restrict__ out, int hidden, size_t total) {
+  pdl_trigger();
+  pdl_wait();
+  const size_t n = total / VEC;
+  for (size_t q = (size_t)blockIdx.x * blockDim.x + threadIdx.x; q < n; q += (size_t)gridDim.x * blockDim.x) {
+    const size_t idx = q * VEC, t = idx / hidden;
+    T* row = out + t * 2 * hidden + (idx - t * hidden);
+    float x[VEC], o[VEC];
+    if constexpr (VEC == 4) { Quad<float>::load(resid + idx, x); Quad<float>::load(origin + idx, o); }
+    else { x[0] = resid[idx]; o[0] = origin[idx]; }
+    if (delta) {
+      float y[VEC];
+      if constexpr (VEC == 4) Quad<T>::load(delta + idx, y); else y[0] = to_float(delta[idx]);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) x[e] += y[e];
+    }
+    if constexpr (VEC == 4) { Quad<T>::store(row, x); Quad<T>::store(row + hidden, o); }
+    else { row[0] = from_float<T>(x[0]); row[hidden] = from_float<T>(o[0]); }
+  }
+}
+
 // ------------------------------------------------------------- a bias on every row
 // y[t, j] <- y[t, j] + bias[j], in 32-bit, rounded once
 template <typename T>
@@ -141,18 +174,38 @@ extern "C" int ts_add_bias(void* y, const void* bias, int num_rows, int n, int d
 
 extern "C" int ts_embed_pos_norm(const int* tokens, const int* positions, const void* table, const void* pos_table,
                                  const void* norm_w, float* out, int num_tokens, int hidden, int vocab, int max_pos,
-                                 float scale, float eps, int dtype, cudaStream_t stream) {
+                                 float scale, float eps, const double* freq, int dtype, cudaStream_t stream) {
   if (num_tokens <= 0) return 0;
-  if (hidden <= 0 || hidden > 12288 || (pos_table && !positions)) return TS_ERR_BAD_ARGUMENT;
+  if (hidden <= 0 || hidden > 12288 || ((pos_table || freq) && !positions)) return TS_ERR_BAD_ARGUMENT;
   const int threads = hidden >= 1024 ? 256 : 128;
   const size_t smem = sizeof(float) * (size_t)hidden;
   if (dtype == TS_DTYPE_F32)
     return launch(embed_pos_norm_kernel<float>, num_tokens, threads, smem, stream, tokens, positions, (const float*)table,
-                  (const float*)pos_table, (const float*)norm_w, out, hidden, vocab, max_pos, scale, eps);
+                  (const float*)pos_table, (const float*)norm_w, out, hidden, vocab, max_pos, scale, eps, freq);
   if (dtype == TS_DTYPE_BF16)
     return launch(embed_pos_norm_kernel<bf16>, num_tokens, threads, smem, stream, tokens, positions, (const bf16*)table,
-                  (const bf16*)pos_table, (const bf16*)norm_w, out, hidden, vocab, max_pos, scale, eps);
+                  (const bf16*)pos_table, (const bf16*)norm_w, out, hidden, vocab, max_pos, scale, eps, freq);
   return TS_ERR_BAD_ARGUMENT;
+}
+
+extern "C" int ts_stream_beside(const float* resid, const void* delta, const float* origin, void* out, int num_tokens, int hidden,
+                                int dtype, cudaStream_t stream) {
+  if (num_tokens <= 0) return 0;
+  if (hidden <= 0 || !resid || !origin || !out) return TS_ERR_BAD_ARGUMENT;
+  if (dtype != TS_DTYPE_F32 && dtype != TS_DTYPE_BF16) return TS_ERR_BAD_ARGUMENT;
+  const size_t total = (size_t)num_tokens * hidden;
+  const bool vec = hidden % 4 == 0 && (((uintptr_t)resid | (uintptr_t)delta | (uintptr_t)origin | (uintptr_t)out) & 15) == 0;
+  size_t blocks = ((vec ? total / 4 : total) + 255) / 256;
+  if (blocks > 148 * 16) blocks = 148 * 16;
+#define TS_BESIDE(T_, V_) \
+  return launch(stream_beside_kernel<T_, V_>, (int)blocks, 256, 0, stream, resid, (const T_*)delta, origin, (T_*)out, hidden, total)
+  if (dtype == TS_DTYPE_F32) {
+    if (vec) TS_BESIDE(float, 4);
+    TS_BESIDE(float, 1);
+  }
+  if (vec) TS_BESIDE(bf16, 4);
+  TS_BESIDE(bf16, 1);
+#undef TS_BESIDE
 }
 
 extern "C" int ts_stream_sum(float* resid, const void* t0, const void* t1, const void* t2, const void* t3, float s0, float s1,

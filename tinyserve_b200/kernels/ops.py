@@ -35,27 +35,30 @@ _SIGNATURES: dict[str, list[Any]] = {
     "ts_silu_mul": [_vp, _vp, _i, _i, _i, _vp],
     "ts_qk_norm_rope_write": [_vp, _vp, _vp, _vp, _f, _vp, _vp, _i, _i, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _vp],
     "ts_paged_attention_simt": [_vp, _vp, _vp, _vp, _vp, _i, _vp, _vp, _vp, _i, _vp, _i, _i, _i, _i, _i, _i,
-                                _f, _i, _i, _vp, _vp, _vp, _i, _i, _i, _vp],
+                                _f, _i, _i, _vp, _vp, _vp, _i, _i, _i, _i, _i, _vp],
+    "ts_pair_combine": [_vp, _vp, _f, _f, _vp, _i, _i, _i, _vp, _vp, _i, _vp],
+    "ts_stream_beside": [_vp, _vp, _vp, _vp, _i, _i, _i, _vp],
+    "ts_activate": [_vp, _c.c_size_t, _i, _i, _vp],
     "ts_hc_mix_norm": [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _f, _i, _vp],
     "ts_hc_collapse": [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _vp],
     "ts_act_mul": [_vp, _vp, _vp, _i, _i, _i, _f, _i, _vp],
     "ts_act_mul_gather": [_vp, _i, _vp, _vp, _i, _i, _i, _vp, _i, _i, _i, _i, _vp],
-    "ts_embed_pos_norm": [_vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _f, _f, _i, _vp],
+    "ts_embed_pos_norm": [_vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _f, _f, _vp, _i, _vp],
     "ts_stream_sum": [_vp, _vp, _vp, _vp, _vp, _f, _f, _f, _f, _i, _vp, _f, _vp, _i, _i, _i, _vp],
     "ts_add_bias": [_vp, _vp, _i, _i, _i, _vp],
     "ts_tanh": [_vp, _c.c_size_t, _i, _vp],
     "ts_linear_scan": [_i, _vp, _i, _vp, _i, _vp, _i, _vp, _i, _vp, _vp, _vp, _vp, _i, _vp, _vp, _i, _i, _i, _i, _vp, _i, _i, _i, _i, _vp, _vp,
-                       _f, _f, _vp, _vp, _i, _i, _f, _vp],
+                       _f, _f, _vp, _vp, _i, _i, _f, _i, _vp],
     "ts_token_shift_mix": [_vp, _i, _vp, _i, _vp, _i, _vp, _vp, _i, _i, _i, _vp, _i, _vp],
     "ts_softcap": [_vp, _c.c_size_t, _f, _vp],
     "ts_rms_norm_rows": [_vp, _c.c_longlong, _vp, _f, _vp, _i, _i, _i, _vp],
-    "ts_head_norm_gate": [_vp, _i, _vp, _i, _vp, _i, _vp, _i, _i, _i, _i, _f, _i, _i, _i, _vp],
+    "ts_head_norm_gate": [_vp, _i, _vp, _i, _vp, _i, _vp, _i, _i, _i, _i, _f, _i, _i, _i, _i, _vp],
     "ts_post_norm_add_rms_norm": [_vp, _vp, _vp, _vp, _f, _i, _f, _vp, _i, _f, _vp, _vp, _i, _i, _vp, _vp, _f, _vp, _vp, _i, _vp],
     "ts_mlstm_scan": [_vp, _i, _i, _i, _i, _vp, _vp, _f, _f, _vp, _i, _vp, _vp, _i, _i, _i, _i, _vp, _i, _vp],
     "ts_delta_scan": [_vp, _i, _i, _i, _i, _vp, _i, _i, _vp, _vp, _vp, _i, _f, _vp, _i, _vp, _vp, _i, _i, _i, _i, _i, _vp, _vp],
-    "ts_causal_conv_silu": [_vp, _i, _vp, _vp, _i, _vp, _vp, _i, _i, _i, _i, _vp, _i, _vp],
+    "ts_causal_conv_silu": [_vp, _i, _vp, _vp, _vp, _i, _vp, _vp, _i, _i, _i, _i, _vp, _i, _i, _vp],
     "ts_qkv_prepare": [_vp, _i, _vp, _i, _vp, _i, _vp, _vp, _vp, _vp, _vp, _f, _vp, _vp, _i, _vp, _vp, _vp, _i, _i, _i, _i,
-                       _i, _i, _vp, _i, _i, _vp],
+                       _i, _i, _vp, _i, _i, _i, _vp],
     "ts_qkv_rotate": [_vp, _i, _vp, _i, _vp, _i, _vp, _vp, _i, _vp, _vp, _i, _i, _i, _f, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _vp,
                       _i, _i, _vp],
     "ts_talking_attention": [_vp, _vp, _vp, _vp, _vp, _i, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _f, _i, _f, _vp, _vp, _i, _vp, _vp,
@@ -63,19 +66,19 @@ _SIGNATURES: dict[str, list[Any]] = {
     "ts_talking_attention_mma": [_vp, _vp, _vp, _vp, _vp, _i, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _f, _i, _f, _vp, _vp, _i, _vp,
                                  _vp, _c.c_longlong, _vp, _vp],
     "ts_talking_attention_mma_takes": [_i, _i, _i, _i],
-    "ts_prefill_attention_mma": [_vp, _vp, _vp, _vp, _vp, _i, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _f, _i, _vp],
-    "ts_decode_attention_mma": [_vp, _vp, _vp, _vp, _vp, _i, _vp, _vp, _vp, _i, _i, _i, _i, _i, _f, _i, _i, _vp, _vp,
+    "ts_prefill_attention_mma": [_vp, _vp, _vp, _vp, _vp, _i, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _f, _i, _i, _i, _vp],
+    "ts_decode_attention_mma": [_vp, _vp, _vp, _vp, _vp, _i, _vp, _vp, _vp, _i, _i, _i, _i, _i, _f, _i, _i, _i, _i, _vp, _vp,
                                 _vp, _vp],
     "ts_decode_attention_mma_slots": [_i],
     "ts_decode_attention_tma": [_vp, _vp, _vp, _vp, _c.c_longlong, _vp, _i, _vp, _vp, _vp, _i, _i, _i, _i, _i, _f, _i,
-                                _i, _vp, _vp, _vp, _vp, _vp],
+                                _i, _vp, _vp, _vp, _vp, _i, _i, _vp],
     "ts_decode_attention_tma_fused": [_vp, _vp, _vp, _f, _vp, _vp, _vp, _vp, _vp, _vp, _c.c_longlong, _vp, _i, _vp,
                                       _vp, _vp, _i, _i, _i, _i, _i, _f, _i, _i, _vp, _vp, _vp, _vp],
     "ts_decode_attention_tma_slots": [_i],
     "ts_prefill_attention_tma": [_vp, _vp, _vp, _vp, _c.c_longlong, _vp, _i, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _f,
-                                 _i, _vp, _vp],
+                                 _i, _i, _vp, _vp],
     "ts_prefill_attention_tcgen05": [_vp, _vp, _vp, _vp, _c.c_longlong, _vp, _i, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i,
-                                     _f, _i, _i, _vp, _vp, _i, _vp],
+                                     _f, _i, _i, _vp, _vp, _i, _i, _i, _vp, _f, _f, _vp],
     "ts_gemm_skinny_normed": [_vp, _vp, _i, _vp, _f, _vp, _vp, _i, _i, _i, _i, _i, _vp],
     "ts_gemm_skinny_to_stream": [_vp, _vp, _vp, _vp, _vp, _i, _i, _i, _vp],
     "ts_gemm_skinny_to_stream_parts": [_i, _i, _i],
@@ -438,7 +441,8 @@ def choose_splits(ctas: int, slots: int, most: int, cluster: bool = False) -> in
 
 def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, page_size: int,
                     block_tables: torch.Tensor, ctx: Any, scale: float, window: int, out: torch.Tensor,
-                    sinks: torch.Tensor | None = None, keep_first: int = 0) -> None:
+                    sinks: torch.Tensor | None = None, keep_first: int = 0, chunk: int = 0, maps: int = 1,
+                    finish: "tuple[torch.Tensor, torch.Tensor, float, float] | None" = None) -> None:
     """Causal attention of this step's queries over each request's cached keys and values.
 
     ``q`` ``[T, Hq, D]`` dt; key cache ``[pages, Hkv, page_size, D]`` dt, value cache the same
@@ -447,8 +451,15 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
     step's maxima. ``window`` 0 means all earlier positions. ``sinks`` (float32 ``[Hq]``,
     optional): a logit per head that joins the softmax's denominator, unscaled, without a value.
     ``keep_first`` (with a window): positions below it stay visible to every later query, whatever
-    the window. ``out`` ``[T, Hq * Dv]`` dt."""
+    the window. ``chunk`` (instead of a window): a query sees only its own run of ``chunk`` positions, counted
+    from position 0. ``out`` ``[T, Hq * Dv]`` dt.
+
+    ``maps=2``: every query head and every key row holds two maps side by side (``D / 2`` elements each), each an
+    attention of its own over the same values: ``out`` is ``[T, Hq * 2 * Dv]``, map innermost. With ``finish =
+    (finished, factor, mult, eps)`` the maps are combined too: ``finished [T, Hq * Dv]`` dt receives ``a1 - factor a2``
+    over its root mean square per head, times ``mult`` (``factor``: one float32 on the device), and ``out`` is scratch."""
     t, hq, d = q.shape
+    hq *= maps
     hkv = k_cache.shape[1]
     dv = v_cache.shape[3]
     dt = q.dtype
@@ -458,6 +469,12 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
         raise KernelError("paged_attention: cache layout must be [pages, kv_heads, page_size, head_dim]")
     if out.numel() != t * hq * dv or hq % hkv:
         raise KernelError("paged_attention: out shape or head grouping")
+    if maps not in (1, 2) or d % maps or (finish is not None) != (maps == 2) or chunk < 0 or (chunk and window):
+        raise KernelError("paged_attention: one map or two (then with what combines them); a window or chunks, not both")
+    if maps == 2:
+        finished, factor, mult, mix_eps = finish
+        if sinks is not None or finished.dtype != dt or finished.numel() != t * hq // 2 * dv or factor.dtype != torch.float32 or factor.numel() != 1:
+            raise KernelError("paged_attention: two maps go without sinks; the finished heads are [T, Hq * Dv], the factor one float32")
     tma_ok = (dt == torch.bfloat16 and d in (64, 128) and dv == d and (page_size == 8 or page_size % 16 == 0)
               and k_cache.shape[0] * hkv * page_size < 2 ** 31)
     # sink logits are known to the tcgen05 prompt kernel, the TMA decode kernel and the CUDA-core
@@ -468,8 +485,8 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
     # kept first positions are known to the tcgen05 prompt kernel and the CUDA-core kernels
     simt_only = (dv != d or d % 16 != 0
                  or ((sinks is not None or keep_first > 0) and not (tma_ok and PREFILL_ATTENTION == "tcgen05")))
-    if d > 256 or dv > 256:
-        raise KernelError(f"paged_attention: head sizes {d}/{dv} must be at most 256")
+    if d > (512 if dv != d else 256) or dv > 256:
+        raise KernelError(f"paged_attention: head sizes {d}/{dv} are beyond what the kernels take")
     if block_tables.dim() != 2 or block_tables.shape[0] != ctx.num_seqs:
         raise KernelError("paged_attention: block_tables must be [requests, width]")
     if sinks is not None and (sinks.shape != (hq,) or sinks.dtype != torch.float32):
@@ -479,30 +496,35 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
     if simt_only:
         # the CUDA-core kernels know sink logits, a value head size of its own and odd head sizes
         _paged_attention_simt(q, k_cache, v_cache, page_size, block_tables, ctx, scale, window, out, sinks, num_prefill,
-                              keep_first)
+                              keep_first, chunk, maps)
+        if maps == 2:
+            pair_combine(out, factor, mix_eps, mult, finished, hq // 2, dv)
         return
+    open_rows = None          # of two maps: the requests whose rows still wait for their combination (None: all of the step)
     if num_prefill and dt == torch.bfloat16 and d <= 128:
         # prefill rows on the tensor cores; the decode rows follow below
-        if tma_ok and PREFILL_ATTENTION == "tcgen05":
+        if tma_ok and PREFILL_ATTENTION == "tcgen05" and (maps == 1 or d == 128):
             # both products as tcgen05.mma with the accumulators in tensor memory
             _check(_fn("ts_prefill_attention_tcgen05")(
-                _dev(q, "q"), _dev(out, "out"), _dev(k_cache, "k_cache"), _dev(v_cache, "v_cache"), k_cache.shape[0],
+                _dev(q, "q"), _dev(finished if maps == 2 else out, "out"), _dev(k_cache, "k_cache"), _dev(v_cache, "v_cache"), k_cache.shape[0],
                 _dev(block_tables, "block_tables", torch.int32), block_tables.shape[1],
                 _dev(ctx.cu_query_lens, "cu_query_lens", torch.int32),
                 _dev(ctx.context_lens_dev, "context_lens", torch.int32),
                 _dev(ctx.prefill_seqs, "prefill_seqs", torch.int32), num_prefill, ctx.max_query_len,
                 hq, hkv, d, page_size, float(scale), int(window),
                 _prefill_heads_per_cta(ctx, hq, hkv),
-                _error_word(q.device).data_ptr(), _opt(sinks, "sinks", torch.float32), keep_first, _stream()),
+                _error_word(q.device).data_ptr(), _opt(sinks, "sinks", torch.float32), keep_first, int(chunk), maps,
+                factor.data_ptr() if maps == 2 else None, float(mult) if maps == 2 else 1.0, float(mix_eps) if maps == 2 else 0.0, _stream()),
                 "prefill_attention_tcgen05")
-        elif tma_ok:
+            open_rows = ctx.decode_seqs
+        elif tma_ok and maps == 1:
             _check(_fn("ts_prefill_attention_tma")(
                 _dev(q, "q"), _dev(out, "out"), _dev(k_cache, "k_cache"), _dev(v_cache, "v_cache"), k_cache.shape[0],
                 _dev(block_tables, "block_tables", torch.int32), block_tables.shape[1],
                 _dev(ctx.cu_query_lens, "cu_query_lens", torch.int32),
                 _dev(ctx.context_lens_dev, "context_lens", torch.int32),
                 _dev(ctx.prefill_seqs, "prefill_seqs", torch.int32), num_prefill, ctx.max_query_len,
-                hq, hkv, d, page_size, float(scale), int(window), _error_word(q.device).data_ptr(), _stream()),
+                hq, hkv, d, page_size, float(scale), int(window), int(chunk), _error_word(q.device).data_ptr(), _stream()),
                 "prefill_attention_tma")
         else:
             _check(_fn("ts_prefill_attention_mma")(
@@ -511,9 +533,11 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
                 _dev(ctx.cu_query_lens, "cu_query_lens", torch.int32),
                 _dev(ctx.context_lens_dev, "context_lens", torch.int32),
                 _dev(ctx.prefill_seqs, "prefill_seqs", torch.int32), num_prefill, ctx.max_query_len,
-                hq, hkv, d, page_size, float(scale), int(window), _stream()), "prefill_attention_mma")
+                hq, hkv, d, page_size, float(scale), int(window), int(chunk), maps, _stream()), "prefill_attention_mma")
         num_prefill = 0
         if not ctx.num_decode:
+            if maps == 2 and open_rows is None:
+                pair_combine(out, factor, mix_eps, mult, finished, hq // 2, dv)
             return
     if keep_first > 0:
         # single tokens over a window and the kept first positions: the CUDA-core kernel, which walks the two
@@ -525,7 +549,8 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
         ctas = ctx.num_decode * hkv * (-(-(hq // hkv) // 16))
         tma = tma_ok
         slots = _decode_slots(d, tma)
-        splits = choose_splits(ctas, slots, ctx.max_context_len // 64, cluster=tma)
+        keys = min(ctx.max_context_len, chunk) if chunk else ctx.max_context_len
+        splits = choose_splits(ctas, slots, keys // 64, cluster=tma)
         part_acc = part_ml = None
         if splits > 1:
             part_acc = ctx.arena.take((ctx.num_decode, hq, splits, d), torch.float32)
@@ -534,26 +559,45 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
                   _dev(ctx.cu_query_lens, "cu_query_lens", torch.int32),
                   _dev(ctx.context_lens_dev, "context_lens", torch.int32),
                   _dev(ctx.decode_seqs, "decode_seqs", torch.int32), ctx.num_decode,
-                  hq, hkv, d, page_size, float(scale), int(window), splits,
-                  _opt(part_acc, "part_acc"), _opt(part_ml, "part_ml"), _error_word(q.device).data_ptr(), _stream())
+                  hq, hkv, d, page_size, float(scale), int(window))
+        scratch = (splits, _opt(part_acc, "part_acc"), _opt(part_ml, "part_ml"), _error_word(q.device).data_ptr())
         if tma:
             # tiles fetched by the TMA unit (tensor copies, 128-byte swizzle)
             _check(_fn("ts_decode_attention_tma")(
                 _dev(q, "q"), _dev(out, "out"), _dev(k_cache, "k_cache"), _dev(v_cache, "v_cache"),
-                k_cache.shape[0], *common[:-1], _opt(sinks, "sinks", torch.float32), common[-1]), "decode_attention_tma")
+                k_cache.shape[0], *common, *scratch, _opt(sinks, "sinks", torch.float32), int(chunk), maps, _stream()), "decode_attention_tma")
         else:
             # tiles fetched row by row with bulk copies
             _check(_fn("ts_decode_attention_mma")(
-                _dev(q, "q"), _dev(out, "out"), _dev(k_cache, "k_cache"), _dev(v_cache, "v_cache"), *common),
+                _dev(q, "q"), _dev(out, "out"), _dev(k_cache, "k_cache"), _dev(v_cache, "v_cache"), *common, int(chunk), maps, *scratch, _stream()),
                 "decode_attention_mma")
-        return
-    _paged_attention_simt(q, k_cache, v_cache, page_size, block_tables, ctx, scale, window, out, None, num_prefill)
+    else:
+        _paged_attention_simt(q, k_cache, v_cache, page_size, block_tables, ctx, scale, window, out, None, num_prefill, 0, chunk, maps)
+    if maps == 2:
+        pair_combine(out, factor, mix_eps, mult, finished, hq // 2, dv, rows_of=None if open_rows is None else (open_rows, ctx))
+
+
+def pair_combine(x: torch.Tensor, factor: torch.Tensor, eps: float, mult: float, out: torch.Tensor, heads: int, dv: int,
+                 rows_of: "tuple[torch.Tensor, Any] | None" = None) -> None:
+    """``out[t, h] = dt(o / sqrt(mean(o^2) + eps) * mult)`` with ``o = x[t, h, 0] - factor * x[t, h, 1]`` in 32-bit; ``x
+    [T, heads, 2, dv]`` and ``out [T, heads, dv]`` dt (any shapes of those sizes), ``factor`` one float32. ``rows_of``:
+    only the rows of these requests (int32 on the device), each of which brings one token of the step ``ctx``."""
+    t = out.numel() // (heads * dv)
+    if x.numel() != 2 * t * heads * dv or x.dtype != out.dtype or factor.numel() != 1:
+        raise KernelError("pair_combine: shape or dtype mismatch")
+    seqs = cu = None
+    rows = t
+    if rows_of is not None:
+        seqs, cu, rows = _dev(rows_of[0], "seqs", torch.int32), _dev(rows_of[1].cu_query_lens, "cu_query_lens", torch.int32), rows_of[1].num_decode
+    _check(_fn("ts_pair_combine")(_dev(x, "x"), _dev(factor, "factor", torch.float32), float(eps), float(mult), _dev(out, "out"), rows,
+                                  heads, dv, seqs, cu, _code(out.dtype), _stream()), "pair_combine")
 
 
 def _paged_attention_simt(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, page_size: int,
                           block_tables: torch.Tensor, ctx: Any, scale: float, window: int, out: torch.Tensor,
-                          sinks: torch.Tensor | None, num_prefill: int, keep_first: int = 0) -> None:
+                          sinks: torch.Tensor | None, num_prefill: int, keep_first: int = 0, chunk: int = 0, maps: int = 1) -> None:
     t, hq, d = q.shape
+    hq *= maps
     hkv, dv, dt = k_cache.shape[1], v_cache.shape[3], q.dtype
     splits, part_acc, part_ml = 1, None, None
     if ctx.num_decode and dv == d and d % 16 == 0:
@@ -570,7 +614,7 @@ def _paged_attention_simt(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch
         _dev(ctx.prefill_seqs, "prefill_seqs", torch.int32), num_prefill, ctx.max_query_len,
         hq, hkv, d, page_size, float(scale), int(window), splits,
         _opt(part_acc, "part_acc"), _opt(part_ml, "part_ml"), _opt(sinks, "sinks", torch.float32), dv,
-        int(keep_first), _code(dt), _stream()), "paged_attention",
+        int(keep_first), int(chunk), maps, _code(dt), _stream()), "paged_attention",
         kernels=(1 if num_prefill else 0) + (1 if ctx.num_decode else 0))
 
 
@@ -1169,7 +1213,21 @@ def hc_collapse(lanes: torch.Tensor, fresh: torch.Tensor | None, delta: torch.Te
 
 
 # --------------------------------------------------------------------------- gates
-ACTIVATIONS = {"silu": 0, "gelu_tanh": 1, "clamped_swish": 2}
+ACTIVATIONS = {"silu": 0, "gelu_tanh": 1, "clamped_swish": 2}         # of a gate (``act_mul``)
+PLAIN_ACTIVATIONS = {"silu": 0, "gelu_tanh": 1, "gelu": 3}            # of a feed-forward without a gate; "gelu" is the exact form
+
+
+def activate(x: torch.Tensor, activation: str) -> None:
+    """In place: ``x <- act(x)`` (32-bit, rounded once); ``activation`` one of ``PLAIN_ACTIVATIONS``."""
+    if activation not in PLAIN_ACTIVATIONS:
+        raise KernelError(f"activate: {activation!r} is not one of {sorted(PLAIN_ACTIVATIONS)}")
+    _check(_fn("ts_activate")(_dev(x, "x"), x.numel(), PLAIN_ACTIVATIONS[activation], _code(x.dtype), _stream()), "activate")
+
+
+def gemm_activated(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, activation: str) -> None:
+    """``out = dt(act(x @ w^T))``: the product and an activation on its result."""
+    gemm(x, w, out)
+    activate(out, activation)
 
 
 def act_mul(gate_up: torch.Tensor, out: torch.Tensor, activation: str, limit: float = 0.0,
@@ -1197,13 +1255,14 @@ def softcap(logits: torch.Tensor, cap: float) -> None:
 
 def head_norm_gate(x: torch.Tensor, weight: torch.Tensor | None, weight_per_head: bool, gate: torch.Tensor | None,
                    normalise: bool, eps: float, out: torch.Tensor, gate_per_head: bool = False,
-                   gate_silu: bool = False) -> None:
+                   gate_silu: bool = False, gate_first: bool = False) -> None:
     """Per (token, head) of ``x [T, H, w]`` (float32 or dt): divide by the root mean square over
     ``w`` (``normalise``), multiply by ``weight`` (``[H * w]`` when ``weight_per_head`` else ``[w]``
     shared by the heads) and by ``sigmoid(gate[t, h, :])`` (``gate`` dt, rows of ``H * w`` values,
     possibly a column slice of a wider matrix; with ``gate_per_head`` the gate has ``H`` values a row
     and head ``h`` is multiplied by ``sigmoid(gate[t, h])``; with ``gate_silu`` the gate's value is
-    ``z sigmoid(z)`` instead of ``sigmoid(z)``); ``out [T, H * w]`` dt."""
+    ``z sigmoid(z)`` instead of ``sigmoid(z)``; with ``gate_first`` the gate is applied before the root mean
+    square is taken); ``out [T, H * w]`` dt."""
     t, heads, w = x.shape
     dt = out.dtype
     if out.numel() != t * heads * w or x.dtype not in (torch.float32, dt):
@@ -1218,7 +1277,7 @@ def head_norm_gate(x: torch.Tensor, weight: torch.Tensor | None, weight_per_head
     _check(_fn("ts_head_norm_gate")(
         _dev(x, "x"), int(x.dtype == torch.float32), _opt(weight, "weight", dt), w if weight_per_head else 0,
         None if gate is None else gate.data_ptr(), gate_stride, _dev(out, "out"), t, heads, w, int(bool(normalise)),
-        float(eps), int(bool(gate_per_head)), int(bool(gate_silu)), _code(dt), _stream()), "head_norm_gate")
+        float(eps), int(bool(gate_per_head)), int(bool(gate_silu)), int(bool(gate_first)), _code(dt), _stream()), "head_norm_gate")
 
 
 def rms_norm_rows(x: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor) -> None:
@@ -1300,20 +1359,24 @@ def delta_scan(qkv: torch.Tensor, q_off: int, k_off: int, v_off: int, a: torch.T
         ctx.num_seqs, heads, kv_heads, d, dv, _dev(out, "out", torch.float32), _stream()), "delta_scan")
 
 
-def causal_conv_silu(x: torch.Tensor, taps: torch.Tensor, state: torch.Tensor, ctx: Any, out: torch.Tensor) -> None:
-    """``out[t, c] = silu(sum_k taps[c, k] * in[t - (K - 1 - k), c])`` (float32) per request, where
+def causal_conv_silu(x: torch.Tensor, taps: torch.Tensor, state: torch.Tensor, ctx: Any, out: torch.Tensor,
+                     bias: torch.Tensor | None = None) -> None:
+    """``out[t, c] = silu(bias[c] + sum_k taps[c, k] * in[t - (K - 1 - k), c])`` (float32; ``bias [C]`` dt, optional) per request, where
     tokens before this step come from ``state [slots, (K - 1) * C]`` float32 (zero at a request's
     start); afterwards the state holds the request's last ``K - 1`` inputs. ``x [T, C]`` dt, ``taps [C, K]`` dt."""
     t, c = x.shape
     k = taps.shape[1]
     if taps.shape[0] != c or tuple(out.shape) != (t, c) or taps.dtype != x.dtype or not x.is_cuda or x.stride(1) != 1:
         raise KernelError("causal_conv_silu: shape or dtype mismatch (x may be a column slice with unit column stride)")
+    if bias is not None and (bias.shape != (c,) or bias.dtype != x.dtype):
+        raise KernelError("causal_conv_silu: one bias per channel")
     state_ptr, state_stride = _state_rows(state, (k - 1) * c, "causal_conv_silu")
+    single = ctx.max_query_len == 1
     _check(_fn("ts_causal_conv_silu")(
-        x.data_ptr(), x.stride(0), _dev(taps, "taps"), state_ptr, state_stride,
+        x.data_ptr(), x.stride(0), _dev(taps, "taps"), _opt(bias, "bias"), state_ptr, state_stride,
         _dev(ctx.cu_query_lens, "cu_query_lens", torch.int32), _dev(ctx.state_slots, "state_slots", torch.int32),
-        ctx.num_seqs, t, c, k, _dev(out, "out", torch.float32), _code(x.dtype), _stream()), "causal_conv_silu",
-        kernels=2 if k > 1 else 1)
+        ctx.num_seqs, t, c, k, _dev(out, "out", torch.float32), int(single), _code(x.dtype), _stream()), "causal_conv_silu",
+        kernels=2 if k > 1 and not single else 1)
 
 
 def linear_scan_bonus(r: torch.Tensor, k: torch.Tensor, v: torch.Tensor, w_pre: torch.Tensor, w_bias: torch.Tensor,
@@ -1358,13 +1421,25 @@ def linear_scan_rotated(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay
                  interleaved=interleaved, k_scale=k_scale)
 
 
+def state_space_scan(c: torch.Tensor, b: torch.Tensor, x: torch.Tensor, dt_pre: torch.Tensor, dt_bias: torch.Tensor, a_log: torch.Tensor,
+                     skip: torch.Tensor, state: torch.Tensor, ctx: Any, heads: int, groups: int, d: int, dv: int, out: torch.Tensor) -> None:
+    """The recurrence of Mamba-2: with ``dt = softplus(dt_pre + dt_bias)`` per head and token, per head ``S <- exp(-exp(a_log) dt) S
+    + b (dt x)^T``, ``o = S^T c + skip x`` (the read-out sees the current token's write). ``c``, ``b`` ``[T, groups * d]`` (head h
+    reads group ``h // (heads / groups)``) and ``x [T, heads * dv]`` float32 with unit column stride, ``dt_pre [T, heads]``
+    float32; ``dt_bias``, ``a_log``, ``skip`` ``[heads]`` float32; ``state [slots, heads * d * dv]`` float32; ``out [T, heads, dv]`` float32."""
+    if heads % groups or c.dtype != torch.float32:
+        raise KernelError("state_space_scan: groups must divide the heads; float32 only")
+    _linear_scan(4, c, b, x, dt_pre, dt_bias, skip, a_log, state, ctx, heads, d, dv, out, groups=groups)
+
+
 def _linear_scan(mode: int, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, w_pre: torch.Tensor | None,
                  w_bias: torch.Tensor | None, bonus: torch.Tensor | None, decay: torch.Tensor | None,
                  state: torch.Tensor, ctx: Any, heads: int, d: int, dv: int, out: torch.Tensor,
                  inv_tau: float = 0.0, q_scale: float = 1.0, cos: torch.Tensor | None = None, sin: torch.Tensor | None = None,
-                 rotary_dim: int = 0, interleaved: bool = False, k_scale: float = 1.0) -> None:
+                 rotary_dim: int = 0, interleaved: bool = False, k_scale: float = 1.0, groups: int | None = None) -> None:
     t, dt = q.shape[0], q.dtype
-    for name, x, width in (("q", q, heads * d), ("k", k, heads * d), ("v", v, heads * dv)):
+    groups = heads if groups is None else groups
+    for name, x, width in (("q", q, groups * d), ("k", k, groups * d), ("v", v, heads * dv)):
         if not x.is_cuda or x.dtype != dt or x.shape != (t, width) or x.stride(1) != 1:
             raise KernelError(f"linear_scan: {name} must be [T, {width}] {dt} with unit column stride on the device")
     if tuple(out.shape) != (t, heads, dv) or d > SCAN_MAX_KEY_DIM:
@@ -1373,6 +1448,10 @@ def _linear_scan(mode: int, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, w
         if (w_pre.shape != (t, heads * d) or w_pre.dtype != torch.float32 or w_pre.stride(1) != 1
                 or w_bias.shape != (heads * d,) or (mode == 0 and bonus.shape != (heads * d,))):
             raise KernelError("linear_scan: decay pre-activations, their bias or the bonus")
+    elif mode == 4:
+        if (w_pre.shape != (t, heads) or w_pre.dtype != torch.float32 or w_pre.stride(1) != 1
+                or any(p.shape != (heads,) for p in (w_bias, bonus, decay))):
+            raise KernelError("linear_scan: one step size, bias, rate and skip per head")
     elif decay.shape != (heads,):
         raise KernelError("linear_scan: one decay per head")
     state_ptr, state_stride = _state_rows(state, heads * d * dv, "linear_scan")
@@ -1382,6 +1461,8 @@ def _linear_scan(mode: int, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, w
         seg_state = ctx.arena.take((ctx.num_seqs * max_segs, heads * d * dv), torch.float32)
         if mode in (0, 2):
             seg_decay = ctx.arena.take((ctx.num_seqs * max_segs, heads * d), torch.float32)
+        elif mode == 4:
+            seg_decay = ctx.arena.take((ctx.num_seqs * max_segs, heads), torch.float32)
     _check(_fn("ts_linear_scan")(
         mode, q.data_ptr(), q.stride(0), k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0),
         None if w_pre is None else w_pre.data_ptr(), 0 if w_pre is None else w_pre.stride(0),
@@ -1391,8 +1472,8 @@ def _linear_scan(mode: int, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, w
         _dev(out, "out", torch.float32), _code(dt), int(ctx.max_query_len), seg_len, max_segs,
         None if seg_state is None else seg_state.data_ptr(), None if seg_decay is None else seg_decay.data_ptr(),
         float(inv_tau), float(q_scale), _opt(cos, "cos", torch.float32), _opt(sin, "sin", torch.float32), int(rotary_dim),
-        int(bool(interleaved)), float(k_scale), _stream()),
-        "linear_scan", kernels=1 if max_segs <= 1 else (4 if mode in (0, 2) else 3))
+        int(bool(interleaved)), float(k_scale), heads // groups, _stream()),
+        "linear_scan", kernels=1 if max_segs <= 1 else (4 if mode in (0, 2, 4) else 3))
 
 
 # A portion of this many tokens or more is cut into segments that run side by side.
@@ -1436,8 +1517,9 @@ def token_shift_mix(x: torch.Tensor, mu: torch.Tensor, state: torch.Tensor, ctx:
 # ------------------------------------------------------- around the residual stream
 def embed_pos_norm(tokens: torch.Tensor, positions: torch.Tensor | None, table: torch.Tensor,
                    pos_table: torch.Tensor | None, norm_weight: torch.Tensor | None, eps: float, out: torch.Tensor,
-                   scale: float = 1.0) -> None:
-    """``x = float32(table[tokens[t]]) * scale (+ pos_table[positions[t]])``, then, with a norm weight,
+                   scale: float = 1.0, freq: torch.Tensor | None = None) -> None:
+    """``x = float32(table[tokens[t]]) * scale (+ pos_table[positions[t]]) (+ sinusoids of the position: with ``freq
+    [ceil(h / 2)]`` float64 the sine of ``positions[t] * freq[i // 2]`` at even columns i, the cosine at odd ones)``, then, with a norm weight,
     ``x / sqrt(mean(x^2) + eps) * weight``; ``out [T, h]`` float32. An id or a position outside its
     table gives a row of NaN."""
     t, h = out.shape
@@ -1446,10 +1528,13 @@ def embed_pos_norm(tokens: torch.Tensor, positions: torch.Tensor | None, table: 
         raise KernelError("embed_pos_norm: shape mismatch")
     if norm_weight is not None and norm_weight.shape != (h,):
         raise KernelError("embed_pos_norm: norm weight size")
+    if freq is not None and (freq.shape != ((h + 1) // 2,) or positions is None):
+        raise KernelError("embed_pos_norm: a frequency per pair of columns, and the positions")
     _check(_fn("ts_embed_pos_norm")(
         _dev(tokens, "tokens", torch.int32), _opt(positions, "positions", torch.int32), _dev(table, "table"),
         _opt(pos_table, "pos_table", dt), _opt(norm_weight, "norm_weight", dt), _dev(out, "out", torch.float32), t, h,
-        table.shape[0], 0 if pos_table is None else pos_table.shape[0], float(scale), float(eps), _code(dt), _stream()),
+        table.shape[0], 0 if pos_table is None else pos_table.shape[0], float(scale), float(eps),
+        _opt(freq, "freq", torch.float64), _code(dt), _stream()),
         "embed_pos_norm")
 
 
@@ -1476,6 +1561,16 @@ def stream_sum(resid: torch.Tensor, terms: Sequence[torch.Tensor], scales: Seque
     sc = [float(x) for x in scales] + [0.0] * (STREAM_SUM_MAX_TERMS - len(scales))
     _check(_fn("ts_stream_sum")(_dev(resid, "resid", torch.float32), *ptrs, *sc, len(terms), _opt(bias, "bias"),
                                 float(bias_scale), _opt(copy, "copy"), t, h, _code(dt), _stream()), "stream_sum")
+
+
+def stream_beside(resid: torch.Tensor, delta: torch.Tensor | None, origin: torch.Tensor, out: torch.Tensor) -> None:
+    """``out[t] = dt([resid[t] + delta[t], origin[t]])``: the stream with its pending output (added in 32-bit) beside another
+    32-bit stream; ``out [T, 2 h]`` dt, ``resid`` stays as it is."""
+    t, h = resid.shape
+    if tuple(origin.shape) != (t, h) or tuple(out.shape) != (t, 2 * h) or (delta is not None and (tuple(delta.shape) != (t, h) or delta.dtype != out.dtype)):
+        raise KernelError("stream_beside: shape or dtype mismatch")
+    _check(_fn("ts_stream_beside")(_dev(resid, "resid", torch.float32), _opt(delta, "delta"), _dev(origin, "origin", torch.float32),
+                                   _dev(out, "out"), t, h, _code(out.dtype), _stream()), "stream_beside")
 
 
 def add_bias(y: torch.Tensor, bias: torch.Tensor) -> None:
@@ -1517,22 +1612,23 @@ def qkv_prepare(q_in: torch.Tensor, k_in: torch.Tensor | None, v_in: torch.Tenso
                 rotary_dim: int, slots: torch.Tensor | None, k_cache: torch.Tensor | None, v_cache: torch.Tensor | None,
                 page_size: int, heads: int, kv_heads: int, d: int, dv: int, q_out: torch.Tensor,
                 q_bias: torch.Tensor | None = None, k_bias: torch.Tensor | None = None,
-                v_bias: torch.Tensor | None = None, norm_whole: bool = False) -> None:
+                v_bias: torch.Tensor | None = None, norm_whole: bool = False, maps: int = 1) -> None:
     """Per (token, head): optional bias (one value per projection row, dt), optional RMSNorm over the head with a plain weight
     (``norm_whole``: over all heads of q, or of k, together, with weights of ``heads * d`` and ``kv_heads * d`` values), rotation of the first
     ``rotary_dim`` elements (i pairs with i + rotary_dim / 2); queries to ``q_out [T, heads, d]``,
     keys and (unchanged) values to the caches at the tokens' slots (when ``k_in`` is given).
     ``q_in``/``k_in``/``v_in`` are 2-D dt with unit column stride (column slices of a merged
-    projection are fine); the value head size ``dv`` may differ from ``d``."""
+    projection are fine); the value head size ``dv`` may differ from ``d``. ``maps``: a key/value head has that many keys
+    side by side, in the projection and in its cache row (``[.., maps * d]``); ``heads`` then counts query (head, map) pairs."""
     t = q_out.shape[0]
     dt = q_out.dtype
-    for name, x, width in (("q_in", q_in, heads * d), ("k_in", k_in, kv_heads * d), ("v_in", v_in, kv_heads * dv)):
+    for name, x, width in (("q_in", q_in, heads * d), ("k_in", k_in, kv_heads * maps * d), ("v_in", v_in, kv_heads * dv)):
         if x is not None and (x.dtype != dt or x.shape != (t, width) or x.stride(1) != 1 or not x.is_cuda):
             raise KernelError(f"qkv_prepare: {name} must be [T, {width}] {dt} with unit column stride on the device")
     if tuple(q_out.shape) != (t, heads, d) or (k_in is None) != (v_in is None):
         raise KernelError("qkv_prepare: q_out shape, or keys without values")
     if k_in is not None:
-        if tuple(k_cache.shape[1:]) != (kv_heads, page_size, d) or tuple(v_cache.shape[1:]) != (kv_heads, page_size, dv):
+        if tuple(k_cache.shape[1:]) != (kv_heads, page_size, maps * d) or tuple(v_cache.shape[1:]) != (kv_heads, page_size, dv):
             raise KernelError("qkv_prepare: cache layout")
         _check_indices("qkv_prepare", None, None, page_size, k_cache.shape[0], slots)
     if rotary_dim and (cos is None or tuple(cos.shape) != (t, rotary_dim // 2) or tuple(sin.shape) != tuple(cos.shape)):
@@ -1543,12 +1639,12 @@ def qkv_prepare(q_in: torch.Tensor, k_in: torch.Tensor | None, v_in: torch.Tenso
     _check(_fn("ts_qkv_prepare")(
         q_in.data_ptr(), q_in.stride(0), None if k_in is None else k_in.data_ptr(), 0 if k_in is None else k_in.stride(0),
         None if v_in is None else v_in.data_ptr(), 0 if v_in is None else v_in.stride(0),
-        _bias(q_bias, heads * d, "q_bias", dt), _bias(k_bias if k_in is not None else None, kv_heads * d, "k_bias", dt),
+        _bias(q_bias, heads * d, "q_bias", dt), _bias(k_bias if k_in is not None else None, kv_heads * maps * d, "k_bias", dt),
         _bias(v_bias if v_in is not None else None, kv_heads * dv, "v_bias", dt),
         _opt(q_weight, "q_weight", dt), _opt(k_weight, "k_weight", dt), float(eps),
         _opt(cos, "cos", torch.float32), _opt(sin, "sin", torch.float32), int(rotary_dim),
         _opt(slots, "slots", torch.int32), _opt(k_cache, "k_cache", dt), _opt(v_cache, "v_cache", dt), page_size, t,
-        heads, kv_heads, d, dv, _dev(q_out, "q_out"), int(bool(norm_whole)), _code(dt), _stream()), "qkv_prepare")
+        heads, kv_heads, d, dv, _dev(q_out, "q_out"), int(bool(norm_whole)), int(maps), _code(dt), _stream()), "qkv_prepare")
 
 
 def qkv_rotate(proj: torch.Tensor, taps: torch.Tensor | None, state: torch.Tensor | None, ctx: Any, cos: torch.Tensor | None,

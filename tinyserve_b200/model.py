@@ -56,7 +56,7 @@ class ModelParts:
         for n, (call, part) in enumerate(zip(spec.order, self.stream_inputs)):
             block = self.layers[call.layer].block
             first_norm = next((block.parts[r] for r, family in type(block).roles.items() if family == "norm" and r in block.parts), None)
-            if part is not None and not getattr(first_norm, "folds_stream_input", False):
+            if part is not None and not part.replaces and not getattr(first_norm, "folds_stream_input", False):
                 raise ValueError(f"order[{n}] has a stream input, but the first norm of its block does not add it")
         self.keeps_origin = any(s is not None and s.needs_origin for s in self.stream_inputs)
         # One cache user per (call of the order, mixer role of its block, need of that mixer), in that order: the

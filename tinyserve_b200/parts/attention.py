@@ -493,6 +493,95 @@ class RotatedAttention(Mixer):
         return out
 
 
+class DifferentialAttention(Mixer):
+    """Attention with two maps per head over the same values, the second subtracted with a learned factor.
+
+    ``q = W_q h`` has ``num_heads * 2 * key_dim`` rows and ``k = W_k h`` ``num_kv_heads * 2 * key_dim``, head by head as
+    [map 1, map 2]; ``v = W_v h`` (``num_kv_heads x value_dim``); no biases. With ``qk_norm`` every map of every q and k
+    head is RMS-normed with a plain weight of ``key_dim`` values shared by heads and maps. q and k turn as the layer's
+    position encoding asks, if it has one. Each map is an attention of its own: scores ``scale * q . k``, causal, with
+    ``window`` only the last ``window`` positions, with ``chunk`` only the query's own run of ``chunk`` positions counted
+    from position 0; ordinary softmax. ``factor = exp(lq1 . lk1) - exp(lq2 . lk2) + diff``, one number for the layer; per
+    head ``o = a1 - factor a2``, divided by its root mean square over the head (no weight), times ``1 - diff``; ``W_o`` on
+    the concatenated heads. ``names`` maps the roles "q", "k", "v", "out", "q_norm", "k_norm", "lq1", "lk1", "lq2", "lk2"
+    to tensor names after the prefix.
+
+    A cached key row holds both maps of a key/value head side by side, so a position costs one row of keys and one of
+    values. The factor is made once, when the weights are bound. Norm, rotation and cache write are one kernel; prompt
+    portions of bfloat16 heads of 2 x 64 over values of 128 are finished inside the tcgen05 attention kernel (both maps of
+    a head in a CTA, over shared value tiles, combined and normed from tensor memory)."""
+
+    recordable = EVERY_STEP
+    _NAMES = {"q": "q", "k": "k", "v": "v", "out": "o", "q_norm": "q.norm", "k_norm": "k.norm", "lq1": "lq1", "lk1": "lk1",
+              "lq2": "lq2", "lk2": "lk2"}
+
+    def __init__(self, prefix: str, hidden_size: int, num_heads: int, num_kv_heads: int, key_dim: int, value_dim: int,
+                 scale: float, diff: float, norm_eps: float, qk_norm: bool = True, window: int | None = None,
+                 chunk: int | None = None, names: Mapping[str, str] | None = None) -> None:
+        if num_heads % num_kv_heads:
+            raise ValueError(f"num_heads={num_heads} is not a multiple of num_kv_heads={num_kv_heads}")
+        if (window is not None and window <= 0) or (chunk is not None and chunk <= 0) or (window is not None and chunk is not None):
+            raise ValueError(f"window={window}, chunk={chunk}: a positive size of one of them, or neither")
+        for what, size in (("key_dim", key_dim), ("value_dim", value_dim)):
+            if not 0 < size <= 256:
+                raise ValueError(f"{what}={size}: the attention kernels take head sizes up to 256")
+        self.prefix, self.h = prefix, int(hidden_size)
+        self.heads, self.groups, self.d, self.dv = int(num_heads), int(num_kv_heads), int(key_dim), int(value_dim)
+        if 2 * self.d == self.dv and self.dv > 256:
+            raise ValueError(f"key_dim={key_dim}: two maps of a head side by side are at most 256 wide when the values are too")
+        self.scale, self.diff, self.eps, self.qk_norm = float(scale), float(diff), float(norm_eps), bool(qk_norm)
+        self.window, self.chunk = None if window is None else int(window), None if chunk is None else int(chunk)
+        self.names = {**self._NAMES, **(names or {})}
+        self.rows = (self.heads * 2 * self.d, self.groups * 2 * self.d, self.groups * self.dv)      # of q, k and v
+        self.q_norm_w = self.k_norm_w = None
+
+    def cache_need(self) -> "KVNeed | SplitKVNeed":
+        if 2 * self.d == self.dv:
+            return KVNeed(self.groups, self.dv, self.window, chunk=self.chunk)
+        return SplitKVNeed(self.groups, 2 * self.d, self.dv, self.window, chunk=self.chunk)
+
+    def tensor_specs(self, prefix: str) -> list[TensorSpec]:
+        p, n, h = prefix + self.prefix, self.names, self.h
+        specs = [TensorSpec(p + "qkv", (sum(self.rows), h), merged_from=tuple(p + n[r] for r in ("q", "k", "v")), merged_rows=self.rows),
+                 TensorSpec(p + n["out"], (h, self.heads * self.dv))]
+        if self.qk_norm:
+            specs += [TensorSpec(p + n[r], (self.d,), init="one_plus_normal") for r in ("q_norm", "k_norm")]
+        return specs + [TensorSpec(p + n[r], (self.d,), std=0.1) for r in ("lq1", "lk1", "lq2", "lk2")]
+
+    def bind(self, prefix: str, tensors: Mapping[str, torch.Tensor]) -> None:
+        p, n = prefix + self.prefix, self.names
+        self.w_in, self.w_o = tensors[p + "qkv"], tensors[p + n["out"]]
+        if self.qk_norm:
+            self.q_norm_w, self.k_norm_w = tensors[p + n["q_norm"]], tensors[p + n["k_norm"]]
+        first, second = (torch.exp((tensors[p + n["lq" + i]].double() * tensors[p + n["lk" + i]].double()).sum()) for i in "12")
+        self.factor = (first - second + self.diff).float().reshape(1)
+
+    def forward(self, x: torch.Tensor, ctx: StepContext, cache: KVCacheEntry, writes_cache: bool, position: Any) -> torch.Tensor:
+        if not writes_cache:
+            raise RuntimeError("this mixer keeps a cache of its own")
+        t, arena = x.shape[0], ctx.arena
+        group = ctx.kv[cache.group]
+        q, k, v = self.rows
+        proj = arena.take((t, q + k + v), ctx.dtype)
+        ops.gemm(x, self.w_in, proj)
+        rot = None if position is None else position.qk_rotation()
+        if rot is not None and rot.interleaved:
+            raise NotImplementedError("this mixer rotates pairs (i, i + rotary_dim / 2) only")
+        queries = arena.take((t, self.heads * 2, self.d), ctx.dtype)
+        ops.qkv_prepare(proj[:, :q], proj[:, q: q + k], proj[:, q + k:], self.q_norm_w, self.k_norm_w, self.eps,
+                        None if rot is None else rot.cos, None if rot is None else rot.sin, 0 if rot is None else rot.rotary_dim,
+                        group.slots, cache.k, cache.v, cache.page_size, self.heads * 2, self.groups, self.d, self.dv, queries, maps=2)
+        both = arena.take((t, self.heads * 2 * self.dv), ctx.dtype)
+        attn = arena.take((t, self.heads * self.dv), ctx.dtype)
+        ops.paged_attention(queries.view(t, self.heads, 2 * self.d), cache.k, cache.v, cache.page_size, group.block_tables, ctx,
+                            self.scale, self.window or 0, both, chunk=self.chunk or 0, maps=2,
+                            finish=(attn, self.factor, 1.0 - self.diff, self.eps))
+        out = arena.take((t, self.h), ctx.dtype)
+        ops.gemm(attn, self.w_o, out)
+        return out
+
+
+register_mixer("differential_attention", DifferentialAttention)
 register_mixer("rotated_attention", RotatedAttention)
 register_mixer("gqa_attention", GQAAttention)
 register_mixer("latent_attention", LatentAttention)

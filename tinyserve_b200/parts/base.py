@@ -22,7 +22,7 @@ Kinds of part and what each must provide:
   (``cache`` is then a tuple too).
 * ``FeedForward``: ``forward(x, ctx) -> [T, hidden]``.
 * ``StreamInput``: adds something to the residual stream in front of a call of the run order
-  (``LayerCall.stream_input``); it is left pending and folded in by the next norm.
+  (``LayerCall.stream_input``), left pending and folded in by the next norm, or replaces the stream.
 * ``Block``: names the roles it wants filled (``roles``: role -> family of part) and arranges
   those parts around the stream; ``PreNormBlock`` wants a mixer, a feed-forward and their norms.
 
@@ -76,10 +76,17 @@ class PagedNeed(CacheNeed):
     of pages, one block table per request). ``window``: only the last ``window`` positions are
     ever read again (pages behind it are given back early); ``None`` keeps every position.
     ``keep_first``: with a window, the first positions that stay readable all the same (their pages
-    are never given back early)."""
+    are never given back early). ``chunk`` (instead of a window): position p reads its own run of ``chunk``
+    positions only, counted from position 0 (pages of finished runs are given back early)."""
 
     window: int | None = None
     keep_first: int = 0
+    chunk: int | None = None
+
+    @property
+    def span(self) -> int | None:
+        """The most positions (the kept first ones apart) that one query reads; ``None``: all."""
+        return self.window if self.window is not None else self.chunk
 
     def bytes_per_token(self, element_size: int) -> int:
         raise NotImplementedError
@@ -120,6 +127,7 @@ class KVNeed(PagedNeed):
     head_dim: int
     window: int | None = None
     keep_first: int = 0
+    chunk: int | None = None
 
     def bytes_per_token(self, element_size: int) -> int:
         return 2 * self.num_kv_heads * self.head_dim * element_size
@@ -143,6 +151,7 @@ class SplitKVNeed(PagedNeed):
     value_dim: int
     window: int | None = None
     keep_first: int = 0
+    chunk: int | None = None
 
     def bytes_per_token(self, element_size: int) -> int:
         return self.num_kv_heads * (self.key_dim + self.value_dim) * element_size
@@ -481,9 +490,11 @@ class TokenInput(Part):
 class StreamInput(Part):
     """Something added to the residual stream right before a call of the run order: ``forward(stream,
     ctx)`` leaves it in ``stream.extra``. ``needs_origin``: it adds the embedding output again
-    (``stream.origin``, which the model then keeps)."""
+    (``stream.origin``, which the model then keeps). ``replaces``: it leaves nothing pending but a new stream (a
+    product of the old one, say)."""
 
     needs_origin: bool = False
+    replaces: bool = False
 
     def forward(self, stream: ResidualStream, ctx: StepContext) -> None:
         raise NotImplementedError

@@ -68,6 +68,34 @@ class PositionedEmbedding(Part):
         return out
 
 
+class SinusoidalEmbedding(Part):
+    """Token embedding plus a fixed vector of the position: ``x = table[token] * scale``, to which column ``2 i`` adds
+    ``sin(p * base^(-2 i / hidden))`` and column ``2 i + 1`` the cosine of the same angle. Positions count from 0 in each
+    request. Angles are formed in 64-bit and reduced before they are rounded; one kernel writes the 32-bit stream."""
+
+    recordable = EVERY_STEP
+
+    def __init__(self, name: str, vocab_size: int, hidden_size: int, scale: float = 1.0, base: float = 10000.0) -> None:
+        if not base > 0:
+            raise ValueError(f"base={base} must be positive")
+        self.name, self.vocab_size, self.hidden_size = name, int(vocab_size), int(hidden_size)
+        self.scale, self.base = float(scale), float(base)
+        self.table = self.freq = None
+
+    def tensor_specs(self, prefix: str) -> list[TensorSpec]:
+        return [TensorSpec(prefix + self.name, (self.vocab_size, self.hidden_size))]
+
+    def bind(self, prefix: str, tensors: Mapping[str, torch.Tensor]) -> None:
+        self.table = tensors[prefix + self.name]
+        pairs = torch.arange((self.hidden_size + 1) // 2, dtype=torch.float64)
+        self.freq = (self.base ** (-2.0 * pairs / self.hidden_size)).to(self.table.device)
+
+    def forward(self, ctx: StepContext) -> torch.Tensor:
+        out = ctx.arena.take((ctx.num_tokens, self.hidden_size), torch.float32)
+        ops.embed_pos_norm(ctx.tokens, ctx.positions, self.table, None, None, 0.0, out, self.scale, freq=self.freq)
+        return out
+
+
 class LMHead(Part):
     recordable = EVERY_STEP
 
@@ -128,7 +156,37 @@ class PassVector(StreamInput):
         stream.extra = (stream.origin if self.needs_origin else None, self.vector)
 
 
+class PassProjection(StreamInput):
+    """In front of a pass of layers that run several times: the stream is replaced by a product of itself beside the
+    embedding output, ``x <- W [x; x0]`` (tensor ``name [hidden, 2 * hidden]``, the same for every pass). What is pending on
+    the stream is added in 32-bit first; the product's sums are the new 32-bit stream."""
+
+    recordable = EVERY_STEP
+    needs_origin = True
+    replaces = True
+
+    def __init__(self, name: str, hidden_size: int) -> None:
+        self.name, self.hidden_size = name, int(hidden_size)
+        self.weight: torch.Tensor | None = None
+
+    def tensor_specs(self, prefix: str) -> list[TensorSpec]:
+        return [TensorSpec(prefix + self.name, (self.hidden_size, 2 * self.hidden_size))]
+
+    def bind(self, prefix: str, tensors: Mapping[str, torch.Tensor]) -> None:
+        self.weight = tensors[prefix + self.name]
+
+    def forward(self, stream: ResidualStream, ctx: StepContext) -> None:
+        if stream.post is not None or stream.second is not None or stream.extra is not None or stream.lanes is not None:
+            raise NotImplementedError("a product of the stream behind anything but one plain pending output")
+        beside = ctx.arena.take((ctx.num_tokens, 2 * self.hidden_size), ctx.dtype)
+        ops.stream_beside(stream.resid, stream.delta, stream.origin, beside)
+        ops.gemm(beside, self.weight, stream.resid)
+        stream.delta = stream.sumsq = None
+
+
+STREAM_INPUTS.register("pass_projection", PassProjection)
 STREAM_INPUTS.register("pass_vector", PassVector)
 EMBEDDINGS.register("token_embedding", TokenEmbedding)
 EMBEDDINGS.register("positioned_embedding", PositionedEmbedding)
+EMBEDDINGS.register("sinusoidal_embedding", SinusoidalEmbedding)
 HEADS.register("lm_head", LMHead)

@@ -120,6 +120,42 @@ class GatedMLP(FeedForward):
         return out
 
 
+class PlainMLP(FeedForward):
+    """A feed-forward without a gate: ``y = act(x Wup^T) Wdown^T``, no biases, with a choice of activation ("gelu": the exact
+    form ``0.5 z (1 + erf(z / sqrt(2)))``, "gelu_tanh", "silu"), applied to the first product's sums where the framework
+    has such a kernel for the step's shape (``ops.gemm_activated``). ``names``: role "up" / "down" -> name after the prefix."""
+
+    recordable = EVERY_STEP
+
+    def __init__(self, prefix: str, hidden_size: int, intermediate_size: int, activation: str = "gelu",
+                 names: "Mapping[str, str] | None" = None) -> None:
+        if activation not in ops.PLAIN_ACTIVATIONS:
+            raise ValueError(f"activation {activation!r} is not one of {sorted(ops.PLAIN_ACTIVATIONS)}")
+        self.prefix, self.activation = prefix, activation
+        self.hidden_size, self.intermediate_size = int(hidden_size), int(intermediate_size)
+        self.names = {"up": "up", "down": "down", **(names or {})}
+        self.w_up = self.w_down = None
+
+    def tensor_specs(self, prefix: str) -> list[TensorSpec]:
+        p, h, i, n = prefix + self.prefix, self.hidden_size, self.intermediate_size, self.names
+        return [TensorSpec(p + n["up"], (i, h)), TensorSpec(p + n["down"], (h, i))]
+
+    def bind(self, prefix: str, tensors: Mapping[str, torch.Tensor]) -> None:
+        p, n = prefix + self.prefix, self.names
+        self.w_up, self.w_down = tensors[p + n["up"]], tensors[p + n["down"]]
+
+    def streamed_weights(self) -> list[torch.Tensor]:
+        return [self.w_up, self.w_down]
+
+    def forward(self, x: torch.Tensor, ctx: StepContext) -> torch.Tensor:
+        t = x.shape[0]
+        act = ctx.arena.take((t, self.intermediate_size), ctx.dtype)
+        ops.gemm_activated(x, self.w_up, act, self.activation)
+        out = ctx.arena.take((t, self.hidden_size), ctx.dtype)
+        ops.gemm(act, self.w_down, out)
+        return out
+
+
 class RoutedExperts(FeedForward):
     """A mixture of ``num_experts`` small SwiGLU feed-forwards of which each token uses ``top``.
 
@@ -261,5 +297,6 @@ class RoutedExperts(FeedForward):
 
 
 register_feed_forward("routed_experts", RoutedExperts)
+register_feed_forward("plain_mlp", PlainMLP)
 register_feed_forward("swiglu", SwiGLU)
 register_feed_forward("gated_mlp", GatedMLP)

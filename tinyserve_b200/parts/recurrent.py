@@ -43,6 +43,11 @@ token's write). Each head's ``o`` is RMS-normed with a weight shared by the head
 head ``S <- decay_h S + k v^T``, ``o = S^T q``; each head's ``o`` is divided by its root mean square (no
 weight), the heads are concatenated, multiplied by ``silu(W_g h)`` and projected by ``W_o``.
 
+``StateSpaceMixer``: Mamba-2 (the state-space duality). ``[z, x, B, C, dt] = W_in h``; x, B and C pass a short causal
+convolution per channel with a bias, and SiLU; ``dt = softplus(dt + dt_bias_h)``; per head, with B and C shared by
+the heads of a group, ``S <- exp(-exp(A_log_h) dt) S + dt B x^T``, ``y = S^T C + D_h x``; the concatenated heads are
+multiplied by ``silu(z)``, then RMS-normed in equal parts, multiplied by a weight per element and projected by ``W_o``.
+
 Gates, decays, step sizes, unit scalings and the state are 32-bit; the projections and the
 convolution's inputs are in the model dtype. Nothing of a step is read on the host: requests are
 found through ``cu_query_lens`` and ``state_slots`` on the device, so every kind of step can be
@@ -480,6 +485,80 @@ class RetentionMixer(Mixer):
         return out
 
 
+class StateSpaceMixer(Mixer):
+    recordable = EVERY_STEP
+    _NAMES = {"in": "in", "conv": "conv", "conv_bias": "conv.b", "step_bias": "dt_bias", "a_log": "A_log", "skip": "D", "norm": "norm",
+              "out": "o"}
+
+    def __init__(self, prefix: str, hidden_size: int, num_heads: int, num_groups: int, state_dim: int, value_dim: int, conv_taps: int,
+                 norm_parts: int, norm_eps: float, names: Mapping[str, str] | None = None) -> None:
+        _check_key_dim("state_space", state_dim)
+        if num_heads % num_groups:
+            raise ValueError(f"num_heads={num_heads} is not a multiple of num_groups={num_groups}")
+        if not 1 <= conv_taps <= ops.SCAN_MAX_TAPS:
+            raise ValueError(f"conv_taps={conv_taps} is outside 1..{ops.SCAN_MAX_TAPS}")
+        if norm_parts < 1 or (num_heads * value_dim) % norm_parts:
+            raise ValueError(f"norm_parts={norm_parts} does not divide the {num_heads * value_dim} inner columns")
+        self.prefix, self.h = prefix, int(hidden_size)
+        self.heads, self.groups, self.d, self.dv = int(num_heads), int(num_groups), int(state_dim), int(value_dim)
+        self.taps, self.parts, self.eps = int(conv_taps), int(norm_parts), float(norm_eps)
+        self.names = {**self._NAMES, **(names or {})}
+        self.inner = self.heads * self.dv
+        self.channels = self.inner + 2 * self.groups * self.d
+        self.state_floats = self.heads * self.d * self.dv
+
+    def cache_need(self) -> StateNeed:
+        # the matrix memory of every head, then the convolution's last taps - 1 inputs of every channel
+        return StateNeed((self.state_floats + (self.taps - 1) * self.channels,), torch.float32)
+
+    def tensor_specs(self, prefix: str) -> list[TensorSpec]:
+        p, n, h = prefix + self.prefix, self.names, self.h
+        return [
+            TensorSpec(p + n["in"], (self.inner + self.channels + self.heads, h)),
+            TensorSpec(p + n["conv"], (self.channels, self.taps), std=0.3),
+            TensorSpec(p + n["conv_bias"], (self.channels,), std=0.1),
+            TensorSpec(p + n["step_bias"], (self.heads,), std=1.0),
+            TensorSpec(p + n["a_log"], (self.heads,), std=0.5),
+            TensorSpec(p + n["skip"], (self.heads,), init="one_plus_normal", std=0.3),
+            TensorSpec(p + n["norm"], (self.inner,), init="one_plus_normal"),
+            TensorSpec(p + n["out"], (h, self.inner)),
+        ]
+
+    def bind(self, prefix: str, tensors: Mapping[str, torch.Tensor]) -> None:
+        p, n = prefix + self.prefix, self.names
+        w_in = tensors[p + n["in"]]
+        # the step sizes enter the recurrence in 32-bit, so their rows are a product of their own
+        self.w_main, self.w_step = w_in[: self.inner + self.channels], w_in[self.inner + self.channels:]
+        if self.heads % 16:
+            # zero rows up to a multiple of 16: the few-row product of decode steps takes such matrices
+            padded = torch.zeros((-(-self.heads // 16) * 16, self.h), dtype=w_in.dtype, device=w_in.device)
+            padded[: self.heads] = self.w_step
+            self.w_step = padded
+        self.w_conv, self.conv_bias = tensors[p + n["conv"]], tensors[p + n["conv_bias"]]
+        self.step_bias, self.a_log, self.skip = (tensors[p + n[r]].float().contiguous() for r in ("step_bias", "a_log", "skip"))
+        self.norm_w, self.w_o = tensors[p + n["norm"]], tensors[p + n["out"]]
+
+    def forward(self, x: torch.Tensor, ctx: StepContext, cache: StateCacheEntry, writes_cache: bool, position: Any) -> torch.Tensor:
+        t, arena = x.shape[0], ctx.arena
+        inner, ch, gn = self.inner, self.channels, self.groups * self.d
+        proj = arena.take((t, inner + ch), ctx.dtype)
+        ops.gemm(x, self.w_main, proj)
+        step = arena.take((t, self.w_step.shape[0]), torch.float32)
+        ops.gemm(x, self.w_step, step)
+        conved = arena.take((t, ch), torch.float32)
+        ops.causal_conv_silu(proj[:, inner:], self.w_conv, cache.state[:, self.state_floats:], ctx, conved, bias=self.conv_bias)
+        read = arena.take((t, self.heads, self.dv), torch.float32)
+        ops.state_space_scan(conved[:, inner + gn:], conved[:, inner: inner + gn], conved[:, :inner], step[:, : self.heads], self.step_bias,
+                             self.a_log, self.skip, cache.state[:, : self.state_floats], ctx, self.heads, self.groups, self.d, self.dv, read)
+        gated = arena.take((t, inner), ctx.dtype)
+        ops.head_norm_gate(read.view(t, self.parts, inner // self.parts), self.norm_w, True, proj[:, :inner], True, self.eps, gated,
+                           gate_silu=True, gate_first=True)
+        out = arena.take((t, self.h), ctx.dtype)
+        ops.gemm(gated, self.w_o, out)
+        return out
+
+
+register_mixer("state_space", StateSpaceMixer)
 register_mixer("retention", RetentionMixer)
 register_mixer("gated_linear_attention", GatedLinearAttention)
 register_mixer("gated_delta", GatedDeltaMixer)
