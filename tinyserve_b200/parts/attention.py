@@ -546,7 +546,7 @@ class DifferentialAttention(Mixer):
                  TensorSpec(p + n["out"], (h, self.heads * self.dv))]
         if self.qk_norm:
             specs += [TensorSpec(p + n[r], (self.d,), init="one_plus_normal") for r in ("q_norm", "k_norm")]
-        return specs + [TensorSpec(p + n[r], (self.d,), std=0.1) for r in ("lq1", "lk1", "lq2", "lk2")]
+        return specs + [TensorSpec(p + n[r], (self.d,), std=0.05) for r in ("lq1", "lk1", "lq2", "lk2")]
 
     def bind(self, prefix: str, tensors: Mapping[str, torch.Tensor]) -> None:
         p, n = prefix + self.prefix, self.names
