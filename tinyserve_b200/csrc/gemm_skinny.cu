@@ -40,6 +40,12 @@
 
 namespace ts {
 
+// An output type that stands for "bf16 after the exact gelu", 0.5 z (1 + erf(z / sqrt(2))) on the 32-bit sums.
+struct SkGelu { bf16 v; };
+template <> __device__ __forceinline__ SkGelu from_float<SkGelu>(float z) {
+  return SkGelu{from_float<bf16>(0.5f * z * (1.f + erff(z * 0.7071067811865476f)))};
+}
+
 // FUSE as a template argument: 0 = a plain product, 1 = silu(gate) * up with the rounding points of the
 // separate kernels, FUSE_GELU_TANH = gelu_tanh(gate) * up in 32-bit, rounded once.
 // FUSE_CLAMPED_SWISH = with g = min(gate, limit), u = clamp(up, -limit, limit): g sigmoid(1.702 g) (u + 1)
@@ -835,6 +841,18 @@ extern "C" int ts_gemm_skinny(const void* x, const void* w, void* out, int M, in
   if (out_dtype == TS_DTYPE_F32)
     return dispatch_skinny<float>((const bf16*)x, (const bf16*)w, (float*)out, M, N, K, stream);
   return TS_ERR_BAD_ARGUMENT;
+}
+
+// gelu(x w^T) (the exact form) in bf16, M <= 16: the activation on the 32-bit sums.
+extern "C" int ts_gemm_skinny_gelu(const void* x, const void* w, void* out, int M, int N, int K, cudaStream_t stream) {
+  if (M <= 0 || N <= 0) return 0;
+  if (M > 16 || K <= 0 || K % 32 != 0 || N % 16 != 0) return TS_ERR_UNSUPPORTED;
+  if (((uintptr_t)x | (uintptr_t)w) & 15) return TS_ERR_UNSUPPORTED;
+  const bf16* xp = (const bf16*)x;
+  const bf16* wp = (const bf16*)w;
+  if (plain_takes_h8(M, N, K)) return launch_h8_plain<SkGelu, false>(xp, wp, (SkGelu*)out, M, N, K, stream);
+  return M <= 8 ? dispatch_skinny_nt<SkGelu, 1>(xp, wp, (SkGelu*)out, M, N, K, stream)
+                : dispatch_skinny_nt<SkGelu, 2>(xp, wp, (SkGelu*)out, M, N, K, stream);
 }
 
 // act[M, inter] = silu(x gate^T) * (x up^T) with w = [gate rows; up rows] of shape [2 inter, K].

@@ -25,6 +25,8 @@
 #define TS_PDL_CLASS PDL_TCGEN05
 #include <cuda.h>
 
+#include <type_traits>
+
 #include "tcgen05.cuh"
 
 namespace ts {
@@ -32,6 +34,19 @@ namespace ts {
 constexpr int TG_BM = 128;
 constexpr int TG_BK = 64;              // 64 bf16 = 128 bytes = one swizzle row
 constexpr int TG_THREADS = 192;     // TMA warp, MMA warp, four epilogue warps
+
+// An output type that stands for "bf16 after the exact gelu": z Phi(z) with the normal distribution's cumulative
+// probability Phi from Abramowitz and Stegun, Handbook of Mathematical Functions, 7.1.26 (error of erf below 1.5e-7, far
+// below the rounding of the result; the small side of Phi is formed without a subtraction).
+struct TgGelu { bf16 v; };
+__device__ __forceinline__ float tg_gelu(float z) {
+  const float a = fabsf(z) * 0.7071067811865476f;
+  const float t = __fdividef(1.f, fmaf(0.3275911f, a, 1.f));
+  const float poly = t * fmaf(t, fmaf(t, fmaf(t, fmaf(t, 1.061405429f, -1.453152027f), 1.421413741f), -0.284496736f), 0.254829592f);
+  const float small = 0.5f * poly * __expf(-a * a);
+  return z * (z < 0.f ? small : 1.f - small);
+}
+template <> __device__ __forceinline__ TgGelu from_float<TgGelu>(float z) { return TgGelu{from_float<bf16>(tg_gelu(z))}; }
 
 // One warp's share of an accumulator tile (its 32 tensor-memory lanes = 32 rows, BN columns from
 // tmem_acc) -> out: cast and store, or silu(gate) * up of the two halves (SWIGLU).
@@ -135,7 +150,10 @@ __device__ __forceinline__ void drain_tile(uint32_t tmem_acc, int row, int M, in
           for (int j = 0; j < 32; j += 8) {
             float f[8];
 #pragma unroll
-            for (int e = 0; e < 8; ++e) f[e] = __uint_as_float(r[j + e]);
+            for (int e = 0; e < 8; ++e) {
+              f[e] = __uint_as_float(r[j + e]);
+              if constexpr (std::is_same_v<TOut, TgGelu>) f[e] = tg_gelu(f[e]);
+            }
             Vec<bf16> v;
             v.pack(f);
             v.store((bf16*)dst + j);
@@ -537,6 +555,19 @@ extern "C" int ts_gemm_tcgen05(const void* x, const void* w, void* out, int M, i
   if (tile_n == 128) { TS_TC(128, 6); }
   TS_TC(256, 4);
 #undef TS_TC
+}
+
+// gelu(x w^T) (the exact form) in bf16: the activation in the epilogue, on the 32-bit sums. tile_n: 256, or 512 for pairs of CTAs.
+extern "C" int ts_gemm_tcgen05_gelu(const void* x, const void* w, void* out, int M, int N, int K, int tile_n, int* error_flag,
+                                    cudaStream_t stream) {
+  if (M <= 0 || N <= 0) return 0;
+  if (K <= 0 || K % 8 != 0 || error_flag == nullptr) return TS_ERR_UNSUPPORTED;
+  if (((uintptr_t)x | (uintptr_t)w) & 15) return TS_ERR_UNSUPPORTED;
+  if (tile_n != 256 && tile_n != 512) return TS_ERR_BAD_ARGUMENT;
+  CUtensorMap mx, mw;
+  if (!make_map(&mx, x, M, K, TG_BM) || !make_map(&mw, w, N, K, tile_n == 512 ? 128 : 256)) return TS_ERR_UNSUPPORTED;
+  if (tile_n == 512) return launch_tc_pair<6, TgGelu, false>(mx, mw, (TgGelu*)out, M, N, K, error_flag, stream);
+  return launch_tc<256, 4, TgGelu>(mx, mw, (TgGelu*)out, M, N, K, error_flag, stream);
 }
 
 // act[M, inter] = silu(x gate^T) * (x up^T) in bf16 with w = [gate rows; up rows], [2 inter, K]:

@@ -38,6 +38,8 @@ _SIGNATURES: dict[str, list[Any]] = {
                                 _f, _i, _i, _vp, _vp, _vp, _i, _i, _i, _i, _i, _vp],
     "ts_pair_combine": [_vp, _vp, _f, _f, _vp, _i, _i, _i, _vp, _vp, _i, _vp],
     "ts_stream_beside": [_vp, _vp, _vp, _vp, _i, _i, _i, _vp],
+    "ts_gemm_skinny_gelu": [_vp, _vp, _vp, _i, _i, _i, _vp],
+    "ts_gemm_tcgen05_gelu": [_vp, _vp, _vp, _i, _i, _i, _i, _vp, _vp],
     "ts_activate": [_vp, _c.c_size_t, _i, _i, _vp],
     "ts_hc_mix_norm": [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _f, _i, _vp],
     "ts_hc_collapse": [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _vp],
@@ -1225,7 +1227,21 @@ def activate(x: torch.Tensor, activation: str) -> None:
 
 
 def gemm_activated(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, activation: str) -> None:
-    """``out = dt(act(x @ w^T))``: the product and an activation on its result."""
+    """``out[M, N] = dt(act(x[M, K] @ w[N, K]^T))``. "gelu" is applied to the 32-bit sums by the product itself where
+    :func:`gemm` would take one of this library's bf16 kernels; otherwise the product is followed by :func:`activate`."""
+    m, k = x.shape
+    n = w.shape[0]
+    if activation == "gelu" and x.dtype == torch.bfloat16 and out.dtype == x.dtype and m:
+        if w.shape[1] != k or tuple(out.shape) != (m, n) or w.dtype != x.dtype:
+            raise KernelError(f"gemm_activated: shapes {tuple(x.shape)} x {tuple(w.shape)} -> {tuple(out.shape)}")
+        if m <= SKINNY_MAX_ROWS and k % 32 == 0 and n % 16 == 0 and n * k <= SKINNY_MAX_WEIGHTS:
+            _check(_fn("ts_gemm_skinny_gelu")(_dev(x, "x"), _dev(w, "w"), _dev(out, "out"), m, n, k, _stream()), "gemm_activated")
+            return
+        tiles = tcgen05_tiles(m, n, 256) if m >= TCGEN05_MIN_ROWS and n >= TCGEN05_MIN_COLS and k % 8 == 0 else ""
+        if tiles:
+            _check(_fn("ts_gemm_tcgen05_gelu")(_dev(x, "x"), _dev(w, "w"), _dev(out, "out"), m, n, k, TCGEN05_PAIR_TILE if tiles == "pairs" else 256,
+                                               _error_word(x.device).data_ptr(), _stream()), "gemm_activated")
+            return
     gemm(x, w, out)
     activate(out, activation)
 
