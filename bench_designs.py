@@ -1,4 +1,4 @@
-"""``python bench.py --designs [--design fegilix|guzovik|gasavik|diderax|sanevik] [--design-beside qwen3|guzovik|...]``:
+"""``python bench.py --designs [--design fegilix|guzovik|gasavik|diderax|sanevik|risonex] [--design-beside qwen3|guzovik|...]``:
 prefill and decode throughput of a design at layer sizes that resemble a real model's (random weights), beside
 the dense Qwen3 decoder (or, with ``--design-beside``, another design of the framework), with the same width,
 attention heads, (active) feed-forward size and number of layers; and where each design's step time goes, kernel class by kernel class, with the
@@ -126,13 +126,31 @@ def sanevik_config(s: dict) -> dict:
             "loop": {"start": 0, "stop": 2, "times": 2}, "layers": [a, p, a, p]}
 
 
+def risonex_config(s: dict) -> dict:
+    """Four layers of which the first two run twice: Mamba-2 + dense feed-forward, differential attention + routed
+    experts, then the same mixers with the feed-forwards exchanged. Two maps of 64 per attention head over values of 128,
+    chunks of 1,536; Mamba-2 with an inner width of twice the model's in heads of 64, a state of 128 in 8 groups; three of
+    the router's outputs per token (experts of a quarter of the dense size, or one of four identity experts) beside a gated
+    shared expert of that size; the ungated dense feed-forward half as wide again, so that its weights are the gated one's."""
+    attn = {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": s["dim"] // 2, "vdim": s["dim"], "scale": (s["dim"] // 2) ** -0.5,
+            "diff": 0.3, "mask": {"size": 1536}}
+    ssd = {"heads": s["width"] // 32, "groups": 8, "state": 128, "vdim": 64, "conv": 4, "norm_groups": 8}
+    ff = s["ff"] // 4
+    moe = {"kind": "moe", "router": {"experts": s["experts"], "identity": 4, "top": 3, "scale": 2.0}, "expert": {"ff": ff}, "shared": {"ff": ff}}
+    dense = {"kind": "dense", "ff": 3 * s["ff"] // 2}
+    return {"architecture": "Risonex", "vocab": VOCAB, "width": s["width"], "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0},
+            "max_positions": 8192, "loop": {"start": 0, "stop": 2, "times": 2},
+            "layers": [{"type": "mamba2", "mlp": dense, "mixer": ssd}, {"type": "attention", "mlp": moe, "mixer": attn},
+                       {"type": "mamba2", "mlp": moe, "mixer": ssd}, {"type": "attention", "mlp": dense, "mixer": attn}]}
+
+
 DESIGNS = {"fegilix": fegilix_config, "guzovik": guzovik_config, "gasavik": gasavik_config, "diderax": diderax_config,
-           "sanevik": sanevik_config}
+           "sanevik": sanevik_config, "risonex": risonex_config}
 NEW_OPS = ["post_norm_add_rms_norm", "latent_prepare", "latent_attention", "bmm", "transpose01", "moe_route_from", "moe_route", "moe_gemm",
            "moe_combine", "gemm_gated", "hc_mix_norm", "hc_collapse", "act_mul", "softcap", "head_norm_gate", "mlstm_scan", "delta_scan",
            "causal_conv_silu", "qkv_prepare", "linear_scan_bonus", "linear_scan_decay", "token_shift_mix", "embed_pos_norm",
            "stream_sum", "add_bias", "tanh_", "act_mul_gather", "gemm_biased_swiglu", "linear_scan_gated", "rms_norm_rows",
-           "qkv_rotate", "talking_attention", "linear_scan_rotated"]
+           "qkv_rotate", "talking_attention", "linear_scan_rotated", "state_space_scan", "gemm_activated", "stream_beside"]
 OLD_OPS = ["embed", "add_rms_norm", "rope_tables", "silu_mul", "qk_norm_rope_write", "paged_attention",
            "decode_attention_fused", "gemm", "gemm_swiglu", "gemm_to_stream", "gemm_normed", "sample"]
 
@@ -200,17 +218,17 @@ class DesignBench(Bench):
         def nbytes(*ts) -> float:
             return float(sum(t.numel() * t.element_size() for t in ts if isinstance(t, torch.Tensor)))
 
-        def seen(ctx, window: int) -> float:
-            """(query, key) pairs of a step under a causal mask and a window (0: none)."""
+        def seen(ctx, window: int, chunk: int = 0) -> float:
+            """(query, key) pairs of a step under a causal mask and a window or chunks (0: none)."""
             total = 0.0
             for n, c in zip(ctx.query_lens, ctx.context_lens):
                 for p in range(c - n, c):
-                    total += min(p + 1, window) if window else p + 1
+                    total += min(p + 1, window) if window else p % chunk + 1 if chunk else p + 1
             return total
 
         def work(name: str, a: tuple, k: dict) -> tuple[float, float]:
             """(bytes, flops) of one call."""
-            if name in ("gemm", "gemm_swiglu", "gemm_to_stream", "gemm_gated"):
+            if name in ("gemm", "gemm_swiglu", "gemm_to_stream", "gemm_gated", "gemm_activated"):
                 return nbytes(a[0], a[1], a[2]), 2.0 * a[0].shape[0] * a[1].shape[0] * a[1].shape[1]
             if name == "gemm_biased_swiglu":      # x, the gate and up rows, the biases, the result
                 return nbytes(a[0], a[1], a[2], a[3]), 2.0 * a[0].shape[0] * a[1].shape[0] * a[1].shape[1]
@@ -243,9 +261,11 @@ class DesignBench(Bench):
                 ctx = a[5] if name == "paged_attention" else a[11]
                 heads = a[0].shape[1] if name == "paged_attention" else a[14]
                 window = a[7] if name == "paged_attention" else 0
-                rows = sum(min(c, (window or c) + n - 1) for n, c in zip(ctx.query_lens, ctx.context_lens))
+                # two maps: each scores with half of the row and weighs the values of its own
+                chunk, maps = k.get("chunk", 0), k.get("maps", 1)
+                rows = sum(c - (c - n) // chunk * chunk if chunk else min(c, (window or c) + n - 1) for n, c in zip(ctx.query_lens, ctx.context_lens))
                 return (float(rows) * kc.shape[1] * (kc.shape[3] + vc.shape[3]) * kc.element_size(),
-                        2.0 * heads * (kc.shape[3] + vc.shape[3]) * seen(ctx, window))
+                        2.0 * heads * (kc.shape[3] + maps * vc.shape[3]) * seen(ctx, window, chunk))
             if name == "qk_norm_rope_write":
                 return 2.0 * nbytes(a[0]), 0.0
             if name == "qkv_prepare":         # q, k and v rows read and written
@@ -272,6 +292,11 @@ class DesignBench(Bench):
             if name == "linear_scan_rotated":     # state in and out, q, k, v read, the read-out written; 4 flops per state element and token
                 ctx, heads, d, dv = a[10], a[11], a[12], a[13]
                 return (2.0 * ctx.num_seqs * heads * d * dv * 4 + nbytes(a[0], a[1], a[2], a[14]), 4.0 * a[0].shape[0] * heads * d * dv)
+            if name == "state_space_scan":    # state in and out, C, B, x read, the read-out written; 4 flops per state element and token
+                ctx, heads, d, dv = a[8], a[9], a[11], a[12]
+                return (2.0 * ctx.num_seqs * heads * d * dv * 4 + nbytes(a[0], a[1], a[2], a[13]), 4.0 * a[0].shape[0] * heads * d * dv)
+            if name == "stream_beside":
+                return nbytes(*a), 0.0
             if name == "qkv_rotate":          # q, k and v rows read and written
                 return 2.0 * a[0].shape[0] * ((a[13] + a[14]) * a[15] + a[14] * a[16]) * a[0].element_size(), 0.0
             if name == "talking_attention":   # keys and values once per request; both products and the mixing of the heads

@@ -164,14 +164,18 @@ def test_keys_of_two_maps_side_by_side(dtype, heads, groups, d, dv, rotary) -> N
         torch.testing.assert_close(got, want, equal_nan=True, **_tol(dtype))
 
 
-@pytest.mark.parametrize("heads, groups, d, dv", [(2, 1, 16, 24), (4, 2, 40, 16), (3, 3, 8, 8), (4, 1, 64, 64), (2, 2, 128, 40), (1, 1, 256, 32), (6, 2, 20, 12)])
-def test_state_space_scan_kernel(heads, groups, d, dv) -> None:
+@pytest.mark.parametrize("chunks", [True, False])
+@pytest.mark.parametrize("heads, groups, d, dv", [(2, 1, 16, 24), (4, 2, 40, 16), (3, 3, 8, 8), (4, 1, 64, 64), (2, 2, 128, 40), (1, 1, 256, 32), (6, 2, 20, 12),
+                                                  (24, 2, 128, 64), (5, 1, 50, 130), (3, 1, 7, 67)])
+def test_state_space_scan_kernel(heads, groups, d, dv, chunks, monkeypatch) -> None:
     """Prompt portions, single tokens and portions long enough to run in segments, from and to state slots out of order;
-    rates from slow to fast, step sizes over several orders of magnitude; C, B and x are column slices."""
+    rates from slow to fast, step sizes over several orders of magnitude; C, B and x are column slices. Long portions as
+    products over chunks of tokens and, with that switched off (and where the state is too wide), token by token."""
     ops = _ops()
+    monkeypatch.setattr(ops, "STATE_SPACE_CHUNKS", chunks)
     a_log, skip = torch.linspace(-4.0, 2.0, heads, device="cuda"), _rand(heads, seed=7)
     bias = torch.linspace(-3.0, 1.0, heads, device="cuda")
-    for lens in ([5, 1, 33, 1, 2], [1, 1, 1], [300, 7, 1], [16, 17], [700, 260]):
+    for lens in ([5, 1, 33, 1, 2], [1, 1, 1], [300, 7, 1], [16, 17], [700, 260], [1, 1, 128, 1, 65, 64, 2], [63, 193]):
         t = sum(lens)
         wide = _rand(t, 2 * groups * d + heads * dv + 3, seed=1, scale=0.5)
         x, b, c = wide[:, : heads * dv], wide[:, heads * dv: heads * dv + groups * d], wide[:, heads * dv + groups * d: heads * dv + 2 * groups * d]
@@ -193,9 +197,11 @@ def test_state_space_scan_kernel(heads, groups, d, dv) -> None:
         assert torch.equal(res[0][1][untouched], start[untouched].double())
 
 
-def test_a_state_a_thousand_tokens_old_is_still_read() -> None:
+@pytest.mark.parametrize("chunks", [True, False])
+def test_a_state_a_thousand_tokens_old_is_still_read(chunks, monkeypatch) -> None:
     """One write that decays slowly, then steps that write next to nothing: the read-out far behind it is its value."""
     ops = _ops()
+    monkeypatch.setattr(ops, "STATE_SPACE_CHUNKS", chunks)
     heads, d, dv, t = 2, 16, 8, 1200
     x, b, c = torch.zeros(t, heads * dv, device="cuda"), torch.zeros(t, heads * d, device="cuda"), torch.zeros(t, heads * d, device="cuda")
     x[0], b[0], c[-1] = 3.0, 1.0, 1.0
@@ -218,13 +224,38 @@ def test_a_state_a_thousand_tokens_old_is_still_read() -> None:
         torch.testing.assert_close(out[-1], torch.full((heads, dv), float(want), device="cuda"), rtol=1e-4, atol=0.0)
 
 
+def test_a_weak_decay_behind_a_strong_one_keeps_its_digits() -> None:
+    """Within a chunk one token decays everything before it to nothing; what is written behind it decays by very little. The
+    differences of large running sums still give those small decays to 32-bit accuracy."""
+    ops = _ops()
+    heads, d, dv, t = 2, 24, 16, 192
+    x, b, c = _rand(t, heads * dv, seed=1), _rand(t, heads * d, seed=2), _rand(t, heads * d, seed=3)
+    step = torch.full((t, heads), -6.0, device="cuda")
+    step[5::40] = 9.0
+    a_log = torch.tensor([6.0, 3.0], device="cuda")
+    zero = torch.zeros(heads, device="cuda")
+    res = []
+    for impl, up in ((ops, torch.float32), (refs, torch.float64)):
+        state = torch.zeros(2, heads * d * dv, dtype=up, device="cuda")
+        ctx = FakeStep([t], [1], device="cuda")
+        ctx.arena = Arena()
+        out = torch.empty(t, heads, dv, dtype=up, device="cuda")
+        impl.state_space_scan(c, b, x, step, zero, a_log, zero, state, ctx, heads, heads, d, dv, out)
+        res.append(out.double())
+    quiet = torch.ones(t, dtype=torch.bool)
+    for n in range(5, t, 40):
+        quiet[n: n + 3] = False               # right behind the strong token its own large write dominates
+    scale = res[1][quiet].abs().median()
+    assert float((res[0] - res[1])[quiet].abs().max()) < 2e-5 * max(1.0, float(res[1].abs().max())) and float(scale) > 0.0
+
+
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("taps", [1, 2, 3, 4, 6, 8])
 def test_convolution_with_a_bias_kernel(dtype, taps) -> None:
     """Portions of several lengths (also shorter than the taps), and a step of single tokens (one kernel then)."""
     ops = _ops()
     channels = 300
-    for lens in ([5, 1, 2, 33, 3], [1, 1, 1]):
+    for lens in ([5, 1, 2, 33, 3], [1, 1, 1], [40, 1, 2, 16, 1, 1, 37]):
         t = sum(lens)
         x = _rand(t, channels + 40, seed=1, dtype=dtype)[:, 24: 24 + channels]
         w, bias = _rand(channels, taps, seed=2, scale=0.5, dtype=dtype), _rand(channels, seed=3, dtype=dtype)

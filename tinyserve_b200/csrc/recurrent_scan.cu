@@ -387,6 +387,76 @@ __global__ void causal_conv_silu_kernel(const T* __restrict__ x, int x_stride, c
   }
 }
 
+// The same for many tokens: a thread takes four channels of CONV_RUN consecutive tokens and keeps the taps and the last
+// inputs in registers (right-aligned: slot KP - 1 is the current token), so an input is read once, eight or sixteen
+// bytes at a time. KP: the taps rounded up to 4 or 8, the missing ones zero.
+constexpr int CONV_RUN = 16, CONV_MIN_TOKENS = 64;
+template <typename T, int KP>
+__global__ void __launch_bounds__(128) causal_conv_silu_run_kernel(const T* __restrict__ x, int x_stride, const T* __restrict__ taps,
+                                                                   const T* __restrict__ bias, const float* __restrict__ state,
+                                                                   int state_stride, const int* __restrict__ cu_q,
+                                                                   const int* __restrict__ state_slots, int num_seqs, int num_tokens, int C,
+                                                                   int K, float* __restrict__ y) {
+  pdl_trigger();
+  pdl_wait();
+  const int c = (blockIdx.x * blockDim.x + threadIdx.x) * 4;
+  if (c >= C) return;
+  const int first = blockIdx.y * CONV_RUN, last = min(first + CONV_RUN, num_tokens);
+  float w[KP][4], b[4] = {0.f, 0.f, 0.f, 0.f}, in[KP][4];
+#pragma unroll
+  for (int j = 0; j < KP; ++j)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) w[j][e] = j >= KP - K ? to_float(taps[(size_t)(c + e) * K + j - (KP - K)]) : 0.f;
+  if (bias) Quad<T>::load(bias + c, b);
+  int lo = 0, hi = num_seqs - 1;
+  while (lo < hi) {
+    const int mid = (lo + hi + 1) >> 1;
+    if (cu_q[mid] <= first) lo = mid; else hi = mid - 1;
+  }
+  int start = cu_q[lo], end = cu_q[lo + 1];
+  const float* st = state + (size_t)state_slots[lo] * state_stride + c;
+  bool fill = true;                       // the inputs before token t are not in the registers yet
+  for (int t = first; t < last; ++t) {
+    while (t >= end && lo + 1 < num_seqs) {
+      ++lo;
+      start = end;
+      end = cu_q[lo + 1];
+      st = state + (size_t)state_slots[lo] * state_stride + c;
+      fill = true;
+    }
+    if (fill) {
+#pragma unroll
+      for (int j = 0; j < KP - 1; ++j) {
+        const int tau = t - (KP - 1 - j);
+        if (j < KP - K) {
+#pragma unroll
+          for (int e = 0; e < 4; ++e) in[j + 1][e] = 0.f;
+        } else if (tau >= start) {
+          Quad<T>::load(x + (size_t)tau * x_stride + c, in[j + 1]);
+        } else {
+#pragma unroll
+          for (int e = 0; e < 4; ++e) in[j + 1][e] = st[(size_t)(K - 1 + tau - start) * C + e];
+        }
+      }
+      fill = false;
+    }
+#pragma unroll
+    for (int j = 0; j < KP - 1; ++j)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) in[j][e] = in[j + 1][e];
+    Quad<T>::load(x + (size_t)t * x_stride + c, in[KP - 1]);
+    float o[4];
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      float acc = b[e];
+#pragma unroll
+      for (int j = 0; j < KP; ++j) acc = fmaf(w[j][e], in[j][e], acc);
+      o[e] = acc / (1.f + expf(-acc));
+    }
+    Quad<float>::store(y + (size_t)t * C + c, o);
+  }
+}
+
 // A step in which no request brings more than one token: output and new state in one pass, a thread per (request, channel).
 template <typename T>
 __global__ void causal_conv_silu_single_kernel(const T* __restrict__ x, int x_stride, const T* __restrict__ taps,
@@ -547,6 +617,23 @@ extern "C" int ts_causal_conv_silu(const void* x, int x_stride, const void* taps
   if (single && dtype == TS_DTYPE_BF16)
     return launch(causal_conv_silu_single_kernel<bf16>, sgrid, threads, 0, stream, (const bf16*)x, x_stride, (const bf16*)taps,
                   (const bf16*)bias, state, state_stride, cu_q, state_slots, channels, num_taps, y);
+  const size_t es = dtype == TS_DTYPE_F32 ? 16 : 8;      // bytes of four inputs
+  if (num_tokens >= CONV_MIN_TOKENS && channels % 4 == 0 && (x_stride % 4) == 0 && (uintptr_t)x % es == 0 && (uintptr_t)bias % es == 0 &&
+      ((uintptr_t)y & 15) == 0 && (dtype == TS_DTYPE_F32 || dtype == TS_DTYPE_BF16)) {
+    const dim3 rgrid((channels / 4 + 127) / 128, (num_tokens + CONV_RUN - 1) / CONV_RUN);
+#define TS_CONV_RUN(T_, KP_)                                                                                                     \
+  launch(causal_conv_silu_run_kernel<T_, KP_>, rgrid, 128, 0, stream, (const T_*)x, x_stride, (const T_*)taps, (const T_*)bias, \
+         (const float*)state, state_stride, cu_q, state_slots, num_seqs, num_tokens, channels, num_taps, y)
+    st = dtype == TS_DTYPE_F32 ? (num_taps <= 4 ? TS_CONV_RUN(float, 4) : TS_CONV_RUN(float, 8))
+                               : (num_taps <= 4 ? TS_CONV_RUN(bf16, 4) : TS_CONV_RUN(bf16, 8));
+#undef TS_CONV_RUN
+    if (st != 0 || num_taps == 1) return st;
+    return dtype == TS_DTYPE_F32
+               ? launch(conv_state_update_kernel<float>, sgrid, threads, 0, stream, (const float*)x, x_stride, state, state_stride, cu_q, state_slots,
+                        channels, num_taps)
+               : launch(conv_state_update_kernel<bf16>, sgrid, threads, 0, stream, (const bf16*)x, x_stride, state, state_stride, cu_q, state_slots,
+                        channels, num_taps);
+  }
   if (dtype == TS_DTYPE_F32) {
     st = launch(causal_conv_silu_kernel<float>, grid, threads, 0, stream, (const float*)x, x_stride, (const float*)taps, (const float*)bias,
                 (const float*)state, state_stride, cu_q, state_slots, num_seqs, num_tokens, channels, num_taps, y);

@@ -51,6 +51,8 @@ _SIGNATURES: dict[str, list[Any]] = {
     "ts_tanh": [_vp, _c.c_size_t, _i, _vp],
     "ts_linear_scan": [_i, _vp, _i, _vp, _i, _vp, _i, _vp, _i, _vp, _vp, _vp, _vp, _i, _vp, _vp, _i, _i, _i, _i, _vp, _i, _i, _i, _i, _vp, _vp,
                        _f, _f, _vp, _vp, _i, _i, _f, _i, _vp],
+    "ts_state_space_chunks": [_vp, _i, _vp, _i, _vp, _i, _vp, _i, _vp, _vp, _vp, _vp, _i, _vp, _vp, _i, _i, _i, _i, _i, _i, _vp, _vp, _vp,
+                              _vp],
     "ts_token_shift_mix": [_vp, _i, _vp, _i, _vp, _i, _vp, _vp, _i, _i, _i, _vp, _i, _vp],
     "ts_softcap": [_vp, _c.c_size_t, _f, _vp],
     "ts_rms_norm_rows": [_vp, _c.c_longlong, _vp, _f, _vp, _i, _i, _i, _vp],
@@ -1445,7 +1447,40 @@ def state_space_scan(c: torch.Tensor, b: torch.Tensor, x: torch.Tensor, dt_pre: 
     float32; ``dt_bias``, ``a_log``, ``skip`` ``[heads]`` float32; ``state [slots, heads * d * dv]`` float32; ``out [T, heads, dv]`` float32."""
     if heads % groups or c.dtype != torch.float32:
         raise KernelError("state_space_scan: groups must divide the heads; float32 only")
+    t = c.shape[0]
+    chunks = t // STATE_SPACE_CHUNK + ctx.num_seqs
+    if (STATE_SPACE_CHUNKS and ctx.max_query_len >= STATE_SPACE_CHUNKS_MIN_TOKENS and d <= STATE_SPACE_CHUNKS_MAX_STATE
+            and 4 * chunks * heads * d * dv <= STATE_SPACE_CHUNKS_SCRATCH_BYTES):
+        _state_space_chunks(c, b, x, dt_pre, dt_bias, a_log, skip, state, ctx, heads, groups, d, dv, out, chunks)
+        return
     _linear_scan(4, c, b, x, dt_pre, dt_bias, skip, a_log, state, ctx, heads, d, dv, out, groups=groups)
+
+
+STATE_SPACE_CHUNKS = True               # long portions as products over chunks; False: token by token always
+STATE_SPACE_CHUNK = 64                  # tokens of a chunk, as the kernel is built
+STATE_SPACE_CHUNKS_MIN_TOKENS = 128
+STATE_SPACE_CHUNKS_MAX_STATE = 128
+STATE_SPACE_CHUNKS_SCRATCH_BYTES = 1 << 30
+
+
+def _state_space_chunks(c: torch.Tensor, b: torch.Tensor, x: torch.Tensor, dt_pre: torch.Tensor, dt_bias: torch.Tensor, a_log: torch.Tensor,
+                        skip: torch.Tensor, state: torch.Tensor, ctx: Any, heads: int, groups: int, d: int, dv: int, out: torch.Tensor,
+                        chunks: int) -> None:
+    """``state_space_scan`` of a step with long portions: 32-bit products over chunks of 64 tokens (``csrc/state_space_chunks.cu``)."""
+    t = c.shape[0]
+    for name, v, width in (("c", c, groups * d), ("b", b, groups * d), ("x", x, heads * dv), ("dt_pre", dt_pre, heads)):
+        if not v.is_cuda or v.dtype != torch.float32 or tuple(v.shape) != (t, width) or v.stride(1) != 1:
+            raise KernelError(f"state_space_scan: {name} must be [T, {width}] float32 with unit column stride on the device")
+    if tuple(out.shape) != (t, heads, dv) or any(p.shape != (heads,) for p in (dt_bias, a_log, skip)):
+        raise KernelError("state_space_scan: out shape, or one bias, rate and skip per head")
+    state_ptr, state_stride = _state_rows(state, heads * d * dv, "state_space_scan")
+    left = ctx.arena.take((chunks, heads * d * dv), torch.float32)
+    decay = ctx.arena.take((chunks, heads), torch.float32)
+    _check(_fn("ts_state_space_chunks")(
+        c.data_ptr(), c.stride(0), b.data_ptr(), b.stride(0), x.data_ptr(), x.stride(0), dt_pre.data_ptr(), dt_pre.stride(0),
+        _dev(dt_bias, "dt_bias", torch.float32), _dev(a_log, "a_log", torch.float32), _dev(skip, "skip", torch.float32), state_ptr, state_stride,
+        _dev(ctx.cu_query_lens, "cu_query_lens", torch.int32), _dev(ctx.state_slots, "state_slots", torch.int32), ctx.num_seqs, t,
+        heads, groups, d, dv, left.data_ptr(), decay.data_ptr(), _dev(out, "out", torch.float32), _stream()), "state_space_scan", kernels=3)
 
 
 def _linear_scan(mode: int, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, w_pre: torch.Tensor | None,
