@@ -126,6 +126,56 @@ __global__ void head_norm_gate_kernel(const IN* __restrict__ x, const T* __restr
   }
 }
 
+// The same with four columns an access and the values kept in registers between the two passes: a warp per (token, head) of
+// up to 128 J columns (a multiple of 4, everything aligned).
+template <typename IN, typename T, int J>
+__global__ void __launch_bounds__(128) head_norm_gate_quads_kernel(const IN* __restrict__ x, const T* __restrict__ weight, int weight_head_stride,
+                                                                   const T* __restrict__ gate, int gate_stride, T* __restrict__ out,
+                                                                   int num_tokens, int heads, int width, int normalise, float eps,
+                                                                   int gate_silu, int gate_first) {
+  pdl_trigger();
+  pdl_wait();
+  const int warp = (int)(((size_t)blockIdx.x * blockDim.x + threadIdx.x) >> 5), lane = threadIdx.x & 31;
+  if (warp >= num_tokens * heads) return;
+  const int t = warp / heads, h = warp - t * heads;
+  const IN* xr = x + (size_t)warp * width;
+  const T* gr = gate ? gate + (size_t)t * gate_stride + h * width : nullptr;
+  float v[J][4], z[J][4];
+#pragma unroll
+  for (int j = 0; j < J; ++j) {
+    const int c = (lane + 32 * j) * 4;
+#pragma unroll
+    for (int e = 0; e < 4; ++e) { v[j][e] = 0.f; z[j][e] = 0.f; }
+    if (c < width) {
+      Quad<IN>::load(xr + c, v[j]);
+      if (gr) Quad<T>::load(gr + c, z[j]);
+    }
+  }
+  float ss = 0.f;
+#pragma unroll
+  for (int j = 0; j < J; ++j)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      z[j][e] = !gr ? 1.f : gate_silu ? z[j][e] * sigmoidf(z[j][e]) : sigmoidf(z[j][e]);
+      if (gate_first) v[j][e] *= z[j][e];
+      ss = fmaf(v[j][e], v[j][e], ss);
+    }
+  const float rstd = normalise ? rsqrtf(warp_sum(ss) / (float)width + eps) : 1.f;
+#pragma unroll
+  for (int j = 0; j < J; ++j) {
+    const int c = (lane + 32 * j) * 4;
+    if (c >= width) continue;
+    float w[4] = {1.f, 1.f, 1.f, 1.f};
+    if (weight) Quad<T>::load(weight + h * weight_head_stride + c, w);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      v[j][e] *= rstd * w[e];
+      if (!gate_first) v[j][e] *= z[j][e];
+    }
+    Quad<T>::store(out + (size_t)warp * width + c, v[j]);
+  }
+}
+
 // The same for wide rows (all heads normed together, say): a CTA per (token, head), the row's sum of squares
 // through shared memory.
 template <typename IN, typename T>
@@ -280,6 +330,26 @@ extern "C" int ts_head_norm_gate(const void* x, int x_is_f32, const void* weight
   const size_t warps = (size_t)num_tokens * heads;
   if (warps == 0) return 0;
   if (gate_first && (!gate || gate_per_head)) return TS_ERR_BAD_ARGUMENT;
+  const uintptr_t elem = dtype == TS_DTYPE_F32 ? 16 : 8, in_elem = dtype == TS_DTYPE_F32 || x_is_f32 ? 16 : 8;      // bytes of four values
+  if (width % 4 == 0 && width <= 1024 && !gate_per_head && gate_stride % 4 == 0 && weight_head_stride % 4 == 0 && (uintptr_t)x % in_elem == 0 &&
+      (((uintptr_t)weight | (uintptr_t)gate | (uintptr_t)out) % elem) == 0 && (dtype == TS_DTYPE_F32 || dtype == TS_DTYPE_BF16)) {
+    const int qb = (int)((warps * 32 + 127) / 128);
+#define TS_HN_QUADS(IN_, T_, J_)                                                                                                      \
+  return launch(head_norm_gate_quads_kernel<IN_, T_, J_>, qb, 128, 0, stream, (const IN_*)x, (const T_*)weight, weight_head_stride,  \
+                (const T_*)gate, gate_stride, (T_*)out, num_tokens, heads, width, normalise, eps, gate_silu, gate_first)
+#define TS_HN_WIDTHS(IN_, T_)                  \
+  {                                            \
+    if (width <= 128) TS_HN_QUADS(IN_, T_, 1); \
+    if (width <= 256) TS_HN_QUADS(IN_, T_, 2); \
+    if (width <= 512) TS_HN_QUADS(IN_, T_, 4); \
+    TS_HN_QUADS(IN_, T_, 8);                   \
+  }
+    if (dtype == TS_DTYPE_F32) TS_HN_WIDTHS(float, float);
+    if (x_is_f32) TS_HN_WIDTHS(float, bf16);
+    TS_HN_WIDTHS(bf16, bf16);
+#undef TS_HN_WIDTHS
+#undef TS_HN_QUADS
+  }
   if (width >= 512) {      // a CTA per row
     const int rows = (int)warps;
     if (dtype == TS_DTYPE_F32)

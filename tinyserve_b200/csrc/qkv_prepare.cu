@@ -212,6 +212,93 @@ __global__ void qkv_prepare_kernel(const T* __restrict__ q_in, int q_stride, con
   }
 }
 
+// bfloat16 heads of up to 8 LPH elements in 16-byte accesses: a head (or an equal piece of a value head) is a group of LPH
+// lanes with eight elements each, so a warp takes 32 / LPH of them at once. Head sizes that are a multiple of 8, a rotation
+// whose pairs lie a whole number of lanes apart, no biases, everything 16-byte aligned.
+template <int LPH>
+__global__ void __launch_bounds__(128) qkv_prepare_packed_kernel(
+    const bf16* __restrict__ q_in, int q_stride, const bf16* __restrict__ k_in, int k_stride, const bf16* __restrict__ v_in, int v_stride,
+    const bf16* __restrict__ q_w, const bf16* __restrict__ k_w, float eps, const float* __restrict__ cos_tab,
+    const float* __restrict__ sin_tab, int rotary_dim, const int* __restrict__ slots, bf16* __restrict__ k_cache,
+    bf16* __restrict__ v_cache, int page_size, int num_tokens, int heads, int kv_heads, int d, int dv, bf16* __restrict__ q_out, int maps) {
+  pdl_trigger();
+  pdl_wait();
+  const int k_heads = k_in ? kv_heads * maps : 0, v_pieces = (dv + 8 * LPH - 1) / (8 * LPH);
+  const int jobs = heads + k_heads + (k_in ? kv_heads * v_pieces : 0);
+  const int l = threadIdx.x % LPH;                     // this lane's place in its group
+  const long long job_id = ((long long)blockIdx.x * blockDim.x + threadIdx.x) / LPH;
+  const bool in = job_id < (long long)num_tokens * jobs;
+  const int t = in ? (int)(job_id / jobs) : 0, job = in ? (int)(job_id - (long long)t * jobs) : 0;
+  const bool is_v = job >= heads + k_heads, is_q = job < heads;
+  const bf16* src = q_in + (size_t)t * q_stride + job * d;
+  bf16* dst = q_out + ((size_t)t * heads + job) * d;
+  int size = d, at = 8 * l;
+  if (!is_q) {
+    const int slot = slots[t], page = slot / page_size, off = slot - page * page_size;
+    if (!is_v) {
+      const int g = job - heads, kvh = g / maps;
+      src = k_in + (size_t)t * k_stride + g * d;
+      dst = k_cache + ((((size_t)page * kv_heads + kvh) * page_size + off) * maps + (g - kvh * maps)) * d;
+    } else {
+      const int vj = job - heads - k_heads, g = vj / v_pieces;
+      src = v_in + (size_t)t * v_stride + g * dv;
+      dst = v_cache + (((size_t)page * kv_heads + g) * page_size + off) * dv;
+      at += (vj - g * v_pieces) * 8 * LPH;
+      size = dv;
+    }
+  }
+  const bool mine = in && at < size;
+  uint4 raw = make_uint4(0u, 0u, 0u, 0u);
+  if (mine) raw = *reinterpret_cast<const uint4*>(src + at);
+  const bf16* w = is_q ? q_w : k_w;
+  // every lane of the warp takes part in the sums and exchanges below; a piece of values keeps its bits
+  const uint32_t* words = reinterpret_cast<const uint32_t*>(&raw);
+  float x[8];
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    x[2 * i] = __uint_as_float(words[i] << 16);
+    x[2 * i + 1] = __uint_as_float(words[i] & 0xffff0000u);
+  }
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < 8; ++i) ss = fmaf(x[i], x[i], ss);
+#pragma unroll
+  for (int o = LPH / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+  if (w != nullptr && !is_v && mine) {
+    const float rstd = rsqrtf(ss / (float)d + eps);
+    const uint4 wr = *reinterpret_cast<const uint4*>(w + at);
+    const uint32_t ww[4] = {wr.x, wr.y, wr.z, wr.w};
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      x[2 * i] *= __uint_as_float(ww[i] << 16) * rstd;
+      x[2 * i + 1] *= __uint_as_float(ww[i] & 0xffff0000u) * rstd;
+    }
+  }
+  if (rotary_dim > 0) {
+    const int half = rotary_dim >> 1;
+    const bool low = at < half, turns = mine && !is_v && at < rotary_dim;
+    const int base = (threadIdx.x & 31) - l;
+    const int partner = turns ? base + (low ? at + half : at - half) / 8 : (threadIdx.x & 31);
+    float y[8];
+#pragma unroll
+    for (int i = 0; i < 8; ++i) y[i] = __shfl_sync(0xffffffffu, x[i], partner);
+    if (turns) {
+      const float* c = cos_tab + (size_t)t * half + (low ? at : at - half);
+      const float* s = sin_tab + (size_t)t * half + (low ? at : at - half);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) x[i] = low ? x[i] * c[i] - y[i] * s[i] : x[i] * c[i] + y[i] * s[i];
+    }
+  }
+  if (!mine) return;
+  if (is_v) {
+    *reinterpret_cast<uint4*>(dst + at) = raw;
+    return;
+  }
+  Vec<bf16> o;
+  o.pack(x);
+  o.store(dst + at);
+}
+
 // The norm over the whole projection: a CTA per token. All its threads form the sums of squares of the token's q row
 // and k row once; then its warps take the heads in turn, each with the row's 1 / rms and its own stretch of the weight.
 constexpr int QW_WARPS = 8;
@@ -299,6 +386,21 @@ extern "C" int ts_qkv_prepare(const void* q_in, int q_stride, const void* k_in, 
                     (const bf16*)q_w, (const bf16*)k_w, eps, cos_tab, sin_tab, rotary_dim, slots, (bf16*)k_cache, (bf16*)v_cache,
                     page_size, heads, kv_heads, d, dv, (bf16*)q_out);
     return TS_ERR_BAD_ARGUMENT;
+  }
+  if (dtype == TS_DTYPE_BF16 && d % 8 == 0 && d <= 128 && dv % 8 == 0 && !q_b && !k_b && !v_b && rotary_dim % 16 == 0 && q_stride % 8 == 0 &&
+      k_stride % 8 == 0 && v_stride % 8 == 0 &&
+      (((uintptr_t)q_in | (uintptr_t)k_in | (uintptr_t)v_in | (uintptr_t)q_w | (uintptr_t)k_w | (uintptr_t)k_cache | (uintptr_t)v_cache | (uintptr_t)q_out) & 15) == 0) {
+    const int lph = d <= 32 ? 4 : d <= 64 ? 8 : 16;
+    const long long jobs = heads + (k_in ? maps * kv_heads + (long long)kv_heads * ((dv + 8 * lph - 1) / (8 * lph)) : 0);
+    const int pb = (int)((num_tokens * jobs * lph + 127) / 128);
+#define TS_QP_PACKED(L_)                                                                                                              \
+  return launch(qkv_prepare_packed_kernel<L_>, pb, 128, 0, stream, (const bf16*)q_in, q_stride, (const bf16*)k_in, k_stride,         \
+                (const bf16*)v_in, v_stride, (const bf16*)q_w, (const bf16*)k_w, eps, cos_tab, sin_tab, rotary_dim, slots, (bf16*)k_cache, \
+                (bf16*)v_cache, page_size, num_tokens, heads, kv_heads, d, dv, (bf16*)q_out, maps)
+    if (lph == 4) TS_QP_PACKED(4);
+    if (lph == 8) TS_QP_PACKED(8);
+    TS_QP_PACKED(16);
+#undef TS_QP_PACKED
   }
   const long long warps = (long long)num_tokens * (heads + (k_in ? (maps + 1) * kv_heads : 0));
   const int threads = QP_WARPS * 32;

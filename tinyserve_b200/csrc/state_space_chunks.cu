@@ -12,13 +12,15 @@
 //                     the weighted scores times x plus C times S_0.
 //
 // Everything is 32-bit on CUDA cores (the state and what enters it must be), but as register-tiled products: a thread
-// holds 8 x 4 sums and spends three 16-byte reads of shared memory on 32 multiply-adds, where the token-by-token form
-// spends a read on four. The running sums are kept in 64-bit: the difference of two of them is what decays a weight, and
+// holds 4 x 4 or 8 x 4 sums and spends a 16-byte read of shared memory on eight or eleven multiply-adds, where the
+// token-by-token form spends one on four. The running sums are kept in 64-bit: the difference of two of them is what decays a weight, and
 // in 32-bit it would lose the digits that a long or fast decaying chunk has accumulated. Every exponent is at most zero.
 //
 // Chunks are numbered over the whole step, request b's from cu_q[b] / 64 + b on (gaps of at most one), so scratch and
 // grid follow the step's tokens, however unequal the requests are; a request of one token costs one chunk of one row.
 #define TS_PDL_CLASS PDL_OTHER
+#include <cuda_pipeline_primitives.h>
+
 #include "common.cuh"
 
 namespace ts {
@@ -81,44 +83,58 @@ __device__ __forceinline__ void chunk_steps(const ScanChunkArgs& a, int h, int t
   cum_s[2 * lane + 1] = run;
 }
 
-// acc[8][4] += A^T B over k rows: A's rows hold the 8-wide operand (row `lda` floats, this thread's 8 from `ar`), B's the
-// 4-wide one. Both 16-byte aligned.
-__device__ __forceinline__ void tile_product(float (&acc)[8][4], const float* ar, int lda, const float* br, int ldb, int k) {
+// acc[4 A][4] += A^T B over k rows: A's rows hold the 4 A-wide operand (row `lda` floats, this thread's part from `ar`), B's
+// the 4-wide one. Both 16-byte aligned.
+template <int A>
+__device__ __forceinline__ void tile_product(float (&acc)[4 * A][4], const float* ar, int lda, const float* br, int ldb, int k) {
 #pragma unroll 4
   for (int i = 0; i < k; ++i) {
-    const float4 a0 = *reinterpret_cast<const float4*>(ar + i * lda);
-    const float4 a1 = *reinterpret_cast<const float4*>(ar + i * lda + 4);
     const float4 b = *reinterpret_cast<const float4*>(br + i * ldb);
-    const float av[8] = {a0.x, a0.y, a0.z, a0.w, a1.x, a1.y, a1.z, a1.w};
 #pragma unroll
-    for (int r = 0; r < 8; ++r) {
-      acc[r][0] = fmaf(av[r], b.x, acc[r][0]);
-      acc[r][1] = fmaf(av[r], b.y, acc[r][1]);
-      acc[r][2] = fmaf(av[r], b.z, acc[r][2]);
-      acc[r][3] = fmaf(av[r], b.w, acc[r][3]);
+    for (int q = 0; q < A; ++q) {
+      const float4 a = *reinterpret_cast<const float4*>(ar + i * lda + 4 * q);
+      const float av[4] = {a.x, a.y, a.z, a.w};
+#pragma unroll
+      for (int r = 0; r < 4; ++r) {
+        acc[4 * q + r][0] = fmaf(av[r], b.x, acc[4 * q + r][0]);
+        acc[4 * q + r][1] = fmaf(av[r], b.y, acc[4 * q + r][1]);
+        acc[4 * q + r][2] = fmaf(av[r], b.z, acc[4 * q + r][2]);
+        acc[4 * q + r][3] = fmaf(av[r], b.w, acc[4 * q + r][3]);
+      }
     }
   }
 }
 
+// Loads in flight per thread before the first is stored to shared memory: one after the other each would wait for memory.
+constexpr int SC_LOADS = 8;
+
 // [nt rows of `width`] -> tile [SC_Q][ld], zero past the edges; four columns an access where the source allows it.
 __device__ __forceinline__ void load_rows(const float* src, int stride, int rows, int width, bool vec, float* dst, int ld, int cols,
                                           int total_rows, int tid, int threads) {
-  const int quads = cols / 4;
-  for (int idx = tid; idx < total_rows * quads; idx += threads) {
-    const int r = idx / quads, c = (idx - r * quads) * 4;
-    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (r < rows) {
-      const float* p = src + (size_t)r * stride + c;
-      if (vec && c + 4 <= width) {
-        v = *reinterpret_cast<const float4*>(p);
-      } else {
-        if (c < width) v.x = p[0];
-        if (c + 1 < width) v.y = p[1];
-        if (c + 2 < width) v.z = p[2];
-        if (c + 3 < width) v.w = p[3];
+  const int quads = cols / 4, total = total_rows * quads;
+  for (int base = tid; base < total; base += threads * SC_LOADS) {
+    float4 v[SC_LOADS];
+#pragma unroll
+    for (int u = 0; u < SC_LOADS; ++u) {
+      const int idx = base + u * threads, r = idx / quads, c = (idx - r * quads) * 4;
+      v[u] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (idx < total && r < rows) {
+        const float* p = src + (size_t)r * stride + c;
+        if (vec && c + 4 <= width) {
+          v[u] = *reinterpret_cast<const float4*>(p);
+        } else {
+          if (c < width) v[u].x = p[0];
+          if (c + 1 < width) v[u].y = p[1];
+          if (c + 2 < width) v[u].z = p[2];
+          if (c + 3 < width) v[u].w = p[3];
+        }
       }
     }
-    *reinterpret_cast<float4*>(dst + r * ld + c) = v;
+#pragma unroll
+    for (int u = 0; u < SC_LOADS; ++u) {
+      const int idx = base + u * threads, r = idx / quads, c = (idx - r * quads) * 4;
+      if (idx < total) *reinterpret_cast<float4*>(dst + r * ld + c) = v[u];
+    }
   }
 }
 
@@ -160,7 +176,7 @@ __global__ void __launch_bounds__(2 * NP) chunk_leave_kernel(ScanChunkArgs a) {
   __syncthreads();
   const int n_at = (tid / 16) * 8, v_at = (tid % 16) * 4;
   float acc[8][4] = {};
-  tile_product(acc, b_s + n_at, NP, x_s + v_at, SC_V, nt);
+  tile_product<2>(acc, b_s + n_at, NP, x_s + v_at, SC_V, nt);
   float* dst = a.left + ((size_t)g * a.H + h) * N * a.dv + v0 + v_at;
   const bool vec = (a.dv & 3) == 0 && v0 + v_at + 4 <= a.dv;
 #pragma unroll
@@ -226,29 +242,41 @@ __global__ void chunk_combine_kernel(ScanChunkArgs a) {
 __device__ __forceinline__ void load_transposed(const float* src, int stride, int nt, int N, int NP, float* dst, int warp, int warps, int lane) {
   const bool vec = rows_aligned(src, stride);
   const int t_local = lane & 7, n4 = (lane >> 3) * 4;      // a warp takes 8 tokens x 16 columns
-  for (int tile = warp; tile < (SC_Q / 8) * (NP / 16); tile += warps) {
-    const int t = (tile & 7) * 8 + t_local, n = (tile >> 3) * 16 + n4;
-    float v[4] = {0.f, 0.f, 0.f, 0.f};
-    if (t < nt) {
-      const float* p = src + (size_t)t * stride + n;
-      if (vec && n + 4 <= N) {
-        const float4 q = *reinterpret_cast<const float4*>(p);
-        v[0] = q.x; v[1] = q.y; v[2] = q.z; v[3] = q.w;
-      } else {
+  const int tiles = (SC_Q / 8) * (NP / 16);
+  for (int base = warp; base < tiles; base += warps * SC_LOADS) {
+    float v[SC_LOADS][4];
 #pragma unroll
-        for (int e = 0; e < 4; ++e)
-          if (n + e < N) v[e] = p[e];
+    for (int u = 0; u < SC_LOADS; ++u) {
+      const int tile = base + u * warps, t = (tile & 7) * 8 + t_local, n = (tile >> 3) * 16 + n4;
+#pragma unroll
+      for (int e = 0; e < 4; ++e) v[u][e] = 0.f;
+      if (tile < tiles && t < nt) {
+        const float* p = src + (size_t)t * stride + n;
+        if (vec && n + 4 <= N) {
+          const float4 q = *reinterpret_cast<const float4*>(p);
+          v[u][0] = q.x; v[u][1] = q.y; v[u][2] = q.z; v[u][3] = q.w;
+        } else {
+#pragma unroll
+          for (int e = 0; e < 4; ++e)
+            if (n + e < N) v[u][e] = p[e];
+        }
       }
     }
 #pragma unroll
-    for (int e = 0; e < 4; ++e) dst[(n + e) * SC_LD + t] = v[e];
+    for (int u = 0; u < SC_LOADS; ++u) {
+      const int tile = base + u * warps, t = (tile & 7) * 8 + t_local, n = (tile >> 3) * 16 + n4;
+      if (tile < tiles) {
+#pragma unroll
+        for (int e = 0; e < 4; ++e) dst[(n + e) * SC_LD + t] = v[u][e];
+      }
+    }
   }
 }
 
 // The read-outs of a chunk. A CTA is (chunk, some heads of one group, 64 value columns).
-constexpr int SC_READ_THREADS = 128;  // (64 / 8) x (64 / 4) tiles of 8 x 4
+constexpr int SC_READ_THREADS = 256;  // (64 / 4) x (64 / 4) tiles of 4 x 4: two CTAs of eight warps an SM
 template <int NP>
-__global__ void __launch_bounds__(SC_READ_THREADS) chunk_read_kernel(ScanChunkArgs a) {
+__global__ void __launch_bounds__(SC_READ_THREADS, 2) chunk_read_kernel(ScanChunkArgs a) {
   extern __shared__ __align__(16) float sc_smem[];
   float* c_s = sc_smem;               // [NP][SC_LD]: C, token fastest
   float* s_s = c_s + NP * SC_LD;      // [NP][SC_LD]: B, token fastest; then [NP][SC_V]: the starting state of a head
@@ -265,49 +293,61 @@ __global__ void __launch_bounds__(SC_READ_THREADS) chunk_read_kernel(ScanChunkAr
   const int h0 = blockIdx.y * a.heads_per_cta, grp = h0 / a.per_group;
   load_transposed(a.c + (size_t)t0 * a.c_stride + grp * N, a.c_stride, nt, N, NP, c_s, warp, SC_READ_THREADS / 32, lane);
   load_transposed(a.b + (size_t)t0 * a.b_stride + grp * N, a.b_stride, nt, N, NP, s_s, warp, SC_READ_THREADS / 32, lane);
+  auto load_x = [&](int h) {
+    const float* xp = a.x + (size_t)t0 * a.x_stride + h * a.dv + v0;
+    load_rows(xp, a.x_stride, nt, min(SC_V, a.dv - v0), rows_aligned(xp, a.x_stride), x_s, SC_V, SC_V, SC_Q, tid, SC_READ_THREADS);
+    if (warp == 0) chunk_steps(a, h, t0, nt, lane, dt_s, cum_s);
+  };
+  load_x(h0);
   __syncthreads();
-  const int t_at = (tid / 16) * 8, col = (tid % 16) * 4;   // this thread's tokens; its keys s, or its value columns
+  const int t_at = (tid / 16) * 4, col = (tid % 16) * 4;   // this thread's tokens; its keys s, or its value columns
   const bool live = t_at < nt;
-  float score[8][4] = {};
-  if (live && col <= t_at + 7) tile_product(score, c_s + t_at, SC_LD, s_s + col, SC_LD, N);
   const int cols = min(SC_V, a.dv - v0);
+  float score[4][4] = {};
+  if (live && col <= t_at + 3) tile_product<1>(score, c_s + t_at, SC_LD, s_s + col, SC_LD, N);
   for (int h = h0; h < h0 + a.heads_per_cta; ++h) {
     __syncthreads();                  // B, or the head before, has been read
-    if (warp == 0) chunk_steps(a, h, t0, nt, lane, dt_s, cum_s);
-    const float* xp = a.x + (size_t)t0 * a.x_stride + h * a.dv + v0;
-    load_rows(xp, a.x_stride, nt, cols, rows_aligned(xp, a.x_stride), x_s, SC_V, SC_V, SC_Q, tid, SC_READ_THREADS);
+    // the head's starting state travels while the weighted scores are made
     const float* sp = a.left + ((size_t)g * a.H + h) * N * a.dv + v0;
-    load_rows(sp, a.dv, N, cols, rows_aligned(sp, a.dv), s_s, SC_V, SC_V, N, tid, SC_READ_THREADS);
-    __syncthreads();
+    if (cols == SC_V && rows_aligned(sp, a.dv)) {
+      for (int idx = tid; idx < N * (SC_V / 4); idx += SC_READ_THREADS)
+        __pipeline_memcpy_async(s_s + idx * 4, sp + (size_t)(idx / (SC_V / 4)) * a.dv + (idx % (SC_V / 4)) * 4, 16);
+    } else {
+      load_rows(sp, a.dv, N, cols, rows_aligned(sp, a.dv), s_s, SC_V, SC_V, N, tid, SC_READ_THREADS);
+    }
+    __pipeline_commit();
+    if (h > h0) {
+      load_x(h);
+      __syncthreads();
+    }
     if (tid < SC_Q) fall_s[tid] = expf((float)cum_s[tid]);
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int s = col + j;
-      float m[8];
+      float m[4];
 #pragma unroll
-      for (int r = 0; r < 8; ++r) {
+      for (int r = 0; r < 4; ++r) {
         const int t = t_at + r;
         m[r] = s <= t && t < nt ? score[r][j] * expf((float)(cum_s[t] - cum_s[s])) * dt_s[s] : 0.f;
       }
-      float4* p = reinterpret_cast<float4*>(m_s + s * SC_LD + t_at);
-      p[0] = make_float4(m[0], m[1], m[2], m[3]);
-      p[1] = make_float4(m[4], m[5], m[6], m[7]);
+      *reinterpret_cast<float4*>(m_s + s * SC_LD + t_at) = make_float4(m[0], m[1], m[2], m[3]);
     }
+    __pipeline_wait_prior(0);
     __syncthreads();
     if (live) {
-      float acc[8][4] = {};
-      tile_product(acc, c_s + t_at, SC_LD, s_s + col, SC_V, N);
+      float acc[4][4] = {};
+      tile_product<1>(acc, c_s + t_at, SC_LD, s_s + col, SC_V, N);
 #pragma unroll
-      for (int r = 0; r < 8; ++r) {
+      for (int r = 0; r < 4; ++r) {
         const float f = fall_s[t_at + r];
 #pragma unroll
         for (int j = 0; j < 4; ++j) acc[r][j] *= f;
       }
-      tile_product(acc, m_s + t_at, SC_LD, x_s + col, SC_V, min(nt, t_at + 8));
+      tile_product<1>(acc, m_s + t_at, SC_LD, x_s + col, SC_V, min(nt, t_at + 4));
       const float skip = a.skip[h];
       const bool vec = (a.dv & 3) == 0 && col + 4 <= cols;
 #pragma unroll
-      for (int r = 0; r < 8; ++r) {
+      for (int r = 0; r < 4; ++r) {
         const int t = t_at + r;
         if (t >= nt) break;
         const float4 xv = *reinterpret_cast<const float4*>(x_s + t * SC_V + col);
