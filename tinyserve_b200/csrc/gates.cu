@@ -47,7 +47,7 @@ __global__ void act_mul_kernel(const T* __restrict__ gate_up, const T* __restric
 
 // x <- act(x), in 32-bit, rounded once: an activation that gates nothing
 template <typename T, int ACT>
-__global__ void activate_kernel(T* __restrict__ x, size_t total) {
+__global__ void activate_kernel(T* x, size_t total) {
   pdl_trigger();
   pdl_wait();
   for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < total; idx += (size_t)gridDim.x * blockDim.x)
@@ -127,10 +127,11 @@ __global__ void head_norm_gate_kernel(const IN* __restrict__ x, const T* __restr
 }
 
 // The same with four columns an access and the values kept in registers between the two passes: a warp per (token, head) of
-// up to 128 J columns (a multiple of 4, everything aligned).
+// up to 128 J columns (a multiple of 4, everything aligned). No __restrict__ on what earlier kernels wrote, so that no read
+// moves in front of the wait for them.
 template <typename IN, typename T, int J>
-__global__ void __launch_bounds__(128) head_norm_gate_quads_kernel(const IN* __restrict__ x, const T* __restrict__ weight, int weight_head_stride,
-                                                                   const T* __restrict__ gate, int gate_stride, T* __restrict__ out,
+__global__ void __launch_bounds__(128) head_norm_gate_quads_kernel(const IN* x, const T* __restrict__ weight, int weight_head_stride,
+                                                                   const T* gate, int gate_stride, T* out,
                                                                    int num_tokens, int heads, int width, int normalise, float eps,
                                                                    int gate_silu, int gate_first) {
   pdl_trigger();

@@ -1,6 +1,7 @@
 // Two attention maps of a head over the same values, combined: o = a1 - factor a2, divided by its root mean square over
 // the head's value columns, times a constant. One warp per (row, head); x is [T, heads, 2, dv], out [T, heads, dv]. The rows
-// are all rows of a step or, with a list of requests, each one's only new row. 32-bit, rounded once.
+// are all rows of a step or, with a list of requests, each one's only new row. 32-bit, rounded once. What earlier kernels
+// wrote is read through pointers without __restrict__, so that no read can move in front of the wait for them.
 #define TS_PDL_CLASS PDL_ELEMENTWISE
 #include "common.cuh"
 
@@ -10,8 +11,8 @@ constexpr int PC_WARPS = 4;
 constexpr int PC_COLS = 8;        // value columns a lane keeps (dv up to 256)
 
 template <typename T>
-__global__ void __launch_bounds__(PC_WARPS * 32) pair_combine_kernel(const T* __restrict__ x, const float* __restrict__ factor, float eps,
-                                                                     float mult, T* __restrict__ out, int num_rows, int heads, int dv,
+__global__ void __launch_bounds__(PC_WARPS * 32) pair_combine_kernel(const T* x, const float* __restrict__ factor, float eps,
+                                                                     float mult, T* out, int num_rows, int heads, int dv,
                                                                      const int* __restrict__ seqs, const int* __restrict__ cu_q) {
   pdl_trigger();
   pdl_wait();

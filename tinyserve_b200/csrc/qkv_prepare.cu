@@ -217,10 +217,9 @@ __global__ void qkv_prepare_kernel(const T* __restrict__ q_in, int q_stride, con
 // whose pairs lie a whole number of lanes apart, no biases, everything 16-byte aligned.
 template <int LPH>
 __global__ void __launch_bounds__(128) qkv_prepare_packed_kernel(
-    const bf16* __restrict__ q_in, int q_stride, const bf16* __restrict__ k_in, int k_stride, const bf16* __restrict__ v_in, int v_stride,
-    const bf16* __restrict__ q_w, const bf16* __restrict__ k_w, float eps, const float* __restrict__ cos_tab,
-    const float* __restrict__ sin_tab, int rotary_dim, const int* __restrict__ slots, bf16* __restrict__ k_cache,
-    bf16* __restrict__ v_cache, int page_size, int num_tokens, int heads, int kv_heads, int d, int dv, bf16* __restrict__ q_out, int maps) {
+    const bf16* q_in, int q_stride, const bf16* k_in, int k_stride, const bf16* v_in, int v_stride, const bf16* __restrict__ q_w,
+    const bf16* __restrict__ k_w, float eps, const float* cos_tab, const float* sin_tab, int rotary_dim, const int* slots, bf16* k_cache,
+    bf16* v_cache, int page_size, int num_tokens, int heads, int kv_heads, int d, int dv, bf16* q_out, int maps) {
   pdl_trigger();
   pdl_wait();
   const int k_heads = k_in ? kv_heads * maps : 0, v_pieces = (dv + 8 * LPH - 1) / (8 * LPH);

@@ -392,11 +392,11 @@ __global__ void causal_conv_silu_kernel(const T* __restrict__ x, int x_stride, c
 // bytes at a time. KP: the taps rounded up to 4 or 8, the missing ones zero.
 constexpr int CONV_RUN = 16, CONV_MIN_TOKENS = 64;
 template <typename T, int KP>
-__global__ void __launch_bounds__(128) causal_conv_silu_run_kernel(const T* __restrict__ x, int x_stride, const T* __restrict__ taps,
-                                                                   const T* __restrict__ bias, const float* __restrict__ state,
+__global__ void __launch_bounds__(128) causal_conv_silu_run_kernel(const T* x, int x_stride, const T* __restrict__ taps,
+                                                                   const T* __restrict__ bias, const float* state,
                                                                    int state_stride, const int* __restrict__ cu_q,
                                                                    const int* __restrict__ state_slots, int num_seqs, int num_tokens, int C,
-                                                                   int K, float* __restrict__ y) {
+                                                                   int K, float* y) {
   pdl_trigger();
   pdl_wait();
   const int c = (blockIdx.x * blockDim.x + threadIdx.x) * 4;
@@ -415,6 +415,8 @@ __global__ void __launch_bounds__(128) causal_conv_silu_run_kernel(const T* __re
   }
   int start = cu_q[lo], end = cu_q[lo + 1];
   const float* st = state + (size_t)state_slots[lo] * state_stride + c;
+  float next[4];                          // the input of token t
+  Quad<T>::load(x + (size_t)first * x_stride + c, next);
   bool fill = true;                       // the inputs before token t are not in the registers yet
   for (int t = first; t < last; ++t) {
     while (t >= end && lo + 1 < num_seqs) {
@@ -444,7 +446,9 @@ __global__ void __launch_bounds__(128) causal_conv_silu_run_kernel(const T* __re
     for (int j = 0; j < KP - 1; ++j)
 #pragma unroll
       for (int e = 0; e < 4; ++e) in[j][e] = in[j + 1][e];
-    Quad<T>::load(x + (size_t)t * x_stride + c, in[KP - 1]);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) in[KP - 1][e] = next[e];
+    if (t + 1 < last) Quad<T>::load(x + (size_t)(t + 1) * x_stride + c, next);      // in flight during this token's arithmetic
     float o[4];
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
@@ -459,10 +463,10 @@ __global__ void __launch_bounds__(128) causal_conv_silu_run_kernel(const T* __re
 
 // A step in which no request brings more than one token: output and new state in one pass, a thread per (request, channel).
 template <typename T>
-__global__ void causal_conv_silu_single_kernel(const T* __restrict__ x, int x_stride, const T* __restrict__ taps,
-                                               const T* __restrict__ bias, float* __restrict__ state, int state_stride,
+__global__ void causal_conv_silu_single_kernel(const T* x, int x_stride, const T* __restrict__ taps,
+                                               const T* __restrict__ bias, float* state, int state_stride,
                                                const int* __restrict__ cu_q, const int* __restrict__ state_slots, int C, int K,
-                                               float* __restrict__ y) {
+                                               float* y) {
   pdl_trigger();
   pdl_wait();
   const int b = blockIdx.x, t = cu_q[b];

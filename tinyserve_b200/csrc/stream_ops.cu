@@ -105,10 +105,10 @@ __global__ void stream_sum_kernel(StreamSumArgs a) {
 }
 
 // --------------------------------------------------- the stream beside the embedding output
-// out[t] = [resid[t] + delta[t], origin[t]]: the sum in 32-bit, both halves rounded once. The stream itself stays.
+// out[t] = [resid[t] + delta[t], origin[t]]: the sum in 32-bit, both halves rounded once. The stream itself stays. (No
+// __restrict__ on what earlier kernels wrote: no read may move in front of the wait for them.)
 template <typename T, int VEC>
-__global__ void stream_beside_kernel(const float* __restrict__ resid, const T* __restrict__ delta, const float* __restrict__ origin,
-                                     T* __restrict__ out, int hidden, size_t total) {
+__global__ void stream_beside_kernel(const float* resid, const T* delta, const float* origin, T* out, int hidden, size_t total) {
   pdl_trigger();
   pdl_wait();
   const size_t n = total / VEC;
