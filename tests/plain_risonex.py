@@ -153,7 +153,7 @@ def state_space_scan(x: torch.Tensor, b: torch.Tensor, c: torch.Tensor, dt: torc
 
 
 def gate_and_norm(y: torch.Tensor, z: torch.Tensor, weight: torch.Tensor, parts: int, eps: float) -> torch.Tensor:
-    """``y``, ``z`` ``[T, inner]``: the gate first, then every part by its own root mean square."""
+    """``y``, ``z`` ``[T, inner]``: gated, then normed part by part."""
     t, inner = y.shape
     g = y * silu(z)
     return over_rms(g.view(t, parts, inner // parts), eps).reshape(t, inner) * weight

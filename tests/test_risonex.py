@@ -213,7 +213,7 @@ def test_reference_state_space_mixer(taps, cuts, heads, groups, n, dv, parts) ->
         assert (other - want).abs().max() > 1e-2, "parts normed together would give the same"
 
 
-def test_the_gate_comes_before_the_norm() -> None:
+def test_gated_before_it_is_normed() -> None:
     y, z, w = _rand(3, 12, seed=1).float(), _rand(3, 12, seed=2).float(), _rand(12, seed=3).float()
     out, late = torch.zeros(3, 12), torch.zeros(3, 12)
     refs.head_norm_gate(y.view(3, 3, 4), w, True, z, True, 1e-5, out, gate_silu=True, gate_first=True)

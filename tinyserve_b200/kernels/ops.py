@@ -458,8 +458,8 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
     the window. ``chunk`` (instead of a window): a query sees only its own run of ``chunk`` positions, counted
     from position 0. ``out`` ``[T, Hq * Dv]`` dt.
 
-    ``maps=2``: every query head and every key row holds two maps side by side (``D / 2`` elements each), each an
-    attention of its own over the same values: ``out`` is ``[T, Hq * 2 * Dv]``, map innermost. With ``finish =
+    ``maps=2``: every query head and every key row holds two maps side by side (``D / 2`` elements each), which
+    attend independently over shared values: ``out`` is ``[T, Hq * 2 * Dv]``, map innermost. With ``finish =
     (finished, factor, mult, eps)`` the maps are combined too: ``finished [T, Hq * Dv]`` dt receives ``a1 - factor a2``
     over its root mean square per head, times ``mult`` (``factor``: one float32 on the device), and ``out`` is scratch."""
     t, hq, d = q.shape

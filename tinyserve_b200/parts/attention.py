@@ -496,12 +496,12 @@ class RotatedAttention(Mixer):
 class DifferentialAttention(Mixer):
     """Attention with two maps per head over the same values, the second subtracted with a learned factor.
 
-    ``q = W_q h`` has ``num_heads * 2 * key_dim`` rows and ``k = W_k h`` ``num_kv_heads * 2 * key_dim``, head by head as
-    [map 1, map 2]; ``v = W_v h`` (``num_kv_heads x value_dim``); no biases. With ``qk_norm`` every map of every q and k
-    head is RMS-normed with a plain weight of ``key_dim`` values shared by heads and maps. q and k turn as the layer's
-    position encoding asks, if it has one. Each map is an attention of its own: scores ``scale * q . k``, causal, with
+    ``q = W_q h`` has ``num_heads * 2 * key_dim`` rows and ``k = W_k h`` ``num_kv_heads * 2 * key_dim``; within a head the
+    first map's rows precede the second's; ``v = W_v h`` (``num_kv_heads x value_dim``); no biases. With ``qk_norm`` every map of
+    every q and k head is RMS-normed with a plain weight of ``key_dim`` values shared by heads and maps. q and k turn as the layer's
+    position encoding asks, if it has one. The two maps attend independently: scores ``scale * q . k``, causal, with
     ``window`` only the last ``window`` positions, with ``chunk`` only the query's own run of ``chunk`` positions counted
-    from position 0; ordinary softmax. ``factor = exp(lq1 . lk1) - exp(lq2 . lk2) + diff``, one number for the layer; per
+    from position 0; ordinary softmax. ``factor = exp(lq1 . lk1) - exp(lq2 . lk2) + diff``, shared by all heads; per
     head ``o = a1 - factor a2``, divided by its root mean square over the head (no weight), times ``1 - diff``; ``W_o`` on
     the concatenated heads. ``names`` maps the roles "q", "k", "v", "out", "q_norm", "k_norm", "lq1", "lk1", "lq2", "lk2"
     to tensor names after the prefix.
